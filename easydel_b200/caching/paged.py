@@ -34,6 +34,7 @@ class PagedBatchMeta:
     request_distribution: tuple[int, int, int] | None = None  # (#decode, #decode+#prefill, #total)
     num_splits: int = 1          # decode-only steps: cut every sequence's keys into this many page ranges
     seq_slots: torch.Tensor | None = None   # int64 [B] engine slot of every sequence (recurrent-state pools)
+    slot_ids: torch.Tensor | None = None    # int32 [B] the same for states that kernels address in place
     # cache groups beyond the first (sliding-window / chunked-local layers with their own pools): per group the page
     # table [B, maxP] and the slot mapping [T]; entry g - 1 belongs to group g
     group_tables: list | None = None
@@ -73,7 +74,8 @@ class PagedKVCache:
             shape = (len(grp.layers), int(grp.num_pages), page_size, grp.spec.num_kv_heads, grp.spec.head_dim)
             k = torch.zeros(shape, dtype=dtype, device=device)      # zeros: the null page must hold finite numbers
             self._k.append(k)
-            self._v.append(k if grp.kind == "latent" else torch.zeros(shape, dtype=dtype, device=device))
+            v_shape = (*shape[:-1], grp.spec.value_dim)
+            self._v.append(k if grp.kind == "latent" else torch.zeros(v_shape, dtype=dtype, device=device))
             for j, layer in enumerate(grp.layers):
                 self.layer_slot[layer] = (g, j)
         # hybrids: layer -> recurrent state with one row per engine slot; ``step_meta`` is the running step's batch
@@ -105,8 +107,16 @@ class PagedKVCache:
         return n
 
     def add_state_pools(self, model, num_slots: int) -> None:
-        layers = getattr(getattr(model, "model", model), "layers", ())
+        backbone = getattr(model, "model", model)
+        layers = getattr(backbone, "layers", ())
+        runs = getattr(backbone, "layer_runs", None)
+        if runs is not None:          # looped layers: every run of a layer has a state of its own
+            layers = [layers[i] for i in runs]
         for i, layer in enumerate(layers):
+            state = layer.make_slot_state(num_slots, self.k.device) if hasattr(layer, "make_slot_state") else None
+            if state is not None:
+                self.linear[i] = state
+                continue
             mixer = getattr(layer, "linear_attn", None) or getattr(layer, "mamba", None)
             if mixer is None and hasattr(getattr(layer, "self_attn", None), "make_state"):
                 mixer = layer.self_attn
@@ -137,6 +147,8 @@ class PagedKVCache:
 
         spec = model.spec
         device = device or model.device
+        if dtype is None and getattr(spec, "residual_f32", False) and model.dtype == torch.float32:
+            dtype = torch.float32       # an all-fp32 model keeps its keys and values in 32 bits too
         dtype = dtype or getattr(model.config, "kvdtype", None) or model.dtype
         es = torch.empty(0, dtype=dtype).element_size()
         latent = getattr(spec, "mla", None) is not None
@@ -177,8 +189,18 @@ class PagedKVCache:
             view = PagedLatentView(self._k[g][j]) if self.groups[g].kind == "latent" else \
                 PagedLayerView(self._k[g][j], self._v[g][j], group=g)
         pool = self.linear.get(layer)
-        view.linear_state = None if pool is None else PagedLinearState(pool, self.step_meta)
+        if pool is None:
+            view.linear_state = None
+        elif getattr(pool, "in_place", False):
+            view.linear_state = pool          # its kernels address the rows of the scheduled sequences themselves
+        else:
+            view.linear_state = PagedLinearState(pool, self.step_meta)
         return view
+
+    @property
+    def states_in_place(self) -> bool:
+        """True when no recurrent state is gathered and scattered around a step (then decode steps can be captured)."""
+        return all(getattr(st, "in_place", False) for st in self.linear.values())
 
     def seq_len(self) -> int:  # the engine passes explicit positions
         return 0
@@ -214,27 +236,89 @@ class PagedLayerView:
 
         q ``[1, T, Hq, D]`` / k, v ``[1, T, Hkv, D]`` (all sequences flattened on the token axis)."""
         meta = attn_meta
-        T = q.shape[1]
         q3, k3, v3 = q[0], k[0], v[0]
-        table = meta.table_of(self.group)
         S.kv_append(k3, v3, self.k_pages, self.v_pages, meta.slots_of(self.group))
         if getattr(attn, "chunk_size", None) or (q3.is_cuda and q3.shape[-1] not in (64, 128)):
-            # block-diagonal attention, or a head size outside the paged kernel's (64 / 128)
+            # block-diagonal attention, or (for these models) a head size other than 64 / 128
             return self._attend_gathered(attn, q3, meta)[None]
-        if meta.max_q == 1 and q3.shape[0] == meta.num_seqs and S.decode_kernel_supports(q3, self.k_pages,
-                                                                                           attn.softcap):
+        return self.attend_pages(attn, q3, meta)[None]
+
+    def attend_pages(self, attn, q3, meta: PagedBatchMeta):
+        """Attention of ``q3 [T, Hq, D]`` over the pages, which already hold this step's keys and values."""
+        table = meta.table_of(self.group)
+        if meta.max_q == 1 and q3.shape[0] == meta.num_seqs and S.decode_kernel_supports(
+                q3, self.k_pages, attn.softcap, self.v_pages.shape[-1]):
             # a pure decode step: the streaming kernel (one CTA per sequence, KV head and key split)
             o = S.decode_attention(q3, self.k_pages, self.v_pages, meta.kv_lens, table, scale=attn.scale,
                                    window=attn.sliding_window or 0, sinks=attn.sinks, num_splits=meta.num_splits)
-            return o[None]
-        if meta.num_splits > 1 and meta.max_q == 1 and not attn.sliding_window and q3.is_cuda:
+            return o
+        if meta.num_splits > 1 and meta.max_q == 1 and not attn.sliding_window and q3.is_cuda and \
+                q3.dtype == torch.bfloat16 and self.v_pages.shape[-1] == q3.shape[-1] and q3.shape[-1] in (64, 128):
             o = S.paged_attention_splitkv(q3, self.k_pages, self.v_pages, meta.kv_lens, table,
                                           meta.num_splits, scale=attn.scale, softcap=attn.softcap, sinks=attn.sinks)
-            return o[None]
-        o = S.paged_attention(q3, self.k_pages, self.v_pages, meta.cu_q, meta.kv_lens, table, meta.max_q,
+            return o
+        return S.paged_attention(q3, self.k_pages, self.v_pages, meta.cu_q, meta.kv_lens, table, meta.max_q,
                               scale=attn.scale, causal=True, window=attn.sliding_window or 0, softcap=attn.softcap,
-                              sinks=attn.sinks)
-        return o[None]
+                                 sinks=attn.sinks)
+
+
+class PagedBatchCache(PagedKVCache):
+    """Pages and states of a fixed batch, for ``model.generate`` and for forward passes without a cache of models that
+    run on flattened token rows (:attr:`ArchSpec.residual_f32`): row b owns a contiguous run of pages and state row b."""
+
+    length = 0             # tokens of the widest row so far (padding included), as the dense cache counts them
+
+    @classmethod
+    def for_model(cls, model, batch: int, max_length: int):
+        backbone = getattr(model, "model", model)
+        per_row = max(1, (max_length + PAGE_SIZE - 1) // PAGE_SIZE)
+        self = cls.init_for_model(backbone, num_pages=max(2, batch * per_row))
+        self.add_state_pools(backbone, batch)
+        dev = self.k.device
+        self.batch, self.max_len = batch, per_row * PAGE_SIZE
+        self._table = torch.arange(batch * per_row, dtype=torch.int32, device=dev).view(batch, per_row)
+        self._slots = torch.arange(batch, dtype=torch.int32, device=dev)
+        self._lens = [0] * batch
+        return self
+
+    def seq_len(self) -> int:
+        return self.length
+
+    def advance(self, n: int) -> None:
+        self.length += n
+
+    def begin(self, new_tokens: list[int]) -> "tuple[PagedBatchMeta, torch.Tensor]":
+        """Metadata of a step that appends ``new_tokens[b]`` tokens to row b, and the position of every new token."""
+        dev = self.k.device
+        pos, cu = [], [0]
+        for b, n in enumerate(new_tokens):
+            pos.append(torch.arange(self._lens[b], self._lens[b] + n))
+            self._lens[b] += n
+            cu.append(cu[-1] + n)
+        if max(self._lens) > self.max_len:
+            raise ValueError(f"KV cache overflow: {max(self._lens)} > {self.max_len}")
+        p = torch.cat(pos).to(device=dev, dtype=torch.int32)
+        row = torch.repeat_interleave(torch.arange(self.batch, device=dev), torch.tensor(new_tokens, device=dev))
+        slots = (self._table[row, (p // PAGE_SIZE).long()] * PAGE_SIZE + p % PAGE_SIZE).to(torch.int32)
+        tables = [self._table] * (self.num_groups - 1)
+        meta = PagedBatchMeta(cu_q=torch.tensor(cu, dtype=torch.int32, device=dev),
+                              kv_lens=torch.tensor(self._lens, dtype=torch.int32, device=dev), page_table=self._table,
+                              slot_mapping=slots, max_q=max(new_tokens), num_seqs=self.batch, slot_ids=self._slots,
+                              group_tables=tables, group_slots=[slots] * (self.num_groups - 1))
+        self.step_meta = meta
+        return meta, p
+
+    def reorder(self, index: torch.Tensor) -> None:
+        """Beam search: row b continues what row ``index[b]`` holds."""
+        pages = self._table[index].reshape(-1).long()
+        for pools in (self._k, self._v):
+            for t in pools:
+                t[:, : pages.numel()] = t[:, pages]
+        for st in self.linear.values():
+            for v in vars(st).values():
+                if isinstance(v, torch.Tensor):
+                    v.copy_(v.index_select(0, index))
+        self._lens = [self._lens[i] for i in index.tolist()]
 
 
 def _pad_queries(q, meta: PagedBatchMeta):

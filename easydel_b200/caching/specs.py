@@ -29,10 +29,15 @@ class KVCacheSpec:
     head_dim: int = 128
     element_size: int = 2
     kind: str = "full"
+    v_head_dim: int = 0          # 0 = values are as wide as keys
+
+    @property
+    def value_dim(self) -> int:
+        return self.v_head_dim or self.head_dim
 
     @property
     def page_size_bytes(self) -> int:
-        return 2 * self.page_size * self.num_kv_heads * self.head_dim * self.element_size
+        return self.page_size * self.num_kv_heads * (self.head_dim + self.value_dim) * self.element_size
 
     def tokens_kept(self, context: int) -> int:
         return context
@@ -50,7 +55,7 @@ class KVCacheSpec:
         return self.pages_per_sequence(max_model_len, max_step_tokens) * self.page_size_bytes
 
     def group_key(self) -> tuple:
-        return (self.kind, 0, self.num_kv_heads, self.head_dim, self.element_size)
+        return (self.kind, 0, self.num_kv_heads, self.head_dim, self.value_dim, self.element_size)
 
 
 @dataclass(frozen=True)
@@ -75,7 +80,7 @@ class SlidingWindowSpec(KVCacheSpec):
         return min(cdiv(max_model_len, self.page_size), cdiv(span, self.page_size) + 1)
 
     def group_key(self) -> tuple:
-        return (self.kind, self.sliding_window, self.num_kv_heads, self.head_dim, self.element_size)
+        return (self.kind, self.sliding_window, self.num_kv_heads, self.head_dim, self.value_dim, self.element_size)
 
 
 @dataclass(frozen=True)
@@ -95,7 +100,7 @@ class ChunkedLocalAttentionSpec(KVCacheSpec):
         return min(cdiv(max_model_len, self.page_size), cdiv(span, self.page_size) + 1)
 
     def group_key(self) -> tuple:
-        return (self.kind, self.attention_chunk_size, self.num_kv_heads, self.head_dim, self.element_size)
+        return (self.kind, self.attention_chunk_size, self.num_kv_heads, self.head_dim, self.value_dim, self.element_size)
 
 
 @dataclass(frozen=True)
@@ -151,7 +156,8 @@ def layer_spec(info, element_size: int = 2, tp_size: int = 1, page_size: int = P
     if not info.requires_kv_cache:
         return None
     kvh = max(1, info.num_kv_heads // max(1, tp_size)) if info.layer_type != "latent_attention" else 1
-    common = dict(page_size=page_size, num_kv_heads=kvh, head_dim=info.head_dim, element_size=element_size)
+    common = dict(page_size=page_size, num_kv_heads=kvh, head_dim=info.head_dim, element_size=element_size,
+                  v_head_dim=info.v_head_dim if info.v_head_dim != info.head_dim else 0)
     if info.layer_type == "latent_attention":
         return MLAAttentionSpec(**common)
     if info.sliding_window:

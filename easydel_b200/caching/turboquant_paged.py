@@ -170,6 +170,8 @@ class TurboQuantPagedKVCache:
         tp_size = getattr(getattr(model.config, "mesh", None), "tp", 1)
         hkv = max(1, spec.num_kv_heads // tp_size)
         probe = cls(1, 2, hkv, spec.head_dim, config, device="cpu")
+        if getattr(spec, "residual_f32", False):
+            raise NotImplementedError("compressed key / value pages are not available for models with an fp32 stream")
         per_page = probe.bytes_per_token_head * hkv * PAGE_SIZE * spec.num_layers
         if num_pages is None:
             if torch.device(device).type == "cuda":

@@ -14,7 +14,9 @@
 //     through shared memory and written as bf16 rows, plus the log-sum-exp when the caller merges key splits.
 //
 // Replaces the decode branch of the reference's ragged / paged attention kernels
-// (easydel/operations/kernels/ragged_page_attention_v3.py, page_attention.py) for head sizes 64 and 128.
+// (easydel/operations/kernels/ragged_page_attention_v3.py, page_attention.py). Query / key and value sizes of a head are
+// separate multiples of 8 up to 128: tiles are DQ / DV = 64 or 128 columns wide and the tensor maps fill the columns
+// past a head's end with zeros.
 #include "common.cuh"
 
 namespace edl {
@@ -34,7 +36,7 @@ constexpr int PAGE = 128;
 constexpr float LOG2E_F = 1.4426950408889634f;
 
 struct DecodeParams {
-  const __nv_bfloat16* q;   // [B, ldq]: head h at columns h * D
+  const __nv_bfloat16* q;   // [B, ldq]: head h at columns h * dq
   long long ldq;
   __nv_bfloat16* o;         // [splits, B, ldo]
   long long ldo;
@@ -43,6 +45,7 @@ struct DecodeParams {
   const int* page_table;    // [B, pt_stride]
   const float* sinks;       // [Hq] or null (only without splits)
   int pt_stride, B, Hq, Hkv, splits, window;
+  int dq, dv;               // real query / key and value sizes of a head
   float scale_log2;
   int* status;
 };
@@ -67,32 +70,31 @@ __device__ __forceinline__ void mma_bf16_16816(float (&d)[4], const uint32_t (&a
 
 // Byte offset of (row, 16-byte chunk) inside a [TK rows x D] tile stored as D/64 boxes of [TK x 128 bytes] with the
 // 128-byte swizzle the tensor maps use (chunk index XOR row % 8 within a box).
-template <int D>
 __device__ __forceinline__ uint32_t tile_off(int row, int chunk) {
   const int box = chunk >> 3, c = chunk & 7;
   return box * (TK * 128) + row * 128 + ((c ^ (row & 7)) << 4);
 }
 
-template <int D>
+template <int DQ, int DV>
 struct DCfg {
-  static constexpr int TILE_BYTES = TK * D * 2;                       // one K or V tile
-  static constexpr int STAGE_BYTES = 2 * TILE_BYTES;                  // K + V
+  static constexpr int K_BYTES = TK * DQ * 2;                         // one K tile
+  static constexpr int STAGE_BYTES = K_BYTES + TK * DV * 2;           // K + V
   static constexpr int WARP_BYTES = DEC_STAGES * STAGE_BYTES;
-  static constexpr int Q_BYTES = 16 * (D * 2 + 16);                   // 16 rows, padded pitch against bank conflicts
+  static constexpr int Q_BYTES = 16 * (DQ * 2 + 16);                  // 16 rows, padded pitch against bank conflicts
   static constexpr int OFF_Q = DEC_WARPS * WARP_BYTES;
   static constexpr int OFF_BAR = OFF_Q + Q_BYTES;
   static constexpr int OFF_RED = OFF_BAR + 128;                       // merge area: per warp m[16], l[16]
   static constexpr int SMEM = OFF_RED + DEC_WARPS * 2 * 16 * 4 + 1024;
 };
 
-template <int D>
+template <int DQ, int DV>
 __global__ void __launch_bounds__(DEC_THREADS)
 attn_decode_kernel(const __grid_constant__ CUtensorMap tk, const __grid_constant__ CUtensorMap tv,
                    const DecodeParams p) {
-  using C = DCfg<D>;
-  constexpr int NKS = D / 16;     // k-steps of the score product
-  constexpr int NDB = D / 8;      // 8-column blocks of the output
-  constexpr int QPITCH = D * 2 + 16;
+  using C = DCfg<DQ, DV>;
+  constexpr int NKS = DQ / 16;     // k-steps of the score product
+  constexpr int NDB = DV / 8;     // 8-column blocks of the output
+  constexpr int QPITCH = DQ * 2 + 16;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   const uint32_t sbase = smem_u32(smem);
@@ -128,13 +130,13 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tk, const __grid_constant
     prefetch_tmap(&tk);
     prefetch_tmap(&tv);
   }
-  // query rows of this KV head's group -> shared memory (rows >= G are zero)
+  // query rows of this KV head's group -> shared memory (rows >= G and columns >= dq are zero)
   {
-    const __nv_bfloat16* qrow = p.q + (long long)b * p.ldq + (long long)hk * G * D;
-    for (int i = threadIdx.x; i < 16 * (D / 8); i += DEC_THREADS) {
-      const int r = i / (D / 8), c = i % (D / 8);
+    const __nv_bfloat16* qrow = p.q + (long long)b * p.ldq + (long long)hk * G * p.dq;
+    for (int i = threadIdx.x; i < 16 * (DQ / 8); i += DEC_THREADS) {
+      const int r = i / (DQ / 8), c = i % (DQ / 8);
       uint4 v = make_uint4(0u, 0u, 0u, 0u);
-      if (r < G) v = *reinterpret_cast<const uint4*>(qrow + (long long)r * D + c * 8);
+      if (r < G && c * 8 < p.dq) v = *reinterpret_cast<const uint4*>(qrow + (long long)r * p.dq + c * 8);
       *reinterpret_cast<uint4*>(smem + C::OFF_Q + r * QPITCH + c * 16) = v;
     }
   }
@@ -150,15 +152,15 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tk, const __grid_constant
     const uint32_t dst = my_ring + st * C::STAGE_BYTES;
     mbar_expect_tx(bar, C::STAGE_BYTES);
 #pragma unroll
-    for (int c = 0; c < D / 64; ++c) {
-      tma_load_3d(dst + c * (TK * 128), &tk, bar, c * 64, hk, row);
-      tma_load_3d(dst + C::TILE_BYTES + c * (TK * 128), &tv, bar, c * 64, hk, row);
-    }
+    for (int c = 0; c < DQ / 64; ++c) tma_load_3d(dst + c * (TK * 128), &tk, bar, c * 64, hk, row);
+#pragma unroll
+    for (int c = 0; c < DV / 64; ++c)
+      tma_load_3d(dst + C::K_BYTES + c * (TK * 128), &tv, bar, c * 64, hk, row);
   };
   if (lane == 0)
     for (int i = 0; i < min(my_n, DEC_STAGES - 1); ++i) issue(i);
 
-  // A fragments of Q (16 rows x D), loaded once
+  // A fragments of Q (16 rows x DQ), loaded once
   uint32_t qa[NKS][4];
   {
     const uint32_t qb = sbase + C::OFF_Q;
@@ -188,7 +190,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tk, const __grid_constant
       break;
     }
     const uint32_t kt = my_ring + st * C::STAGE_BYTES;
-    const uint32_t vt = kt + C::TILE_BYTES;
+    const uint32_t vt = kt + C::K_BYTES;
     const int tile = t0 + warp + i * DEC_WARPS;
     const int key0 = tile * TK;
 
@@ -203,7 +205,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tk, const __grid_constant
         // four matrices of key block j: d-chunks 2ks, 2ks+1 (k-step ks) and 2ks+2, 2ks+3 (k-step ks+1)
         uint32_t kb[4];
         const int row = j * 8 + (lane & 7);
-        ldmatrix_x4(kt + tile_off<D>(row, ks * 2 + (lane >> 3)), kb);
+        ldmatrix_x4(kt + tile_off(row, ks * 2 + (lane >> 3)), kb);
         mma_bf16_16816(s[j], qa[ks], kb[0], kb[1]);
         mma_bf16_16816(s[j], qa[ks + 1], kb[2], kb[3]);
       }
@@ -263,7 +265,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tk, const __grid_constant
         // transposed loads: (keys 16t..+7, chunk j), (keys 16t+8..+15, chunk j), the same two for chunk j+1
         uint32_t vb[4];
         const int row = t * 16 + (lane & 7) + ((lane >> 3) & 1) * 8;
-        ldmatrix_x4_trans(vt + tile_off<D>(row, j + (lane >> 4)), vb);
+        ldmatrix_x4_trans(vt + tile_off(row, j + (lane >> 4)), vb);
         mma_bf16_16816(o_acc[j], pa[t], vb[0], vb[1]);
         mma_bf16_16816(o_acc[j + 1], pa[t], vb[2], vb[3]);
       }
@@ -300,15 +302,15 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tk, const __grid_constant
     l_all[h] = l;
     w_mine[h] = exp2f(m_run[h] - m);
   }
-  // each warp scales its O by its weight and adds it into a shared fp32 [16 x D] accumulator, one warp after another
-  float* o_sh = reinterpret_cast<float*>(smem);   // 16 * D * 4 bytes <= one warp's ring
+  // each warp scales its O by its weight and adds it into a shared fp32 [16 x DV] accumulator, one warp after another
+  float* o_sh = reinterpret_cast<float*>(smem);   // 16 * DV * 4 bytes <= one warp's ring
   for (int w = 0; w < DEC_WARPS; ++w) {
     if (warp == w) {
 #pragma unroll
       for (int j = 0; j < NDB; ++j) {
         const int col = j * 8 + (lane & 3) * 2;
-        float2* lo2 = reinterpret_cast<float2*>(o_sh + r0 * D + col);
-        float2* hi2 = reinterpret_cast<float2*>(o_sh + (r0 + 8) * D + col);
+        float2* lo2 = reinterpret_cast<float2*>(o_sh + r0 * DV + col);
+        float2* hi2 = reinterpret_cast<float2*>(o_sh + (r0 + 8) * DV + col);
         float2 a = w == 0 ? make_float2(0.f, 0.f) : *lo2;
         float2 c = w == 0 ? make_float2(0.f, 0.f) : *hi2;
         a.x += o_acc[j][0] * w_mine[0];
@@ -321,23 +323,24 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tk, const __grid_constant
     }
     __syncthreads();
   }
-  // ---- write: G rows of D bf16 (+ LSE). Row r <-> query head hk * G + r.
+  // ---- write: G rows of dv bf16 (+ LSE). Row r <-> query head hk * G + r.
   const long long orow = (long long)split * p.B + b;   // split-major: the layout edl_attn_combine reads
-  for (int i = threadIdx.x; i < G * (D / 8); i += DEC_THREADS) {
-    const int r = i / (D / 8), c = i % (D / 8);
+  for (int i = threadIdx.x; i < G * (DV / 8); i += DEC_THREADS) {
+    const int r = i / (DV / 8), c = i % (DV / 8);
+    if (c * 8 >= p.dv) continue;
     float m = -1e30f, l = 0.f;
     for (int w = 0; w < DEC_WARPS; ++w) m = fmaxf(m, red[w * 32 + r]);
     for (int w = 0; w < DEC_WARPS; ++w) l += red[w * 32 + 16 + r] * exp2f(red[w * 32 + r] - m);
     const int head = hk * G + r;
     if (p.sinks && p.splits == 1) l += exp2f(p.sinks[head] * LOG2E_F - m);
     const float inv = l > 0.f ? 1.f / l : 0.f;
-    const float* src = o_sh + r * D + c * 8;
+    const float* src = o_sh + r * DV + c * 8;
     uint4 v;
     v.x = pack_bf16x2(src[0] * inv, src[1] * inv);
     v.y = pack_bf16x2(src[2] * inv, src[3] * inv);
     v.z = pack_bf16x2(src[4] * inv, src[5] * inv);
     v.w = pack_bf16x2(src[6] * inv, src[7] * inv);
-    *reinterpret_cast<uint4*>(p.o + orow * p.ldo + (long long)head * D + c * 8) = v;
+    *reinterpret_cast<uint4*>(p.o + orow * p.ldo + (long long)head * p.dv + c * 8) = v;
     if (c == 0 && p.lse)
       p.lse[((long long)split * p.Hq + head) * p.B + b] = l > 0.f ? (m + log2f(l)) * 0.6931471805599453f : -INFINITY;
   }
@@ -350,15 +353,15 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tk, const __grid_constant
   }
 }
 
-template <int D>
-int launch_decode(const void* k_pages, const void* v_pages, long long ld_page, long long num_pages,
-                  const DecodeParams& p, cudaStream_t stream) {
-  using C = DCfg<D>;
+template <int DQ, int DV>
+int launch_decode(const void* k_pages, const void* v_pages, long long ld_kpage, long long ld_vpage,
+                  long long num_pages, const DecodeParams& p, cudaStream_t stream) {
+  using C = DCfg<DQ, DV>;
   CUtensorMap tk, tv;
   const long long total_k = num_pages * PAGE;
-  if (make_tmap_3d_16b(&tk, k_pages, D, p.Hkv, total_k, D, ld_page, 64, 1, TK, 3)) return -1;
-  if (make_tmap_3d_16b(&tv, v_pages, D, p.Hkv, total_k, D, ld_page, 64, 1, TK, 3)) return -1;
-  auto kern = attn_decode_kernel<D>;
+  if (make_tmap_3d_16b(&tk, k_pages, p.dq, p.Hkv, total_k, p.dq, ld_kpage, 64, 1, TK, 3)) return -1;
+  if (make_tmap_3d_16b(&tv, v_pages, p.dv, p.Hkv, total_k, p.dv, ld_vpage, 64, 1, TK, 3)) return -1;
+  auto kern = attn_decode_kernel<DQ, DV>;
   static bool attr_set[64] = {false};
   int dev = 0;
   cudaGetDevice(&dev);
@@ -378,19 +381,21 @@ int launch_decode(const void* k_pages, const void* v_pages, long long ld_page, l
 }  // namespace edl
 
 // Decode attention over a paged KV cache: q [B, ldq] (one token per sequence, head h at columns h * D),
-// pages [num_pages * 128, ld_page] with the KV heads packed in a row, page_table [B, pt_stride], kv_lens [B]
+// pages [num_pages * 128, ld_kpage / ld_vpage] with the KV heads packed in a row, page_table [B, pt_stride], kv_lens [B]
 // (keys per sequence, the new token included). o [splits, B, ldo]; with splits > 1 part s holds the result over
 // the s-th part of every sequence's keys and lse [splits, Hq, B] its log-sum-exp, for edl_attn_combine.
-// Hq / Hkv <= 16; D is 64 or 128; window = 0 or the sliding-window length.
+// Hq / Hkv <= 16; D (queries, keys) and Dv (values) are multiples of 8 up to 128; window = 0 or the sliding-window length.
 EDL_HOST_API int edl_attn_decode(const void* q, const void* k_pages, const void* v_pages, void* o, float* lse,
-                                 long long ldq, long long ld_page, long long ldo, const int* kv_lens,
+                                 long long ldq, long long ld_kpage, long long ld_vpage, long long ldo, const int* kv_lens,
                                  const int* page_table, int pt_stride, int B, long long num_pages, int Hq, int Hkv,
-                                 int D, float scale, int window, int splits, const float* sinks, int* status,
+                                 int D, int Dv, float scale, int window, int splits, const float* sinks, int* status,
                                  void* stream) {
   using namespace edl;
   if (B <= 0) return 0;
-  if ((D != 64 && D != 128) || Hq % Hkv || Hq / Hkv > 16 || splits < 1) {
-    set_last_error("edl_attn_decode: unsupported layout (D=%d, Hq=%d, Hkv=%d, splits=%d)", D, Hq, Hkv, splits);
+  if (D < 8 || D > 128 || (D & 7) || Dv < 8 || Dv > 128 || (Dv & 7) || Hkv < 1 || Hq % Hkv || Hq / Hkv > 16 ||
+      splits < 1) {
+    set_last_error("edl_attn_decode: unsupported layout (D=%d, Dv=%d, Hq=%d, Hkv=%d, splits=%d)", D, Dv, Hq, Hkv,
+                   splits);
     return -1;
   }
   if ((ldq & 7) || (ldo & 7) || (reinterpret_cast<uintptr_t>(q) & 15) || (reinterpret_cast<uintptr_t>(o) & 15)) {
@@ -415,6 +420,11 @@ EDL_HOST_API int edl_attn_decode(const void* q, const void* k_pages, const void*
   p.scale_log2 = scale * 1.4426950408889634f;
   p.status = status;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-  if (D == 128) return launch_decode<128>(k_pages, v_pages, ld_page, num_pages, p, s);
-  return launch_decode<64>(k_pages, v_pages, ld_page, num_pages, p, s);
+  p.dq = D;
+  p.dv = Dv;
+  if (D > 64)
+    return Dv > 64 ? launch_decode<128, 128>(k_pages, v_pages, ld_kpage, ld_vpage, num_pages, p, s)
+                   : launch_decode<128, 64>(k_pages, v_pages, ld_kpage, ld_vpage, num_pages, p, s);
+  return Dv > 64 ? launch_decode<64, 128>(k_pages, v_pages, ld_kpage, ld_vpage, num_pages, p, s)
+                 : launch_decode<64, 64>(k_pages, v_pages, ld_kpage, ld_vpage, num_pages, p, s);
 }

@@ -1,5 +1,9 @@
-// Flash-attention forward on tcgen05 tensor cores (head_dim 64 or 128, bf16, GQA,
+// Flash-attention forward on tcgen05 tensor cores (tiles of 64 or 128 columns per head, bf16, GQA,
 // causal, variable-length batches, sliding window, logit soft-cap, attention sinks).
+//
+// The query / key size and the value size of a head are separate and may be any multiple of 8 up to 128: a tile is
+// DQ (or DV) columns wide, 64 or 128, and the tensor maps carry the real sizes, so the columns past a head's end
+// arrive as zeros and only the real value columns are stored. Memory holds no padding.
 //
 // One CTA per (block of 256 query rows = two tiles A and B, query head, sequence):
 //   warp 0      TMA producer: both Q tiles once, then K and V tiles of 128 keys through
@@ -71,17 +75,20 @@ struct AttnFwdParams {
   const int* kv_lens;    // [B] keys per sequence (context length including the new tokens), paged mode
   int pt_stride;
   int pack;              // query heads per tile row group (1 = one head per CTA)
+  int dq, dv;            // real query / key and value sizes of a head (<= the tile widths)
   int nx, ny;            // launch geometry: query blocks and heads (the grid itself is one-dimensional)
 };
 
-template <int D>
+template <int DQ, int DV>
 struct ACfg {
-  static constexpr int DCH = D / 64;              // 128-byte chunks along head_dim
-  static constexpr int Q_BYTES = BQ * D * 2;      // one query tile
-  static constexpr int KV_BYTES = BKV * D * 2;
+  static constexpr int QCH = DQ / 64;             // 128-byte chunks along a query / key head
+  static constexpr int VCH = DV / 64;             // ... and along a value head
+  static constexpr int Q_BYTES = BQ * DQ * 2;     // one query tile
+  static constexpr int K_BYTES = BKV * DQ * 2;
+  static constexpr int V_BYTES = BKV * DV * 2;
   static constexpr int OFF_K = 2 * Q_BYTES;
-  static constexpr int OFF_V = OFF_K + 2 * KV_BYTES;
-  static constexpr int OFF_BAR = OFF_V + 2 * KV_BYTES;
+  static constexpr int OFF_V = OFF_K + 2 * K_BYTES;
+  static constexpr int OFF_BAR = OFF_V + 2 * V_BYTES;
   static constexpr int OFF_XCH = OFF_BAR + 256;   // float [tile][parity][half][row]: row maxima / sums of a half
   static constexpr int SMEM = OFF_XCH + 2 * 2 * 2 * BQ * 4 + 1024;
 };
@@ -105,11 +112,11 @@ __device__ __forceinline__ TileRange tile_range(int q0, int tq, int len_q, int l
   return r;
 }
 
-template <int D>
+template <int DQ, int DV>
 __global__ void __launch_bounds__(ATT_THREADS, 1)
 attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CUtensorMap tk,
                 const __grid_constant__ CUtensorMap tv, const AttnFwdParams p) {
-  using C = ACfg<D>;
+  using C = ACfg<DQ, DV>;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   const uint32_t sQ = smem_u32(smem);
@@ -138,9 +145,8 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
   const int pack = p.pack;                       // power of two, divides BQ
   const int pshift = 31 - __clz(pack);
   const int TQ = BQ >> pshift;                   // query tokens per tile
-  const int h = rem_id % p.ny;                   // query head (pack == 1) or KV head (packed)
-  const int hk = pack == 1 ? h / (p.Hq / p.Hkv) : h;
-  const int h_first = pack == 1 ? h : hk * pack; // first query head of this CTA's rows
+  const int h_first = (rem_id % p.ny) * pack;    // first query head of this CTA's rows
+  const int hk = h_first / (p.Hq / p.Hkv);       // their KV head (pack divides the group)
 
   const int q_start = p.cu_q ? p.cu_q[b] : b * p.Tq;
   const int k_start = p.page_table ? 0 : (p.cu_k ? p.cu_k[b] : b * p.Tk);
@@ -199,7 +205,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
 #pragma unroll
       for (int t = 0; t < 2; ++t)
 #pragma unroll
-        for (int c = 0; c < C::DCH; ++c)
+        for (int c = 0; c < C::QCH; ++c)
           tma_load_3d(sQ + t * C::Q_BYTES + c * (BQ * 128), &tq, b_qfull, c * 64, h_first, q_start + qblock0 + t * TQ);
       for (int j = jmin; j < jmax; ++j) {
         const int it = j - jmin;
@@ -208,17 +214,17 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
         if (it >= 2 &&
             !mbar_wait(b_kempty + 8 * s, ((it >> 1) - 1) & 1, abort_flag, p.status, EDL_TIMEOUT_PRODUCER))
           break;
-        mbar_expect_tx(b_kfull + 8 * s, C::KV_BYTES);
+        mbar_expect_tx(b_kfull + 8 * s, C::K_BYTES);
 #pragma unroll
-        for (int c = 0; c < C::DCH; ++c)
-          tma_load_3d(sK0 + s * C::KV_BYTES + c * (BKV * 128), &tk, b_kfull + 8 * s, c * 64, hk, krow);
+        for (int c = 0; c < C::QCH; ++c)
+          tma_load_3d(sK0 + s * C::K_BYTES + c * (BKV * 128), &tk, b_kfull + 8 * s, c * 64, hk, krow);
         if (it >= 2 &&
             !mbar_wait(b_vempty + 8 * s, ((it >> 1) - 1) & 1, abort_flag, p.status, EDL_TIMEOUT_PRODUCER))
           break;
-        mbar_expect_tx(b_vfull + 8 * s, C::KV_BYTES);
+        mbar_expect_tx(b_vfull + 8 * s, C::V_BYTES);
 #pragma unroll
-        for (int c = 0; c < C::DCH; ++c)
-          tma_load_3d(sV0 + s * C::KV_BYTES + c * (BKV * 128), &tv, b_vfull + 8 * s, c * 64, hk, krow);
+        for (int c = 0; c < C::VCH; ++c)
+          tma_load_3d(sV0 + s * C::V_BYTES + c * (BKV * 128), &tv, b_vfull + 8 * s, c * 64, hk, krow);
       }
     }
   } else if (warp == 1) {
@@ -229,16 +235,16 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
       const bool trace_on = blockIdx.x == 0 && leader;
 #endif
       constexpr uint32_t idesc_qk = umma_idesc_bf16(BQ, BKV, 0, 0);
-      constexpr uint32_t idesc_pv = umma_idesc_bf16(BQ, D, 0, 1);
+      constexpr uint32_t idesc_pv = umma_idesc_bf16(BQ, DV, 0, 1);
       bool ok = mbar_wait(b_qfull, 0, abort_flag, p.status, EDL_TIMEOUT_MMA);
       int pv_cnt[2] = {0, 0};
       auto valid = [&](int t, int j) { return t == 0 ? (j >= rgA.lo && j < rgA.hi) : (j >= rgB.lo && j < rgB.hi); };
       auto issue_qk = [&](int t, int j) {
         const int s = (j - jmin) & 1;
-        const uint32_t kb = sK0 + s * C::KV_BYTES;
+        const uint32_t kb = sK0 + s * C::K_BYTES;
         const uint32_t qbase = sQ + t * C::Q_BYTES;
 #pragma unroll
-        for (int c = 0; c < C::DCH; ++c)
+        for (int c = 0; c < C::QCH; ++c)
 #pragma unroll
           for (int k = 0; k < 4; ++k) {
             uint64_t ad = umma_smem_desc_sw128(qbase + c * (BQ * 128) + k * 32, 16, 1024);
@@ -251,7 +257,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
         const int s = (j - jmin) & 1;
         if (!mbar_wait(b_pfull + 8 * t, pv_cnt[t] & 1, abort_flag, p.status, EDL_TIMEOUT_MMA)) return false;
         tc_fence_after();
-        const uint32_t vb = sV0 + s * C::KV_BYTES;
+        const uint32_t vb = sV0 + s * C::V_BYTES;
 #pragma unroll
         for (int k = 0; k < BKV / 16; ++k) {
           uint64_t bd = umma_smem_desc_sw128(vb + k * 2048, BKV * 128, 1024);
@@ -383,7 +389,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
       }
       mx = fmaxf(mx, mx_other) * mul;  // mul > 0, so scaling commutes with the maximum
       // lazy rescale. Both halves of a row see the same maxima, so they take the same decision (warp-uniform,
-      // as tcgen05.ld/st are warp-wide) and each rescales its own 64 columns of O. The QK^T product of this
+      // as tcgen05.ld/st are warp-wide) and each rescales its own half of O's columns. The QK^T product of this
       // step was issued after the PV product of the previous one, so O is quiescent here.
       const float m_new = fmaxf(m_used, mx);
       if (__any_sync(0xffffffffu, m_new > m_used + 8.f)) {
@@ -391,13 +397,13 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
         l *= alpha;
         if (n > 0) {
 #pragma unroll 1
-          for (int c = 0; c < D / 64; ++c) {
+          for (int c = 0; c < DV / 64; ++c) {
             uint32_t rr[32];
-            tmem_ld_32x32b_x32(tO + half * (D / 2) + c * 32, rr);
+            tmem_ld_32x32b_x32(tO + half * (DV / 2) + c * 32, rr);
             tc_wait_ld();
 #pragma unroll
             for (int i = 0; i < 32; ++i) rr[i] = __float_as_uint(__uint_as_float(rr[i]) * alpha);
-            tmem_st_32x32b_x32(tO + half * (D / 2) + c * 32, rr);
+            tmem_st_32x32b_x32(tO + half * (DV / 2) + c * 32, rr);
           }
         }
         m_used = m_new;
@@ -432,7 +438,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
       TRACE(t, n, 6);
     }
 
-    // epilogue: O / l -> bf16, plus LSE. Each half writes its own D / 2 columns; the row sum is the two halves'.
+    // epilogue: O / l -> bf16, plus LSE. Each half writes its own DV / 2 columns; the row sum is the two halves'.
     const bool any = rg.hi > rg.lo;
     if (any && alive) {
       float l_other;
@@ -447,12 +453,12 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
       if (p.sinks) l += exp2f(p.sinks[qhead] * LOG2E - m_used);
       const float inv_l = l > 0.f ? 1.f / l : 0.f;
       const bool row_ok = qrow < len_q;
-      __nv_bfloat16* op = p.o + (long long)(q_start + qrow) * p.ldo + (long long)qhead * D + half * (D / 2);
+      __nv_bfloat16* op = p.o + (long long)(q_start + qrow) * p.ldo + (long long)qhead * p.dv + half * (DV / 2);
 #pragma unroll 1
-      for (int c = 0; c < D / 64; ++c) {
+      for (int c = 0; c < DV / 64; ++c) {
         uint32_t rr[32];
         if (any) {
-          tmem_ld_32x32b_x32(tO + half * (D / 2) + c * 32, rr);
+          tmem_ld_32x32b_x32(tO + half * (DV / 2) + c * 32, rr);
           tc_wait_ld();
         } else {
 #pragma unroll
@@ -461,6 +467,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
         if (row_ok) {
 #pragma unroll
           for (int i = 0; i < 32; i += 8) {
+            if (half * (DV / 2) + c * 32 + i >= p.dv) break;   // dv is a multiple of 8
             uint4 o;
             o.x = pack_bf16x2(__uint_as_float(rr[i]) * inv_l, __uint_as_float(rr[i + 1]) * inv_l);
             o.y = pack_bf16x2(__uint_as_float(rr[i + 2]) * inv_l, __uint_as_float(rr[i + 3]) * inv_l);
@@ -485,15 +492,15 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
   if (warp == 1) tmem_dealloc(tmem_base, 512);
 }
 
-template <int D>
+template <int DQ, int DV>
 int launch_fwd(const void* q, const void* k, const void* v, long long ldq, long long ldk, long long ldv,
                long long total_q, long long total_k, const AttnFwdParams& p, cudaStream_t stream) {
-  using C = ACfg<D>;
+  using C = ACfg<DQ, DV>;
   CUtensorMap tq, tk, tv;
-  if (make_tmap_3d_16b(&tq, q, D, p.Hq, total_q, D, ldq, 64, p.pack, BQ / p.pack, 3)) return -1;
-  if (make_tmap_3d_16b(&tk, k, D, p.Hkv, total_k, D, ldk, 64, 1, BKV, 3)) return -1;
-  if (make_tmap_3d_16b(&tv, v, D, p.Hkv, total_k, D, ldv, 64, 1, BKV, 3)) return -1;
-  auto kern = attn_fwd_kernel<D>;
+  if (make_tmap_3d_16b(&tq, q, p.dq, p.Hq, total_q, p.dq, ldq, 64, p.pack, BQ / p.pack, 3)) return -1;
+  if (make_tmap_3d_16b(&tk, k, p.dq, p.Hkv, total_k, p.dq, ldk, 64, 1, BKV, 3)) return -1;
+  if (make_tmap_3d_16b(&tv, v, p.dv, p.Hkv, total_k, p.dv, ldv, 64, 1, BKV, 3)) return -1;
+  auto kern = attn_fwd_kernel<DQ, DV>;
   static bool attr_set[64] = {false};  // per device
   int dev = 0;
   cudaGetDevice(&dev);
@@ -507,10 +514,20 @@ int launch_fwd(const void* q, const void* k, const void* v, long long ldq, long 
   const int tq_block = 2 * BQ / p.pack;  // query tokens per CTA
   AttnFwdParams pl = p;
   pl.nx = (p.Tq + tq_block - 1) / tq_block;
-  pl.ny = p.pack == 1 ? p.Hq : p.Hkv;
+  pl.ny = p.Hq / p.pack;
   const long long blocks = (long long)pl.nx * pl.ny * p.B;
   kern<<<(unsigned)blocks, ATT_THREADS, C::SMEM, stream>>>(tq, tk, tv, pl);
   return check_cuda(cudaGetLastError(), "attn_fwd launch");
+}
+
+// Tile widths from the real head sizes.
+int dispatch_fwd(const void* q, const void* k, const void* v, long long ldq, long long ldk, long long ldv,
+                 long long total_q, long long total_k, const AttnFwdParams& p, cudaStream_t s) {
+  if (p.dq > 64)
+    return p.dv > 64 ? launch_fwd<128, 128>(q, k, v, ldq, ldk, ldv, total_q, total_k, p, s)
+                     : launch_fwd<128, 64>(q, k, v, ldq, ldk, ldv, total_q, total_k, p, s);
+  return p.dv > 64 ? launch_fwd<64, 128>(q, k, v, ldq, ldk, ldv, total_q, total_k, p, s)
+                   : launch_fwd<64, 64>(q, k, v, ldq, ldk, ldv, total_q, total_k, p, s);
 }
 
 }  // namespace
@@ -568,32 +585,34 @@ EDL_HOST_API int edl_attn_fwd(const void* q, const void* k, const void* v, void*
   p.kv_lens = nullptr;
   p.pt_stride = 0;
   p.pack = 1;
-  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-  if (D == 128) return launch_fwd<128>(q, k, v, ldq, ldk, ldv, total_q, total_k, p, s);
-  return launch_fwd<64>(q, k, v, ldq, ldk, ldv, total_q, total_k, p, s);
+  p.dq = p.dv = D;
+  return dispatch_fwd(q, k, v, ldq, ldk, ldv, total_q, total_k, p, reinterpret_cast<cudaStream_t>(stream));
 }
 
 // Paged attention for serving (mixed prefill + decode in one launch).
 //   q:        [total_q, ldq] new query tokens of all sequences, concatenated; cu_q [B+1] their offsets
-//   k_pages / v_pages: [num_pages * 128, ld_page] page pools (page size 128 tokens), heads packed in a row;
+//   k_pages / v_pages: [num_pages * 128, ld_kpage / ld_vpage] page pools (page size 128 tokens), heads packed in a row;
 //             the new tokens' keys/values must already be written to their pages
 //   page_table [B, pt_stride]: page ids of each sequence in order; kv_lens [B]: keys per sequence
 //             (cached + new). Query token i of a sequence sits at key position kv_len - len_q + i.
 //   max_q:    largest number of new tokens of any sequence (sizes the grid)
 // All query heads of a KV head share one tile (rows = token x head), so one pass over a page
-// serves the whole GQA group. Hq / Hkv must be a power of two <= 128.
+// serves the whole GQA group; a group whose size is not a power of two is cut into equal power-of-two parts.
+// Head sizes D (queries, keys) and Dv (values): multiples of 8 up to 128.
 static int attn_paged_impl(const void* q, const void* k_pages, const void* v_pages, void* o, float* lse,
-                           long long ldq, long long ld_page, long long ldo, const int* cu_q, const int* kv_lens,
+                           long long ldq, long long ld_kpage, long long ld_vpage, long long ldo, const int* cu_q, const int* kv_lens,
                            const int* page_table, int pt_stride, int B, int max_q, long long total_q,
-                           long long num_pages, int Hq, int Hkv, int D, float scale, int causal, int window,
+                           long long num_pages, int Hq, int Hkv, int D, int Dv, float scale, int causal, int window,
                            float softcap, const float* sinks, int* status, void* stream) {
   using namespace edl;
   if (B <= 0 || max_q <= 0 || total_q <= 0) return 0;
-  const int G = Hq / Hkv;
-  if ((D != 64 && D != 128) || Hq % Hkv || (G & (G - 1)) || G > 128) {
-    set_last_error("edl_attn_paged: unsupported head layout (D=%d, Hq=%d, Hkv=%d)", D, Hq, Hkv);
+  if (D < 8 || D > 128 || (D & 7) || Dv < 8 || Dv > 128 || (Dv & 7) || Hkv < 1 || Hq % Hkv) {
+    set_last_error("edl_attn_paged: unsupported head layout (D=%d, Dv=%d, Hq=%d, Hkv=%d)", D, Dv, Hq, Hkv);
     return -1;
   }
+  const int group = Hq / Hkv;
+  int G = group & -group;            // largest power of two that divides the group
+  if (G > 128) G = 128;
   if ((ldo & 7) || (reinterpret_cast<uintptr_t>(o) & 15)) {
     set_last_error("edl_attn_paged: output must be 16-byte aligned with ldo %% 8 == 0");
     return -1;
@@ -620,29 +639,29 @@ static int attn_paged_impl(const void* q, const void* k_pages, const void* v_pag
   p.kv_lens = kv_lens;
   p.pt_stride = pt_stride;
   p.pack = G;
-  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-  const long long total_k = num_pages * 128;
-  if (D == 128) return launch_fwd<128>(q, k_pages, v_pages, ldq, ld_page, ld_page, total_q, total_k, p, s);
-  return launch_fwd<64>(q, k_pages, v_pages, ldq, ld_page, ld_page, total_q, total_k, p, s);
+  p.dq = D;
+  p.dv = Dv;
+  return dispatch_fwd(q, k_pages, v_pages, ldq, ld_kpage, ld_vpage, total_q, num_pages * 128, p,
+                      reinterpret_cast<cudaStream_t>(stream));
 }
 
 EDL_HOST_API int edl_attn_paged(const void* q, const void* k_pages, const void* v_pages, void* o, long long ldq,
-                                long long ld_page, long long ldo, const int* cu_q, const int* kv_lens,
-                                const int* page_table, int pt_stride, int B, int max_q, long long total_q,
-                                long long num_pages, int Hq, int Hkv, int D, float scale, int causal, int window,
+                                long long ld_kpage, long long ld_vpage, long long ldo, const int* cu_q,
+                                const int* kv_lens, const int* page_table, int pt_stride, int B, int max_q, long long total_q,
+                                long long num_pages, int Hq, int Hkv, int D, int Dv, float scale, int causal, int window,
                                 float softcap, const float* sinks, int* status, void* stream) {
-  return attn_paged_impl(q, k_pages, v_pages, o, nullptr, ldq, ld_page, ldo, cu_q, kv_lens, page_table, pt_stride, B,
-                         max_q, total_q, num_pages, Hq, Hkv, D, scale, causal, window, softcap, sinks, status, stream);
+  return attn_paged_impl(q, k_pages, v_pages, o, nullptr, ldq, ld_kpage, ld_vpage, ldo, cu_q, kv_lens, page_table, pt_stride, B,
+                         max_q, total_q, num_pages, Hq, Hkv, D, Dv, scale, causal, window, softcap, sinks, status, stream);
 }
 
 // Same, also writing lse [Hq, total_q] (natural log of the softmax denominator; -inf for a row without keys):
 // the partial results of split-KV decode and of context-parallel attention are merged from (o, lse) pairs.
 EDL_HOST_API int edl_attn_paged_lse(const void* q, const void* k_pages, const void* v_pages, void* o, float* lse,
-                                    long long ldq, long long ld_page, long long ldo, const int* cu_q,
+                                    long long ldq, long long ld_kpage, long long ld_vpage, long long ldo, const int* cu_q,
                                     const int* kv_lens, const int* page_table, int pt_stride, int B, int max_q,
-                                    long long total_q, long long num_pages, int Hq, int Hkv, int D, float scale,
+                                    long long total_q, long long num_pages, int Hq, int Hkv, int D, int Dv, float scale,
                                     int causal, int window, float softcap, const float* sinks, int* status,
                                     void* stream) {
-  return attn_paged_impl(q, k_pages, v_pages, o, lse, ldq, ld_page, ldo, cu_q, kv_lens, page_table, pt_stride, B,
-                         max_q, total_q, num_pages, Hq, Hkv, D, scale, causal, window, softcap, sinks, status, stream);
+  return attn_paged_impl(q, k_pages, v_pages, o, lse, ldq, ld_kpage, ld_vpage, ldo, cu_q, kv_lens, page_table, pt_stride, B,
+                         max_q, total_q, num_pages, Hq, Hkv, D, Dv, scale, causal, window, softcap, sinks, status, stream);
 }

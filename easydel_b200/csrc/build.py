@@ -18,6 +18,7 @@ from __future__ import annotations
 import argparse
 import concurrent.futures as cf
 import hashlib
+import json
 import os
 import shutil
 import subprocess
@@ -44,6 +45,17 @@ NVCC_FLAGS = [
     "--expt-relaxed-constexpr",
 ]
 
+# Kernels whose job is 32-bit arithmetic (fp32 residual stream, gates and recurrences, attention of fp32 models) are
+# compiled without fast-math.
+PRECISE = frozenset({"stream_ops", "hgrn2", "attention_simt"})
+
+# What serving a model family needs, by model type, for a first call on a machine without a built library.
+SERVING_PARTS = {
+    "rakevik": ("common", "gemm", "attention_fwd", "attention_decode", "attn_combine", "attention_simt", "serving",
+                "host_native", "stream_ops", "hgrn2"),
+}
+MANIFEST_SUFFIX = ".sources.json"      # beside a linked library: the digest of every source it was built from
+
 
 def _nvcc() -> str:
     cand = os.environ.get("NVCC") or shutil.which("nvcc") or "/usr/local/cuda/bin/nvcc"
@@ -52,7 +64,12 @@ def _nvcc() -> str:
     return cand
 
 
+def _flags_for(src: Path, flags: list[str]) -> list[str]:
+    return [f for f in flags if f != "--use_fast_math"] if src.stem in PRECISE else flags
+
+
 def _digest(src: Path, flags: list[str]) -> str:
+    flags = _flags_for(src, flags)
     h = hashlib.sha256()
     h.update(" ".join(flags).encode())
     h.update(src.read_bytes())
@@ -67,7 +84,7 @@ def _compile_one(nvcc: str, src: Path, flags: list[str], force: bool, verbose: b
     dig = _digest(src, flags)
     if not force and obj.exists() and stamp.exists() and stamp.read_text() == dig:
         return obj, False, ""
-    cmd = [nvcc, *flags, "-I", str(CSRC), "-c", str(src), "-o", str(obj)]
+    cmd = [nvcc, *_flags_for(src, flags), "-I", str(CSRC), "-c", str(src), "-o", str(obj)]
     proc = subprocess.run(cmd, capture_output=True, text=True)
     if proc.returncode != 0:
         raise RuntimeError(f"nvcc failed for {src.name}:\n{proc.stdout}\n{proc.stderr}")
@@ -79,9 +96,33 @@ def sources() -> list[Path]:
     return sorted(CSRC.glob("*.cu"))
 
 
-def build(force: bool = False, verbose: bool = False, jobs: int | None = None, out: str | None = None) -> Path:
+def _manifest(lib: Path) -> dict[str, str]:
+    try:
+        return json.loads(lib.with_name(lib.name + MANIFEST_SUFFIX).read_text())
+    except (OSError, ValueError):
+        return {}
+
+
+def ensure(model_type: str) -> Path:
+    """A library with current kernels for serving ``model_type``: the full one if it is up to date in the parts the
+    family needs, else a smaller one with those parts only (compiled and linked now if it is missing or stale)."""
+    parts = SERVING_PARTS.get(model_type)
+    if parts is None:
+        return build()
+    want = {n: _digest(CSRC / f"{n}.cu", list(NVCC_FLAGS)) for n in parts}
+    partial = LIB_DIR / f"libedl_b200_{model_type}.so"
+    for lib in (LIB_PATH, partial):
+        have = _manifest(lib)
+        if lib.exists() and all(have.get(n) == d for n, d in want.items()):
+            return lib
+    return build(only=parts, link=partial)
+
+
+def build(force: bool = False, verbose: bool = False, jobs: int | None = None, out: str | None = None,
+          only: tuple[str, ...] | None = None, link: Path | None = None) -> Path:
     """Compiles what changed and links the shared library; returns its path. ``out``: link there instead of the
-    in-tree location, with the objects in a directory of their own (a build with other flags beside the main one)."""
+    in-tree location, with the objects in a directory of their own (a build with other flags beside the main one).
+    ``only``: the sources to take, by stem; ``link``: where to link them."""
     global BUILD, LIB_PATH
     nvcc = _nvcc()
     if out is not None:
@@ -96,7 +137,8 @@ def build(force: bool = False, verbose: bool = False, jobs: int | None = None, o
     flags += extra
     if verbose:
         flags += ["-Xptxas", "-v"]
-    srcs = sources()
+    srcs = sources() if only is None else [CSRC / f"{n}.cu" for n in only]
+    target = LIB_PATH if link is None else link
     objs: list[Path] = []
     changed = False
     with cf.ThreadPoolExecutor(max_workers=jobs or min(8, os.cpu_count() or 4)) as ex:
@@ -107,15 +149,17 @@ def build(force: bool = False, verbose: bool = False, jobs: int | None = None, o
             changed |= did
             if log:
                 print(log, file=sys.stderr)
-    if changed or not LIB_PATH.exists():
-        tmp = LIB_PATH.with_suffix(".so.tmp")
+    digests = {x.stem: _digest(x, flags) for x in srcs}
+    if changed or not target.exists() or _manifest(target) != digests:
+        tmp = target.with_suffix(".so.tmp")
         cmd = [nvcc, "-shared", "-o", str(tmp), *map(str, objs), "-gencode", "arch=compute_100a,code=sm_100a",
                "-lcudart_static", "-Xcompiler", "-fPIC"]
         proc = subprocess.run(cmd, capture_output=True, text=True)
         if proc.returncode != 0:
             raise RuntimeError(f"link failed:\n{proc.stdout}\n{proc.stderr}")
-        os.replace(tmp, LIB_PATH)
-    return LIB_PATH
+        os.replace(tmp, target)
+        target.with_name(target.name + MANIFEST_SUFFIX).write_text(json.dumps(digests))
+    return target
 
 
 def main() -> None:

@@ -885,9 +885,11 @@ EDL_HOST_API int edl_gemm_grouped(int kind, const void* X, const void* W, void* 
 
 namespace edl {
 namespace {
-// out[m, n] = sum_s ws[s, m, n] (+ bias[n]), fp32 partials -> bf16.
-__global__ void splitk_reduce_kernel(const float* __restrict__ ws, __nv_bfloat16* __restrict__ out,
-                                     const __nv_bfloat16* __restrict__ bias, int M, int N, long long ldc, int splits) {
+// out[m, n] (+)= sum_s ws[s, m, n] (+ bias[n]), fp32 partials -> bf16, or fp32 with GEMM_OUT_F32 (added to what is
+// there with GEMM_ACCUMULATE).
+__global__ void splitk_reduce_kernel(const float* __restrict__ ws, void* __restrict__ out_v,
+                                     const __nv_bfloat16* __restrict__ bias, int M, int N, long long ldc, int splits,
+                                     int flags) {
   const long long vec_per_row = N / 4;
   const long long total = (long long)M * vec_per_row;
   const long long plane = (long long)M * N;
@@ -909,10 +911,22 @@ __global__ void splitk_reduce_kernel(const float* __restrict__ ws, __nv_bfloat16
       a.z += __bfloat162float(bias[n + 2]);
       a.w += __bfloat162float(bias[n + 3]);
     }
+    if (flags & GEMM_OUT_F32) {
+      float4* dst = reinterpret_cast<float4*>(reinterpret_cast<float*>(out_v) + m * ldc + n);
+      if (flags & GEMM_ACCUMULATE) {
+        const float4 c = *dst;
+        a.x += c.x;
+        a.y += c.y;
+        a.z += c.z;
+        a.w += c.w;
+      }
+      *dst = a;
+      continue;
+    }
     uint2 o;
     o.x = pack_bf16x2(a.x, a.y);
     o.y = pack_bf16x2(a.z, a.w);
-    *reinterpret_cast<uint2*>(out + m * ldc + n) = o;
+    *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(out_v) + m * ldc + n) = o;
   }
 }
 }  // namespace
@@ -923,13 +937,19 @@ __global__ void splitk_reduce_kernel(const float* __restrict__ ws, __nv_bfloat16
 // The K range is cut into `splits` slices, each (tile, slice) pair is one unit of work writing an fp32 partial
 // into `workspace` [splits, M, N]; a second small kernel sums the slices and casts to bf16.
 //   k_offsets: device int[splits + 1], multiples of 64 from 0 to K. N must be a multiple of 8.
+//   flags: GEMM_OUT_F32 = C is fp32, with GEMM_ACCUMULATE = C += (fp32 only; a branch's output projection adds into
+//   an fp32 residual stream this way).
 EDL_HOST_API int edl_gemm_splitk(const void* A, const void* B, void* C, const void* bias, int M, int N, int K,
                                  long long lda, long long ldb, long long ldc, int splits, void* workspace,
-                                 const int* k_offsets, int* status, void* stream) {
+                                 const int* k_offsets, int flags, int* status, void* stream) {
   using namespace edl;
   if (M <= 0 || N <= 0 || K <= 0) return 0;
   if ((lda & 7) || (ldb & 7) || (ldc & 7) || (N & 7) || splits < 1) {
     set_last_error("edl_gemm_splitk: lda, ldb, ldc, N must be multiples of 8 and splits >= 1");
+    return -1;
+  }
+  if ((flags & GEMM_ACCUMULATE) && !(flags & GEMM_OUT_F32)) {
+    set_last_error("edl_gemm_splitk: accumulation needs an fp32 output");
     return -1;
   }
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
@@ -941,9 +961,8 @@ EDL_HOST_API int edl_gemm_splitk(const void* A, const void* B, void* C, const vo
   const long long vecs = (long long)M * (N / 4);
   int blocks = (int)((vecs + 255) / 256);
   if (blocks > 4 * sm_count()) blocks = 4 * sm_count();
-  splitk_reduce_kernel<<<blocks, 256, 0, s>>>(reinterpret_cast<const float*>(workspace),
-                                              reinterpret_cast<__nv_bfloat16*>(C),
-                                              reinterpret_cast<const __nv_bfloat16*>(bias), M, N, ldc, splits);
+  splitk_reduce_kernel<<<blocks, 256, 0, s>>>(reinterpret_cast<const float*>(workspace), C,
+                                              reinterpret_cast<const __nv_bfloat16*>(bias), M, N, ldc, splits, flags);
   return check_cuda(cudaGetLastError(), "splitk_reduce launch");
 }
 

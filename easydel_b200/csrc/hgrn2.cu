@@ -1,0 +1,384 @@
+// HGRN2: linear attention whose forget gate also decides what is written. Per head, with a [D, V] state S in fp32,
+//
+//   f_t = lower + (1 - lower) * sigmoid(z_t + bias)          (one gate per head and channel)
+//   S_t = diag(f_t) S_{t-1} + (1 - f_t) v_t^T,   o_t = S_t^T silu(q_t)
+//
+// The kernels read the packed projection rows [q (H D) | z (H D) | v (H V)] and keep everything between them and the
+// output in 32 bits. States live in a pool addressed by slot and are updated where they lie.
+//
+//   * hgrn2_decode: one token per sequence. A CTA per (sequence, head) streams the state once (it is all the traffic
+//     there is), and finishes the row with the per-head RMS norm.
+//   * hgrn2_scan: any number of tokens per sequence. The columns of a state never meet, so a CTA owns (sequence, head,
+//     column tile) and walks the tokens with its part of the state in registers: 8 rows x 4 columns per thread, packed
+//     fp32 arithmetic, gates of 16 tokens at a time in shared memory.
+//   * When (sequences x heads x tiles) cannot fill the GPU and sequences are long, the token axis is cut into segments:
+//     one pass leaves every segment's end state from a zero start and the product of its gates, a small kernel chains
+//     them into the state each segment starts from, and the scan then runs all segments at once.
+//
+// Compiled without fast-math.
+#include "common.cuh"
+
+namespace edl {
+namespace {
+
+__device__ __forceinline__ float g_of(float v) { return v; }
+__device__ __forceinline__ float g_of(__nv_bfloat16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ void g_put(float* p, float v) { *p = v; }
+__device__ __forceinline__ void g_put(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
+
+__device__ __forceinline__ float gate_f(float z, float lower) { return lower + (1.f - lower) / (1.f + expf(-z)); }
+__device__ __forceinline__ float silu_p(float x) { return x / (1.f + expf(-x)); }
+
+struct Hgrn2Params {
+  const void* proj;          // [T, ld]: q | z | v
+  long long ld;
+  const float* bias;         // [H * D]
+  const float* lower;        // [H * D]
+  const int* cu;             // [B + 1]
+  const int* slots;          // [B] pool rows, or null: row b of the pool is sequence b
+  float* state;              // pool [*, H, D, V], or null: start from zero, keep nothing
+  void* out;                 // scan: fp32 [T, H * V]; decode: operand type
+  int B, H, D, V;
+  // segmented form
+  float* ws;                 // [B * nseg, H, D, V]: end states, then start states, of the segments
+  float* prod;               // [B * nseg, H, D]: products of the gates
+  int seg_len, nseg;
+  // decode
+  const float* norm;         // [V]
+  float eps;
+};
+
+enum { SCAN_WHOLE = 0, SCAN_ENDS = 1, SCAN_SEGMENTS = 2 };
+constexpr int SCT = 128;     // threads of a scan CTA
+constexpr int CPT = 4;       // columns per thread
+
+// DP: D rounded up to a tile; RPT rows per thread; DP / RPT lanes share a column group.
+template <typename TI, int DP, int RPT, int MODE>
+__global__ void __launch_bounds__(SCT)
+hgrn2_scan_kernel(const Hgrn2Params p) {
+  constexpr int SPLIT = DP / RPT;               // 4 .. 32 adjacent lanes
+  constexpr int CT = (SCT / SPLIT) * CPT;       // columns of this CTA
+  constexpr int TC = DP <= 256 ? 16 : 8;        // tokens per stage
+  constexpr int NK = RPT / 4;
+  static_assert(SPLIT >= 4 && SPLIT <= 32 && RPT % 4 == 0, "");
+  __shared__ __align__(16) float sf[TC][DP];
+  __shared__ __align__(16) float sq[MODE == SCAN_ENDS ? 1 : TC][DP];
+  __shared__ __align__(16) float sv[TC][CT];
+  const int tid = threadIdx.x;
+  const int part = tid % SPLIT, grp = tid / SPLIT;
+  const int h = blockIdx.y;
+  const int col0 = blockIdx.x * CT, col = col0 + grp * CPT;
+  int b, seg = 0, t0, t1;
+  if (MODE == SCAN_WHOLE) {
+    b = blockIdx.z;
+    t0 = p.cu[b];
+    t1 = p.cu[b + 1];
+  } else {
+    b = blockIdx.z / p.nseg;
+    seg = blockIdx.z % p.nseg;
+    t0 = p.cu[b] + seg * p.seg_len;
+    t1 = min(p.cu[b + 1], t0 + p.seg_len);
+  }
+  if (t0 >= t1) return;
+  const bool final_seg = MODE == SCAN_WHOLE || t1 == p.cu[b + 1];
+  if (MODE == SCAN_ENDS && final_seg) return;   // nothing follows the last segment
+  const TI* proj = reinterpret_cast<const TI*>(p.proj);
+  const int HD = p.H * p.D;
+  const long long mat = (long long)p.D * p.V;
+  float* pool = nullptr;
+  if (p.state) pool = p.state + ((long long)(p.slots ? p.slots[b] : b) * p.H + h) * mat;
+  float* seg_state = MODE == SCAN_WHOLE ? nullptr : p.ws + ((long long)(b * p.nseg + seg) * p.H + h) * mat;
+
+  // rows of this thread: 4 * (part + SPLIT * k) + j, k < NK, j < 4; S2[k][j / 2][c] holds rows j, j + 1 as a pair
+  float S[NK][4][CPT];
+  float pr[NK][4];
+  {
+    const float* src = MODE == SCAN_WHOLE ? pool : (MODE == SCAN_SEGMENTS ? seg_state : nullptr);
+#pragma unroll
+    for (int k = 0; k < NK; ++k)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int row = 4 * (part + SPLIT * k) + j;
+        pr[k][j] = 1.f;
+#pragma unroll
+        for (int c = 0; c < CPT; ++c)
+          S[k][j][c] = (src && row < p.D && col + c < p.V) ? src[(long long)row * p.V + col + c] : 0.f;
+      }
+  }
+  for (int tb = t0; tb < t1; tb += TC) {
+    const int n = min(TC, t1 - tb);
+    __syncthreads();
+    for (int i = tid; i < n * DP; i += SCT) {
+      const int t = i / DP, d = i % DP;
+      float f = 0.f, qv = 0.f;
+      if (d < p.D) {
+        const TI* row = proj + (tb + t) * p.ld + h * p.D + d;
+        f = gate_f(g_of(row[HD]) + p.bias[h * p.D + d], p.lower[h * p.D + d]);
+        if (MODE != SCAN_ENDS) qv = silu_p(g_of(row[0]));
+      }
+      sf[t][d] = f;
+      if (MODE != SCAN_ENDS) sq[t][d] = qv;
+    }
+    for (int i = tid; i < n * CT; i += SCT) {
+      const int t = i / CT, c = i % CT;
+      sv[t][c] = col0 + c < p.V ? g_of(proj[(tb + t) * p.ld + 2 * HD + h * p.V + col0 + c]) : 0.f;
+    }
+    __syncthreads();
+#pragma unroll 2
+    for (int t = 0; t < n; ++t) {
+      const float4 v4 = *reinterpret_cast<const float4*>(&sv[t][grp * CPT]);
+      const float v[CPT] = {v4.x, v4.y, v4.z, v4.w};
+      float a0[CPT], a1[CPT];
+#pragma unroll
+      for (int c = 0; c < CPT; ++c) a0[c] = a1[c] = 0.f;
+#pragma unroll
+      for (int k = 0; k < NK; ++k) {
+        const float4 f4 = *reinterpret_cast<const float4*>(&sf[t][4 * (part + SPLIT * k)]);
+        float4 q4 = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (MODE != SCAN_ENDS) q4 = *reinterpret_cast<const float4*>(&sq[t][4 * (part + SPLIT * k)]);
+#pragma unroll
+        for (int c = 0; c < CPT; ++c) {
+          // S = f S + (1 - f) v as v + f (S - v), two rows per instruction
+          float d0 = S[k][0][c], d1 = S[k][1][c], d2 = S[k][2][c], d3 = S[k][3][c];
+          add2(d0, d1, -v[c], -v[c]);
+          add2(d2, d3, -v[c], -v[c]);
+          fma2(S[k][0][c], S[k][1][c], f4.x, f4.y, d0, d1, v[c], v[c]);
+          fma2(S[k][2][c], S[k][3][c], f4.z, f4.w, d2, d3, v[c], v[c]);
+          if (MODE != SCAN_ENDS) {
+            fma2(a0[c], a1[c], q4.x, q4.y, S[k][0][c], S[k][1][c], a0[c], a1[c]);
+            fma2(a0[c], a1[c], q4.z, q4.w, S[k][2][c], S[k][3][c], a0[c], a1[c]);
+          }
+        }
+        if (MODE == SCAN_ENDS) {
+          pr[k][0] *= f4.x;
+          pr[k][1] *= f4.y;
+          pr[k][2] *= f4.z;
+          pr[k][3] *= f4.w;
+        }
+      }
+      if (MODE != SCAN_ENDS) {
+        // sum over the lanes of the group: the first two exchanges also spread the four columns over four lanes
+        float s[CPT];
+#pragma unroll
+        for (int c = 0; c < CPT; ++c) s[c] = a0[c] + a1[c];
+        const bool hi0 = part & 1, hi1 = part & 2;
+        const float x0 = __shfl_xor_sync(0xffffffffu, hi0 ? s[0] : s[2], 1);
+        const float x1 = __shfl_xor_sync(0xffffffffu, hi0 ? s[1] : s[3], 1);
+        const float y0 = (hi0 ? s[2] : s[0]) + x0, y1 = (hi0 ? s[3] : s[1]) + x1;
+        float z = (hi1 ? y1 : y0) + __shfl_xor_sync(0xffffffffu, hi1 ? y0 : y1, 2);
+#pragma unroll
+        for (int o = 4; o < SPLIT; o <<= 1) z += __shfl_xor_sync(0xffffffffu, z, o);
+        const int c = (part & 1) * 2 + ((part >> 1) & 1);
+        if (part < 4 && col + c < p.V)
+          reinterpret_cast<float*>(p.out)[(long long)(tb + t) * p.H * p.V + (long long)h * p.V + col + c] = z;
+      }
+    }
+  }
+  float* dst = MODE == SCAN_ENDS ? seg_state : (final_seg ? pool : nullptr);
+  if (dst) {
+#pragma unroll
+    for (int k = 0; k < NK; ++k)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int row = 4 * (part + SPLIT * k) + j;
+        if (row < p.D) {
+#pragma unroll
+          for (int c = 0; c < CPT; ++c)
+            if (col + c < p.V) dst[(long long)row * p.V + col + c] = S[k][j][c];
+          if (MODE == SCAN_ENDS && col == 0)
+            p.prod[((long long)(b * p.nseg + seg) * p.H + h) * p.D + row] = pr[k][j];
+        }
+      }
+  }
+}
+
+// Start state of every segment from the pool state, the end states and the gate products.
+__global__ void hgrn2_chain_kernel(const Hgrn2Params p) {
+  const int b = blockIdx.z, h = blockIdx.y;
+  const int len = p.cu[b + 1] - p.cu[b];
+  if (len <= 0) return;
+  const int segs = (len + p.seg_len - 1) / p.seg_len;
+  const long long mat = (long long)p.D * p.V;
+  const float* pool = p.state ? p.state + ((long long)(p.slots ? p.slots[b] : b) * p.H + h) * mat : nullptr;
+  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < mat;
+       i += (long long)gridDim.x * blockDim.x) {
+    const int row = (int)(i / p.V);
+    float s = pool ? pool[i] : 0.f;
+    for (int g = 0; g < segs; ++g) {
+      const long long at = (long long)(b * p.nseg + g) * p.H + h;
+      float* w = p.ws + at * mat + i;
+      const float end = *w;
+      *w = s;
+      if (g + 1 < segs) s = fmaf(p.prod[at * p.D + row], s, end);
+    }
+  }
+}
+
+constexpr int DCT = 256;
+
+// One token per sequence; VEC columns per thread.
+template <typename TI, int VEC>
+__global__ void __launch_bounds__(DCT)
+hgrn2_decode_kernel(const Hgrn2Params p) {
+  extern __shared__ __align__(16) float dsm[];   // f [D] | q [D] | partial sums [groups][V]
+  __shared__ float red[32];
+  const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x;
+  const TI* row = reinterpret_cast<const TI*>(p.proj) + (long long)p.cu[b] * p.ld;
+  if (p.cu[b + 1] <= p.cu[b]) return;
+  const int HD = p.H * p.D, D = p.D, V = p.V;
+  float* sf = dsm;
+  float* sq = dsm + D;
+  float* sums = dsm + ((2 * D + 3) & ~3);
+  const int vcols = V / VEC;                     // column groups
+  const int groups = max(1, DCT / vcols);        // row groups
+  float* st = p.state + ((long long)(p.slots ? p.slots[b] : b) * p.H + h) * (long long)D * V;
+  for (int d = tid; d < D; d += DCT) {
+    sf[d] = gate_f(g_of(row[HD + h * D + d]) + p.bias[h * D + d], p.lower[h * D + d]);
+    sq[d] = silu_p(g_of(row[h * D + d]));
+  }
+  __syncthreads();
+  for (int u = tid; u < vcols * groups; u += DCT) {   // one round unless V / VEC > DCT
+    const int cg = u % vcols, rg = u / vcols;
+    float v[VEC], acc[VEC];
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) {
+      v[j] = g_of(row[2 * HD + h * V + cg * VEC + j]);
+      acc[j] = 0.f;
+    }
+    constexpr int BATCH = 8;                     // rows in flight: all loads of a batch are issued before its stores
+    for (int d0 = rg; d0 < D; d0 += groups * BATCH) {
+      float s[BATCH][VEC];
+#pragma unroll
+      for (int i = 0; i < BATCH; ++i) {
+        const int d = d0 + i * groups;
+        const float* sp = st + (long long)d * V + cg * VEC;
+        if (d < D) {
+          if constexpr (VEC == 4) {
+            const float4 x = *reinterpret_cast<const float4*>(sp);
+            s[i][0] = x.x; s[i][1] = x.y; s[i][2] = x.z; s[i][3] = x.w;
+          } else {
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) s[i][j] = sp[j];
+          }
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < BATCH; ++i) {
+        const int d = d0 + i * groups;
+        if (d >= D) break;
+        float* sp = st + (long long)d * V + cg * VEC;
+        const float f = sf[d], q = sq[d];
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) {
+          s[i][j] = fmaf(f, s[i][j] - v[j], v[j]);
+          acc[j] = fmaf(q, s[i][j], acc[j]);
+        }
+        if constexpr (VEC == 4) {
+          *reinterpret_cast<float4*>(sp) = make_float4(s[i][0], s[i][1], s[i][2], s[i][3]);
+        } else {
+#pragma unroll
+          for (int j = 0; j < VEC; ++j) sp[j] = s[i][j];
+        }
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) sums[rg * V + cg * VEC + j] = acc[j];
+  }
+  __syncthreads();
+  float ss = 0.f;
+  for (int c = tid; c < V; c += DCT) {
+    float o = 0.f;
+    for (int g = 0; g < groups; ++g) o += sums[g * V + c];
+    sums[c] = o;                                 // group 0's own place
+    ss += o * o;
+  }
+  const float rs = 1.f / sqrtf(block_sum(ss, red) / (float)V + p.eps);
+  TI* out = reinterpret_cast<TI*>(p.out) + (long long)p.cu[b] * p.H * V + (long long)h * V;
+  for (int c = tid; c < V; c += DCT) g_put(out + c, sums[c] * rs * p.norm[c]);
+}
+
+template <typename TI, int MODE>
+int launch_scan(const Hgrn2Params& p, int z, cudaStream_t s) {
+#define EDL_HS(DP, RPT)                                                                          \
+  {                                                                                              \
+    constexpr int CT = (SCT / (DP / RPT)) * CPT;                                                 \
+    hgrn2_scan_kernel<TI, DP, RPT, MODE><<<dim3((p.V + CT - 1) / CT, p.H, z), SCT, 0, s>>>(p);   \
+  }
+  if (p.D <= 32) EDL_HS(32, 8)
+  else if (p.D <= 64) EDL_HS(64, 8)
+  else if (p.D <= 128) EDL_HS(128, 8)
+  else if (p.D <= 256) EDL_HS(256, 8)
+  else EDL_HS(512, 16)
+#undef EDL_HS
+  return check_cuda(cudaGetLastError(), "hgrn2_scan launch");
+}
+
+template <typename TI>
+int run_scan(Hgrn2Params& p, cudaStream_t s) {
+  if (p.seg_len <= 0) return launch_scan<TI, SCAN_WHOLE>(p, p.B, s);
+  if (launch_scan<TI, SCAN_ENDS>(p, p.B * p.nseg, s)) return -1;
+  const long long mat = (long long)p.D * p.V;
+  hgrn2_chain_kernel<<<dim3((unsigned)((mat + 255) / 256), p.H, p.B), 256, 0, s>>>(p);
+  if (check_cuda(cudaGetLastError(), "hgrn2_chain launch")) return -1;
+  return launch_scan<TI, SCAN_SEGMENTS>(p, p.B * p.nseg, s);
+}
+
+bool bad_sizes(const char* who, int B, int H, int D, int V) {
+  if (H < 1 || H > 65535 || D < 1 || D > 512 || V < 1 || V > 1024 || B > 65535) {
+    set_last_error("%s: unsupported sizes (B=%d, H=%d, D=%d, V=%d)", who, B, H, D, V);
+    return true;
+  }
+  return false;
+}
+
+}  // namespace
+}  // namespace edl
+
+using namespace edl;
+
+// o [T, H * V] fp32 (no output norm). seg_len > 0: segmented form, nseg >= ceil(longest sequence / seg_len), with
+// ws [B * nseg, H, D, V] and prod [B * nseg, H, D] fp32.
+EDL_HOST_API int edl_hgrn2_scan(const void* proj, int f32, long long ld, const float* bias, const float* lower,
+                                const int* cu, const int* slots, float* state, float* o, int B, int H, int D, int V,
+                                int seg_len, int nseg, float* ws, float* prod, void* stream) {
+  if (B <= 0) return 0;
+  if (bad_sizes("edl_hgrn2_scan", B, H, D, V)) return -1;
+  if (seg_len > 0 && (nseg < 1 || !ws || !prod || (long long)B * nseg > 65535)) {
+    set_last_error("edl_hgrn2_scan: bad segmentation (seg_len=%d, nseg=%d)", seg_len, nseg);
+    return -1;
+  }
+  Hgrn2Params p{};
+  p.proj = proj; p.ld = ld; p.bias = bias; p.lower = lower; p.cu = cu; p.slots = slots; p.state = state; p.out = o;
+  p.B = B; p.H = H; p.D = D; p.V = V; p.seg_len = seg_len; p.nseg = nseg; p.ws = ws; p.prod = prod;
+  cudaStream_t s = (cudaStream_t)stream;
+  return f32 ? run_scan<float>(p, s) : run_scan<__nv_bfloat16>(p, s);
+}
+
+// One token per sequence (row cu[b] of proj), output norm included; out [T, H * V] in the projection's type.
+EDL_HOST_API int edl_hgrn2_decode(const void* proj, int f32, long long ld, const float* bias, const float* lower,
+                                  const int* cu, const int* slots, float* state, const float* norm, float eps,
+                                  void* out, int B, int H, int D, int V, void* stream) {
+  if (B <= 0) return 0;
+  if (bad_sizes("edl_hgrn2_decode", B, H, D, V)) return -1;
+  if (!state) {
+    set_last_error("edl_hgrn2_decode: needs a state pool");
+    return -1;
+  }
+  Hgrn2Params p{};
+  p.proj = proj; p.ld = ld; p.bias = bias; p.lower = lower; p.cu = cu; p.slots = slots; p.state = state; p.out = out;
+  p.B = B; p.H = H; p.D = D; p.V = V; p.norm = norm; p.eps = eps;
+  cudaStream_t s = (cudaStream_t)stream;
+  const bool v4 = V % 4 == 0 && (reinterpret_cast<uintptr_t>(state) & 15) == 0;
+  const int vcols = v4 ? V / 4 : V;
+  const int groups = vcols >= DCT ? 1 : DCT / vcols;
+  const size_t smem = (size_t)(((2 * D + 3) & ~3) + groups * V) * sizeof(float);   // <= 2 * 512 + 1024 + V floats
+  const dim3 grid(H, B);
+#define EDL_HD(T, V_) hgrn2_decode_kernel<T, V_><<<grid, DCT, smem, s>>>(p)
+  if (f32) {
+    if (v4) EDL_HD(float, 4); else EDL_HD(float, 1);
+  } else {
+    if (v4) EDL_HD(__nv_bfloat16, 4); else EDL_HD(__nv_bfloat16, 1);
+  }
+#undef EDL_HD
+  return check_cuda(cudaGetLastError(), "hgrn2_decode launch");
+}

@@ -1,0 +1,477 @@
+// Element-wise and row kernels around an fp32 residual stream.
+//
+// Models that keep the sum of their branches in 32 bits hold x [T, W] as fp32; every branch reads it through a norm
+// that writes the operand of the next product (bf16, or fp32 for an all-fp32 model) and its output projection
+// accumulates straight into x. The kernels here are what sits between those products:
+//
+//   * embedding rows into the stream (and, for models whose passes read [x ; x0], into the right half of that operand);
+//   * RMS norm, optionally followed by a token shift (each row is blended with the normalised row before it; the row
+//     before a step's first row lives in a per-slot state that the same launch brings up to date);
+//   * the left half of a pass's [x ; x0] operand;
+//   * xIELU, a two-branch activation with two learned numbers;
+//   * the attention prologue: per-head RMS norm of q and k, position-dependent query temperature and the page append,
+//     in one pass over the packed projection.
+//
+// Compiled without fast-math: these are the parts of such a model that are computed in 32 bits.
+#include "common.cuh"
+
+namespace edl {
+namespace {
+
+template <typename T>
+__device__ __forceinline__ float ld1(const T* p);
+template <>
+__device__ __forceinline__ float ld1<float>(const float* p) { return *p; }
+template <>
+__device__ __forceinline__ float ld1<__nv_bfloat16>(const __nv_bfloat16* p) { return __bfloat162float(*p); }
+__device__ __forceinline__ void st1(float* p, float v) { *p = v; }
+__device__ __forceinline__ void st1(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
+
+template <int VEC, typename T>
+__device__ __forceinline__ void ldv(const T* p, float (&v)[VEC]) {
+  if constexpr (VEC == 4 && sizeof(T) == 4) {
+    const float4 a = *reinterpret_cast<const float4*>(p);
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+  } else if constexpr (VEC == 4) {
+    const uint2 a = *reinterpret_cast<const uint2*>(p);
+    const float2 lo = unpack_bf16x2(a.x), hi = unpack_bf16x2(a.y);
+    v[0] = lo.x; v[1] = lo.y; v[2] = hi.x; v[3] = hi.y;
+  } else {
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) v[i] = ld1<T>(p + i);
+  }
+}
+template <int VEC, typename T>
+__device__ __forceinline__ void stv(T* p, const float (&v)[VEC]) {
+  if constexpr (VEC == 4 && sizeof(T) == 4) {
+    *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+  } else if constexpr (VEC == 4) {
+    *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]));
+  } else {
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) st1(p + i, v[i]);
+  }
+}
+
+// Largest b with cu[b] <= r (cu is a non-decreasing prefix sum).
+__device__ __forceinline__ int seq_of_row(const int* cu, int nseq, int r) {
+  int lo = 0, hi = nseq;
+  while (hi - lo > 1) {
+    const int mid = (lo + hi) >> 1;
+    if (cu[mid] <= r) lo = mid; else hi = mid;
+  }
+  return lo;
+}
+
+// ---- embedding -------------------------------------------------------------------------------------------------
+template <typename T, int VEC>
+__global__ void embed_stream_kernel(const T* __restrict__ table, const long long* __restrict__ ids,
+                                    float* __restrict__ x, T* __restrict__ right, long long ld_right, int rows, int W,
+                                    int V, int* status) {
+  const int per = W / VEC;
+  const long long total = (long long)rows * per;
+  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total;
+       i += (long long)gridDim.x * blockDim.x) {
+    const int r = (int)(i / per), c = (int)(i - (long long)r * per) * VEC;
+    const long long id = ids[r];
+    float v[VEC];
+    if (id < 0 || id >= V) {
+      if (status) atomicCAS(status, 0, EDL_BAD_INDEX);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) v[j] = 0.f;
+    } else {
+      ldv<VEC>(table + id * W + c, v);
+    }
+    stv<VEC>(x + (long long)r * W + c, v);
+    if (right) stv<VEC>(right + r * ld_right + c, v);
+  }
+}
+
+// ---- left half of [x ; x0] -------------------------------------------------------------------------------------
+template <typename T, int VEC>
+__global__ void cast_rows_kernel(const float* __restrict__ x, T* __restrict__ out, long long ld_out, int rows, int W) {
+  const int per = W / VEC;
+  const long long total = (long long)rows * per;
+  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total;
+       i += (long long)gridDim.x * blockDim.x) {
+    const int r = (int)(i / per), c = (int)(i - (long long)r * per) * VEC;
+    float v[VEC];
+    ldv<VEC>(x + (long long)r * W + c, v);
+    stv<VEC>(out + r * ld_out + c, v);
+  }
+}
+
+// ---- RMS norm (+ token shift) -----------------------------------------------------------------------------------
+constexpr int NT = 256;
+
+// Two block-wide sums at once.
+__device__ __forceinline__ float2 block_sum2(float a, float b, float2* red) {
+  const int lane = threadIdx.x & 31, w = threadIdx.x >> 5;
+  a = warp_sum(a);
+  b = warp_sum(b);
+  __syncthreads();
+  if (lane == 0) red[w] = make_float2(a, b);
+  __syncthreads();
+  float2 t = red[0];
+#pragma unroll
+  for (int i = 1; i < NT / 32; ++i) {
+    t.x += red[i].x;
+    t.y += red[i].y;
+  }
+  return t;
+}
+
+// One CTA per row. NV: vectors of VEC elements each thread keeps of a row (0: rows too wide for registers are read
+// twice). Without `mu` this is a plain norm.
+template <typename TO, int VEC, int NV>
+__global__ void __launch_bounds__(NT)
+norm_shift_kernel(const float* __restrict__ x, const float* __restrict__ w, const float* __restrict__ mu, float eps,
+                  int rows, int W, const int* __restrict__ cu, int nseq, const int* __restrict__ slots,
+                  float* __restrict__ state, long long ld_state, TO* __restrict__ out) {
+  __shared__ float2 red[NT / 32];
+  const int r = blockIdx.x;
+  const float inv_w = 1.f / (float)W;
+  const float* xr = x + (long long)r * W;
+  const float* xp = nullptr;   // the row before, when this step brought it
+  float* st = nullptr;
+  int last = -1;
+  if (mu) {
+    const int b = seq_of_row(cu, nseq, r);
+    if (r > cu[b]) {
+      xp = xr - W;
+    } else if (state) {
+      st = state + (long long)slots[b] * ld_state;
+      last = cu[b + 1] - 1;
+    }
+  }
+  constexpr int STEP = NT * VEC;
+  constexpr int KEEP = NV > 0 ? NV : 1;
+  float a[KEEP][VEC], p[KEEP][VEC];
+  float sa = 0.f, sp = 0.f;
+  if constexpr (NV > 0) {
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+      const int c = threadIdx.x * VEC + k * STEP;
+      if (c < W) {
+        ldv<VEC>(xr + c, a[k]);
+        if (xp) ldv<VEC>(xp + c, p[k]);
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) {
+          sa += a[k][j] * a[k][j];
+          if (xp) sp += p[k][j] * p[k][j];
+        }
+      }
+    }
+  } else {
+    for (int c = threadIdx.x * VEC; c < W; c += STEP) {
+      ldv<VEC>(xr + c, a[0]);
+      if (xp) ldv<VEC>(xp + c, p[0]);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) {
+        sa += a[0][j] * a[0][j];
+        if (xp) sp += p[0][j] * p[0][j];
+      }
+    }
+  }
+  const float2 s = block_sum2(sa, sp, red);
+  const float ra = 1.f / sqrtf(s.x * inv_w + eps), rp = 1.f / sqrtf(s.y * inv_w + eps);
+  auto emit = [&](int c, const float (&av)[VEC], const float (&pv)[VEC]) {
+    float wv[VEC], h[VEC];
+    ldv<VEC>(w + c, wv);
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) h[j] = av[j] * ra * wv[j];
+    if (mu) {
+      float m[VEC], before[VEC], o[VEC];
+      ldv<VEC>(mu + c, m);
+      if (st) {
+        ldv<VEC>(st + c, before);
+      } else {
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) before[j] = xp ? pv[j] * rp * wv[j] : 0.f;
+      }
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) o[j] = h[j] + (before[j] - h[j]) * m[j];
+      stv<VEC>(out + (long long)r * W + c, o);
+      if (st && last == r) stv<VEC>(st + c, h);
+    } else {
+      stv<VEC>(out + (long long)r * W + c, h);
+    }
+  };
+  if constexpr (NV > 0) {
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+      const int c = threadIdx.x * VEC + k * STEP;
+      if (c < W) emit(c, a[k], p[k]);
+    }
+  } else {
+    for (int c = threadIdx.x * VEC; c < W; c += STEP) {
+      ldv<VEC>(xr + c, a[0]);
+      if (xp) ldv<VEC>(xp + c, p[0]);
+      emit(c, a[0], p[0]);
+    }
+  }
+  if (st && last != r) {
+    // The CTA of a sequence's first row is the only reader of its state; having read it, it also normalises the last
+    // row and leaves that one for the next step. Nobody else touches the state, so no launch has to follow.
+    const float* xl = x + (long long)last * W;
+    float sl = 0.f, v[VEC], wv[VEC];
+    for (int c = threadIdx.x * VEC; c < W; c += STEP) {
+      ldv<VEC>(xl + c, v);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) sl += v[j] * v[j];
+    }
+    const float rl = 1.f / sqrtf(block_sum2(sl, 0.f, red).x * inv_w + eps);
+    for (int c = threadIdx.x * VEC; c < W; c += STEP) {
+      ldv<VEC>(xl + c, v);
+      ldv<VEC>(w + c, wv);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) v[j] = v[j] * rl * wv[j];
+      stv<VEC>(st + c, v);
+    }
+  }
+}
+
+// ---- RMS norm over the heads of a [T, H * V] matrix with one weight vector for all heads ------------------------------
+template <typename TO>
+__global__ void __launch_bounds__(NT)
+head_norm_kernel(const float* __restrict__ o, const float* __restrict__ w, float eps, long long items, int V,
+                 TO* __restrict__ out) {
+  const int lane = threadIdx.x & 31;
+  const long long stride = (long long)gridDim.x * (NT / 32);
+  for (long long it = blockIdx.x * (long long)(NT / 32) + (threadIdx.x >> 5); it < items; it += stride) {
+    const float* src = o + it * V;
+    float s = 0.f;
+    for (int c = lane; c < V; c += 32) s += src[c] * src[c];
+    s = warp_sum(s);
+    const float rs = 1.f / sqrtf(s / (float)V + eps);
+    for (int c = lane; c < V; c += 32) st1(out + it * V + c, src[c] * rs * w[c]);
+  }
+}
+
+// ---- xIELU ------------------------------------------------------------------------------------------------------------
+__device__ __forceinline__ float softplus1(float x) { return x > 20.f ? x : log1pf(expf(x)); }
+
+template <typename T, int VEC>
+__global__ void xielu_kernel(const T* __restrict__ z, const float* __restrict__ act, T* __restrict__ y,
+                             long long n_vec) {
+  const float ap = softplus1(act[0]), an = 0.5f + softplus1(act[1]);
+  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < n_vec;
+       i += (long long)gridDim.x * blockDim.x) {
+    float v[VEC];
+    ldv<VEC>(z + i * VEC, v);
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) {
+      const float t = v[j];
+      v[j] = t > 0.f ? ap * t * t + 0.5f * t : an * (expm1f(t) - t) + 0.5f * t;
+    }
+    stv<VEC>(y + i * VEC, v);
+  }
+}
+
+// ---- attention prologue -------------------------------------------------------------------------------------------------
+// qkv [T, ld]: Hq query heads of D, Hkv key heads of D, Hkv value heads of Dv. One warp per (token, head): q and k are
+// RMS-normed over D (weights may be null: no norm), q is multiplied by its position's temperature
+// 1 + coef * ln(floor((p + 1) / every) + 1) (every <= 0: none) and written to q_out; k and v go to their page slot.
+template <typename T, int VEC>
+__global__ void __launch_bounds__(NT)
+qkv_prologue_kernel(const T* __restrict__ qkv, long long ld, const int* __restrict__ pos,
+                    const int* __restrict__ slots, const float* __restrict__ qw, const float* __restrict__ kw,
+                    float eps, float coef, float every, int T_rows, int Hq, int Hkv, int D, int Dv,
+                    T* __restrict__ q_out, T* __restrict__ k_pages, T* __restrict__ v_pages, long long ld_kpage,
+                    long long ld_vpage, long long num_slots, int* status) {
+  const int lane = threadIdx.x & 31;
+  const int heads = Hq + 2 * Hkv;
+  const long long items = (long long)T_rows * heads;
+  const long long stride = (long long)gridDim.x * (NT / 32);
+  for (long long it = blockIdx.x * (long long)(NT / 32) + (threadIdx.x >> 5); it < items; it += stride) {
+    const int t = (int)(it / heads), h = (int)(it - (long long)t * heads);
+    const T* row = qkv + t * ld;
+    const int hk = h < Hq ? -1 : (h < Hq + Hkv ? h - Hq : h - Hq - Hkv);
+    long long slot = 0;
+    if (h >= Hq) {
+      slot = slots[t];
+      if (slot < 0) continue;
+      if (slot >= num_slots) {
+        if (status) atomicCAS(status, 0, EDL_BAD_INDEX);
+        continue;
+      }
+    }
+    if (h >= Hq + Hkv) {   // value head: copied
+      const T* src = row + (long long)(Hq + Hkv) * D + (long long)hk * Dv;
+      T* dst = v_pages + slot * ld_vpage + (long long)hk * Dv;
+      for (int c = lane * VEC; c < Dv; c += 32 * VEC) {
+        float v[VEC];
+        ldv<VEC>(src + c, v);
+        stv<VEC>(dst + c, v);
+      }
+      continue;
+    }
+    const bool is_q = h < Hq;
+    const T* src = row + (long long)h * D;          // key heads follow the query heads
+    const float* w = is_q ? qw : kw;
+    float scale = 1.f;
+    if (w) {
+      float s = 0.f;
+      for (int c = lane * VEC; c < D; c += 32 * VEC) {
+        float v[VEC];
+        ldv<VEC>(src + c, v);
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) s += v[j] * v[j];
+      }
+      s = warp_sum(s);
+      scale = 1.f / sqrtf(s / (float)D + eps);
+    }
+    float temp = 1.f;
+    if (is_q && every > 0.f) temp = 1.f + coef * logf(floorf(((float)pos[t] + 1.f) / every) + 1.f);
+    T* dst = is_q ? q_out + ((long long)t * Hq + h) * D : k_pages + slot * ld_kpage + (long long)hk * D;
+    for (int c = lane * VEC; c < D; c += 32 * VEC) {
+      float v[VEC], wv[VEC];
+      ldv<VEC>(src + c, v);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) wv[j] = w ? w[c + j] : 1.f;
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) v[j] = v[j] * scale * wv[j] * temp;
+      stv<VEC>(dst + c, v);
+    }
+  }
+}
+
+int blocks_for(long long work, int per_block, int waves) {
+  long long b = (work + per_block - 1) / per_block, cap = (long long)sm_count() * waves;
+  return (int)(b < 1 ? 1 : (b > cap ? cap : b));
+}
+
+template <typename TO, int VEC>
+int launch_norm_shift(const float* x, const float* w, const float* mu, float eps, int rows, int W, const int* cu,
+                      int nseq, const int* slots, float* state, long long ld_state, TO* out, cudaStream_t s) {
+  const int nv = (W + NT * VEC - 1) / (NT * VEC);
+#define EDL_NS(N) \
+  norm_shift_kernel<TO, VEC, N><<<rows, NT, 0, s>>>(x, w, mu, eps, rows, W, cu, nseq, slots, state, ld_state, out)
+  if (nv <= 1) EDL_NS(1);
+  else if (nv <= 2) EDL_NS(2);
+  else if (nv <= 4) EDL_NS(4);
+  else if (nv <= 8) EDL_NS(8);
+  else EDL_NS(0);
+#undef EDL_NS
+  return check_cuda(cudaGetLastError(), "norm_shift launch");
+}
+
+bool al(const void* p, size_t n) { return (reinterpret_cast<uintptr_t>(p) & (n - 1)) == 0; }
+
+}  // namespace
+}  // namespace edl
+
+using namespace edl;
+
+// x [rows, W] fp32 = table[ids]; right (may be null): the same rows in the table's type at pitch ld_right.
+EDL_HOST_API int edl_embed_stream(const void* table, int f32, const long long* ids, float* x, void* right,
+                                  long long ld_right, int rows, int W, int V, int* status, void* stream) {
+  if (rows <= 0) return 0;
+  cudaStream_t s = (cudaStream_t)stream;
+  const bool v4 = W % 4 == 0 && ld_right % 4 == 0 && al(table, 16) && al(x, 16) && (!right || al(right, 8));
+  const int vec = v4 ? 4 : 1;
+  const int blocks = blocks_for((long long)rows * (W / vec), 256, 8);
+#define EDL_E(T, V_)                                                                                               \
+  embed_stream_kernel<T, V_><<<blocks, 256, 0, s>>>((const T*)table, ids, x, (T*)right, ld_right, rows, W, V, status)
+  if (f32) {
+    if (v4 && (!right || al(right, 16))) EDL_E(float, 4); else EDL_E(float, 1);
+  } else {
+    if (v4) EDL_E(__nv_bfloat16, 4); else EDL_E(__nv_bfloat16, 1);
+  }
+#undef EDL_E
+  return check_cuda(cudaGetLastError(), "embed_stream launch");
+}
+
+// out [rows, :W] at pitch ld_out = x [rows, W] in the operand type.
+EDL_HOST_API int edl_cast_rows(const float* x, void* out, int f32, long long ld_out, int rows, int W, void* stream) {
+  if (rows <= 0) return 0;
+  cudaStream_t s = (cudaStream_t)stream;
+  const bool v4 = W % 4 == 0 && ld_out % 4 == 0 && al(x, 16) && al(out, f32 ? 16 : 8);
+  const int blocks = blocks_for((long long)rows * (W / (v4 ? 4 : 1)), 256, 8);
+#define EDL_C(T, V_) cast_rows_kernel<T, V_><<<blocks, 256, 0, s>>>(x, (T*)out, ld_out, rows, W)
+  if (f32) {
+    if (v4) EDL_C(float, 4); else EDL_C(float, 1);
+  } else {
+    if (v4) EDL_C(__nv_bfloat16, 4); else EDL_C(__nv_bfloat16, 1);
+  }
+#undef EDL_C
+  return check_cuda(cudaGetLastError(), "cast_rows launch");
+}
+
+// out [rows, W] = rms_norm(x) * w, blended with the previous row's norm by mu when mu is given. cu [nseq + 1] bounds the
+// sequences on the row axis; state [*, ld_state] fp32 holds, per slot, the normalised row before the step's first one
+// (null: sequences start here) and is updated to the step's last row.
+EDL_HOST_API int edl_norm_shift(const float* x, const float* w, const float* mu, float eps, int rows, int W,
+                                const int* cu, int nseq, const int* slots, float* state, long long ld_state, void* out,
+                                int f32, void* stream) {
+  if (rows <= 0) return 0;
+  if (mu && (!cu || nseq <= 0 || (state && !slots))) {
+    set_last_error("edl_norm_shift: a token shift needs sequence bounds, and slots for a state");
+    return -1;
+  }
+  cudaStream_t s = (cudaStream_t)stream;
+  const bool v4 = W % 4 == 0 && ld_state % 4 == 0 && al(x, 16) && al(w, 16) && (!mu || al(mu, 16)) &&
+                  (!state || al(state, 16)) && al(out, f32 ? 16 : 8);
+  if (f32)
+    return v4 ? launch_norm_shift<float, 4>(x, w, mu, eps, rows, W, cu, nseq, slots, state, ld_state, (float*)out, s)
+              : launch_norm_shift<float, 1>(x, w, mu, eps, rows, W, cu, nseq, slots, state, ld_state, (float*)out, s);
+  return v4 ? launch_norm_shift<__nv_bfloat16, 4>(x, w, mu, eps, rows, W, cu, nseq, slots, state, ld_state,
+                                                  (__nv_bfloat16*)out, s)
+            : launch_norm_shift<__nv_bfloat16, 1>(x, w, mu, eps, rows, W, cu, nseq, slots, state, ld_state,
+                                                  (__nv_bfloat16*)out, s);
+}
+
+// o [items, V] fp32 -> rms_norm over V times w.
+EDL_HOST_API int edl_head_norm(const float* o, const float* w, float eps, long long items, int V, void* out, int f32,
+                               void* stream) {
+  if (items <= 0) return 0;
+  cudaStream_t s = (cudaStream_t)stream;
+  const int blocks = blocks_for(items, NT / 32, 16);
+  if (f32) head_norm_kernel<float><<<blocks, NT, 0, s>>>(o, w, eps, items, V, (float*)out);
+  else head_norm_kernel<__nv_bfloat16><<<blocks, NT, 0, s>>>(o, w, eps, items, V, (__nv_bfloat16*)out);
+  return check_cuda(cudaGetLastError(), "head_norm launch");
+}
+
+// y = xielu(z), n elements; act = the two raw parameters (fp32, on the device).
+EDL_HOST_API int edl_xielu(const void* z, const float* act, void* y, int f32, long long n, void* stream) {
+  if (n <= 0) return 0;
+  cudaStream_t s = (cudaStream_t)stream;
+  const bool v4 = n % 4 == 0 && al(z, f32 ? 16 : 8) && al(y, f32 ? 16 : 8);
+  const int blocks = blocks_for(n / (v4 ? 4 : 1), 256, 8);
+#define EDL_X(T, V_) xielu_kernel<T, V_><<<blocks, 256, 0, s>>>((const T*)z, act, (T*)y, n / V_)
+  if (f32) {
+    if (v4) EDL_X(float, 4); else EDL_X(float, 1);
+  } else {
+    if (v4) EDL_X(__nv_bfloat16, 4); else EDL_X(__nv_bfloat16, 1);
+  }
+#undef EDL_X
+  return check_cuda(cudaGetLastError(), "xielu launch");
+}
+
+EDL_HOST_API int edl_qkv_prologue(const void* qkv, int f32, long long ld, const int* pos, const int* slots,
+                                  const float* qw, const float* kw, float eps, float coef, float every, int T, int Hq,
+                                  int Hkv, int D, int Dv, void* q_out, void* k_pages, void* v_pages,
+                                  long long ld_kpage, long long ld_vpage, long long num_slots, int* status,
+                                  void* stream) {
+  if (T <= 0) return 0;
+  if (Hq <= 0 || Hkv <= 0 || D <= 0 || Dv <= 0 || !slots || (every > 0.f && !pos)) {
+    set_last_error("edl_qkv_prologue: bad arguments (Hq=%d, Hkv=%d, D=%d, Dv=%d)", Hq, Hkv, D, Dv);
+    return -1;
+  }
+  cudaStream_t s = (cudaStream_t)stream;
+  const size_t a = f32 ? 16 : 8;
+  const bool v4 = D % 4 == 0 && Dv % 4 == 0 && ld % 4 == 0 && ld_kpage % 4 == 0 && ld_vpage % 4 == 0 && al(qkv, a) &&
+                  al(q_out, a) && al(k_pages, a) && al(v_pages, a);
+  const int blocks = blocks_for((long long)T * (Hq + 2 * Hkv), NT / 32, 8);
+#define EDL_P(TT, V_)                                                                                                \
+  qkv_prologue_kernel<TT, V_><<<blocks, NT, 0, s>>>((const TT*)qkv, ld, pos, slots, qw, kw, eps, coef, every, T, Hq, \
+                                                    Hkv, D, Dv, (TT*)q_out, (TT*)k_pages, (TT*)v_pages, ld_kpage,    \
+                                                    ld_vpage, num_slots, status)
+  if (f32) {
+    if (v4) EDL_P(float, 4); else EDL_P(float, 1);
+  } else {
+    if (v4) EDL_P(__nv_bfloat16, 4); else EDL_P(__nv_bfloat16, 1);
+  }
+#undef EDL_P
+  return check_cuda(cudaGetLastError(), "qkv_prologue launch");
+}

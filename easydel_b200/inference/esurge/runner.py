@@ -88,8 +88,9 @@ class ModelRunner:
 
         self.use_graphs = dev.type == "cuda" and os.environ.get("EDL_ESURGE_CUDA_GRAPHS", "1") != "0"
         latent_kernel = bool(cache.latent and cache.k.shape[-1] == 576)    # the 512 + 64 layout has a decode kernel
-        if cache.linear or getattr(cache, "compressed", False) or (cache.latent and not latent_kernel) or \
-                (not cache.latent and model.spec.head_dim not in (64, 128)):
+        stream32 = getattr(self._lm.spec, "residual_f32", False)   # every head size has a capturable kernel there
+        if not getattr(cache, "states_in_place", True) or getattr(cache, "compressed", False) or (cache.latent and not latent_kernel) or \
+                (not cache.latent and not stream32 and model.spec.head_dim not in (64, 128)):
             self.use_graphs = False     # these serving paths are tensor code with host-side steps: run eagerly
         self._seq_slots = torch.zeros(max_num_seqs, dtype=torch.int64, device=dev)
         self._graphs: dict[int, tuple[tp.Any, torch.Tensor]] = {}
@@ -155,16 +156,19 @@ class ModelRunner:
             return 1
         return int(min(8, self.max_pages_per_seq // 4, max(1, self._sms // units)))
 
-    def _forward(self, B: int, T: int, max_q: int, num_decode: int, mm_rows=None) -> torch.Tensor:
-        """Backbone over the first ``T`` staged tokens of ``B`` sequences, LM head on each sequence's last row.
-        ``mm_rows``: ``[(first staged row, features [n, hidden])]`` to write over the token embeddings."""
+    def _forward(self, B: int, T: int, max_q: int, num_decode: int, mm_rows=None,
+                 logit_rows: torch.Tensor | None = None) -> torch.Tensor:
+        """Backbone over the first ``T`` staged tokens of ``B`` sequences, LM head on each sequence's last row (or on the
+        staged rows ``logit_rows``). ``mm_rows``: ``[(first staged row, features [n, hidden])]`` to write over the token
+        embeddings."""
         d_ids, d_pos, d_slots, d_cu, d_kv, d_last, d_table = self._dviews[:7]
         MP = self.max_pages_per_seq
         meta = PagedBatchMeta(cu_q=d_cu[:B + 1], kv_lens=d_kv[:B], page_table=d_table.view(self.max_num_seqs, MP)[:B],
                               slot_mapping=d_slots[:T], max_q=max_q, num_seqs=B, last_token_index=d_last[:B],
                               request_distribution=(num_decode, B, B),
                               num_splits=self._decode_splits(B) if (max_q == 1 and T == B) else 1,
-                              seq_slots=self._seq_slots[:B] if self.cache.linear else None)
+                              seq_slots=self._seq_slots[:B] if self.cache.linear else None,
+                              slot_ids=self._dviews[7][:B])
         if self.num_groups > 1:
             extra = self._dviews[10:]
             meta.group_slots = [extra[2 * g][:T] for g in range(self.num_groups - 1)]
@@ -184,7 +188,7 @@ class ModelRunner:
         else:
             res = model(input_ids=d_ids[:T][None].long(), position_ids=d_pos, past_key_values=self.cache,
                         cache_metadata=meta, apply_lm_head=False)
-        rows = S.gather_rows(res.last_hidden_state[0], d_last[:B])
+        rows = S.gather_rows(res.last_hidden_state[0], d_last[:B] if logit_rows is None else logit_rows)
         if self.tp_group is not None and hasattr(model, "apply_lm_head_vocab_parallel"):
             return model.apply_lm_head_vocab_parallel(rows, self.tp_group)
         return model.apply_lm_head(rows)
@@ -210,22 +214,50 @@ class ModelRunner:
 
     def _decode_step_graphed(self, Bp: int) -> torch.Tensor:
         """Greedy decode step for ``Bp`` rows: eager the first time (warm-up), captured the second, replayed after."""
+        return self._decode_graph(Bp)[0]
+
+    def _decode_graph(self, Bp: int) -> tuple[torch.Tensor, torch.Tensor]:
+        """``(tokens, logits)`` of the greedy decode step for ``Bp`` rows, see :meth:`_decode_step_graphed`."""
         entry = self._graphs.get(Bp)
         if entry is not None:
             entry[0].replay()
-            return entry[1]
+            return entry[1], entry[2]
         if Bp not in self._warm:
             self._warm.add(Bp)
-            return S.sample(self._forward(Bp, Bp, 1, Bp))[0]
+            logits = self._forward(Bp, Bp, 1, Bp)
+            return S.sample(logits)[0], logits
         torch.cuda.synchronize(self.device)
         g = torch.cuda.CUDAGraph()
         with torch.cuda.graph(g, pool=self._graph_pool):
-            toks = S.sample(self._forward(Bp, Bp, 1, Bp))[0]
+            logits = self._forward(Bp, Bp, 1, Bp)
+            toks = S.sample(logits)[0]
         if self._graph_pool is None:
             self._graph_pool = g.pool()
-        self._graphs[Bp] = (g, toks)
+        self._graphs[Bp] = (g, toks, logits)
         g.replay()
-        return toks
+        return toks, logits
+
+    @torch.no_grad()
+    def step_logits(self, out: SchedulerOutput, rows: tp.Sequence[int]) -> torch.Tensor | None:
+        """Runs one engine step like :meth:`launch` (same staging, same kernels, same decode graphs) without sampling:
+        returns the fp32 logits of the step's token rows ``rows`` (offsets on the flat token axis) on the host, or None
+        if no row is asked for. Synchronises, and raises if a kernel reported a failure."""
+        st = self._stage(out)
+        if st is None:
+            return None
+        sched, B, Bp, T, max_q, decode_only, mm_rows = st[:7]
+        if self.use_graphs and decode_only:
+            logits = self._decode_graph(Bp)[1]            # row b is sequence b
+            logits = logits[torch.tensor(list(rows), dtype=torch.long, device=self.device)] if len(rows) else None
+        else:
+            idx = torch.tensor(list(rows) or [T - 1], dtype=torch.int32, device=self.device)
+            logits = self._forward(B, T, max_q, out.num_decode, mm_rows, logit_rows=idx)
+        host = logits.float().cpu() if len(rows) else None
+        if self.device.type == "cuda":
+            from ...ops import _lib
+
+            _lib.check_status(self.device)
+        return host
 
     @torch.no_grad()
     def execute(self, out: SchedulerOutput) -> dict[str, int]:
@@ -254,6 +286,20 @@ class ModelRunner:
     def launch(self, out: SchedulerOutput):
         """Enqueues one engine step on the device and returns a handle for :meth:`collect`; does not wait for it."""
         t0 = time.perf_counter()
+        st = self._stage(out)
+        if st is None:
+            return None
+        sched, B, Bp, T, max_q, decode_only, mm_rows, any_pen, any_random = st
+        t1 = time.perf_counter()
+        from ...utils.helpers import nvtx_range
+
+        with nvtx_range(f"esurge_step_B{B}_T{T}"):
+            tokens, t2, t3 = self._run_model(out, sched, B, Bp, T, max_q, decode_only, any_pen, any_random, mm_rows)
+        return self._finish_launch(sched, B, tokens, t0, t1, t2, t3)
+
+    def _stage(self, out: SchedulerOutput):
+        """Fills the batch metadata of one step and uploads it; returns what the device step needs to know (None for an
+        empty step)."""
         sched = out.scheduled
         B = len(sched)
         T = out.total_tokens
@@ -380,7 +426,7 @@ class ModelRunner:
                 for g in range(self.num_groups - 1):
                     self._hviews[10 + 2 * g].numpy()[B:Bp] = 0
                     self._hviews[11 + 2 * g].numpy().reshape(self.max_num_seqs, MP)[B:Bp, :] = 0
-        if self.cache.linear:
+        if self.cache.linear and not getattr(self.cache, "states_in_place", False):
             # recurrent-state rows of the scheduled sequences; padding rows of a batch bucket share the spare row
             sl = [s.request.slot for s in sched] + [self.max_num_seqs] * (Bp - B)
             self._seq_slots[:Bp].copy_(torch.tensor(sl, dtype=torch.int64), non_blocking=True)
@@ -389,12 +435,7 @@ class ModelRunner:
         if nfix:
             d_fixpos, d_fixslot = self._dviews[8][:nfix].long(), self._dviews[9][:nfix].long()
             self._dviews[0].index_copy_(0, d_fixpos, self._last_tokens.index_select(0, d_fixslot).to(torch.int32))
-        t1 = time.perf_counter()
-        from ...utils.helpers import nvtx_range
-
-        with nvtx_range(f"esurge_step_B{B}_T{T}"):
-            tokens, t2, t3 = self._run_model(out, sched, B, Bp, T, max_q, decode_only, any_pen, any_random, mm_rows)
-        return self._finish_launch(sched, B, tokens, t0, t1, t2, t3)
+        return sched, B, Bp, T, max_q, decode_only, mm_rows, any_pen, any_random
 
     def _run_model(self, out, sched, B, Bp, T, max_q, decode_only, any_pen, any_random, mm_rows):
         if self.use_graphs and decode_only:

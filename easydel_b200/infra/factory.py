@@ -48,9 +48,14 @@ class ModuleRegistration:
 class Registry:
     _configs: dict[str, dict[str, type]] = field(default_factory=lambda: {ConfigType.MODULE_CONFIG.value: {}})
     _modules: dict[str, dict[str, ModuleRegistration]] = field(default_factory=dict)
+    _architectures: dict[str, str] = field(default_factory=dict)      # architecture name -> model type
 
-    def register_config(self, config_type: str, config_field: ConfigType = ConfigType.MODULE_CONFIG):
+    def register_config(self, config_type: str, config_field: ConfigType = ConfigType.MODULE_CONFIG,
+                        architecture: str | None = None):
+        """``architecture``: the name under which checkpoint configurations without a ``model_type`` name the family."""
         def deco(cls):
+            if architecture is not None:
+                self._architectures[architecture] = config_type
             self._configs.setdefault(str(config_field), {})[config_type] = cls
             cls.model_type = getattr(cls, "model_type", None) or config_type
             return cls
@@ -84,6 +89,17 @@ class Registry:
         except KeyError:
             known = sorted(self._modules.get(task, {}))
             raise KeyError(f"no {task} module registered for model_type {model_type!r}; known: {known}") from None
+
+    def model_type_of(self, config: dict) -> str:
+        """Model type of a checkpoint configuration: its ``model_type``, or the type registered for the architecture it
+        names."""
+        if config.get("model_type"):
+            return config["model_type"]
+        names = [config.get("architecture"), *(config.get("architectures") or ())]
+        for n in names:
+            if n in self._architectures:
+                return self._architectures[n]
+        raise KeyError(f"the configuration names no model_type and no known architecture (found {names})")
 
     def alias(self, alias: str, target: str) -> None:
         """Makes ``alias`` resolve to everything registered as ``target``: composite checkpoints name their halves

@@ -19,6 +19,10 @@ class EasyGenerationMixin:
         from ...caching.transformer import TransformerCache
 
         spec = getattr(self, "spec", None)
+        if spec is not None and getattr(spec, "residual_f32", False):
+            from ...caching.paged import PagedBatchCache
+
+            return PagedBatchCache.for_model(self, batch_size, max_length)
         if spec is not None and getattr(spec, "mla", None) is not None:
             from ...layers.mla import MLACache
 

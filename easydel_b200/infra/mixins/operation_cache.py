@@ -46,6 +46,7 @@ class LayerOperationInfo:
     chunk_size: int | None = None
     num_kv_heads: int = 0
     head_dim: int = 0
+    v_head_dim: int = 0                   # 0 = values are as wide as keys
 
     @property
     def is_attention_layer(self) -> bool:
@@ -139,7 +140,7 @@ class OperationsCacheInfo:
         """Average bytes of keys + values kept per token of a ``context``-token sequence, over all layers."""
         total = 0
         for l in self.layers:
-            total += 2 * l.tokens_kept(context) * l.num_kv_heads * l.head_dim * element_size
+            total += l.tokens_kept(context) * l.num_kv_heads * (l.head_dim + (l.v_head_dim or l.head_dim)) * element_size
         return total / max(1, context)
 
 
@@ -149,7 +150,9 @@ class OperationCacheMixin:
     def _decoder_layers(self):
         backbone = getattr(self, "language_model", self)
         backbone = getattr(backbone, "model", backbone)
-        return list(getattr(backbone, "layers", ()))
+        layers = list(getattr(backbone, "layers", ()))
+        runs = getattr(backbone, "layer_runs", None)      # looped layers: one entry per run, each with its own cache
+        return layers if runs is None else [layers[i] for i in runs]
 
     def get_operations_cache_info(self, mode: ExecutionMode = ExecutionMode.MIXED) -> OperationsCacheInfo:
         infos: list[LayerOperationInfo] = []
@@ -204,7 +207,7 @@ def _describe_layer(i: int, layer) -> list[LayerOperationInfo]:
                                       CacheType.RECURRENT | CacheType.HYBRID, False, True))
         return out
     if getattr(layer, "is_linear", False):
-        name = "kimi_delta_attention" if ltype == "kda" else "gated_delta_rule"
+        name = {"kda": "kimi_delta_attention", "hgrn2": "hgrn2"}.get(ltype, "gated_delta_rule")
         out.append(LayerOperationInfo(i, "linear_attention", name, None, None, CacheType.RECURRENT | CacheType.HYBRID,
                                       False, True))
         return out
@@ -218,8 +221,13 @@ def _describe_layer(i: int, layer) -> list[LayerOperationInfo]:
         chunk = getattr(attn, "chunk_size", None) or None
         kind = "sliding_attention" if window else ("chunked_attention" if chunk else "full_attention")
         out.append(LayerOperationInfo(i, kind, "flash_attention", "paged_decode_attention",
-                                      0 if hasattr(layer, "mamba") else None, paged, True, False, window, chunk,
-                                      getattr(attn, "num_kv_heads", 0), getattr(attn, "head_dim", 0)))
+                                      0 if hasattr(layer, "mamba") or getattr(layer, "shift", None) is not None
+                                      else None, paged, True, False, window, chunk,
+                                      getattr(attn, "num_kv_heads", 0), getattr(attn, "head_dim", 0),
+                                      getattr(attn, "v_head_dim", 0)))
+    if getattr(layer, "shift", None) is not None:         # the previous token's normalised row, per sequence
+        out.append(LayerOperationInfo(i, "token_shift", "norm_shift", None, 1, CacheType.RECURRENT | CacheType.HYBRID,
+                                      False, True))
     if hasattr(layer, "mamba"):
         out.append(LayerOperationInfo(i, "ssm", "ssd_scan", None, 1, CacheType.RECURRENT | CacheType.HYBRID, False,
                                       True))

@@ -254,7 +254,8 @@ def load_config(path: str, config_kwargs: dict | None = None, **overrides):
     _ensure_models_imported()
     with open(os.path.join(path, CONFIG_NAME), encoding="utf-8") as f:
         d = json.load(f)
-    mtype = d.pop("model_type")
+    mtype = registry.model_type_of(d)
+    d.pop("model_type", None)
     for k in ("architectures", "transformers_version", "torch_dtype", "dtype"):
         d.pop(k, None) if k != "architectures" else None
     arch = d.pop("architectures", None)

@@ -20,7 +20,7 @@ import typing as tp
 import torch
 from torch import nn
 
-from ..ops import functional as F
+from ..ops import functional as F, stream
 from .linears import ColumnParallelLinear, RowParallelLinear
 from .norms import LayerNorm, RMSNorm
 from .rotary import get_rope
@@ -60,7 +60,8 @@ class Attention(nn.Module):
                  clip_qkv: float | None = None, dtype: torch.dtype = torch.float32, init_std: float = 0.02,
                  tp_size: int = 1, tp_rank: int = 0, tp_group=None, qk_norm_offset: float = 0.0,
                  output_gate: bool = False, chunk_size: int | None = None,
-                 temp_tuning: tuple[float, float] | None = None, head_scale_init: float | None = None):
+                 temp_tuning: tuple[float, float] | None = None, head_scale_init: float | None = None,
+                 v_head_dim: int | None = None, norm_dtype: torch.dtype | None = None):
         super().__init__()
         # GIDD: one learned multiplier per query head on top of ``scale`` (with L2-normalised q / k it is the whole
         # temperature of the head)
@@ -84,24 +85,25 @@ class Attention(nn.Module):
         self.num_heads = num_heads // tp_size
         self.num_kv_heads = max(1, num_kv_heads // tp_size)
         self.head_dim = head_dim
+        self.v_head_dim = v_head_dim or head_dim       # value heads may have a width of their own
         self.tp_size, self.tp_rank = tp_size, tp_rank
         self.sliding_window = sliding_window
         self.softcap = softcap
         self.causal = causal
         self.clip_qkv = clip_qkv
         self.scale = scale if scale is not None else 1.0 / math.sqrt(head_dim)
-        kv_out = num_kv_heads * head_dim if not self.kv_replicated else self.num_kv_heads * head_dim * tp_size
-        self.qkv_proj = ColumnParallelLinear(hidden_size, (num_heads * head_dim * (2 if output_gate else 1), kv_out,
-                                                           kv_out), bias=bias,
+        kv_heads = num_kv_heads if not self.kv_replicated else self.num_kv_heads * tp_size
+        self.qkv_proj = ColumnParallelLinear(hidden_size, (num_heads * head_dim * (2 if output_gate else 1),
+                                                           kv_heads * head_dim, kv_heads * self.v_head_dim), bias=bias,
                                              dtype=dtype, init_std=init_std, tp_size=tp_size, tp_rank=tp_rank,
                                              tp_group=tp_group)
-        self.o_proj = RowParallelLinear(num_heads * head_dim, hidden_size, bias=o_bias, dtype=dtype,
+        self.o_proj = RowParallelLinear(num_heads * self.v_head_dim, hidden_size, bias=o_bias, dtype=dtype,
                                         init_std=init_std, tp_size=tp_size, tp_rank=tp_rank, tp_group=tp_group)
         self.qkv_proj.remat_name, self.o_proj.remat_name = "attn_qkv", "attn_output"
         self.qk_norm, self.qk_norm_eps = qk_norm, qk_norm_eps
         if qk_norm == "rms_head":      # per-head RMSNorm over head_dim (Qwen3, Gemma3, OLMo... per-head flavour)
-            self.q_norm = RMSNorm(head_dim, qk_norm_eps, dtype, offset=qk_norm_offset)
-            self.k_norm = RMSNorm(head_dim, qk_norm_eps, dtype, offset=qk_norm_offset)
+            self.q_norm = RMSNorm(head_dim, qk_norm_eps, norm_dtype or dtype, offset=qk_norm_offset)
+            self.k_norm = RMSNorm(head_dim, qk_norm_eps, norm_dtype or dtype, offset=qk_norm_offset)
         elif qk_norm == "rms_full":    # RMSNorm over the whole projection (OLMo2, Cohere-style full width)
             self.q_norm = RMSNorm(self.num_heads * head_dim, qk_norm_eps, dtype)
             self.k_norm = RMSNorm(self.num_kv_heads * head_dim, qk_norm_eps, dtype)
@@ -214,6 +216,34 @@ class Attention(nn.Module):
         if gate is not None:
             o = o * torch.sigmoid(gate)
         return self.o_proj(o)
+
+    def mix_stream(self, h: torch.Tensor, step, cache_view=None) -> torch.Tensor:
+        """Form for layers over an fp32 residual stream: h ``[T, hidden]`` (all sequences on one axis) ->
+        ``[T, heads * v_head_dim]`` before the output projection, which the layer accumulates into the stream. Per-head
+        q / k norms, the query temperature and the page append are one kernel over the packed projection. ``step``:
+        :class:`..modules._base.decoder.StreamStep`."""
+        if self.rotary is not None or self.alibi is not None or self.output_gate or self.clip_qkv is not None or \
+                self.head_scale is not None or self.chunk_size or self.qk_norm not in (None, "rms_head"):
+            raise NotImplementedError("fp32-stream attention covers plain, per-head-normed and tempered heads")
+        qkv = stream.linear(h, self.qkv_proj.weight, self.qkv_proj.bias)
+        T = h.shape[0]
+        Hq, Hkv, D, Dv = self.num_heads, self.num_kv_heads, self.head_dim, self.v_head_dim
+        qw, kw = (self.q_norm.weight, self.k_norm.weight) if self.qk_norm else (None, None)
+        if cache_view is not None:
+            q = stream.qkv_prologue(qkv, (Hq, Hkv, D, Dv), qw, kw, self.qk_norm_eps, step.positions, self.temp_tuning,
+                                    step.meta.slots_of(cache_view.group), cache_view.k_pages, cache_view.v_pages)
+            return cache_view.attend_pages(self, q, step.meta).reshape(T, Hq * Dv)
+        # no cache (autograd): the batch's rows are equally long
+        from ..ops import reference as R
+
+        q, k, v = torch.split(qkv, [Hq * D, Hkv * D, Hkv * Dv], -1)
+        q, k = stream.qk_norm_temper(q.reshape(T, Hq, D), k.reshape(T, Hkv, D), qw, kw, self.qk_norm_eps,
+                                     step.positions, self.temp_tuning)
+        B = step.batch
+        o = R.attention(q.view(B, T // B, Hq, D), k.view(B, T // B, Hkv, D), v.reshape(B, T // B, Hkv, Dv),
+                        causal=self.causal, scale=self.scale, segment_ids=step.segment_ids,
+                        sliding_window=self.sliding_window, softcap=self.softcap, sinks=self.sinks)
+        return o.reshape(T, Hq * Dv)
 
     def _alibi_attention(self, q, k, v, segment_ids):
         # ALiBi families (Falcon-RW, MPT, BLOOM-style) are served by the dense oracle path: a

@@ -5,7 +5,7 @@ from __future__ import annotations
 import torch
 from torch import nn
 
-from ..ops import functional as F
+from ..ops import functional as F, stream
 from ..ops.reference import ACT2FN
 from .linears import ColumnParallelLinear, RowParallelLinear
 
@@ -52,6 +52,13 @@ class PlainMLP(nn.Module):
         self.fc2 = RowParallelLinear(intermediate_size, hidden_size, bias=bias, dtype=dtype, init_std=init_std,
                                      tp_size=tp_size, tp_rank=tp_rank, tp_group=tp_group)
         self.fc1.remat_name, self.fc2.remat_name = "mlp_gate_up", "mlp_down"
+        if act == "xielu":        # two learned numbers, kept (and evaluated) in fp32
+            self.act_params = nn.Parameter(torch.tensor([0.3, 0.3], dtype=torch.float32))
+
+    def hidden(self, x: torch.Tensor) -> torch.Tensor:
+        """The activations between the two products."""
+        z = self.fc1(x)
+        return stream.xielu(z, self.act_params) if self.act == "xielu" else ACT2FN[self.act](z)
 
     def forward(self, x: torch.Tensor) -> torch.Tensor:
-        return self.fc2(ACT2FN[self.act](self.fc1(x)))
+        return self.fc2(self.hidden(x))

@@ -40,6 +40,8 @@ from . import kimi_vl  # noqa: F401
 from .kimi_vl import *  # noqa: F401,F403
 from . import llama4  # noqa: F401
 from .llama4 import *  # noqa: F401,F403
+from . import rakevik  # noqa: F401
+from .rakevik import *  # noqa: F401,F403
 
 # The halves of composite checkpoints under the model types their own configs carry.
 from ..infra.factory import registry as _registry  # noqa: E402

@@ -20,6 +20,7 @@ import torch
 from torch import nn
 from torch.utils.checkpoint import checkpoint
 
+from ...caching.paged import PagedBatchCache, PagedBatchMeta
 from ...infra.base_module import EasyDeLBaseModule
 from ...infra.loss_utils import (LossConfig, LossMetrics, ForSequenceClassificationLoss,
                                  auxiliary_load_balancing_loss_func, causal_lm_loss_from_hidden)
@@ -31,7 +32,7 @@ from ...layers.linears import ColumnParallelLinear
 from ...layers.mlp import GatedMLP, PlainMLP
 from ...layers.moe import MoEBlock
 from ...layers.norms import LayerNorm, RMSNorm
-from ...ops import functional as F
+from ...ops import functional as F, stream
 
 
 @dataclass
@@ -126,11 +127,42 @@ class ArchSpec:
     ssm_branch: dict | None = None    # kwargs of layers.ssm_branch.SSDMixer: a Mamba-2 mixer beside attention (Falcon-H1)
     branch_multipliers: tuple[float, float, float] = (1.0, 1.0, 1.0)  # attention input, attention output, SSM output
     mlp_multipliers: tuple[float, float] = (1.0, 1.0)                  # gate pre-activation, MLP output
+    residual_f32: bool = False        # the residual stream is fp32 [tokens, hidden]; branches accumulate into it
+    token_shift: bool = False         # every mixer reads h + (h of the previous token - h) * shift (fp32-stream models)
+    v_head_dim: int | None = None     # width of a value head when it differs from head_dim (fp32-stream models)
+    hgrn2: dict | None = None         # heads / dim / vdim of layers.hgrn2.HGRN2Mixer for layers of type "hgrn2"
+    loop: tuple[int, int, int] | None = None  # (start, stop, times): layers start .. stop-1 run ``times`` times in a row
+                                      # with the same weights, each run with a cache of its own; before a pass the
+                                      # stream becomes W [x ; embedding output] + step[pass] (fp32-stream models)
     residual_mlp: bool = False        # Arctic: MoE layers add a dense hidden-sized MLP branch after attention while
                                       # the experts read the layer input (norm of x, not of x + attention)
 
 
+@dataclass
+class StreamStep:
+    """What the layers of an fp32-stream model need to know about the running step: all sequences lie on one token axis."""
+
+    cu: torch.Tensor                      # int32 [B + 1] sequence bounds
+    positions: torch.Tensor               # int32 [T]
+    max_len: int                          # longest sequence of the step
+    batch: int
+    slots: torch.Tensor | None = None     # int32 [B] state rows of the sequences
+    meta: tp.Any = None                   # PagedBatchMeta, with a paged cache
+    segment_ids: torch.Tensor | None = None
+
+
+@dataclass
+class LayerSlotState:
+    """Per-slot state of one layer run of an fp32-stream model, read and written in place by its kernels."""
+
+    shift: torch.Tensor | None            # fp32 [slots, hidden]: the previous token's normalised row
+    recurrent: torch.Tensor | None        # fp32 [slots, heads, dim, vdim]: HGRN2
+    in_place: tp.ClassVar[bool] = True
+
+
 def _norm(spec: ArchSpec, dtype) -> nn.Module:
+    if spec.residual_f32:
+        return RMSNorm(spec.hidden_size, spec.norm_eps, torch.float32)
     if spec.norm == "rms":
         return RMSNorm(spec.hidden_size, spec.norm_eps, dtype, offset=spec.norm_offset)
     if spec.norm == "layer_noparam":
@@ -170,7 +202,10 @@ class DecoderLayer(nn.Module):
             rope = spec.rope_local
         if ltype == "nope":
             rope = None
-        self.is_linear = ltype in ("linear", "lightning", "kda")
+        self.is_linear = ltype in ("linear", "lightning", "kda", "hgrn2")
+        if spec.residual_f32 and tp_size > 1:
+            raise NotImplementedError("models with an fp32 residual stream run with tensor parallelism 1")
+        self.shift = nn.Parameter(torch.zeros(spec.hidden_size, dtype=torch.float32)) if spec.token_shift else None
         self.ltype = ltype
         if ltype == "lightning":
             from ...layers.lightning_attention import LightningAttention
@@ -178,6 +213,11 @@ class DecoderLayer(nn.Module):
             self.self_attn = LightningAttention(spec.hidden_size, spec.num_heads, spec.head_dim, spec.num_layers,
                                                 act=spec.act, layer_idx=layer_idx,
                                                 dtype=dtype, init_std=spec.init_std, **spec.lightning)
+        elif ltype == "hgrn2":
+            from ...layers.hgrn2 import HGRN2Mixer
+
+            self.linear_attn = HGRN2Mixer(spec.hidden_size, layer_idx=layer_idx, dtype=dtype, init_std=spec.init_std,
+                                          norm_eps=spec.norm_eps, **spec.hgrn2)
         elif ltype == "kda":
             from ...layers.linear_attention import KimiDeltaAttention
 
@@ -229,7 +269,8 @@ class DecoderLayer(nn.Module):
             sliding_window=window, softcap=spec.attn_softcap, scale=spec.attn_scale, use_sinks=spec.use_sinks,
             use_alibi=spec.pos_emb == "alibi", clip_qkv=spec.clip_qkv, dtype=dtype, init_std=spec.init_std,
             tp_size=tp_size, tp_rank=tp_rank, tp_group=tp_group, qk_norm_offset=spec.norm_offset,
-            output_gate=spec.attn_output_gate)
+            output_gate=spec.attn_output_gate, v_head_dim=spec.v_head_dim,
+            norm_dtype=torch.float32 if spec.residual_f32 else None)
 
     def _build_mlp(self, config, spec, layer_idx, dtype, tp_size, tp_rank, tp_group):
         moe = spec.moe
@@ -252,6 +293,8 @@ class DecoderLayer(nn.Module):
                                 expert_init_std=moe.expert_init_std, ep_size=ep_size, ep_rank=ep_rank,
                                 ep_group=ep_group, tp_size=tp_size, tp_rank=tp_rank, tp_group=tp_group,
                                 expert_tensor_mode=bool(getattr(config, "use_expert_tensor_mode", False)))
+        elif spec.intermediate_size == 0:      # a layer with a mixer only
+            self.mlp = None
         elif spec.mlp == "gated":
             self.mlp = GatedMLP(spec.hidden_size, spec.intermediate_size, spec.act, spec.mlp_bias, dtype,
                                 spec.init_std, tp_size, tp_rank, tp_group)
@@ -268,6 +311,8 @@ class DecoderLayer(nn.Module):
             self.post_feedforward_layernorm = _norm(spec, dtype)
         else:
             self.input_layernorm = _norm(spec, dtype)
+            if self.mlp is None:
+                return
             if (spec.residual == "pre" and not spec.sandwich_norm) or \
                     (spec.residual == "parallel" and not spec.shared_parallel_norm):
                 self.post_attention_layernorm = _norm(spec, dtype)
@@ -298,8 +343,39 @@ class DecoderLayer(nn.Module):
                 state.commit()
         return self.self_attn(h, positions, segment_ids=segment_ids, cache_view=cache_view, attn_meta=attn_meta)
 
+    def make_slot_state(self, num_slots: int, device) -> LayerSlotState | None:
+        """State pool of this layer for ``num_slots`` sequences (fp32-stream models; None for the others)."""
+        spec = self.spec
+        if not spec.residual_f32 or (self.shift is None and self.ltype != "hgrn2"):
+            return None
+        zeros = lambda *s: torch.zeros(num_slots, *s, dtype=torch.float32, device=device)  # noqa: E731
+        m = self.linear_attn if self.ltype == "hgrn2" else None
+        return LayerSlotState(zeros(spec.hidden_size) if self.shift is not None else None,
+                              zeros(m.heads, m.dim, m.vdim) if m is not None else None)
+
+    def _forward_stream(self, x: torch.Tensor, step: StreamStep, view):
+        """One layer on the fp32 stream ``x [T, hidden]``: norm (+ token shift) -> mixer -> the output projection
+        accumulates into the stream; then norm -> MLP likewise."""
+        spec = self.spec
+        mixer = self.linear_attn if self.ltype == "hgrn2" else self.self_attn
+        dt = mixer.o_proj.weight.dtype
+        state = view.linear_state if view is not None else None
+        h = stream.norm_shift(x, self.input_layernorm.weight, spec.norm_eps, dt, mu=self.shift, cu=step.cu,
+                              slots=step.slots, state=None if state is None else state.shift)
+        if self.ltype == "hgrn2":
+            o = mixer(h, step, None if state is None else state.recurrent)
+        else:
+            o = mixer.mix_stream(h, step, view)
+        x = stream.linear_add_(x, o, mixer.o_proj.weight)
+        if self.mlp is not None:
+            h = stream.norm_shift(x, self.post_attention_layernorm.weight, spec.norm_eps, dt)
+            x = stream.linear_add_(x, self.mlp.hidden(h), self.mlp.fc2.weight)
+        return x
+
     def forward(self, x, pending, positions, segment_ids=None, cache_view=None, attn_meta=None):
         spec = self.spec
+        if spec.residual_f32:
+            return self._forward_stream(x, attn_meta, cache_view), None, None
         rl = None
         fused = spec.norm == "rms" and spec.residual == "pre" and not spec.sandwich_norm \
             and spec.residual_multiplier is None and not self.has_residual_mlp
@@ -393,12 +469,20 @@ class DecoderModel(EasyDeLBaseModule):
         self.layers = nn.ModuleList([DecoderLayer(config, layer_spec(i), i, pd) for i in range(spec.num_layers)])
         if spec.final_norm:
             self.norm = _norm(spec, pd)
+        if spec.loop is not None:
+            lo, hi, times = spec.loop
+            self.layer_runs = [*range(lo), *(list(range(lo, hi)) * times), *range(hi, spec.num_layers)]
+            self.loop_in = ColumnParallelLinear(2 * spec.hidden_size, spec.hidden_size, bias=False, dtype=pd,
+                                                init_std=spec.init_std)
+            self.loop_step = nn.Parameter(torch.zeros(times, spec.hidden_size, dtype=pd))
         self._setup_sequence_parallel(config)
         self._setup_context_parallel(config)
 
     #: process group over which the sequence dimension of a batch is sharded (``attn_mechanism="ring"``), or None
     cp_group = None
     cp_layout = "zigzag"
+    #: layer index of every layer run, in order, when layers run several times (None: every layer once)
+    layer_runs: list[int] | None = None
 
     def _setup_context_parallel(self, config) -> None:
         """``attn_mechanism="ring"`` on a mesh whose ``sp`` axis is larger than one: every rank of the ``sp`` group
@@ -428,7 +512,8 @@ class DecoderModel(EasyDeLBaseModule):
         tp_size, _, tp_group = _tp_of(config)
         self._sp_group = tp_group
         plain = all(not l.is_moe and not l.is_linear and l.ltype != "lightning" and l.spec.mla is None
-                    and l.spec.ssm_branch is None and l.spec.normed_residual is None for l in self.layers)
+                    and l.spec.ssm_branch is None and l.spec.normed_residual is None and not l.spec.residual_f32
+                    for l in self.layers)
         self.sp_capable = bool(tp_size > 1 and plain and getattr(config, "tp_sequence_parallel", True))
         if self.sp_capable:
             for m in self.layers.modules():
@@ -465,6 +550,9 @@ class DecoderModel(EasyDeLBaseModule):
         ``sequence_parallel``: the caller takes ``last_hidden_state`` as this rank's row shard ``[1, B*T/tp, H]``
         (rows of the flattened ``[B*T]`` token axis) when ``self.sp.active`` is set on return."""
         spec = self.spec
+        if spec.residual_f32:
+            return self._forward_stream(input_ids, inputs_embeds, attention_mask, position_ids, segment_ids,
+                                        past_key_values, cache_metadata, output_hidden_states)
         if inputs_embeds is None:
             if input_ids.dim() == 1:
                 input_ids = input_ids[None]
@@ -539,6 +627,103 @@ class DecoderModel(EasyDeLBaseModule):
         return cls(**kw)
 
 
+def _stream_batch(self, shape, attention_mask, segment_ids, cache, metadata, device):
+    """Rows of a ``[B, T]`` batch as sequences on one token axis: (step, cache, index of the kept tokens or None).
+    Padding marked by ``attention_mask`` (or by the generation loop's segment ids) takes no part; without a cache the
+    batch gets a throw-away one, so that one set of kernels serves every caller outside autograd."""
+    B, T = shape
+    keep = attention_mask
+    if isinstance(metadata, dict) and metadata.get("kv_segment_ids") is not None:
+        s = cache.seq_len()
+        keep = metadata["kv_segment_ids"][:, s:s + T] != 0
+    if torch.is_grad_enabled() and cache is None:
+        if segment_ids is None and keep is not None and not bool(keep.all()):
+            segment_ids = keep.to(torch.int32)
+        cu = torch.arange(0, (B + 1) * T, T, dtype=torch.int32, device=device)
+        positions = torch.arange(T, device=device)[None].expand(B, T)
+        if segment_ids is not None:
+            from ...ops.attention import segment_ids_to_cu_seqlens
+
+            cu, _ = segment_ids_to_cu_seqlens(segment_ids)
+            positions = _positions_from_segments(segment_ids)
+        return StreamStep(cu, positions.reshape(-1).to(torch.int32), T, B, segment_ids=segment_ids), None, None
+    if segment_ids is not None:
+        raise NotImplementedError("packed segments run under autograd only: pass the documents as separate rows")
+    if cache is None:
+        cache = PagedBatchCache.for_model(self, B, T)
+    index, counts = None, [T] * B
+    if keep is not None and T > 1 and not bool(keep.all()):
+        index = keep.reshape(-1).nonzero().squeeze(1)
+        counts = keep.sum(1).tolist()
+    meta, positions = cache.begin([int(n) for n in counts])
+    return StreamStep(meta.cu_q, positions, meta.max_q, B, meta.slot_ids, meta), cache, index
+
+
+def _forward_stream(self, input_ids, inputs_embeds, attention_mask, position_ids, segment_ids, cache, metadata,
+                    output_hidden_states):
+    """Forward pass of a model with an fp32 residual stream: the tokens of all sequences on one axis, looped layers run
+    as often as they are listed in ``layer_runs``."""
+    spec = self.spec
+    ids = input_ids if input_ids is None or input_ids.dim() == 2 else input_ids[None]
+    B, T = ids.shape if ids is not None else inputs_embeds.shape[:2]
+    index = None
+    if isinstance(metadata, PagedBatchMeta):
+        step = StreamStep(metadata.cu_q, position_ids.reshape(-1).to(torch.int32), metadata.max_q, metadata.num_seqs,
+                          metadata.slot_ids, metadata)
+    else:
+        dev = ids.device if ids is not None else inputs_embeds.device
+        step, cache, index = _stream_batch(self, (B, T), attention_mask, segment_ids, cache, metadata, dev)
+    dt, W = self.dtype, spec.hidden_size
+    flat = None if ids is None else ids.reshape(-1)
+    if index is not None and flat is not None:
+        flat = flat[index]
+    n = flat.numel() if flat is not None else (index.numel() if index is not None else B * T)
+    operand = right = None
+    if spec.loop is not None:             # [x ; x0]: x0 is written once, x before every pass
+        operand = torch.empty(n, 2 * W, dtype=self.loop_in.weight.dtype, device=self.device)
+        right = operand[:, W:]
+    if inputs_embeds is None:
+        x = stream.embed(self.embed_tokens.weight, flat, right)
+    else:
+        x = inputs_embeds.reshape(B * T, W)
+        x = (x if index is None else x[index]).float()
+        if right is not None:
+            stream.cast_rows(x, right)
+        x = x.clone()
+    lo, hi, _ = spec.loop or (0, 0, 0)
+    hidden = [] if output_hidden_states else None
+    done = 0
+    for run, i in enumerate(self.layer_runs if self.layer_runs is not None else range(spec.num_layers)):
+        if spec.loop is not None and i == lo and lo <= run < lo + (hi - lo) * spec.loop[2]:
+            bias = self.loop_step[done]
+            if torch.is_grad_enabled():
+                x = stream.linear(torch.cat([x.to(dt), right], -1), self.loop_in.weight, bias, torch.float32)
+            else:
+                stream.cast_rows(x, operand[:, :W])
+                x = stream.linear(operand, self.loop_in.weight, bias, torch.float32)
+            done += 1
+        if hidden is not None:
+            hidden.append(x.clone())
+        view = cache.view(run) if cache is not None else None
+        x, _, _ = self.layers[i](x, None, step.positions, None, view, step)
+    x = stream.norm_shift(x, self.norm.weight, spec.norm_eps, dt)
+
+    def unflatten(t):
+        if index is not None:
+            full = t.new_zeros(B * T, W)
+            full[index] = t
+            t = full
+        return t.view(B, T, W)
+
+    x = unflatten(x)
+    if hidden is not None:
+        hidden = [*map(unflatten, hidden), x]
+    return BaseModelOutput(last_hidden_state=x, hidden_states=tuple(hidden) if hidden else None, past_key_values=cache)
+
+
+DecoderModel._forward_stream = _forward_stream
+
+
 def _positions_from_segments(segment_ids: torch.Tensor) -> torch.Tensor:
     """Positions restart at 0 at every segment boundary of a packed row."""
     B, T = segment_ids.shape
@@ -581,6 +766,10 @@ class DecoderForCausalLM(EasyDeLBaseModule):
 
     def apply_lm_head(self, hidden: torch.Tensor) -> torch.Tensor:
         spec = self.spec
+        if spec.residual_f32:      # the head's accumulators are the logits: no 16-bit rounding of them
+            out = stream.linear(hidden.reshape(-1, hidden.shape[-1]), self.lm_head_weight(), self.lm_head_bias(),
+                                torch.float32)
+            return out.view(*hidden.shape[:-1], out.shape[-1])
         logits = F.linear(hidden, self.lm_head_weight(), self.lm_head_bias())
         if spec.logit_scale is not None:
             logits = logits * spec.logit_scale

@@ -24,7 +24,8 @@ def _read_model_type(path: str) -> tuple[str, list[str] | None]:
     path = _resolve_dir(path)
     with open(os.path.join(path, CONFIG_NAME), encoding="utf-8") as f:
         d = json.load(f)
-    return d["model_type"], d.get("architectures")
+    _ensure_models_imported()
+    return registry.model_type_of(d), d.get("architectures")
 
 
 def resolve_model_class(path: str, task: TaskType = TaskType.CAUSAL_LM):

@@ -33,7 +33,7 @@ _SIGS = {
     "edl_sm_count": (i32, []),
     "edl_abi_version": (i32, []),
     "edl_gemm_bf16": (i32, [vp, vp, vp, vp, i32, i32, i32, i64, i64, i64, i32, i32, i32, vp, vp, i32, i32]),
-    "edl_gemm_splitk": (i32, [vp, vp, vp, vp, i32, i32, i32, i64, i64, i64, i32, vp, vp, vp, vp]),
+    "edl_gemm_splitk": (i32, [vp, vp, vp, vp, i32, i32, i32, i64, i64, i64, i32, vp, vp, i32, vp, vp]),
     "edl_gemm_pair_splitk": (i32, [vp, vp, vp, vp, i32, i32, i32, i64, i64, i64, i32, vp, vp, vp, vp]),
     "edl_gemm_pair_splitk_workspace": (i64, [i32, i32]),
     "edl_rmsnorm_fwd": (i32, [vp, vp, vp, vp, vp, vp, i32, i32, f32, f32, vp]),
@@ -56,6 +56,15 @@ _SIGS = {
 
 def lib_path() -> Path:
     return _LIB_PATH
+
+
+def use_library(path) -> None:
+    """Names the library file to load (before anything is loaded)."""
+    global _LIB_PATH
+    if _lib is None:
+        _LIB_PATH = Path(path)
+    elif Path(path) != _LIB_PATH:
+        raise RuntimeError(f"{_LIB_PATH} is loaded already")
 
 
 def _load():

@@ -63,6 +63,10 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = None,
     """y = x @ w.T + bias with ``w`` in torch Linear layout ``[out, in]``. ``name``: the activation-checkpoint
     name of this product (see :mod:`.remat`)."""
     if _lib.use_kernels(x):
+        if x.dtype == torch.float32:
+            from . import stream      # an all-fp32 model: true 32-bit products
+
+            return stream.linear(_as_2d(x), w, bias).view(*x.shape[:-1], w.shape[0])
         if x.dtype != torch.bfloat16:
             raise TypeError(f"GPU linear expects bf16 activations, got {x.dtype}")
         if (w.shape[0] % 8) or (w.shape[1] % 8):

@@ -161,12 +161,12 @@ def gemm(a: torch.Tensor, b: torch.Tensor, *, a_mn: bool = False, b_mn: bool = F
     if not (a_mn or b_mn or accumulate or max_ctas or force_bn) and out.dtype == torch.bfloat16 \
             and _pair128_plan(M, N, K, a.device):
         force_bn = 384
-    if not (a_mn or b_mn or accumulate or max_ctas or force_bn) and out.dtype == torch.bfloat16:
+    if not (a_mn or b_mn or max_ctas or force_bn) and (out.dtype == torch.float32 or not accumulate):
         splits = _splitk_plan(M, N, K, a.device)
         if splits > 1:
             ws = torch.empty((splits, M, N), dtype=torch.float32, device=a.device)
             _lib.call("edl_gemm_splitk", a.data_ptr(), b.data_ptr(), out.data_ptr(), _lib.ptr(bias), M, N, K, lda, ldb,
-                      ldc, splits, ws.data_ptr(), _splitk_offsets(K, splits, a.device).data_ptr(),
+                      ldc, splits, ws.data_ptr(), _splitk_offsets(K, splits, a.device).data_ptr(), flags,
                       _lib.status_word(a.device).data_ptr(), _lib.stream_ptr())
             return out
     _lib.call("edl_gemm_bf16", a.data_ptr(), b.data_ptr(), out.data_ptr(), _lib.ptr(bias), M, N, K, lda, ldb, ldc,

@@ -9,16 +9,17 @@ import torch
 from . import _lib
 
 vp, i32, i64, f32 = _lib.vp, _lib.i32, _lib.i64, _lib.f32
-_lib.register("edl_attn_paged_lse", i32, [vp, vp, vp, vp, vp, i64, i64, i64, vp, vp, vp, i32, i32, i32, i64, i64, i32,
-                                          i32, i32, _lib.f32, i32, i32, _lib.f32, vp, vp, vp])
+_lib.register("edl_attn_paged_lse", i32, [vp, vp, vp, vp, vp, i64, i64, i64, i64, vp, vp, vp, i32, i32, i32, i64, i64,
+                                          i32, i32, i32, i32, _lib.f32, i32, i32, _lib.f32, vp, vp, vp])
 _lib.register("edl_attn_combine", i32, [vp, i64, vp, i32, i32, i32, i32, vp, vp, vp, vp])
-_lib.register("edl_attn_paged", i32, [vp, vp, vp, vp, i64, i64, i64, vp, vp, vp, i32, i32, i32, i64, i64, i32, i32,
-                                      i32, f32, i32, i32, f32, vp, vp, vp])
+_lib.register("edl_attn_paged", i32, [vp, vp, vp, vp, i64, i64, i64, i64, vp, vp, vp, i32, i32, i32, i64, i64, i32, i32,
+                                      i32, i32, f32, i32, i32, f32, vp, vp, vp])
 _lib.register("edl_paged_kv_append", i32, [vp, vp, vp, vp, vp, i32, i32, i64, i64, i64, i64, vp, vp])
 _lib.register("edl_sample", i32, [vp, i32, i64, i32, i32, vp, vp, vp, vp, vp, vp, vp, vp, i64, vp, vp, vp, vp, vp])
 _lib.register("edl_count_update", i32, [vp, i64, vp, vp, i32, i32, vp])
 _lib.register("edl_gather_rows", i32, [vp, vp, vp, i32, i32, i64, vp])
-_lib.register("edl_attn_decode", i32, [vp, vp, vp, vp, vp, i64, i64, i64, vp, vp, i32, i32, i64, i32, i32, i32, f32,
+_lib.register("edl_attn_decode", i32, [vp, vp, vp, vp, vp, i64, i64, i64, i64, vp, vp, i32, i32, i64, i32, i32, i32, i32,
+                                       f32,
                                        i32, i32, vp, vp, vp])
 
 _lib.register("edl_attn_mla_decode", i32, [vp, vp, vp, vp, i64, i64, vp, vp, i32, i32, i64, i32, f32, i32, vp, vp])
@@ -32,6 +33,7 @@ def kv_append(k: torch.Tensor, v: torch.Tensor, k_pages: torch.Tensor, v_pages: 
     T = k.shape[0]
     width = k.shape[-2] * k.shape[-1]
     if k.is_cuda:
+        assert v.shape == k.shape, "keys and values of different widths are appended by stream.qkv_prologue"
         assert k.stride(-1) == 1 and k.stride(-2) == k.shape[-1] and v.stride(-2) == v.shape[-1]
         ld_page = k_pages.stride(1)
         _lib.call("edl_paged_kv_append", k.data_ptr(), v.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(),
@@ -52,43 +54,76 @@ def paged_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tenso
                     out: torch.Tensor | None = None) -> torch.Tensor:
     """Mixed prefill/decode attention over a paged KV cache.
 
-    q ``[T, Hq, D]`` (new tokens of all sequences, concatenated), pages ``[P, 128, Hkv, D]``,
-    ``cu_q`` int32 ``[B+1]``, ``kv_lens`` int32 ``[B]`` (cached + new keys), ``page_table`` int32 ``[B, maxP]``.
+    q ``[T, Hq, D]`` (new tokens of all sequences, concatenated), key pages ``[P, 128, Hkv, D]``, value pages
+    ``[P, 128, Hkv, Dv]`` (``Dv`` may differ from ``D``), ``cu_q`` int32 ``[B+1]``, ``kv_lens`` int32 ``[B]`` (cached +
+    new keys), ``page_table`` int32 ``[B, maxP]``. Layouts outside :func:`paged_kernel_supports` (32-bit floats,
+    heads wider than 128) run the plain SIMT kernel.
     """
     T, Hq, D = q.shape
-    Hkv = k_pages.shape[2]
+    Hkv, Dv = k_pages.shape[2], v_pages.shape[-1]
     B = kv_lens.numel()
     scale = scale if scale is not None else 1.0 / math.sqrt(D)
+    if q.is_cuda and not paged_kernel_supports(q, k_pages, v_pages):
+        if not causal or softcap:
+            raise NotImplementedError("the SIMT attention kernel is causal and has no soft-cap")
+        return simt_attention(q, k_pages, v_pages, cu_q, kv_lens, page_table, scale=scale, window=window, sinks=sinks,
+                              out=out)
     if q.is_cuda:
         assert k_pages.shape[1] == PAGE_SIZE, "the paged kernels use pages of 128 tokens"
         assert q.stride(-1) == 1 and q.stride(-2) == D
         if out is None:
-            out = torch.empty((T, Hq, D), dtype=q.dtype, device=q.device)
+            out = torch.empty((T, Hq, Dv), dtype=q.dtype, device=q.device)
         _lib.call("edl_attn_paged", q.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), out.data_ptr(),
-                  q.stride(0), k_pages.stride(1), out.stride(0), cu_q.data_ptr(), kv_lens.data_ptr(),
-                  page_table.data_ptr(), page_table.stride(0), B, int(max_q), T, k_pages.shape[0], Hq, Hkv, D,
-                  float(scale), int(causal), int(window or 0), float(softcap or 0.0), _lib.ptr(sinks),
+                  q.stride(0), k_pages.stride(1), v_pages.stride(1), out.stride(0), cu_q.data_ptr(),
+                  kv_lens.data_ptr(), page_table.data_ptr(), page_table.stride(0), B, int(max_q), T, k_pages.shape[0],
+                  Hq, Hkv, D, Dv, float(scale), int(causal), int(window or 0), float(softcap or 0.0), _lib.ptr(sinks),
                   _lib.status_word(q.device).data_ptr(), _lib.stream_ptr())
         return out
     return paged_attention_reference(q, k_pages, v_pages, cu_q, kv_lens, page_table, scale=scale, causal=causal,
                                      window=window, softcap=softcap, sinks=sinks)
 
 
+_lib.register("edl_attn_simt", i32, [vp, vp, vp, vp, i32, i64, i64, i64, vp, vp, vp, i32, i32, i32, i64, i32, i32, i32, i32,
+                                     f32, i32, vp, vp, vp])
+
+
+def simt_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, cu_q: torch.Tensor,
+                   kv_lens: torch.Tensor, page_table: torch.Tensor, *, scale: float, window: int = 0, sinks=None,
+                   out: torch.Tensor | None = None) -> torch.Tensor:
+    """Causal paged attention in fp32 arithmetic (``csrc/attention_simt.cu``): fp32 models, and head sizes outside the
+    tensor-core kernels'. Arguments as :func:`paged_attention`."""
+    T, Hq, D = q.shape
+    Hkv, Dv = k_pages.shape[2], v_pages.shape[-1]
+    if q.dtype != k_pages.dtype or q.dtype != v_pages.dtype or q.dtype not in (torch.bfloat16, torch.float32):
+        raise TypeError(f"queries and pages must share one type (bf16 or fp32), got {q.dtype} / {k_pages.dtype}")
+    assert k_pages.shape[1] == PAGE_SIZE and q.stride(-1) == 1 and q.stride(-2) == D
+    if out is None:
+        out = torch.empty((T, Hq, Dv), dtype=q.dtype, device=q.device)
+    assert out.is_contiguous()
+    _lib.call("edl_attn_simt", q.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), out.data_ptr(),
+              int(q.dtype == torch.float32), q.stride(0), k_pages.stride(1), v_pages.stride(1), cu_q.data_ptr(),
+              kv_lens.data_ptr(), page_table.data_ptr(), page_table.stride(0), kv_lens.numel(), T, k_pages.shape[0], Hq,
+              Hkv, D, Dv, float(scale), int(window or 0), _lib.ptr(sinks), _lib.status_word(q.device).data_ptr(),
+              _lib.stream_ptr())
+    return out
+
+
 def decode_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, kv_lens: torch.Tensor,
                      page_table: torch.Tensor, *, scale: float | None = None, window: int = 0, sinks=None,
                      num_splits: int = 1) -> torch.Tensor:
     """Decode-step attention (one query token per sequence) with the streaming kernel of
-    ``csrc/attention_decode.cu``. q ``[B, Hq, D]``; pages ``[P, 128, Hkv, D]``; ``num_splits`` cuts every
+    ``csrc/attention_decode.cu``. q ``[B, Hq, D]``; pages ``[P, 128, Hkv, D]`` (values may have another width than
+    keys); ``num_splits`` cuts every
     sequence's keys into that many parts that run as separate CTAs and are merged by :func:`attn_combine`."""
     B, Hq, D = q.shape
-    Hkv = k_pages.shape[2]
+    Hkv, Dv = k_pages.shape[2], v_pages.shape[-1]
     scale = scale if scale is not None else 1.0 / math.sqrt(D)
     S_ = max(1, int(num_splits))
-    out = torch.empty((S_, B, Hq, D), dtype=q.dtype, device=q.device)
+    out = torch.empty((S_, B, Hq, Dv), dtype=q.dtype, device=q.device)
     lse = torch.empty((S_, Hq, B), dtype=torch.float32, device=q.device) if S_ > 1 else None
     _lib.call("edl_attn_decode", q.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), out.data_ptr(), _lib.ptr(lse),
-              q.stride(0), k_pages.stride(1), Hq * D, kv_lens.data_ptr(), page_table.data_ptr(),
-              page_table.stride(0), B, k_pages.shape[0], Hq, Hkv, D, float(scale), int(window or 0), S_,
+              q.stride(0), k_pages.stride(1), v_pages.stride(1), Hq * Dv, kv_lens.data_ptr(), page_table.data_ptr(),
+              page_table.stride(0), B, k_pages.shape[0], Hq, Hkv, D, Dv, float(scale), int(window or 0), S_,
               _lib.ptr(sinks) if S_ == 1 else None, _lib.status_word(q.device).data_ptr(), _lib.stream_ptr())
     if S_ == 1:
         return out[0]
@@ -120,11 +155,21 @@ def mla_decode_kernel_supports(q: torch.Tensor, pages: torch.Tensor) -> bool:
             and pages.shape[-1] == 576 and pages.shape[1] == PAGE_SIZE and pages.is_contiguous())
 
 
-def decode_kernel_supports(q: torch.Tensor, k_pages: torch.Tensor, softcap: float) -> bool:
+def _tile_width(n: int) -> bool:
+    return 8 <= n <= 128 and n % 8 == 0
+
+
+def paged_kernel_supports(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor) -> bool:
+    """Layouts of the tensor-core paged attention kernels: bf16, head sizes that are multiples of 8 up to 128."""
+    return (q.is_cuda and q.dtype == torch.bfloat16 and k_pages.dtype == torch.bfloat16
+            and _tile_width(q.shape[-1]) and _tile_width(v_pages.shape[-1]) and q.stride(0) % 8 == 0)
+
+
+def decode_kernel_supports(q: torch.Tensor, k_pages: torch.Tensor, softcap: float, v_dim: int | None = None) -> bool:
     Hq, D = q.shape[-2], q.shape[-1]
     Hkv = k_pages.shape[2]
-    return (q.is_cuda and q.dtype == torch.bfloat16 and D in (64, 128) and Hq % Hkv == 0 and Hq // Hkv <= 16
-            and not softcap and k_pages.shape[1] == PAGE_SIZE and q.stride(-1) == 1 and q.stride(-2) == D)
+    return (q.is_cuda and q.dtype == torch.bfloat16 and _tile_width(D) and _tile_width(v_dim or D) and Hq % Hkv == 0
+            and Hq // Hkv <= 16 and not softcap and k_pages.shape[1] == PAGE_SIZE and q.stride(-1) == 1 and q.stride(-2) == D)
 
 
 def attn_combine(o_parts: torch.Tensor, lse_parts: torch.Tensor, sinks=None, want_lse: bool = False):
@@ -178,9 +223,9 @@ def paged_attention_splitkv(q: torch.Tensor, k_pages: torch.Tensor, v_pages: tor
     o_parts = torch.empty(B * S_, Hq, D, dtype=q.dtype, device=q.device)
     lse = torch.empty(Hq, B * S_, dtype=torch.float32, device=q.device)
     _lib.call("edl_attn_paged_lse", qr.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), o_parts.data_ptr(),
-              lse.data_ptr(), qr.stride(0), k_pages.stride(1), o_parts.stride(0), cu.data_ptr(), lens.data_ptr(),
-              pt.data_ptr(), pt.stride(0), B * S_, 1, B * S_, k_pages.shape[0], Hq, k_pages.shape[2], D, float(scale),
-              1, 0, float(softcap or 0.0), None, _lib.status_word(q.device).data_ptr(), _lib.stream_ptr())
+              lse.data_ptr(), qr.stride(0), k_pages.stride(1), v_pages.stride(1), o_parts.stride(0), cu.data_ptr(),
+              lens.data_ptr(), pt.data_ptr(), pt.stride(0), B * S_, 1, B * S_, k_pages.shape[0], Hq, k_pages.shape[2],
+              D, D, float(scale), 1, 0, float(softcap or 0.0), None, _lib.status_word(q.device).data_ptr(), _lib.stream_ptr())
     # [B*S, Hq, D] -> [S, B, Hq, D]; lse [Hq, B*S] -> [S, Hq, B]
     op = o_parts.view(B, S_, Hq, D).transpose(0, 1).contiguous()
     lp = lse.view(Hq, B, S_).permute(2, 0, 1).contiguous()

@@ -1,5 +1,5 @@
 """State-space and linear-attention recurrences: Mamba-1 selective scan, Mamba-2 SSD, gated delta rule, KDA and
-the ragged causal conv1d in front of them (``csrc/ssm.cu``).
+the ragged causal conv1d in front of them (``csrc/ssm.cu``), HGRN2 (``csrc/hgrn2.cu``).
 
 Every op has a PyTorch reference (also its autograd path: training differentiates the reference, chunk by chunk,
 while inference and evaluation call the CUDA recurrences). Sequences are packed on the token axis with
@@ -18,6 +18,8 @@ _lib.register("edl_selective_scan", i32, [vp, vp, vp, vp, vp, vp, vp, vp, i32, v
 _lib.register("edl_ssd_scan", i32, [vp, vp, vp, vp, vp, vp, vp, i32, vp, i32, i32, i32, i32, i32, vp, vp, vp])
 _lib.register("edl_delta_rule", i32, [vp, vp, vp, vp, vp, i32, vp, i32, i32, i32, i32, f32, vp, vp, vp])
 _lib.register("edl_ragged_conv1d", i32, [vp, vp, vp, vp, vp, i32, i32, i32, i32, vp, vp, vp])
+_lib.register("edl_hgrn2_scan", i32, [vp, i32, _lib.i64, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, vp, vp, vp])
+_lib.register("edl_hgrn2_decode", i32, [vp, i32, _lib.i64, vp, vp, vp, vp, vp, vp, f32, vp, i32, i32, i32, i32, vp])
 _lib.register("edl_wkv4", i32, [vp, vp, vp, vp, vp, i32, i32, vp, vp, vp])
 
 
@@ -484,3 +486,89 @@ def wkv4(time_decay, time_first, k, v, cu_seqlens=None, state=None):
     if k.is_cuda and k.shape[0] > 16:      # launch-bound on a GPU; on the host the per-token loop does less arithmetic
         return wkv4_chunked(time_decay, time_first, k, v, cu_seqlens, state)
     return wkv4_reference(time_decay, time_first, k, v, cu_seqlens, state)
+
+
+# ----------------------------------------------------------------------------------------- HGRN2
+def hgrn2_gates(q, z, bias, lower):
+    """fp32 ``(silu(q), f)`` with ``f = lower + (1 - lower) sigmoid(z + bias)``; all ``[T, H, D]`` / ``[H, D]``."""
+    return tF.silu(q.float()), lower.float() + (1.0 - lower.float()) * torch.sigmoid(z.float() + bias.float())
+
+
+def hgrn2_reference(proj, heads, bias, lower, cu, slots=None, state=None):
+    """Token by token: ``S = diag(f) S + (1 - f) v^T``, ``o = S^T silu(q)`` (fp32 ``[T, H, V]``). ``state``
+    ``[*, H, D, V]`` fp32 is read and updated at rows ``slots``."""
+    H, D, V = heads
+    T = proj.shape[0]
+    q, z, v = torch.split(proj, [H * D, H * D, H * V], -1)
+    q, f = hgrn2_gates(q.reshape(T, H, D), z.reshape(T, H, D), bias.view(H, D), lower.view(H, D))
+    v = v.reshape(T, H, V).float()
+    bounds = cu.tolist()
+    rows = list(range(len(bounds) - 1)) if slots is None else slots.tolist()
+    outs = []
+    for b in range(len(bounds) - 1):
+        if bounds[b + 1] <= bounds[b]:
+            continue
+        s = state[rows[b]].clone() if state is not None else proj.new_zeros(H, D, V, dtype=torch.float32)
+        for t in range(bounds[b], bounds[b + 1]):
+            s = f[t][:, :, None] * s + (1.0 - f[t])[:, :, None] * v[t][:, None, :]
+            outs.append((s * q[t][:, :, None]).sum(1))
+        if state is not None:
+            with torch.no_grad():
+                state[rows[b]] = s
+    return torch.stack(outs)
+
+
+#: tokens per segment of the segmented scan, and the most fp32 elements its workspace may hold
+HGRN2_SEGMENT = 256
+HGRN2_WORKSPACE = 1 << 27
+_SMS: dict[int, int] = {}
+
+
+def _hgrn2_segments(B: int, H: int, D: int, V: int, max_len: int, device) -> int:
+    """Segments to cut every sequence into (0 = walk each sequence in one go)."""
+    if max_len < 2 * HGRN2_SEGMENT:
+        return 0
+    idx = device.index or 0
+    if idx not in _SMS:
+        _SMS[idx] = torch.cuda.get_device_properties(device).multi_processor_count
+    width = 128 if D <= 32 else 64 if D <= 64 else 32 if D <= 128 else 16      # columns per CTA
+    if B * H * ((V + width - 1) // width) >= 6 * _SMS[idx]:
+        return 0
+    n = (max_len + HGRN2_SEGMENT - 1) // HGRN2_SEGMENT
+    return n if B * n <= 65535 and B * n * H * D * V <= HGRN2_WORKSPACE else 0
+
+
+def hgrn2(proj: torch.Tensor, heads: tuple[int, int, int], bias: torch.Tensor, lower: torch.Tensor,
+          norm: torch.Tensor, eps: float, cu: torch.Tensor, max_len: int, slots: torch.Tensor | None = None,
+          state: torch.Tensor | None = None, segments: int | None = None) -> torch.Tensor:
+    """HGRN2 over packed projections ``proj [T, 2 H D + H V]`` (q | gate | value), with the per-head output norm.
+
+    ``heads = (H, D, V)``; ``bias``, ``lower`` fp32 ``[H D]``; ``norm`` fp32 ``[V]``; ``cu`` int32 ``[B + 1]``; ``state``
+    fp32 ``[*, H, D, V]``, rows ``slots`` (int32 ``[B]``) read and updated in place; ``max_len``: longest sequence of the
+    step. Returns ``[T, H V]`` in the projection's type."""
+    from . import stream as ST
+
+    H, D, V = heads
+    T, B = proj.shape[0], cu.numel() - 1
+    if not ST.on_kernels(proj):
+        o = hgrn2_reference(proj, heads, bias, lower, cu, slots, state)
+        return ST.head_norm(o, norm, eps, proj.dtype).reshape(T, H * V)
+    f32_in = int(proj.dtype == torch.float32)
+    sp = _lib.stream_ptr()
+    if max_len == 1 and state is not None:
+        out = torch.empty(T, H * V, dtype=proj.dtype, device=proj.device)
+        _lib.call("edl_hgrn2_decode", proj.data_ptr(), f32_in, proj.stride(0), bias.data_ptr(), lower.data_ptr(),
+                  cu.data_ptr(), _lib.ptr(slots), state.data_ptr(), norm.data_ptr(), float(eps), out.data_ptr(), B, H, D,
+                  V, sp)
+        return out
+    n = _hgrn2_segments(B, H, D, V, max_len, proj.device) if segments is None else segments
+    ws = prod = None
+    if n:
+        ws = torch.empty(B * n * H * D * V, dtype=torch.float32, device=proj.device)
+        prod = torch.empty(B * n * H * D, dtype=torch.float32, device=proj.device)
+    seg_len = -(-max_len // n) if n else 0
+    o = torch.empty(T, H, V, dtype=torch.float32, device=proj.device)
+    _lib.call("edl_hgrn2_scan", proj.data_ptr(), f32_in, proj.stride(0), bias.data_ptr(), lower.data_ptr(),
+              cu.data_ptr(), _lib.ptr(slots), _lib.ptr(state), o.data_ptr(), B, H, D, V, seg_len, n, _lib.ptr(ws),
+              _lib.ptr(prod), sp)
+    return ST.head_norm(o, norm, eps, proj.dtype).view(T, H * V)
