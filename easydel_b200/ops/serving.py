@@ -336,7 +336,7 @@ def count_update(counts: torch.Tensor, tokens: torch.Tensor, row_slots: torch.Te
 
 def gather_rows(src: torch.Tensor, idx: torch.Tensor) -> torch.Tensor:
     """``src[idx]`` for a 2-D bf16 matrix (last hidden state of every sequence)."""
-    if src.is_cuda and src.dtype == torch.bfloat16:
+    if src.is_cuda and src.dtype == torch.bfloat16 and src.shape[1] % 8 == 0:
         out = torch.empty((idx.numel(), src.shape[1]), dtype=src.dtype, device=src.device)
         _lib.call("edl_gather_rows", src.data_ptr(), idx.data_ptr(), out.data_ptr(), idx.numel(), src.shape[1],
                   src.stride(0), _lib.stream_ptr())
