@@ -17,6 +17,8 @@ At 8 GPUs (``--serving auto``; ``on`` forces it at any N) the same JSON line car
 output tokens/s and TTFT / TPOT percentiles for Llama-3-70B at TP = N on the Poisson workload of the baseline
 (``easydel_b200/inference/esurge/bench_serving.py``), measured after the training state has been freed.
 
+``--model rakevik`` measures that family instead (kernels and serving throughput beside the closest existing models).
+
 ``--impl reference`` reports whether the unmodified reference can run here.
 ``--impl library`` runs the same config through stock PyTorch parts only (cuBLAS linears, SDPA,
 FSDP2 over NCCL, unfused AdamW; ``benchmarks/library_llama.py``) and prints the same JSON line with
@@ -248,7 +250,15 @@ def main() -> None:
     ap.add_argument("--serving-rate", type=float, default=8.0, help="Poisson arrival rate, requests/s")
     ap.add_argument("--serving-seconds", type=float, default=270.0,
                     help="requests stop being admitted after this long; the ones admitted are finished")
+    ap.add_argument("--model", default=None, choices=["rakevik"],
+                    help="instead of the headline workload: kernels and serving throughput of this family beside the "
+                         "closest existing models (benchmarks/bench_rakevik.py), one JSON line per row")
     args = ap.parse_args()
+    if args.model == "rakevik":
+        from benchmarks import bench_rakevik
+
+        bench_rakevik.main(["all"])
+        return
     if args.impl == "reference":
         reference_arm(args)
         return
