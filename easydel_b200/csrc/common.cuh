@@ -358,7 +358,7 @@ __device__ __forceinline__ float exp2_poly(float x) {
 // with 16 bytes each; instead the block goes through a swizzled 4 KB shared-memory stage and leaves as four whole
 // 128-byte row segments per instruction. `gbase` points at (first row, first column) of the block in global
 // memory, `ld_bytes` is the row pitch, rows >= valid_rows and 16-byte chunks >= valid_chunks are skipped.
-// ACC_F32 adds the staged fp32 values to what is in memory (gradient accumulation).
+// ACC_F32 adds the staged fp32 values to what is in memory (gradient accumulation, fp32 residual streams).
 template <bool ACC_F32>
 __device__ __forceinline__ void store_rows_coalesced(uint8_t* stage, const uint4 (&pk)[8], uint8_t* gbase,
                                                      long long ld_bytes, int valid_rows, int valid_chunks, int lane) {
@@ -373,14 +373,13 @@ __device__ __forceinline__ void store_rows_coalesced(uint8_t* stage, const uint4
     uint4 v = *reinterpret_cast<const uint4*>(stage + r * 128 + ((ch ^ (r & 7)) << 4));
     if (col_ok && r < valid_rows) {
       uint4* g = reinterpret_cast<uint4*>(gbase + r * ld_bytes + ch * 16);
-      if (ACC_F32) {
-        const uint4 o = *g;
-        v.x = __float_as_uint(__uint_as_float(v.x) + __uint_as_float(o.x));
-        v.y = __float_as_uint(__uint_as_float(v.y) + __uint_as_float(o.y));
-        v.z = __float_as_uint(__uint_as_float(v.z) + __uint_as_float(o.z));
-        v.w = __float_as_uint(__uint_as_float(v.w) + __uint_as_float(o.w));
+      if (ACC_F32) {   // added in L2: nothing to wait for (every element has one writer, so the sum is reproducible)
+        asm volatile("red.global.add.v4.f32 [%0], {%1, %2, %3, %4};" ::"l"(g), "f"(__uint_as_float(v.x)),
+                     "f"(__uint_as_float(v.y)), "f"(__uint_as_float(v.z)), "f"(__uint_as_float(v.w))
+                     : "memory");
+      } else {
+        *g = v;
       }
-      *g = v;
     }
   }
   __syncwarp();

@@ -26,8 +26,35 @@ __device__ __forceinline__ float g_of(__nv_bfloat16 v) { return __bfloat162float
 __device__ __forceinline__ void g_put(float* p, float v) { *p = v; }
 __device__ __forceinline__ void g_put(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
 
-__device__ __forceinline__ float gate_f(float z, float lower) { return lower + (1.f - lower) / (1.f + expf(-z)); }
-__device__ __forceinline__ float silu_p(float x) { return x / (1.f + expf(-x)); }
+// sigmoid in fp32. With bf16 projections the hardware exponential and divide (about 2 ulp each, far below the step of
+// their operand) keep the gates off the critical path; fp32 projections take the accurate functions.
+template <typename TI>
+__device__ __forceinline__ float sigm(float z) {
+  if constexpr (sizeof(TI) == 4) return 1.f / (1.f + expf(-z));
+  else return __fdividef(1.f, 1.f + __expf(-fmaxf(z, -80.f)));
+}
+template <typename TI>
+__device__ __forceinline__ float gate_f(float z, float lower) { return fmaf(1.f - lower, sigm<TI>(z), lower); }
+template <typename TI>
+__device__ __forceinline__ float silu_p(float x) { return x * sigm<TI>(x); }
+
+// four consecutive elements of a row (vec: 4-element aligned), `n` of them real, zeros behind
+template <typename TI>
+__device__ __forceinline__ void load4(const TI* p, int n, bool vec, float (&v)[4]) {
+  if (vec && n >= 4) {
+    if constexpr (sizeof(TI) == 4) {
+      const float4 a = *reinterpret_cast<const float4*>(p);
+      v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+    } else {
+      const uint2 a = *reinterpret_cast<const uint2*>(p);
+      const float2 lo = unpack_bf16x2(a.x), hi = unpack_bf16x2(a.y);
+      v[0] = lo.x; v[1] = lo.y; v[2] = hi.x; v[3] = hi.y;
+    }
+    return;
+  }
+#pragma unroll
+  for (int j = 0; j < 4; ++j) v[j] = j < n ? g_of(p[j]) : 0.f;
+}
 
 struct Hgrn2Params {
   const void* proj;          // [T, ld]: q | z | v
@@ -43,6 +70,7 @@ struct Hgrn2Params {
   float* ws;                 // [B * nseg, H, D, V]: end states, then start states, of the segments
   float* prod;               // [B * nseg, H, D]: products of the gates
   int seg_len, nseg;
+  bool vec;                  // heads and rows start on 4-element boundaries
   // decode
   const float* norm;         // [V]
   float eps;
@@ -108,20 +136,29 @@ hgrn2_scan_kernel(const Hgrn2Params p) {
   for (int tb = t0; tb < t1; tb += TC) {
     const int n = min(TC, t1 - tb);
     __syncthreads();
-    for (int i = tid; i < n * DP; i += SCT) {
-      const int t = i / DP, d = i % DP;
-      float f = 0.f, qv = 0.f;
-      if (d < p.D) {
-        const TI* row = proj + (tb + t) * p.ld + h * p.D + d;
-        f = gate_f(g_of(row[HD]) + p.bias[h * p.D + d], p.lower[h * p.D + d]);
-        if (MODE != SCAN_ENDS) qv = silu_p(g_of(row[0]));
+    // 4 channels (then 4 columns) per thread and turn; a thread's channels are the same in every turn
+#pragma unroll 4
+    for (int i = tid; i < n * (DP / 4); i += SCT) {
+      const int t = i / (DP / 4), d = (i % (DP / 4)) * 4;
+      const TI* row = proj + (tb + t) * p.ld + h * p.D + d;
+      float z[4], f[4];
+      load4(row + HD, p.D - d, p.vec, z);
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+        f[j] = d + j < p.D ? gate_f<TI>(z[j] + p.bias[h * p.D + d + j], p.lower[h * p.D + d + j]) : 0.f;
+      *reinterpret_cast<float4*>(&sf[t][d]) = make_float4(f[0], f[1], f[2], f[3]);
+      if (MODE != SCAN_ENDS) {
+        load4(row, p.D - d, p.vec, z);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) z[j] = silu_p<TI>(z[j]);
+        *reinterpret_cast<float4*>(&sq[t][d]) = make_float4(z[0], z[1], z[2], z[3]);
       }
-      sf[t][d] = f;
-      if (MODE != SCAN_ENDS) sq[t][d] = qv;
     }
-    for (int i = tid; i < n * CT; i += SCT) {
-      const int t = i / CT, c = i % CT;
-      sv[t][c] = col0 + c < p.V ? g_of(proj[(tb + t) * p.ld + 2 * HD + h * p.V + col0 + c]) : 0.f;
+    for (int i = tid; i < n * (CT / 4); i += SCT) {
+      const int t = i / (CT / 4), c = (i % (CT / 4)) * 4;
+      float v[4];
+      load4(proj + (tb + t) * p.ld + 2 * HD + h * p.V + col0 + c, p.V - col0 - c, p.vec, v);
+      *reinterpret_cast<float4*>(&sv[t][c]) = make_float4(v[0], v[1], v[2], v[3]);
     }
     __syncthreads();
 #pragma unroll 2
@@ -233,8 +270,8 @@ hgrn2_decode_kernel(const Hgrn2Params p) {
   const int groups = max(1, DCT / vcols);        // row groups
   float* st = p.state + ((long long)(p.slots ? p.slots[b] : b) * p.H + h) * (long long)D * V;
   for (int d = tid; d < D; d += DCT) {
-    sf[d] = gate_f(g_of(row[HD + h * D + d]) + p.bias[h * D + d], p.lower[h * D + d]);
-    sq[d] = silu_p(g_of(row[h * D + d]));
+    sf[d] = gate_f<TI>(g_of(row[HD + h * D + d]) + p.bias[h * D + d], p.lower[h * D + d]);
+    sq[d] = silu_p<TI>(g_of(row[h * D + d]));
   }
   __syncthreads();
   for (int u = tid; u < vcols * groups; u += DCT) {   // one round unless V / VEC > DCT
@@ -350,6 +387,7 @@ EDL_HOST_API int edl_hgrn2_scan(const void* proj, int f32, long long ld, const f
   Hgrn2Params p{};
   p.proj = proj; p.ld = ld; p.bias = bias; p.lower = lower; p.cu = cu; p.slots = slots; p.state = state; p.out = o;
   p.B = B; p.H = H; p.D = D; p.V = V; p.seg_len = seg_len; p.nseg = nseg; p.ws = ws; p.prod = prod;
+  p.vec = D % 4 == 0 && V % 4 == 0 && ld % 4 == 0 && (reinterpret_cast<uintptr_t>(proj) & (f32 ? 15 : 7)) == 0;
   cudaStream_t s = (cudaStream_t)stream;
   return f32 ? run_scan<float>(p, s) : run_scan<__nv_bfloat16>(p, s);
 }

@@ -36,6 +36,15 @@ __device__ __forceinline__ void ldv(const T* p, float (&v)[VEC]) {
     const uint2 a = *reinterpret_cast<const uint2*>(p);
     const float2 lo = unpack_bf16x2(a.x), hi = unpack_bf16x2(a.y);
     v[0] = lo.x; v[1] = lo.y; v[2] = hi.x; v[3] = hi.y;
+  } else if constexpr (VEC == 8 && sizeof(T) == 2) {
+    const uint4 a = *reinterpret_cast<const uint4*>(p);
+    const uint32_t w[4] = {a.x, a.y, a.z, a.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float2 f = unpack_bf16x2(w[i]);
+      v[2 * i] = f.x;
+      v[2 * i + 1] = f.y;
+    }
   } else {
 #pragma unroll
     for (int i = 0; i < VEC; ++i) v[i] = ld1<T>(p + i);
@@ -47,6 +56,9 @@ __device__ __forceinline__ void stv(T* p, const float (&v)[VEC]) {
     *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
   } else if constexpr (VEC == 4) {
     *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]));
+  } else if constexpr (VEC == 8 && sizeof(T) == 2) {
+    *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]),
+                                              pack_bf16x2(v[4], v[5]), pack_bf16x2(v[6], v[7]));
   } else {
 #pragma unroll
     for (int i = 0; i < VEC; ++i) st1(p + i, v[i]);
@@ -119,6 +131,112 @@ __device__ __forceinline__ float2 block_sum2(float a, float b, float2* red) {
     t.y += red[i].y;
   }
   return t;
+}
+
+// Many rows, a whole row in registers: a CTA walks `per` consecutive rows and keeps the normalised row before the
+// current one, so each row is read once (plus the one in front of the CTA's first).
+template <typename TO, int NV>
+__global__ void __launch_bounds__(NT)
+norm_shift_rows_kernel(const float* __restrict__ x, const float* __restrict__ w, const float* __restrict__ mu, float eps,
+                       int rows, int W, const int* __restrict__ cu, int nseq, const int* __restrict__ slots,
+                       float* __restrict__ state, long long ld_state, TO* __restrict__ out, int per) {
+  __shared__ float2 red[NT / 32];
+  constexpr int STEP = NT * 4;
+  const int r0 = blockIdx.x * per, r1 = min(rows, r0 + per);
+  const float inv_w = 1.f / (float)W;
+  int b = mu ? seq_of_row(cu, nseq, r0) : 0;
+  float wv[NV][4], mv[NV][4], h[NV][4], before[NV][4], next[NV][4];
+#pragma unroll
+  for (int k = 0; k < NV; ++k) {
+    const int c = threadIdx.x * 4 + k * STEP;
+    if (c < W) {
+      ldv<4>(w + c, wv[k]);
+      if (mu) ldv<4>(mu + c, mv[k]);
+    }
+  }
+  auto load = [&](int r, float (&d)[NV][4]) {
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+      const int c = threadIdx.x * 4 + k * STEP;
+      if (c < W) ldv<4>(x + (long long)r * W + c, d[k]);
+    }
+  };
+  // h = rms_norm of the row in d
+  auto norm = [&](const float (&d)[NV][4]) {
+    float s = 0.f;
+#pragma unroll
+    for (int k = 0; k < NV; ++k)
+      if (threadIdx.x * 4 + k * STEP < W)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) s += d[k][j] * d[k][j];
+    const float rs = 1.f / sqrtf(block_sum2(s, 0.f, red).x * inv_w + eps);
+#pragma unroll
+    for (int k = 0; k < NV; ++k)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) h[k][j] = d[k][j] * rs * wv[k][j];
+  };
+  if (mu && r0 > cu[b]) {
+    load(r0 - 1, next);
+    norm(next);
+#pragma unroll
+    for (int k = 0; k < NV; ++k)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) before[k][j] = h[k][j];
+  }
+  load(r0, next);
+  for (int r = r0; r < r1; ++r) {
+    norm(next);
+    if (r + 1 < r1) load(r + 1, next);
+    float* st = nullptr;
+    int last = -1;
+    if (mu) {
+      while (b + 1 < nseq && r >= cu[b + 1]) ++b;
+      if (r == cu[b]) {                 // first row of a sequence: the row before it is the slot's state, or zeros
+        st = state ? state + (long long)slots[b] * ld_state : nullptr;
+        last = cu[b + 1] - 1;
+#pragma unroll
+        for (int k = 0; k < NV; ++k) {
+          const int c = threadIdx.x * 4 + k * STEP;
+#pragma unroll
+          for (int j = 0; j < 4; ++j) before[k][j] = 0.f;
+          if (st && c < W) ldv<4>(st + c, before[k]);
+        }
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+      const int c = threadIdx.x * 4 + k * STEP;
+      if (c < W) {
+        float o[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) o[j] = mu ? h[k][j] + (before[k][j] - h[k][j]) * mv[k][j] : h[k][j];
+        stv<4>(out + (long long)r * W + c, o);
+        if (st && last == r) stv<4>(st + c, h[k]);
+      }
+#pragma unroll
+      for (int j = 0; j < 4; ++j) before[k][j] = h[k][j];
+    }
+    if (st && last != r) {              // the state's only reader also leaves the step's last row in it
+      float s = 0.f, v[4];
+      const float* xl = x + (long long)last * W;
+      for (int c = threadIdx.x * 4; c < W; c += STEP) {
+        ldv<4>(xl + c, v);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) s += v[j] * v[j];
+      }
+      const float rl = 1.f / sqrtf(block_sum2(s, 0.f, red).x * inv_w + eps);
+#pragma unroll
+      for (int k = 0; k < NV; ++k) {
+        const int c = threadIdx.x * 4 + k * STEP;
+        if (c < W) {
+          ldv<4>(xl + c, v);
+#pragma unroll
+          for (int j = 0; j < 4; ++j) v[j] = v[j] * rl * wv[k][j];
+          stv<4>(st + c, v);
+        }
+      }
+    }
+  }
 }
 
 // One CTA per row. NV: vectors of VEC elements each thread keeps of a row (0: rows too wide for registers are read
@@ -262,7 +380,14 @@ __global__ void xielu_kernel(const T* __restrict__ z, const float* __restrict__ 
 #pragma unroll
     for (int j = 0; j < VEC; ++j) {
       const float t = v[j];
-      v[j] = t > 0.f ? ap * t * t + 0.5f * t : an * (expm1f(t) - t) + 0.5f * t;
+      float e;   // e^t - 1 - t for t <= 0
+      if constexpr (sizeof(T) == 4) {
+        e = expm1f(t) - t;
+      } else {   // the operand has 8 bits: a short Taylor sum near zero, the hardware exponential elsewhere
+        const float near = 0.5f * t * t * fmaf(t * (1.f / 3.f), fmaf(t, 0.25f, 1.f), 1.f);
+        e = t > -0.06f ? near : __expf(t) - 1.f - t;
+      }
+      v[j] = t > 0.f ? ap * t * t + 0.5f * t : an * e + 0.5f * t;
     }
     stv<VEC>(y + i * VEC, v);
   }
@@ -336,6 +461,78 @@ qkv_prologue_kernel(const T* __restrict__ qkv, long long ld, const int* __restri
   }
 }
 
+// The same for heads of up to 128 elements in 4-element pieces: a lane holds its piece of four heads at a time in
+// registers, so that four rows are in flight per warp and nothing is read twice.
+template <typename T>
+__global__ void __launch_bounds__(NT)
+qkv_prologue_small_kernel(const T* __restrict__ qkv, long long ld, const int* __restrict__ pos,
+                          const int* __restrict__ slots, const float* __restrict__ qw, const float* __restrict__ kw,
+                          float eps, float coef, float every, int T_rows, int Hq, int Hkv, int D, int Dv,
+                          T* __restrict__ q_out, T* __restrict__ k_pages, T* __restrict__ v_pages, long long ld_kpage,
+                          long long ld_vpage, long long num_slots, int* status) {
+  constexpr int U = 4;
+  const int lane = threadIdx.x & 31, c = lane * 4;
+  const int heads = Hq + 2 * Hkv, per_token = (heads + U - 1) / U;
+  const bool in_d = c < D, in_v = c < Dv;
+  float wq[4] = {1.f, 1.f, 1.f, 1.f}, wk[4] = {1.f, 1.f, 1.f, 1.f};
+  if (in_d) {
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      if (qw) wq[j] = qw[c + j];
+      if (kw) wk[j] = kw[c + j];
+    }
+  }
+  const float inv_d = 1.f / (float)D;
+  const unsigned groups = (unsigned)T_rows * per_token, stride = gridDim.x * (NT / 32);
+  for (unsigned it = blockIdx.x * (NT / 32) + (threadIdx.x >> 5); it < groups; it += stride) {
+    const int t = it / per_token, h0 = (it - t * per_token) * U;
+    const T* row = qkv + t * ld;
+    float v[U][4], s[U];
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int h = h0 + u;
+      const bool val = h >= Hq + Hkv;
+      s[u] = 0.f;
+      if (h < heads && (val ? in_v : in_d)) {
+        ldv<4>(row + (val ? (Hq + Hkv) * D + (h - Hq - Hkv) * Dv : h * D) + c, v[u]);
+        s[u] = v[u][0] * v[u][0] + v[u][1] * v[u][1] + v[u][2] * v[u][2] + v[u][3] * v[u][3];
+      }
+    }
+    long long slot = 0;
+    float temp = 1.f;
+    if (h0 + U > Hq) {
+      slot = slots[t];
+      if (slot >= num_slots) {
+        if (status) atomicCAS(status, 0, EDL_BAD_INDEX);
+        slot = -1;
+      }
+    }
+    if (h0 < Hq && every > 0.f) temp = 1.f + coef * logf(floorf(((float)pos[t] + 1.f) / every) + 1.f);
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+      for (int u = 0; u < U; ++u) s[u] += __shfl_xor_sync(0xffffffffu, s[u], o);
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int h = h0 + u;
+      if (h >= heads) break;
+      if (h < Hq) {
+        const float r = (qw ? 1.f / sqrtf(s[u] * inv_d + eps) : 1.f) * temp;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) v[u][j] *= r * wq[j];
+        if (in_d) stv<4>(q_out + ((long long)t * Hq + h) * D + c, v[u]);
+      } else if (slot >= 0 && h < Hq + Hkv) {
+        const float r = kw ? 1.f / sqrtf(s[u] * inv_d + eps) : 1.f;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) v[u][j] *= r * wk[j];
+        if (in_d) stv<4>(k_pages + slot * ld_kpage + (h - Hq) * D + c, v[u]);
+      } else if (slot >= 0) {
+        if (in_v) stv<4>(v_pages + slot * ld_vpage + (h - Hq - Hkv) * Dv + c, v[u]);
+      }
+    }
+  }
+}
+
 int blocks_for(long long work, int per_block, int waves) {
   long long b = (work + per_block - 1) / per_block, cap = (long long)sm_count() * waves;
   return (int)(b < 1 ? 1 : (b > cap ? cap : b));
@@ -345,6 +542,17 @@ template <typename TO, int VEC>
 int launch_norm_shift(const float* x, const float* w, const float* mu, float eps, int rows, int W, const int* cu,
                       int nseq, const int* slots, float* state, long long ld_state, TO* out, cudaStream_t s) {
   const int nv = (W + NT * VEC - 1) / (NT * VEC);
+  if (VEC == 4 && nv <= 4 && rows >= 16 * sm_count()) {
+    const int per = mu ? 8 : 2;
+    const int grid = (rows + per - 1) / per;
+#define EDL_NR(N) \
+  norm_shift_rows_kernel<TO, N><<<grid, NT, 0, s>>>(x, w, mu, eps, rows, W, cu, nseq, slots, state, ld_state, out, per)
+    if (nv <= 1) EDL_NR(1);
+    else if (nv <= 2) EDL_NR(2);
+    else EDL_NR(4);
+#undef EDL_NR
+    return check_cuda(cudaGetLastError(), "norm_shift launch");
+  }
 #define EDL_NS(N) \
   norm_shift_kernel<TO, VEC, N><<<rows, NT, 0, s>>>(x, w, mu, eps, rows, W, cu, nseq, slots, state, ld_state, out)
   if (nv <= 1) EDL_NS(1);
@@ -437,12 +645,15 @@ EDL_HOST_API int edl_xielu(const void* z, const float* act, void* y, int f32, lo
   if (n <= 0) return 0;
   cudaStream_t s = (cudaStream_t)stream;
   const bool v4 = n % 4 == 0 && al(z, f32 ? 16 : 8) && al(y, f32 ? 16 : 8);
-  const int blocks = blocks_for(n / (v4 ? 4 : 1), 256, 8);
+  const bool v8 = !f32 && n % 8 == 0 && al(z, 16) && al(y, 16);
+  const int blocks = blocks_for(n / (v8 ? 8 : v4 ? 4 : 1), 256, 8);
 #define EDL_X(T, V_) xielu_kernel<T, V_><<<blocks, 256, 0, s>>>((const T*)z, act, (T*)y, n / V_)
   if (f32) {
     if (v4) EDL_X(float, 4); else EDL_X(float, 1);
   } else {
-    if (v4) EDL_X(__nv_bfloat16, 4); else EDL_X(__nv_bfloat16, 1);
+    if (v8) EDL_X(__nv_bfloat16, 8);
+    else if (v4) EDL_X(__nv_bfloat16, 4);
+    else EDL_X(__nv_bfloat16, 1);
   }
 #undef EDL_X
   return check_cuda(cudaGetLastError(), "xielu launch");
@@ -462,6 +673,19 @@ EDL_HOST_API int edl_qkv_prologue(const void* qkv, int f32, long long ld, const 
   const size_t a = f32 ? 16 : 8;
   const bool v4 = D % 4 == 0 && Dv % 4 == 0 && ld % 4 == 0 && ld_kpage % 4 == 0 && ld_vpage % 4 == 0 && al(qkv, a) &&
                   al(q_out, a) && al(k_pages, a) && al(v_pages, a);
+  if (v4 && D <= 128 && Dv <= 128 && (long long)T * (Hq + 2 * Hkv) < (1LL << 30)) {
+    const int nb = blocks_for((long long)T * ((Hq + 2 * Hkv + 3) / 4), NT / 32, 8);
+    if (f32)
+      qkv_prologue_small_kernel<float><<<nb, NT, 0, s>>>((const float*)qkv, ld, pos, slots, qw, kw, eps, coef, every, T,
+                                                         Hq, Hkv, D, Dv, (float*)q_out, (float*)k_pages,
+                                                         (float*)v_pages, ld_kpage, ld_vpage, num_slots, status);
+    else
+      qkv_prologue_small_kernel<__nv_bfloat16><<<nb, NT, 0, s>>>(
+          (const __nv_bfloat16*)qkv, ld, pos, slots, qw, kw, eps, coef, every, T, Hq, Hkv, D, Dv,
+          (__nv_bfloat16*)q_out, (__nv_bfloat16*)k_pages, (__nv_bfloat16*)v_pages, ld_kpage, ld_vpage, num_slots,
+          status);
+    return check_cuda(cudaGetLastError(), "qkv_prologue launch");
+  }
   const int blocks = blocks_for((long long)T * (Hq + 2 * Hkv), NT / 32, 8);
 #define EDL_P(TT, V_)                                                                                                \
   qkv_prologue_kernel<TT, V_><<<blocks, NT, 0, s>>>((const TT*)qkv, ld, pos, slots, qw, kw, eps, coef, every, T, Hq, \

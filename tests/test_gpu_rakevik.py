@@ -56,6 +56,27 @@ def test_norm_shift(W, dtype):
     _close(first[1:6], O.token_shift(O.rms_norm(x[1:6], w, 1e-5), mu), dtype)
 
 
+@pytest.mark.parametrize("W", [320, 1536, 4096])
+@pytest.mark.parametrize("dtype", DT)
+def test_norm_shift_over_many_rows(W, dtype):
+    """Enough rows for the form that walks several rows per CTA: sequence bounds in every place of such a group."""
+    from easydel_b200.ops import stream
+
+    lens = [1, 1, 2, 3, 4, 5, 6, 7, 8, 9, 1, 15, 1000, 1, 1500, 17]
+    cu = _i32(*torch.tensor([0, *lens]).cumsum(0).tolist())
+    x, w, mu = 3 * _r(sum(lens), W), 1 + 0.1 * _r(W, seed=1), torch.rand(W).cuda()
+    slots = torch.randperm(len(lens)).to(torch.int32).cuda()
+    state = _r(len(lens), W, seed=2)
+    want, ends = [], state.clone()
+    for s, c in zip(slots.tolist(), torch.split(x, lens)):
+        h = O.rms_norm(c, w, 1e-5)
+        want.append(O.token_shift(torch.cat([state[s:s + 1], h]), mu)[1:])
+        ends[s] = h[-1]
+    _close(stream.norm_shift(x, w, 1e-5, dtype, mu, cu, slots, state), torch.cat(want), dtype)
+    _close(state, ends, torch.float32)
+    _close(stream.norm_shift(x, w, 1e-5, dtype), O.rms_norm(x, w, 1e-5), dtype)
+
+
 @pytest.mark.parametrize("dtype", DT)
 def test_embedding_operand_and_activation(dtype):
     from easydel_b200.ops import stream
