@@ -8,9 +8,10 @@
 //
 //   * hgrn2_decode: one token per sequence. A CTA per (sequence, head) streams the state once (it is all the traffic
 //     there is), and finishes the row with the per-head RMS norm.
-//   * hgrn2_scan: any number of tokens per sequence. The columns of a state never meet, so a CTA owns (sequence, head,
+//   * hgrn2_scan: any number of tokens per sequence. An element-wise pass turns the projection rows into fp32 rows
+//     [f (D) | silu q (D) | v (V)] per token and head. The columns of a state never meet, so a CTA owns (sequence, head,
 //     column tile) and walks the tokens with its part of the state in registers: 8 rows x 4 columns per thread, packed
-//     fp32 arithmetic, gates of 16 tokens at a time in shared memory.
+//     fp32 arithmetic, the rows of up to 16 tokens at a time brought into shared memory one stage ahead (cp.async).
 //   * When (sequences x heads x tiles) cannot fill the GPU and sequences are long, the token axis is cut into segments:
 //     one pass leaves every segment's end state from a zero start and the product of its gates, a small kernel chains
 //     them into the state each segment starts from, and the scan then runs all segments at once.
@@ -70,6 +71,8 @@ struct Hgrn2Params {
   float* ws;                 // [B * nseg, H, D, V]: end states, then start states, of the segments
   float* prod;               // [B * nseg, H, D]: products of the gates
   int seg_len, nseg;
+  float* rows;               // scan: [T, H, 2 D + V] fp32 rows f | silu q | v
+  int T;
   bool vec;                  // heads and rows start on 4-element boundaries
   // decode
   const float* norm;         // [V]
@@ -80,18 +83,62 @@ enum { SCAN_WHOLE = 0, SCAN_ENDS = 1, SCAN_SEGMENTS = 2 };
 constexpr int SCT = 128;     // threads of a scan CTA
 constexpr int CPT = 4;       // columns per thread
 
+__device__ __forceinline__ void cp_async16(float* dst, const float* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+
+// Projection rows -> fp32 rows. A thread keeps its (head, channel) and walks the tokens.
+template <typename TI, int VEC>
+__global__ void __launch_bounds__(256)
+hgrn2_rows_kernel(const Hgrn2Params p) {
+  const int D = p.D, V = p.V, width = 2 * D + V;
+  const int u = blockIdx.x * 256 + threadIdx.x;
+  if (u >= p.H * (width / VEC)) return;
+  const int h = u / (width / VEC), c = (u - h * (width / VEC)) * VEC;
+  const int kind = c < D ? 0 : (c < 2 * D ? 1 : 2);        // gate, query, value
+  const int ch = h * D + (kind == 0 ? c : c - D);
+  const int HD = p.H * D;
+  const TI* src = reinterpret_cast<const TI*>(p.proj) +
+                  (kind == 0 ? HD + ch : kind == 1 ? ch : 2 * HD + h * V + c - 2 * D);
+  float b[VEC], low[VEC];
+#pragma unroll
+  for (int j = 0; j < VEC; ++j) {
+    b[j] = kind == 0 ? p.bias[ch + j] : 0.f;
+    low[j] = kind == 0 ? p.lower[ch + j] : 0.f;
+  }
+  float* dst = p.rows + (long long)h * width + c;
+  const long long pitch = (long long)p.H * width;
+#pragma unroll 4
+  for (int t = blockIdx.y; t < p.T; t += gridDim.y) {
+    float v[VEC];
+    if constexpr (VEC == 4) load4(src + t * p.ld, 4, true, v);
+    else v[0] = g_of(src[t * p.ld]);
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) {
+      if (kind == 0) v[j] = gate_f<TI>(v[j] + b[j], low[j]);
+      else if (kind == 1) v[j] = silu_p<TI>(v[j]);
+    }
+    if constexpr (VEC == 4) *reinterpret_cast<float4*>(dst + t * pitch) = make_float4(v[0], v[1], v[2], v[3]);
+    else dst[t * pitch] = v[0];
+  }
+}
+
 // DP: D rounded up to a tile; RPT rows per thread; DP / RPT lanes share a column group.
-template <typename TI, int DP, int RPT, int MODE>
-__global__ void __launch_bounds__(SCT)
+template <int DP, int RPT, int MODE>
+__global__ void __launch_bounds__(SCT, RPT == 8 ? 6 : 3)
 hgrn2_scan_kernel(const Hgrn2Params p) {
   constexpr int SPLIT = DP / RPT;               // 4 .. 32 adjacent lanes
   constexpr int CT = (SCT / SPLIT) * CPT;       // columns of this CTA
-  constexpr int TC = DP <= 256 ? 16 : 8;        // tokens per stage
+  constexpr int TC = DP <= 128 ? 16 : 2048 / DP;   // tokens per stage
   constexpr int NK = RPT / 4;
+  constexpr bool Q = MODE != SCAN_ENDS;
   static_assert(SPLIT >= 4 && SPLIT <= 32 && RPT % 4 == 0, "");
-  __shared__ __align__(16) float sf[TC][DP];
-  __shared__ __align__(16) float sq[MODE == SCAN_ENDS ? 1 : TC][DP];
-  __shared__ __align__(16) float sv[TC][CT];
+  __shared__ __align__(16) float sf[2][TC][DP];
+  __shared__ __align__(16) float sq[2][Q ? TC : 1][DP];
+  __shared__ __align__(16) float sv[2][TC][CT];
   const int tid = threadIdx.x;
   const int part = tid % SPLIT, grp = tid / SPLIT;
   const int h = blockIdx.y;
@@ -110,14 +157,55 @@ hgrn2_scan_kernel(const Hgrn2Params p) {
   if (t0 >= t1) return;
   const bool final_seg = MODE == SCAN_WHOLE || t1 == p.cu[b + 1];
   if (MODE == SCAN_ENDS && final_seg) return;   // nothing follows the last segment
-  const TI* proj = reinterpret_cast<const TI*>(p.proj);
-  const int HD = p.H * p.D;
   const long long mat = (long long)p.D * p.V;
   float* pool = nullptr;
   if (p.state) pool = p.state + ((long long)(p.slots ? p.slots[b] : b) * p.H + h) * mat;
   float* seg_state = MODE == SCAN_WHOLE ? nullptr : p.ws + ((long long)(b * p.nseg + seg) * p.H + h) * mat;
 
-  // rows of this thread: 4 * (part + SPLIT * k) + j, k < NK, j < 4; S2[k][j / 2][c] holds rows j, j + 1 as a pair
+  // the stages' columns past the real sizes are zeros: the copies never touch them
+  if (p.D < DP) {
+    for (int i = tid; i < 2 * TC * DP; i += SCT) {
+      (&sf[0][0][0])[i] = 0.f;
+      if (Q) (&sq[0][0][0])[i] = 0.f;
+    }
+  }
+  if (col0 + CT > p.V)
+    for (int i = tid; i < 2 * TC * CT; i += SCT) (&sv[0][0][0])[i] = 0.f;
+  __syncthreads();
+  const int width = 2 * p.D + p.V;
+  auto fetch = [&](int tb, int buf) {
+    const int n = min(TC, t1 - tb);
+    const float* base = p.rows + ((long long)tb * p.H + h) * width;
+    const long long pitch = (long long)p.H * width;
+    for (int i = tid; i < n * (DP / 4); i += SCT) {
+      const int t = i / (DP / 4), d = (i % (DP / 4)) * 4;
+      const float* row = base + t * pitch + d;
+      if (p.vec) {
+        if (d < p.D) {
+          cp_async16(&sf[buf][t][d], row);
+          if (Q) cp_async16(&sq[buf][t][d], row + p.D);
+        }
+      } else {
+        for (int j = 0; j < 4 && d + j < p.D; ++j) {
+          sf[buf][t][d + j] = row[j];
+          if (Q) sq[buf][t][d + j] = row[p.D + j];
+        }
+      }
+    }
+    for (int i = tid; i < n * (CT / 4); i += SCT) {
+      const int t = i / (CT / 4), c = (i % (CT / 4)) * 4;
+      const float* row = base + t * pitch + 2 * p.D + col0 + c;
+      if (p.vec) {
+        if (col0 + c < p.V) cp_async16(&sv[buf][t][c], row);
+      } else {
+        for (int j = 0; j < 4 && col0 + c + j < p.V; ++j) sv[buf][t][c + j] = row[j];
+      }
+    }
+    cp_async_commit();
+  };
+  fetch(t0, 0);
+
+  // rows of this thread: 4 * (part + SPLIT * k) + j, k < NK, j < 4; packed arithmetic takes rows j, j + 1 as a pair
   float S[NK][4][CPT];
   float pr[NK][4];
   {
@@ -133,46 +221,30 @@ hgrn2_scan_kernel(const Hgrn2Params p) {
           S[k][j][c] = (src && row < p.D && col + c < p.V) ? src[(long long)row * p.V + col + c] : 0.f;
       }
   }
-  for (int tb = t0; tb < t1; tb += TC) {
+  float* out = reinterpret_cast<float*>(p.out) + ((long long)t0 * p.H + h) * p.V + col + (part & 1) * 2 + ((part >> 1) & 1);
+  const bool writes = part < 4 && col + (part & 1) * 2 + ((part >> 1) & 1) < p.V;
+  int buf = 0;
+  for (int tb = t0; tb < t1; tb += TC, buf ^= 1) {
     const int n = min(TC, t1 - tb);
-    __syncthreads();
-    // 4 channels (then 4 columns) per thread and turn; a thread's channels are the same in every turn
-#pragma unroll 4
-    for (int i = tid; i < n * (DP / 4); i += SCT) {
-      const int t = i / (DP / 4), d = (i % (DP / 4)) * 4;
-      const TI* row = proj + (tb + t) * p.ld + h * p.D + d;
-      float z[4], f[4];
-      load4(row + HD, p.D - d, p.vec, z);
-#pragma unroll
-      for (int j = 0; j < 4; ++j)
-        f[j] = d + j < p.D ? gate_f<TI>(z[j] + p.bias[h * p.D + d + j], p.lower[h * p.D + d + j]) : 0.f;
-      *reinterpret_cast<float4*>(&sf[t][d]) = make_float4(f[0], f[1], f[2], f[3]);
-      if (MODE != SCAN_ENDS) {
-        load4(row, p.D - d, p.vec, z);
-#pragma unroll
-        for (int j = 0; j < 4; ++j) z[j] = silu_p<TI>(z[j]);
-        *reinterpret_cast<float4*>(&sq[t][d]) = make_float4(z[0], z[1], z[2], z[3]);
-      }
-    }
-    for (int i = tid; i < n * (CT / 4); i += SCT) {
-      const int t = i / (CT / 4), c = (i % (CT / 4)) * 4;
-      float v[4];
-      load4(proj + (tb + t) * p.ld + 2 * HD + h * p.V + col0 + c, p.V - col0 - c, p.vec, v);
-      *reinterpret_cast<float4*>(&sv[t][c]) = make_float4(v[0], v[1], v[2], v[3]);
+    if (tb + TC < t1) {
+      fetch(tb + TC, buf ^ 1);     // every warp left that stage at the barrier below
+      cp_async_wait<1>();
+    } else {
+      cp_async_wait<0>();
     }
     __syncthreads();
 #pragma unroll 2
     for (int t = 0; t < n; ++t) {
-      const float4 v4 = *reinterpret_cast<const float4*>(&sv[t][grp * CPT]);
+      const float4 v4 = *reinterpret_cast<const float4*>(&sv[buf][t][grp * CPT]);
       const float v[CPT] = {v4.x, v4.y, v4.z, v4.w};
       float a0[CPT], a1[CPT];
 #pragma unroll
       for (int c = 0; c < CPT; ++c) a0[c] = a1[c] = 0.f;
 #pragma unroll
       for (int k = 0; k < NK; ++k) {
-        const float4 f4 = *reinterpret_cast<const float4*>(&sf[t][4 * (part + SPLIT * k)]);
+        const float4 f4 = *reinterpret_cast<const float4*>(&sf[buf][t][4 * (part + SPLIT * k)]);
         float4 q4 = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (MODE != SCAN_ENDS) q4 = *reinterpret_cast<const float4*>(&sq[t][4 * (part + SPLIT * k)]);
+        if (MODE != SCAN_ENDS) q4 = *reinterpret_cast<const float4*>(&sq[buf][t][4 * (part + SPLIT * k)]);
 #pragma unroll
         for (int c = 0; c < CPT; ++c) {
           // S = f S + (1 - f) v as v + f (S - v), two rows per instruction
@@ -205,11 +277,11 @@ hgrn2_scan_kernel(const Hgrn2Params p) {
         float z = (hi1 ? y1 : y0) + __shfl_xor_sync(0xffffffffu, hi1 ? y0 : y1, 2);
 #pragma unroll
         for (int o = 4; o < SPLIT; o <<= 1) z += __shfl_xor_sync(0xffffffffu, z, o);
-        const int c = (part & 1) * 2 + ((part >> 1) & 1);
-        if (part < 4 && col + c < p.V)
-          reinterpret_cast<float*>(p.out)[(long long)(tb + t) * p.H * p.V + (long long)h * p.V + col + c] = z;
+        if (writes) *out = z;
+        out += (long long)p.H * p.V;
       }
     }
+    __syncthreads();
   }
   float* dst = MODE == SCAN_ENDS ? seg_state : (final_seg ? pool : nullptr);
   if (dst) {
@@ -241,12 +313,23 @@ __global__ void hgrn2_chain_kernel(const Hgrn2Params p) {
        i += (long long)gridDim.x * blockDim.x) {
     const int row = (int)(i / p.V);
     float s = pool ? pool[i] : 0.f;
-    for (int g = 0; g < segs; ++g) {
-      const long long at = (long long)(b * p.nseg + g) * p.H + h;
-      float* w = p.ws + at * mat + i;
-      const float end = *w;
-      *w = s;
-      if (g + 1 < segs) s = fmaf(p.prod[at * p.D + row], s, end);
+    constexpr int AHEAD = 8;                     // segments whose loads are in flight together
+    for (int g0 = 0; g0 < segs; g0 += AHEAD) {
+      float end[AHEAD], f[AHEAD];
+#pragma unroll
+      for (int j = 0; j < AHEAD; ++j) {
+        const long long at = (long long)(b * p.nseg + g0 + j) * p.H + h;
+        if (g0 + j + 1 < segs) {
+          end[j] = p.ws[at * mat + i];
+          f[j] = p.prod[at * p.D + row];
+        }
+      }
+#pragma unroll
+      for (int j = 0; j < AHEAD; ++j) {
+        if (g0 + j >= segs) break;
+        p.ws[((long long)(b * p.nseg + g0 + j) * p.H + h) * mat + i] = s;
+        if (g0 + j + 1 < segs) s = fmaf(f[j], s, end[j]);
+      }
     }
   }
 }
@@ -334,12 +417,12 @@ hgrn2_decode_kernel(const Hgrn2Params p) {
   for (int c = tid; c < V; c += DCT) g_put(out + c, sums[c] * rs * p.norm[c]);
 }
 
-template <typename TI, int MODE>
+template <int MODE>
 int launch_scan(const Hgrn2Params& p, int z, cudaStream_t s) {
 #define EDL_HS(DP, RPT)                                                                          \
   {                                                                                              \
     constexpr int CT = (SCT / (DP / RPT)) * CPT;                                                 \
-    hgrn2_scan_kernel<TI, DP, RPT, MODE><<<dim3((p.V + CT - 1) / CT, p.H, z), SCT, 0, s>>>(p);   \
+    hgrn2_scan_kernel<DP, RPT, MODE><<<dim3((p.V + CT - 1) / CT, p.H, z), SCT, 0, s>>>(p);   \
   }
   if (p.D <= 32) EDL_HS(32, 8)
   else if (p.D <= 64) EDL_HS(64, 8)
@@ -352,12 +435,19 @@ int launch_scan(const Hgrn2Params& p, int z, cudaStream_t s) {
 
 template <typename TI>
 int run_scan(Hgrn2Params& p, cudaStream_t s) {
-  if (p.seg_len <= 0) return launch_scan<TI, SCAN_WHOLE>(p, p.B, s);
-  if (launch_scan<TI, SCAN_ENDS>(p, p.B * p.nseg, s)) return -1;
+  const int per_token = p.H * ((2 * p.D + p.V) / (p.vec ? 4 : 1));
+  const int gx = (per_token + 255) / 256;
+  int gy = (8 * sm_count() + gx - 1) / gx;
+  if (gy > p.T) gy = p.T;
+  if (p.vec) hgrn2_rows_kernel<TI, 4><<<dim3(gx, gy), 256, 0, s>>>(p);
+  else hgrn2_rows_kernel<TI, 1><<<dim3(gx, gy), 256, 0, s>>>(p);
+  if (check_cuda(cudaGetLastError(), "hgrn2_rows launch")) return -1;
+  if (p.seg_len <= 0) return launch_scan<SCAN_WHOLE>(p, p.B, s);
+  if (launch_scan<SCAN_ENDS>(p, p.B * p.nseg, s)) return -1;
   const long long mat = (long long)p.D * p.V;
   hgrn2_chain_kernel<<<dim3((unsigned)((mat + 255) / 256), p.H, p.B), 256, 0, s>>>(p);
   if (check_cuda(cudaGetLastError(), "hgrn2_chain launch")) return -1;
-  return launch_scan<TI, SCAN_SEGMENTS>(p, p.B * p.nseg, s);
+  return launch_scan<SCAN_SEGMENTS>(p, p.B * p.nseg, s);
 }
 
 bool bad_sizes(const char* who, int B, int H, int D, int V) {
@@ -373,12 +463,12 @@ bool bad_sizes(const char* who, int B, int H, int D, int V) {
 
 using namespace edl;
 
-// o [T, H * V] fp32 (no output norm). seg_len > 0: segmented form, nseg >= ceil(longest sequence / seg_len), with
+// o [T, H * V] fp32 (no output norm); rows: workspace [T, H, 2 D + V] fp32. seg_len > 0: segmented form, nseg >= ceil(longest sequence / seg_len), with
 // ws [B * nseg, H, D, V] and prod [B * nseg, H, D] fp32.
 EDL_HOST_API int edl_hgrn2_scan(const void* proj, int f32, long long ld, const float* bias, const float* lower,
-                                const int* cu, const int* slots, float* state, float* o, int B, int H, int D, int V,
-                                int seg_len, int nseg, float* ws, float* prod, void* stream) {
-  if (B <= 0) return 0;
+                                const int* cu, const int* slots, float* state, float* o, float* rows, int T, int B,
+                                int H, int D, int V, int seg_len, int nseg, float* ws, float* prod, void* stream) {
+  if (B <= 0 || T <= 0) return 0;
   if (bad_sizes("edl_hgrn2_scan", B, H, D, V)) return -1;
   if (seg_len > 0 && (nseg < 1 || !ws || !prod || (long long)B * nseg > 65535)) {
     set_last_error("edl_hgrn2_scan: bad segmentation (seg_len=%d, nseg=%d)", seg_len, nseg);
@@ -387,7 +477,9 @@ EDL_HOST_API int edl_hgrn2_scan(const void* proj, int f32, long long ld, const f
   Hgrn2Params p{};
   p.proj = proj; p.ld = ld; p.bias = bias; p.lower = lower; p.cu = cu; p.slots = slots; p.state = state; p.out = o;
   p.B = B; p.H = H; p.D = D; p.V = V; p.seg_len = seg_len; p.nseg = nseg; p.ws = ws; p.prod = prod;
-  p.vec = D % 4 == 0 && V % 4 == 0 && ld % 4 == 0 && (reinterpret_cast<uintptr_t>(proj) & (f32 ? 15 : 7)) == 0;
+  p.rows = rows; p.T = T;
+  p.vec = D % 4 == 0 && V % 4 == 0 && ld % 4 == 0 && (reinterpret_cast<uintptr_t>(proj) & (f32 ? 15 : 7)) == 0 &&
+          (reinterpret_cast<uintptr_t>(rows) & 15) == 0;
   cudaStream_t s = (cudaStream_t)stream;
   return f32 ? run_scan<float>(p, s) : run_scan<__nv_bfloat16>(p, s);
 }

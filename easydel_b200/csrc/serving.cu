@@ -108,22 +108,30 @@ sample_kernel(const void* __restrict__ logits, int is_f32, long long ld, int V, 
   const bool greedy = temp <= 0.f || k == 1;
   if (k <= 0 || k > MAX_CAND) k = MAX_CAND;
   const int rounds = greedy ? 1 : k;
-  if (greedy && !pen && !is_f32 && (V & 7) == 0 && (ld & 7) == 0) {
+  if (greedy && !pen && (V & 7) == 0 && (ld & 7) == 0 && (reinterpret_cast<uintptr_t>(logits) & 15) == 0) {
     // Greedy rows without penalties: one pass of 16-byte loads computes the arg-max and, online, the
     // log-sum-exp that the reported log-probability needs.
-    const uint4* rowp = reinterpret_cast<const uint4*>(reinterpret_cast<const __nv_bfloat16*>(logits) + row * ld);
+    const uint4* rowp = reinterpret_cast<const uint4*>(reinterpret_cast<const char*>(logits) +
+                                                       row * ld * (is_f32 ? 4 : 2));
     ArgMax best{-INFINITY, 0x7fffffff};
     float m = -INFINITY, ssum = 0.f;
     const int nvec = V >> 3;
     for (int i = threadIdx.x; i < nvec; i += SAMP_THREADS) {
-      const uint4 q = rowp[i];
-      const uint32_t w[4] = {q.x, q.y, q.z, q.w};
       float z[8];
+      if (is_f32) {
+        const uint4 a = rowp[2 * i], b = rowp[2 * i + 1];
+        const uint32_t w[8] = {a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w};
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const float2 f = unpack_bf16x2(w[j]);
-        z[2 * j] = f.x;
-        z[2 * j + 1] = f.y;
+        for (int j = 0; j < 8; ++j) z[j] = __uint_as_float(w[j]);
+      } else {
+        const uint4 q = rowp[i];
+        const uint32_t w[4] = {q.x, q.y, q.z, q.w};
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const float2 f = unpack_bf16x2(w[j]);
+          z[2 * j] = f.x;
+          z[2 * j + 1] = f.y;
+        }
       }
       float cm = z[0];
 #pragma unroll

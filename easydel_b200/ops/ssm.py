@@ -18,7 +18,7 @@ _lib.register("edl_selective_scan", i32, [vp, vp, vp, vp, vp, vp, vp, vp, i32, v
 _lib.register("edl_ssd_scan", i32, [vp, vp, vp, vp, vp, vp, vp, i32, vp, i32, i32, i32, i32, i32, vp, vp, vp])
 _lib.register("edl_delta_rule", i32, [vp, vp, vp, vp, vp, i32, vp, i32, i32, i32, i32, f32, vp, vp, vp])
 _lib.register("edl_ragged_conv1d", i32, [vp, vp, vp, vp, vp, i32, i32, i32, i32, vp, vp, vp])
-_lib.register("edl_hgrn2_scan", i32, [vp, i32, _lib.i64, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, vp, vp, vp])
+_lib.register("edl_hgrn2_scan", i32, [vp, i32, _lib.i64, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, vp, vp, vp])
 _lib.register("edl_hgrn2_decode", i32, [vp, i32, _lib.i64, vp, vp, vp, vp, vp, vp, f32, vp, i32, i32, i32, i32, vp])
 _lib.register("edl_wkv4", i32, [vp, vp, vp, vp, vp, i32, i32, vp, vp, vp])
 
@@ -518,24 +518,27 @@ def hgrn2_reference(proj, heads, bias, lower, cu, slots=None, state=None):
     return torch.stack(outs)
 
 
-#: tokens per segment of the segmented scan, and the most fp32 elements its workspace may hold
-HGRN2_SEGMENT = 256
+#: shortest segment of the segmented scan, and the most fp32 elements its workspace may hold
+HGRN2_SEGMENT = 128
 HGRN2_WORKSPACE = 1 << 27
 _SMS: dict[int, int] = {}
 
 
 def _hgrn2_segments(B: int, H: int, D: int, V: int, max_len: int, device) -> int:
-    """Segments to cut every sequence into (0 = walk each sequence in one go)."""
+    """Segments to cut every sequence into (0 = walk each sequence in one go). Cutting costs a second pass over the
+    tokens, so it is for steps whose (sequence, head, column tile) units leave most of the GPU idle; then there are as
+    many segments as fill six CTAs per SM."""
     if max_len < 2 * HGRN2_SEGMENT:
         return 0
     idx = device.index or 0
     if idx not in _SMS:
         _SMS[idx] = torch.cuda.get_device_properties(device).multi_processor_count
     width = 128 if D <= 32 else 64 if D <= 64 else 32 if D <= 128 else 16      # columns per CTA
-    if B * H * ((V + width - 1) // width) >= 6 * _SMS[idx]:
+    units = B * H * ((V + width - 1) // width)
+    if units >= 3 * _SMS[idx]:
         return 0
-    n = (max_len + HGRN2_SEGMENT - 1) // HGRN2_SEGMENT
-    return n if B * n <= 65535 and B * n * H * D * V <= HGRN2_WORKSPACE else 0
+    n = min(-(-6 * _SMS[idx] // units), max_len // HGRN2_SEGMENT)
+    return n if n > 1 and B * n <= 65535 and B * n * H * D * V <= HGRN2_WORKSPACE else 0
 
 
 def hgrn2(proj: torch.Tensor, heads: tuple[int, int, int], bias: torch.Tensor, lower: torch.Tensor,
@@ -568,7 +571,8 @@ def hgrn2(proj: torch.Tensor, heads: tuple[int, int, int], bias: torch.Tensor, l
         prod = torch.empty(B * n * H * D, dtype=torch.float32, device=proj.device)
     seg_len = -(-max_len // n) if n else 0
     o = torch.empty(T, H, V, dtype=torch.float32, device=proj.device)
+    rows = torch.empty(T * H * (2 * D + V), dtype=torch.float32, device=proj.device)
     _lib.call("edl_hgrn2_scan", proj.data_ptr(), f32_in, proj.stride(0), bias.data_ptr(), lower.data_ptr(),
-              cu.data_ptr(), _lib.ptr(slots), _lib.ptr(state), o.data_ptr(), B, H, D, V, seg_len, n, _lib.ptr(ws),
+              cu.data_ptr(), _lib.ptr(slots), _lib.ptr(state), o.data_ptr(), rows.data_ptr(), T, B, H, D, V, seg_len, n, _lib.ptr(ws),
               _lib.ptr(prod), sp)
     return ST.head_norm(o, norm, eps, proj.dtype).view(T, H * V)

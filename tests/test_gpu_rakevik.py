@@ -135,6 +135,19 @@ def test_attention_prologue(heads, dtype):
     assert int((kp.view(384, -1).abs().sum(1) > 0).sum()) == T - 1
 
 
+@pytest.mark.parametrize("V", [512, 1000, 77])
+@pytest.mark.parametrize("dtype", DT)
+def test_greedy_sampling_of_either_logit_type(V, dtype):
+    from easydel_b200.ops import serving as S
+
+    lg = _r(9, V, dtype=dtype)
+    lg[2, 5] = lg[2, V - 1] = lg[2].max() + 1           # a tie: the first one wins
+    tok, lp = S.sample(lg, want_logprob=True)
+    assert tok.tolist() == lg.float().argmax(-1).tolist() and int(tok[2]) == 5
+    want = torch.log_softmax(lg.float(), -1).gather(1, tok.long()[:, None])[:, 0]
+    assert torch.allclose(lp, want, atol=1e-3)
+
+
 # ------------------------------------------------------------------------------------------------ attention
 def _paged(lens_kv, Hkv, D, Dv, dtype, seed=0):
     """Random keys / values of several sequences on shuffled pages; returns dense lists and the paged form."""
