@@ -257,7 +257,10 @@ def main() -> None:
     if args.model == "rakevik":
         from benchmarks import bench_rakevik
 
+        sampler = ClockSampler(0)
+        sampler.start()
         bench_rakevik.main(["all"])
+        print(json.dumps({"clocks": sampler.stop()}))
         return
     if args.impl == "reference":
         reference_arm(args)

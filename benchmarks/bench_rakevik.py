@@ -81,7 +81,7 @@ def bench_rows(t: Table, T: int, W: int, H: int, G: int, D: int, V: int, F: int)
     cos = torch.rand(T, D // 2, device="cuda")
     out = torch.empty_like(packed)
     t.add("qkv_prologue (norm q k, temperature, append)", size,
-          (lambda: stream.qkv_prologue(qkv, heads, qn, qn, 1e-6, pos, (0.3, 64.0), sl, kp, vp), nb),
+          (lambda: stream.qkv_prologue(qkv, heads, qn, qn, 1e-6, pos, (0.5, 1024.0), sl, kp, vp), nb),
           "rope over packed qkv (no norm, no append)",
           (lambda: K.rope_copy(packed, out, pos, cos, cos, H + G, D), 2 * T * (H + 2 * G) * D * 2))
     z, act, gu = _rand(T, F), torch.tensor([0.3, 0.3], device="cuda"), _rand(T, 2 * F)
@@ -161,7 +161,7 @@ def bench_kernels() -> list[dict]:
             bench_recurrence(t, 8, 1024, H, 128, 128)
             for B in (8, 64, 256):
                 bench_recurrence(t, B, 1, H, 128, 128)
-        for D, V in ((128, 128), (64, 80), (96, 128)):
+        for D, V in ((128, 128), (64, 96), (96, 128)):
             bench_attention(t, 1, 8192, 8192, 32, 8, D, V)
             bench_attention(t, 64, 1, 2048, 32, 8, D, V)
     return t.rows
@@ -185,7 +185,7 @@ def _models(W: int, H: int, G: int, F: int, layers: int):
     rec = {"type": "hgrn2", "mixer": {"heads": H, "dim": 128, "vdim": 128}, "mlp": mlp}
     att = {"type": "attention", "mlp": mlp,
            "mixer": {"heads": H, "kv_heads": G, "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
-                     "q_temp": {"coef": 0.3, "every": 1024}}}
+                     "q_temp": {"coef": 0.5, "every": 1024}}}
     gated = 2 * F // 3 // 64 * 64
     common = dict(vocab_size=VOCAB, hidden_size=W, intermediate_size=gated, num_hidden_layers=layers,
                   num_attention_heads=H, num_key_value_heads=G, head_dim=128, tie_word_embeddings=False)

@@ -1,4 +1,5 @@
-// HGRN2: linear attention whose forget gate also decides what is written. Per head, with a [D, V] state S in fp32,
+// HGRN2, a gated linear recurrence without keys: a channel's write strength is the complement of its forget gate. Per
+// head, with a [D, V] state S in fp32,
 //
 //   f_t = lower + (1 - lower) * sigmoid(z_t + bias)          (one gate per head and channel)
 //   S_t = diag(f_t) S_{t-1} + (1 - f_t) v_t^T,   o_t = S_t^T silu(q_t)

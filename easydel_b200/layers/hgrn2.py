@@ -1,4 +1,5 @@
-"""HGRN2 token mixer: gated linear attention whose forget gate also decides what is written (``ops.ssm.hgrn2``).
+"""HGRN2 token mixer, a gated linear recurrence without keys: channels write with the complement of their forget gate
+(``ops.ssm.hgrn2``).
 
 Per head, with a ``[dim, vdim]`` state: ``q = silu(W_q h)``, ``v = W_v h``, ``f = lower + (1 - lower) sigmoid(W_f h + b)``,
 ``S <- diag(f) S + (1 - f) v^T``, ``o = S^T q``; each head's ``o`` is RMS-normed with a weight shared by the heads. The

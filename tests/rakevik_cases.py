@@ -16,7 +16,7 @@ def hgrn2(heads, dim, vdim, ff=None):
             "mlp": {"kind": "dense", "ff": ff} if ff else None}
 
 
-def attention(heads, kv_heads, dim, vdim, scale, coef=None, every=64, ff=None):
+def attention(heads, kv_heads, dim, vdim, scale, coef=None, every=50, ff=None):
     m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale}
     if coef is not None:
         m["q_temp"] = {"coef": coef, "every": every}
