@@ -226,3 +226,17 @@ def test_trace_command(tmp_path, monkeypatch, capsys):
     got = np.concatenate([np.fromfile(tmp_path / f"{n}.f32", dtype="<f4") for n in (0, 2)]).reshape(3, -1)
     assert not (tmp_path / "1.f32").exists()
     assert C.error(torch.from_numpy(got), want[[0, 9, 11]]) < TOL
+
+
+def test_builder_serves_a_checkpoint_folder(tmp_path):
+    """The builder behind ``python -m easydel_b200.elarge`` (serve / eval), without a tokenizer in the folder."""
+    from easydel_b200.elarge import eLargeModel
+    from easydel_b200.inference import SamplingParams
+
+    cfg, w, _ = C.make(tmp_path, "plain", torch.float32, "cpu")
+    elm = eLargeModel.from_pretrained(str(tmp_path / "plain")).set_dtype("float32")
+    elm.update("loader", device="cpu").set_esurge(max_model_len=128, max_num_seqs=2)
+    assert elm.validate() == []
+    prompt = C.tokens(7, cfg["vocab"])
+    out = elm.build_esurge().generate([prompt], SamplingParams(max_tokens=3, temperature=0.0, ignore_eos=True))
+    assert out[0].outputs[0].token_ids == _greedy(cfg, w, prompt, 3)
