@@ -13,7 +13,7 @@ ragged_page/cache.py:1157-1250): query start offsets, context lengths, page tabl
 from __future__ import annotations
 
 import typing as tp
-from dataclasses import dataclass
+from dataclasses import dataclass, field
 
 import torch
 
@@ -39,6 +39,19 @@ class PagedBatchMeta:
     # table [B, maxP] and the slot mapping [T]; entry g - 1 belongs to group g
     group_tables: list | None = None
     group_slots: list | None = None
+    # host copy of (new tokens, keys after this step's append) of every sequence; None in captured decode steps
+    spans: list[tuple[int, int]] | None = None
+    # what latent layers of one step share about the pages its portions can see, by (group, window, first sequence)
+    visible: dict = field(default_factory=dict)
+
+    def leading_singles(self) -> int:
+        """How many sequences at the head of the batch bring exactly one token."""
+        n = 0
+        for new, _ in self.spans or ():
+            if new != 1:
+                break
+            n += 1
+        return n
 
     def table_of(self, group: int) -> torch.Tensor:
         return self.page_table if group == 0 or not self.group_tables else self.group_tables[group - 1]
@@ -75,7 +88,7 @@ class PagedKVCache:
             k = torch.zeros(shape, dtype=dtype, device=device)      # zeros: the null page must hold finite numbers
             self._k.append(k)
             v_shape = (*shape[:-1], grp.spec.value_dim)
-            self._v.append(k if grp.kind == "latent" else torch.zeros(v_shape, dtype=dtype, device=device))
+            self._v.append(k if grp.spec.latent else torch.zeros(v_shape, dtype=dtype, device=device))
             for j, layer in enumerate(grp.layers):
                 self.layer_slot[layer] = (g, j)
         # hybrids: layer -> recurrent state with one row per engine slot; ``step_meta`` is the running step's batch
@@ -186,7 +199,7 @@ class PagedKVCache:
             view = PagedLayerView(None, None)        # a layer without keys / values (recurrent mixer only)
         else:
             g, j = slot
-            view = PagedLatentView(self._k[g][j]) if self.groups[g].kind == "latent" else \
+            view = PagedLatentView(self._k[g][j], group=g) if self.groups[g].spec.latent else \
                 PagedLayerView(self._k[g][j], self._v[g][j], group=g)
         pool = self.linear.get(layer)
         if pool is None:
@@ -304,6 +317,7 @@ class PagedBatchCache(PagedKVCache):
         meta = PagedBatchMeta(cu_q=torch.tensor(cu, dtype=torch.int32, device=dev),
                               kv_lens=torch.tensor(self._lens, dtype=torch.int32, device=dev), page_table=self._table,
                               slot_mapping=slots, max_q=max(new_tokens), num_seqs=self.batch, slot_ids=self._slots,
+                              spans=list(zip(new_tokens, self._lens)),
                               group_tables=tables, group_slots=[slots] * (self.num_groups - 1))
         self.step_meta = meta
         return meta, p
@@ -378,8 +392,8 @@ class PagedLatentView:
 
     linear_state = None
 
-    def __init__(self, pages: torch.Tensor):
-        self.pages = pages                  # [P, page, 1, kv_lora_rank + rope_dim]
+    def __init__(self, pages: torch.Tensor, group: int = 0):
+        self.pages, self.group = pages, group        # [P, page, 1, kv_lora_rank + rope_dim]
 
     def attend_latent(self, mla, q_nope, q_rope, latent, k_rope, meta: PagedBatchMeta):
         """q_nope ``[1,T,H,nope]``, q_rope ``[1,T,H,rope]`` (rotated), latent ``[1,T,L]`` (normalised), k_rope

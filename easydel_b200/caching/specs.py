@@ -12,6 +12,7 @@ group.
 from __future__ import annotations
 
 from dataclasses import dataclass, field
+from typing import ClassVar
 
 PAGE_TOKENS = 128
 
@@ -31,13 +32,17 @@ class KVCacheSpec:
     kind: str = "full"
     v_head_dim: int = 0          # 0 = values are as wide as keys
 
+    #: rows are keys and values at once (latent attention): no value pool
+    latent: ClassVar[bool] = False
+
     @property
     def value_dim(self) -> int:
         return self.v_head_dim or self.head_dim
 
     @property
     def page_size_bytes(self) -> int:
-        return self.page_size * self.num_kv_heads * (self.head_dim + self.value_dim) * self.element_size
+        width = self.head_dim if self.latent else self.head_dim + self.value_dim
+        return self.page_size * self.num_kv_heads * width * self.element_size
 
     def tokens_kept(self, context: int) -> int:
         return context
@@ -108,10 +113,17 @@ class MLAAttentionSpec(KVCacheSpec):
     """One row ``[latent | rotary key]`` per token, shared by every head; no separate value pool."""
 
     kind: str = "latent"
+    latent: ClassVar[bool] = True
 
-    @property
-    def page_size_bytes(self) -> int:
-        return self.page_size * self.num_kv_heads * self.head_dim * self.element_size
+
+@dataclass(frozen=True)
+class SlidingLatentSpec(SlidingWindowSpec):
+    """Latent rows of which only the last ``sliding_window`` are ever read."""
+
+    latent: ClassVar[bool] = True
+
+    def group_key(self) -> tuple:
+        return ("sliding_latent", *super().group_key()[1:])
 
 
 @dataclass(frozen=True)
@@ -159,6 +171,8 @@ def layer_spec(info, element_size: int = 2, tp_size: int = 1, page_size: int = P
     common = dict(page_size=page_size, num_kv_heads=kvh, head_dim=info.head_dim, element_size=element_size,
                   v_head_dim=info.v_head_dim if info.v_head_dim != info.head_dim else 0)
     if info.layer_type == "latent_attention":
+        if info.sliding_window:
+            return SlidingLatentSpec(sliding_window=int(info.sliding_window), **common)
         return MLAAttentionSpec(**common)
     if info.sliding_window:
         return SlidingWindowSpec(sliding_window=int(info.sliding_window), **common)

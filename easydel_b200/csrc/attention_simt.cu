@@ -1,4 +1,4 @@
-// Paged causal attention on the general-purpose cores: any head sizes up to 512 (query / key) and 1024 (value), bf16 or
+// Paged causal attention on the general-purpose cores: any head sizes up to 2048 (query / key) and 1024 (value), bf16 or
 // fp32 storage, all arithmetic in fp32. It serves fp32 models (true 32-bit products, which the tensor cores do not have)
 // and head sizes outside the tensor-core kernels' tiles.
 //
@@ -11,7 +11,7 @@ namespace edl {
 namespace {
 
 constexpr int ST = 128;      // threads = keys per tile = tokens per page
-constexpr int MAX_D = 512;
+constexpr int MAX_D = 2048;
 constexpr int MAX_VC = 8;    // value columns per thread (Dv <= 1024)
 
 __device__ __forceinline__ float f_of(float v) { return v; }

@@ -139,7 +139,7 @@ template <typename TO, int NV>
 __global__ void __launch_bounds__(NT)
 norm_shift_rows_kernel(const float* __restrict__ x, const float* __restrict__ w, const float* __restrict__ mu, float eps,
                        int rows, int W, const int* __restrict__ cu, int nseq, const int* __restrict__ slots,
-                       float* __restrict__ state, long long ld_state, TO* __restrict__ out, int per) {
+                       float* __restrict__ state, long long ld_state, float offset, TO* __restrict__ out, int per) {
   __shared__ float2 red[NT / 32];
   constexpr int STEP = NT * 4;
   const int r0 = blockIdx.x * per, r1 = min(rows, r0 + per);
@@ -151,6 +151,8 @@ norm_shift_rows_kernel(const float* __restrict__ x, const float* __restrict__ w,
     const int c = threadIdx.x * 4 + k * STEP;
     if (c < W) {
       ldv<4>(w + c, wv[k]);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) wv[k][j] += offset;
       if (mu) ldv<4>(mu + c, mv[k]);
     }
   }
@@ -245,7 +247,7 @@ template <typename TO, int VEC, int NV>
 __global__ void __launch_bounds__(NT)
 norm_shift_kernel(const float* __restrict__ x, const float* __restrict__ w, const float* __restrict__ mu, float eps,
                   int rows, int W, const int* __restrict__ cu, int nseq, const int* __restrict__ slots,
-                  float* __restrict__ state, long long ld_state, TO* __restrict__ out) {
+                  float* __restrict__ state, long long ld_state, float offset, TO* __restrict__ out) {
   __shared__ float2 red[NT / 32];
   const int r = blockIdx.x;
   const float inv_w = 1.f / (float)W;
@@ -297,7 +299,10 @@ norm_shift_kernel(const float* __restrict__ x, const float* __restrict__ w, cons
     float wv[VEC], h[VEC];
     ldv<VEC>(w + c, wv);
 #pragma unroll
-    for (int j = 0; j < VEC; ++j) h[j] = av[j] * ra * wv[j];
+    for (int j = 0; j < VEC; ++j) {
+      wv[j] += offset;
+      h[j] = av[j] * ra * wv[j];
+    }
     if (mu) {
       float m[VEC], before[VEC], o[VEC];
       ldv<VEC>(mu + c, m);
@@ -343,7 +348,7 @@ norm_shift_kernel(const float* __restrict__ x, const float* __restrict__ w, cons
       ldv<VEC>(xl + c, v);
       ldv<VEC>(w + c, wv);
 #pragma unroll
-      for (int j = 0; j < VEC; ++j) v[j] = v[j] * rl * wv[j];
+      for (int j = 0; j < VEC; ++j) v[j] = v[j] * rl * (wv[j] + offset);
       stv<VEC>(st + c, v);
     }
   }
@@ -540,13 +545,14 @@ int blocks_for(long long work, int per_block, int waves) {
 
 template <typename TO, int VEC>
 int launch_norm_shift(const float* x, const float* w, const float* mu, float eps, int rows, int W, const int* cu,
-                      int nseq, const int* slots, float* state, long long ld_state, TO* out, cudaStream_t s) {
+                      int nseq, const int* slots, float* state, long long ld_state, float offset, TO* out,
+                      cudaStream_t s) {
   const int nv = (W + NT * VEC - 1) / (NT * VEC);
   if (VEC == 4 && nv <= 4 && rows >= 16 * sm_count()) {
     const int per = mu ? 8 : 2;
     const int grid = (rows + per - 1) / per;
 #define EDL_NR(N) \
-  norm_shift_rows_kernel<TO, N><<<grid, NT, 0, s>>>(x, w, mu, eps, rows, W, cu, nseq, slots, state, ld_state, out, per)
+  norm_shift_rows_kernel<TO, N><<<grid, NT, 0, s>>>(x, w, mu, eps, rows, W, cu, nseq, slots, state, ld_state, offset, out, per)
     if (nv <= 1) EDL_NR(1);
     else if (nv <= 2) EDL_NR(2);
     else EDL_NR(4);
@@ -554,7 +560,7 @@ int launch_norm_shift(const float* x, const float* w, const float* mu, float eps
     return check_cuda(cudaGetLastError(), "norm_shift launch");
   }
 #define EDL_NS(N) \
-  norm_shift_kernel<TO, VEC, N><<<rows, NT, 0, s>>>(x, w, mu, eps, rows, W, cu, nseq, slots, state, ld_state, out)
+  norm_shift_kernel<TO, VEC, N><<<rows, NT, 0, s>>>(x, w, mu, eps, rows, W, cu, nseq, slots, state, ld_state, offset, out)
   if (nv <= 1) EDL_NS(1);
   else if (nv <= 2) EDL_NS(2);
   else if (nv <= 4) EDL_NS(4);
@@ -606,12 +612,12 @@ EDL_HOST_API int edl_cast_rows(const float* x, void* out, int f32, long long ld_
   return check_cuda(cudaGetLastError(), "cast_rows launch");
 }
 
-// out [rows, W] = rms_norm(x) * w, blended with the previous row's norm by mu when mu is given. cu [nseq + 1] bounds the
+// out [rows, W] = rms_norm(x) * (w + offset), blended with the previous row's norm by mu when mu is given. cu [nseq + 1] bounds the
 // sequences on the row axis; state [*, ld_state] fp32 holds, per slot, the normalised row before the step's first one
 // (null: sequences start here) and is updated to the step's last row.
 EDL_HOST_API int edl_norm_shift(const float* x, const float* w, const float* mu, float eps, int rows, int W,
-                                const int* cu, int nseq, const int* slots, float* state, long long ld_state, void* out,
-                                int f32, void* stream) {
+                                const int* cu, int nseq, const int* slots, float* state, long long ld_state, float offset,
+                                void* out, int f32, void* stream) {
   if (rows <= 0) return 0;
   if (mu && (!cu || nseq <= 0 || (state && !slots))) {
     set_last_error("edl_norm_shift: a token shift needs sequence bounds, and slots for a state");
@@ -621,11 +627,11 @@ EDL_HOST_API int edl_norm_shift(const float* x, const float* w, const float* mu,
   const bool v4 = W % 4 == 0 && ld_state % 4 == 0 && al(x, 16) && al(w, 16) && (!mu || al(mu, 16)) &&
                   (!state || al(state, 16)) && al(out, f32 ? 16 : 8);
   if (f32)
-    return v4 ? launch_norm_shift<float, 4>(x, w, mu, eps, rows, W, cu, nseq, slots, state, ld_state, (float*)out, s)
-              : launch_norm_shift<float, 1>(x, w, mu, eps, rows, W, cu, nseq, slots, state, ld_state, (float*)out, s);
-  return v4 ? launch_norm_shift<__nv_bfloat16, 4>(x, w, mu, eps, rows, W, cu, nseq, slots, state, ld_state,
+    return v4 ? launch_norm_shift<float, 4>(x, w, mu, eps, rows, W, cu, nseq, slots, state, ld_state, offset, (float*)out, s)
+              : launch_norm_shift<float, 1>(x, w, mu, eps, rows, W, cu, nseq, slots, state, ld_state, offset, (float*)out, s);
+  return v4 ? launch_norm_shift<__nv_bfloat16, 4>(x, w, mu, eps, rows, W, cu, nseq, slots, state, ld_state, offset,
                                                   (__nv_bfloat16*)out, s)
-            : launch_norm_shift<__nv_bfloat16, 1>(x, w, mu, eps, rows, W, cu, nseq, slots, state, ld_state,
+            : launch_norm_shift<__nv_bfloat16, 1>(x, w, mu, eps, rows, W, cu, nseq, slots, state, ld_state, offset,
                                                   (__nv_bfloat16*)out, s);
 }
 

@@ -82,6 +82,7 @@ class ModelRunner:
         self._tok_host = [torch.zeros(B + 1, dtype=torch.int64, pin_memory=pin) for _ in range(2)]
         self._tok_dev = torch.zeros(B + 1, dtype=torch.int64, device=dev)
         self._launches = 0
+        self._spans: list[tuple[int, int]] | None = None     # (new tokens, keys) of the staged step's sequences
         # Decode-only greedy steps are replayed from CUDA graphs, one per power-of-two batch bucket
         # (the reference compiles (tokens, requests) buckets ahead of time: runners/execution_manager.py:1291-1405).
         import os
@@ -89,7 +90,7 @@ class ModelRunner:
         self.use_graphs = dev.type == "cuda" and os.environ.get("EDL_ESURGE_CUDA_GRAPHS", "1") != "0"
         latent_kernel = bool(cache.latent and cache.k.shape[-1] == 576)    # the 512 + 64 layout has a decode kernel
         stream32 = getattr(self._lm.spec, "residual_f32", False)   # every head size has a capturable kernel there
-        if not getattr(cache, "states_in_place", True) or getattr(cache, "compressed", False) or (cache.latent and not latent_kernel) or \
+        if not getattr(cache, "states_in_place", True) or getattr(cache, "compressed", False) or (cache.latent and not latent_kernel and not stream32) or \
                 (not cache.latent and not stream32 and model.spec.head_dim not in (64, 128)):
             self.use_graphs = False     # these serving paths are tensor code with host-side steps: run eagerly
         self._seq_slots = torch.zeros(max_num_seqs, dtype=torch.int64, device=dev)
@@ -168,7 +169,7 @@ class ModelRunner:
                               request_distribution=(num_decode, B, B),
                               num_splits=self._decode_splits(B) if (max_q == 1 and T == B) else 1,
                               seq_slots=self._seq_slots[:B] if self.cache.linear else None,
-                              slot_ids=self._dviews[7][:B])
+                              slot_ids=self._dviews[7][:B], spans=self._spans)
         if self.num_groups > 1:
             extra = self._dviews[10:]
             meta.group_slots = [extra[2 * g][:T] for g in range(self.num_groups - 1)]
@@ -360,6 +361,7 @@ class ModelRunner:
                 cu_np[:B + 1] = np.arange(B + 1, dtype=np.int32)
                 last_np[:B] = np.arange(B, dtype=np.int32)
             max_q = 1
+        spans = []
         for b, s in enumerate(sched if not fast else ()):
             req = s.request
             n, st = s.num_new_tokens, s.start
@@ -396,6 +398,7 @@ class ModelRunner:
                 self._slot_npages[req.slot] = len(pg)
                 self._slot_epoch[req.slot] = req.pages_epoch
             kv_np[b] = st + n
+            spans.append((n, st + n))
             o += n
             cu_np[b + 1] = o
             last_np[b] = o - 1
@@ -403,6 +406,7 @@ class ModelRunner:
             sp = req.sampling_params
             any_pen |= sp.needs_penalties
             any_random |= not sp.is_greedy
+        self._spans = spans if max_q > 1 else None
         if self.num_groups > 1:
             self._fill_extra_groups(sched, B)
         decode_only = max_q == 1 and not any_pen and not any_random

@@ -212,9 +212,11 @@ def _describe_layer(i: int, layer) -> list[LayerOperationInfo]:
                                       False, True))
         return out
     if spec is not None and getattr(spec, "mla", None) is not None:
+        m = spec.mla
+        width = m["kv_rank"] + m["rot_dim"] if "kv_rank" in m else m["kv_lora_rank"] + m["qk_rope_head_dim"]
         out.append(LayerOperationInfo(i, "latent_attention", "flash_attention", "latent_paged_attention", None,
                                       CacheType.TRANSFORMER | CacheType.LATENT_PAGES | CacheType.HYBRID, True, False,
-                                      num_kv_heads=1, head_dim=spec.mla["kv_lora_rank"] + spec.mla["qk_rope_head_dim"]))
+                                      getattr(attn, "sliding_window", None) or None, num_kv_heads=1, head_dim=width))
         return out
     if attn is not None:
         window = getattr(attn, "sliding_window", None) or None

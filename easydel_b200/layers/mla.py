@@ -13,7 +13,7 @@ from __future__ import annotations
 import torch
 from torch import nn
 
-from ..ops import functional as F
+from ..ops import functional as F, latent, stream
 from ..ops import reference as R
 from .linears import ColumnParallelLinear, RowParallelLinear
 from .norms import RMSNorm
@@ -196,3 +196,77 @@ class MLAttention(nn.Module):
             # library attention for them on a GPU and the dense form on CPU
             o = F.attention(qf, k, v, causal=True, scale=self.scale, segment_ids=segment_ids)
         return self.o_proj(o.reshape(B, T, self.H * self.vd).to(hidden.dtype))
+
+
+class LatentStreamAttention(nn.Module):
+    """Latent attention of layers over an fp32 residual stream, with a sliding window, a sink per head, rotary pairs on
+    neighbouring channels of the rotary part and an output gate (each optional).
+
+    One packed product gives the queries of every head, the latent, the shared rotary key and the gate; the two
+    up-projections (unrotated keys, values) are stacked. The cache holds rows ``[normalised latent | rotated key]``;
+    :mod:`..ops.latent` runs the attention. The output projection is applied by the decoder layer."""
+
+    def __init__(self, hidden_size: int, heads: int, *, dim: int, rot_dim: int, vdim: int, kv_rank: int, scale: float,
+                 rope_base: float = 10000.0, rope_dims: int | None = None, sliding_window: int | None = None,
+                 use_sinks: bool = False, output_gate: bool = False, norm_eps: float = 1e-6, layer_idx: int = 0,
+                 dtype=torch.bfloat16, init_std: float = 0.02):
+        super().__init__()
+        self.heads, self.dim, self.rot_dim, self.vdim, self.kv_rank = heads, dim, rot_dim, vdim, kv_rank
+        self.scale, self.sliding_window, self.output_gate = scale, sliding_window, output_gate
+        self.eps, self.layer_idx = norm_eps, layer_idx
+        widths = (heads * (dim + rot_dim), kv_rank + rot_dim) + ((heads * vdim,) if output_gate else ())
+        kw = dict(dtype=dtype, init_std=init_std)
+        proj = ColumnParallelLinear(hidden_size, widths, bias=False, **kw)
+        if output_gate:
+            self.qdg_proj = proj
+        else:
+            self.qd_proj = proj
+        self.kv_norm = RMSNorm(kv_rank, norm_eps, torch.float32)
+        self.ukv_proj = ColumnParallelLinear(kv_rank, (heads * dim, heads * vdim), bias=False, **kw)
+        self.o_proj = RowParallelLinear(heads * vdim, hidden_size, bias=False, **kw)
+        self.sinks = nn.Parameter(torch.zeros(heads, dtype=torch.float32)) if use_sinks else None
+        dims = rot_dim if rope_dims is None else rope_dims
+        if dims % 2 or dims > rot_dim:
+            raise ValueError(f"{dims} rotated channels of a rotary part of {rot_dim}")
+        self.rope_base, self.rope_dims = float(rope_base), dims
+        self.tiles = latent.tiles_support(self)
+        self._freq: torch.Tensor | None = None
+        self._expansion: tuple | None = None
+
+    def frequencies(self, device) -> torch.Tensor:
+        if self._freq is None or self._freq.device != device:
+            self._freq = latent.pair_frequencies(self.rope_base, self.rope_dims, device)
+        return self._freq
+
+    def expansion(self) -> torch.Tensor:
+        """The product that turns cache rows into keys and values, rebuilt when the up-projections change."""
+        w = self.ukv_proj.weight
+        key = (w.data_ptr(), w._version)
+        if self._expansion is None or self._expansion[0] != key:
+            self._expansion = (key, latent.expansion_weight(w.detach(), self.heads, self.dim, self.rot_dim, self.vdim,
+                                                            self.kv_rank))
+        return self._expansion[1]
+
+    def mix_stream(self, h: torch.Tensor, step, cache_view=None) -> torch.Tensor:
+        """h ``[T, hidden]`` (all sequences on one axis) -> gated heads ``[T, heads * vdim]``. ``step``:
+        :class:`..modules._base.decoder.StreamStep`."""
+        H, D, R, L = self.heads, self.dim, self.rot_dim, self.kv_rank
+        proj = stream.linear(h, (self.qdg_proj if self.output_gate else self.qd_proj).weight)
+        freq = self.frequencies(proj.device)
+        if cache_view is not None:
+            meta, pages = step.meta, cache_view.pages
+            latent.prologue(proj, (H, D, R, L), self.kv_norm.weight, self.eps, freq, step.positions,
+                            meta.slots_of(cache_view.group), pages)
+            return latent.attend(self, proj, pages, meta, meta.table_of(cache_view.group), cache_view.group)
+        # no cache (autograd): the batch's rows are equally long
+        q, c, kr, gate = latent.split_packed(proj, H, D, R, L)
+        pos = step.positions
+        q = torch.cat([q[..., :D], latent.rotate_pairs(q[..., D:], pos, freq)], -1)
+        c, kr = latent.latent_norm(c, self.kv_norm.weight, self.eps), latent.rotate_pairs(kr, pos, freq)
+        B = step.batch
+        fold = lambda t: t.reshape(B, t.shape[0] // B, *t.shape[1:])  # noqa: E731
+        up = self.ukv_proj.weight
+        o = latent.expanded_attention(self, fold(q), fold(c), fold(kr), up[:H * D].view(H, D, L),
+                                      up[H * D:].view(H, self.vdim, L), step.segment_ids)
+        o = o.reshape(h.shape[0], H * self.vdim).to(proj.dtype)
+        return o * torch.sigmoid(gate.float()).to(o.dtype) if self.output_gate else o

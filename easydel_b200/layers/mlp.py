@@ -58,7 +58,13 @@ class PlainMLP(nn.Module):
     def hidden(self, x: torch.Tensor) -> torch.Tensor:
         """The activations between the two products."""
         z = self.fc1(x)
-        return stream.xielu(z, self.act_params) if self.act == "xielu" else ACT2FN[self.act](z)
+        if self.act == "xielu":
+            return stream.xielu(z, self.act_params)
+        return stream.gelu_erf(z) if self.act == "gelu" and stream.on_kernels(z) else ACT2FN[self.act](z)
+
+    def stream_rows(self, h: torch.Tensor) -> torch.Tensor:
+        """Branch of a layer over an fp32 residual stream: fp32 rows for :func:`..ops.stream.post_norm`."""
+        return stream.linear(self.hidden(h), self.fc2.weight, self.fc2.bias, torch.float32)
 
     def forward(self, x: torch.Tensor) -> torch.Tensor:
         return self.fc2(self.hidden(x))

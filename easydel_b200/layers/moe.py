@@ -22,7 +22,7 @@ import torch
 from torch import nn
 
 from ..ops import functional as F
-from ..ops import grouped as G
+from ..ops import grouped as G, reference as R, stream
 from .linears import ColumnParallelLinear
 from .mlp import GatedMLP
 
@@ -128,8 +128,12 @@ class MoEBlock(nn.Module):
                  router_jitter_eps: float = 0.01, routing_strategy: str | None = None,
                  capacity_factor: float | None = None,
                  load_balancing_strategy: str = MoeLoadBalancingStrategy.STANDARD, lbl_coef: float | None = None,
-                 rzl_coef: float | None = None, expert_tensor_mode: bool = False):
+                 rzl_coef: float | None = None, expert_tensor_mode: bool = False, act_limit: float | None = None):
         super().__init__()
+        # clamped gated units ("gptoss_swiglu"): where the gate and the linear branch are cut off
+        if act_limit is not None:
+            act = R.clamped_swiglu(act_limit)
+        self.act_limit = act_limit
         # Expert tensor mode (the reference's ``use_expert_tensor_mode``, easydel/layers/linears/_linear_moe.py:113,
         # :330): the experts are spread over the TENSOR-parallel group instead of an expert-parallel one. Every rank
         # of that group sees the same tokens, so nothing is exchanged: a rank runs its own experts on all tokens and
@@ -331,3 +335,21 @@ class MoEBlock(nn.Module):
                 s = s * torch.sigmoid(self.shared_expert_gate(x2).float()).to(s.dtype)
             y = y + s
         return y.view(shape), logits
+
+    # ------------------------------------------------------------------ fp32-stream layers
+    def stream_rows(self, h: torch.Tensor):
+        """Branch of a layer over an fp32 residual stream: h ``[T, H]`` -> what :func:`..ops.stream.post_norm` adds to the
+        stream, either expert rows with their weights (kernels) or fp32 rows. Router logits and scores are fp32."""
+        logits = stream.linear(h, self.gate.weight, self.gate.bias, torch.float32)
+        plain = self.scoring == "sigmoid" and self.norm_topk_prob and self.routing_strategy is None and \
+            self.n_group == 1 and self.capacity_factor is None and self.routed_scaling_factor == 1.0
+        if self.act_limit is None or not plain or self.shared_experts is not None or self.ep_size > 1 or \
+                self.gate_up_proj.bias is not None:
+            raise NotImplementedError("fp32-stream experts: sigmoid scores, renormalised, clamped gated units")
+        if stream.on_kernels(h):
+            from ..ops import moe_kernels as MK
+
+            r = MK.SigmoidRouting(logits, self.e_score_correction_bias, self.top_k)
+            return MK.clamped_experts(h, r, self.gate_up_proj.weight, self.down_proj.weight, self.act_limit)
+        w, idx, _ = self.route(logits)
+        return G.moe_ffn(h, self.gate_up_proj.weight, self.down_proj.weight, w, idx, self.act).float()

@@ -40,6 +40,8 @@ from . import kimi_vl  # noqa: F401
 from .kimi_vl import *  # noqa: F401,F403
 from . import llama4  # noqa: F401
 from .llama4 import *  # noqa: F401,F403
+from . import disunex  # noqa: F401
+from .disunex import *  # noqa: F401,F403
 from . import rakevik  # noqa: F401
 from .rakevik import *  # noqa: F401,F403
 

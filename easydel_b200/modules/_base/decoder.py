@@ -54,6 +54,7 @@ class MoESpec:
     expert_init_std: float = 0.01
     expert_bias: bool = False         # per-expert biases on both expert projections (GPT-OSS)
     expert_act: str | None = None     # gated activation of the experts when it differs from the dense MLP's
+    expert_limit: float | None = None  # clamped gated units: the limit of both branches (replaces ``expert_act``)
     scale_input: bool = False         # routing score applied to the experts' input (Llama-4)
     router_jitter_eps: float = 0.01   # margin of the sparsemixer routing (Phi-3.5-MoE)
     routing_strategy: str | None = None          # top_k | top_k_ndiv | switch | expert_choice | hash; None = by scoring
@@ -98,7 +99,8 @@ class ArchSpec:
     attn_scale: float | None = None
     sliding_window: int | None = None
     layer_types: tuple[str, ...] | None = None  # per layer: "full" | "sliding" | "nope" (full, no rope)
-    residual: str = "pre"             # pre | parallel | post (norm applied to the branch output, OLMo2)
+    residual: str = "pre"             # pre | parallel | post (norm applied to the branch output, OLMo2) | post_sum
+                                      # (x <- norm(residual_alpha x + branch), branches read x; fp32-stream models)
     sandwich_norm: bool = False       # extra norms after attention / MLP outputs (Gemma2/3)
     shared_parallel_norm: bool = True  # parallel residual with one norm (GPT-J, Phi) vs two (NeoX)
     use_sinks: bool = False
@@ -111,7 +113,9 @@ class ArchSpec:
     logit_scale: float | None = None  # Cohere / Granite style multiplier on logits
     residual_multiplier: float | None = None
     embedding_multiplier: float | None = None
-    mla: dict | None = None           # kwargs of layers.mla.MLAttention: latent attention instead of MHA / GQA
+    residual_alpha: float = 1.0       # weight of the stream in a "post_sum" layer
+    mla: dict | None = None           # kwargs of layers.mla.MLAttention (fp32-stream models: of LatentStreamAttention):
+                                      # latent attention instead of MHA / GQA
     linear_attn: dict | None = None   # kwargs of layers.linear_attention.GatedDeltaNet for layers of type "linear"
     attn_output_gate: bool = False    # sigmoid gate on the attention output, emitted by the query projection
     attn_chunk_size: int | None = None  # block-diagonal attention on the rotary layers of a rope / nope mix (Llama-4)
@@ -134,6 +138,8 @@ class ArchSpec:
     loop: tuple[int, int, int] | None = None  # (start, stop, times): layers start .. stop-1 run ``times`` times in a row
                                       # with the same weights, each run with a cache of its own; before a pass the
                                       # stream becomes W [x ; embedding output] + step[pass] (fp32-stream models)
+    layer_runs: tuple[int, ...] | None = None  # layer of every run, in order, when layers are used more than once (each
+                                      # run with a cache of its own; fp32-stream models)
     residual_mlp: bool = False        # Arctic: MoE layers add a dense hidden-sized MLP branch after attention while
                                       # the experts read the layer input (norm of x, not of x + attention)
 
@@ -162,7 +168,7 @@ class LayerSlotState:
 
 def _norm(spec: ArchSpec, dtype) -> nn.Module:
     if spec.residual_f32:
-        return RMSNorm(spec.hidden_size, spec.norm_eps, torch.float32)
+        return RMSNorm(spec.hidden_size, spec.norm_eps, torch.float32, offset=spec.norm_offset)
     if spec.norm == "rms":
         return RMSNorm(spec.hidden_size, spec.norm_eps, dtype, offset=spec.norm_offset)
     if spec.norm == "layer_noparam":
@@ -228,6 +234,11 @@ class DecoderLayer(nn.Module):
 
             self.linear_attn = GatedDeltaNet(spec.hidden_size, layer_idx=layer_idx, dtype=dtype,
                                              init_std=spec.init_std, norm_eps=spec.norm_eps, **spec.linear_attn)
+        elif spec.mla is not None and spec.residual_f32:
+            from ...layers.mla import LatentStreamAttention
+
+            self.self_attn = LatentStreamAttention(spec.hidden_size, spec.num_heads, norm_eps=spec.norm_eps,
+                                                   layer_idx=layer_idx, dtype=dtype, init_std=spec.init_std, **spec.mla)
         elif spec.mla is not None:
             from ...layers.mla import MLAttention
 
@@ -292,7 +303,8 @@ class DecoderLayer(nn.Module):
                                 shared_gate=moe.shared_gate, dtype=dtype, init_std=spec.init_std,
                                 expert_init_std=moe.expert_init_std, ep_size=ep_size, ep_rank=ep_rank,
                                 ep_group=ep_group, tp_size=tp_size, tp_rank=tp_rank, tp_group=tp_group,
-                                expert_tensor_mode=bool(getattr(config, "use_expert_tensor_mode", False)))
+                                expert_tensor_mode=bool(getattr(config, "use_expert_tensor_mode", False)),
+                                act_limit=moe.expert_limit)
         elif spec.intermediate_size == 0:      # a layer with a mixer only
             self.mlp = None
         elif spec.mlp == "gated":
@@ -306,7 +318,11 @@ class DecoderLayer(nn.Module):
             self.residual_layernorm = _norm(spec, dtype)
             self.residual_mlp = GatedMLP(spec.hidden_size, spec.hidden_size, spec.act, False, dtype, spec.init_std,
                                          tp_size, tp_rank, tp_group)
-        if spec.residual == "post":
+        if spec.residual == "post_sum":
+            self.post_attention_layernorm = _norm(spec, dtype)
+            if self.mlp is not None:
+                self.post_feedforward_layernorm = _norm(spec, dtype)
+        elif spec.residual == "post":
             self.post_attention_layernorm = _norm(spec, dtype)
             self.post_feedforward_layernorm = _norm(spec, dtype)
         else:
@@ -372,8 +388,24 @@ class DecoderLayer(nn.Module):
             x = stream.linear_add_(x, self.mlp.hidden(h), self.mlp.fc2.weight)
         return x
 
+    def _forward_post_sum(self, x: torch.Tensor, h: torch.Tensor, step: StreamStep, view):
+        """One layer on the fp32 stream ``x [T, hidden]`` that normalises after the sum. ``h`` holds the same rows in the
+        operand type: the norm that closes a branch writes both, so a branch reads nothing else."""
+        spec = self.spec
+        attn, n1 = self.self_attn, self.post_attention_layernorm
+        o = attn.mix_stream(h, step, view)
+        branch = stream.linear(o, attn.o_proj.weight, out_dtype=torch.float32)
+        x, h = stream.post_norm(x, branch, spec.residual_alpha, n1.weight, spec.norm_eps, h.dtype, n1.offset)
+        if self.mlp is not None:
+            n2 = self.post_feedforward_layernorm
+            branch = self.mlp.stream_rows(h)
+            x, h = stream.post_norm(x, branch, spec.residual_alpha, n2.weight, spec.norm_eps, h.dtype, n2.offset)
+        return x, h
+
     def forward(self, x, pending, positions, segment_ids=None, cache_view=None, attn_meta=None):
         spec = self.spec
+        if spec.residual == "post_sum":
+            return *self._forward_post_sum(x, pending, attn_meta, cache_view), None
         if spec.residual_f32:
             return self._forward_stream(x, attn_meta, cache_view), None, None
         rl = None
@@ -475,6 +507,8 @@ class DecoderModel(EasyDeLBaseModule):
             self.loop_in = ColumnParallelLinear(2 * spec.hidden_size, spec.hidden_size, bias=False, dtype=pd,
                                                 init_std=spec.init_std)
             self.loop_step = nn.Parameter(torch.zeros(times, spec.hidden_size, dtype=pd))
+        elif spec.layer_runs is not None:
+            self.layer_runs = list(spec.layer_runs)
         self._setup_sequence_parallel(config)
         self._setup_context_parallel(config)
 
@@ -679,6 +713,9 @@ def _forward_stream(self, input_ids, inputs_embeds, attention_mask, position_ids
         flat = flat[index]
     n = flat.numel() if flat is not None else (index.numel() if index is not None else B * T)
     operand = right = None
+    h = None                              # "post_sum" layers: the stream's rows in the operand type
+    if spec.residual == "post_sum":
+        right = h = torch.empty(n, W, dtype=self.embed_tokens.weight.dtype, device=self.device)
     if spec.loop is not None:             # [x ; x0]: x0 is written once, x before every pass
         operand = torch.empty(n, 2 * W, dtype=self.loop_in.weight.dtype, device=self.device)
         right = operand[:, W:]
@@ -705,8 +742,8 @@ def _forward_stream(self, input_ids, inputs_embeds, attention_mask, position_ids
         if hidden is not None:
             hidden.append(x.clone())
         view = cache.view(run) if cache is not None else None
-        x, _, _ = self.layers[i](x, None, step.positions, None, view, step)
-    x = stream.norm_shift(x, self.norm.weight, spec.norm_eps, dt)
+        x, h, _ = self.layers[i](x, h, step.positions, None, view, step)
+    x = stream.norm_shift(x, self.norm.weight, spec.norm_eps, dt, offset=self.norm.offset)
 
     def unflatten(t):
         if index is not None:

@@ -30,6 +30,13 @@ _SPLITK_OFFSETS: dict[tuple, torch.Tensor] = {}
 _SM_COUNT: dict[int, int] = {}
 
 
+def sm_count(device) -> int:
+    idx = device.index or 0
+    if idx not in _SM_COUNT:
+        _SM_COUNT[idx] = torch.cuda.get_device_properties(device).multi_processor_count
+    return _SM_COUNT[idx]
+
+
 def _splitk_plan(M: int, N: int, K: int, device) -> int:
     """Number of K slices for a skinny GEMM (1 = use the plain kernel).
 

@@ -234,3 +234,78 @@ def grouped_linear(x_sorted, w, group_sizes):
     xs = r.gather(x_sorted.contiguous())
     ys = _grouped_fwd(r, xs, w)
     return ys[r.slot_pos.long()]
+
+
+# ------------------------------------------------------------------------------------------------ fp32-stream inference
+_lib.register("edl_moe_sigmoid_route", i32, [vp, vp, i32, i32, i32, vp, vp, vp])
+_lib.register("edl_moe_sigmoid_route_small", i32, [vp, vp, i32, i32, i32, vp, vp, i32, vp, vp, vp, vp])
+_lib.register("edl_moe_clamped_glu", i32, [vp, i32, vp, vp, vp, i32, i64, _lib.f32, _lib.f32, vp])
+_lib.register("edl_moe_grouped_simt", i32, [vp, i32, i64, vp, i32, vp, vp, vp, vp, i32, i32, i32, vp])
+
+SMALL_ROUTE_PAIRS = 4096      # (token, choice) pairs that one launch routes and buckets
+
+
+class ExpertRows:
+    """Outputs of the routed experts before they are combined: token t's branch is ``sum_s weights[t, s] *
+    ys[pos[t, s]]``. The norm that follows an fp32-stream layer's branch takes them in this form
+    (:func:`.stream.post_norm`)."""
+
+    def __init__(self, ys: torch.Tensor, weights: torch.Tensor, pos: torch.Tensor):
+        self.ys, self.weights, self.pos = ys, weights, pos
+        self.k = weights.shape[1]
+
+    def combine(self) -> torch.Tensor:
+        p = self.pos.view(self.weights.shape).long()
+        return (self.ys[p.clamp_min(0)].float() * (self.weights * (p >= 0))[..., None]).sum(1)
+
+
+class SigmoidRouting(Routing):
+    """Routing tables straight from fp32 router logits ``[T, E]``: sigmoid scores, choice by score + ``correction``,
+    weights = the chosen scores over their sum. A decode step's few tokens take one launch."""
+
+    def __init__(self, logits: torch.Tensor, correction: torch.Tensor | None, top_k: int):
+        T, E = logits.shape
+        dev = logits.device
+        self.weights = torch.empty(T, top_k, dtype=torch.float32, device=dev)
+        corr = _lib.ptr(correction)
+        if T * top_k > SMALL_ROUTE_PAIRS:
+            idx = torch.empty(T, top_k, dtype=torch.int64, device=dev)
+            _lib.call("edl_moe_sigmoid_route", logits.data_ptr(), corr, T, E, top_k, idx.data_ptr(),
+                      self.weights.data_ptr(), _lib.stream_ptr())
+            super().__init__(idx, E)
+            return
+        self.T, self.k, self.E = T, top_k, E
+        # every expert in use pads one ragged tile, and no more experts than pairs are in use
+        self.max_tiles = (T * top_k + 127) // 128 + min(E, T * top_k)
+        self.max_rows = self.max_tiles * 128
+        ints = torch.empty(self.max_tiles + 2 + T * top_k + self.max_rows, dtype=torch.int32, device=dev)
+        self.tile_expert, self.meta, self.slot_pos, self.row_token = torch.split(
+            ints, [self.max_tiles, 2, T * top_k, self.max_rows])
+        self.offsets = self.meta         # only the weight-gradient product reads segment offsets
+        _lib.call("edl_moe_sigmoid_route_small", logits.data_ptr(), corr, T, E, top_k, self.weights.data_ptr(),
+                  self.tile_expert.data_ptr(), self.max_tiles, self.meta.data_ptr(), self.slot_pos.data_ptr(),
+                  self.row_token.data_ptr(), _lib.stream_ptr())
+
+
+def clamped_experts(x: torch.Tensor, r: SigmoidRouting, w_gate_up: torch.Tensor, w_down: torch.Tensor, limit: float,
+                    alpha: float = 1.702) -> ExpertRows:
+    """Routed experts with the clamped gated unit, inference only: rows in use are computed, padding rows of the
+    segments stay undefined and are never read back."""
+    F2, H = w_gate_up.shape[1:]
+    f32_ = int(x.dtype == torch.float32)
+    tiles = not f32_ and F2 % 16 == 0 and H % 8 == 0 and x.stride(0) % 8 == 0
+
+    def product(a, w, gather):
+        out = torch.empty(r.max_rows, w.shape[1], dtype=x.dtype, device=x.device)
+        if tiles:
+            return r.grouped(0, r.gather(a) if gather else a, w, out, N=w.shape[1], Kd=w.shape[2])
+        _lib.call("edl_moe_grouped_simt", a.data_ptr(), f32_, a.stride(0), r.row_token.data_ptr(), int(gather),
+                  w.data_ptr(), r.tile_expert.data_ptr(), r.meta.data_ptr(), out.data_ptr(), r.max_rows, w.shape[1],
+                  w.shape[2], _lib.stream_ptr())
+        return out
+
+    gu = product(x, w_gate_up, True)
+    a = torch.empty(r.max_rows, F2 // 2, dtype=x.dtype, device=x.device)
+    _lib.call("edl_moe_clamped_glu", gu.data_ptr(), f32_, r.row_token.data_ptr(), r.meta.data_ptr(), a.data_ptr(), F2 // 2,
+              r.max_rows, float(limit), float(alpha), _lib.stream_ptr())
+    return ExpertRows(product(a, w_down, False), r.weights, r.slot_pos)

@@ -8,6 +8,7 @@ written for clarity, not speed, and are differentiable through autograd.
 
 from __future__ import annotations
 
+import functools
 import math
 
 import torch
@@ -56,8 +57,17 @@ def _gptoss_swiglu(g, u, alpha: float = 1.702, limit: float = 7.0):
 GATED_FNS = {"gptoss_swiglu": _gptoss_swiglu}
 
 
-def gated_act(gu, act: str = "silu"):
+@functools.lru_cache(maxsize=None)
+def clamped_swiglu(limit: float, alpha: float = 1.702):
+    """The clamped unit with another limit, as an activation for :func:`gated_act`."""
+    return functools.partial(_gptoss_swiglu, alpha=alpha, limit=limit)
+
+
+def gated_act(gu, act="silu"):
+    """``act``: an activation's name (the unit is ``act(gate) * up`` unless listed above) or a function of (gate, up)."""
     g, u = gu.chunk(2, dim=-1)
+    if callable(act):
+        return act(g, u)
     if act in GATED_FNS:
         return GATED_FNS[act](g, u)
     return ACT2FN[act](g) * u

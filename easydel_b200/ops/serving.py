@@ -22,9 +22,11 @@ _lib.register("edl_attn_decode", i32, [vp, vp, vp, vp, vp, i64, i64, i64, i64, v
                                        f32,
                                        i32, i32, vp, vp, vp])
 
-_lib.register("edl_attn_mla_decode", i32, [vp, vp, vp, vp, i64, i64, vp, vp, i32, i32, i64, i32, f32, i32, vp, vp])
+_lib.register("edl_attn_mla_decode", i32, [vp, i64, i64, vp, i64, i64, vp, vp, vp, i64, vp, vp, i32, i32, i64, i32, i32, i32,
+                                            f32, i32, vp, i32, vp, vp])
 
 PAGE_SIZE = 128
+MAX_QK_DIM = 128      # widest query / key head of the tensor-core prefill kernel
 
 
 def kv_append(k: torch.Tensor, v: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor,
@@ -89,11 +91,13 @@ _lib.register("edl_attn_simt", i32, [vp, vp, vp, vp, i32, i64, i64, i64, vp, vp,
 
 def simt_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, cu_q: torch.Tensor,
                    kv_lens: torch.Tensor, page_table: torch.Tensor, *, scale: float, window: int = 0, sinks=None,
-                   out: torch.Tensor | None = None) -> torch.Tensor:
+                   out: torch.Tensor | None = None, v_dim: int | None = None) -> torch.Tensor:
     """Causal paged attention in fp32 arithmetic (``csrc/attention_simt.cu``): fp32 models, and head sizes outside the
-    tensor-core kernels'. Arguments as :func:`paged_attention`."""
+    tensor-core kernels'. Arguments as :func:`paged_attention`; ``v_dim``: only the first elements of a value row count
+    (latent rows, which are keys and values at once; one KV head)."""
     T, Hq, D = q.shape
-    Hkv, Dv = k_pages.shape[2], v_pages.shape[-1]
+    Hkv, Dv = k_pages.shape[2], v_dim or v_pages.shape[-1]
+    assert v_dim is None or Hkv == 1
     if q.dtype != k_pages.dtype or q.dtype != v_pages.dtype or q.dtype not in (torch.bfloat16, torch.float32):
         raise TypeError(f"queries and pages must share one type (bf16 or fp32), got {q.dtype} / {k_pages.dtype}")
     assert k_pages.shape[1] == PAGE_SIZE and q.stride(-1) == 1 and q.stride(-2) == D
@@ -138,16 +142,28 @@ def mla_decode_attention(q: torch.Tensor, pages: torch.Tensor, kv_lens: torch.Te
     ``[P, 128, 1, 576]`` rows (compressed key/value | rotated rotary key). Returns ``[B, H, 512]``: the
     softmax-weighted sums of the rows' compressed part, to be sent through the value up-projection."""
     B, H, W = q.shape
-    assert W == 576 and pages.shape[-1] == 576 and pages.shape[1] == PAGE_SIZE and q.is_contiguous()
+    assert W == 576 and pages.shape[-1] == 576 and q.is_contiguous()
+    return latent_decode(q[..., :512], q[..., 512:], pages, kv_lens, page_table, scale=scale, num_splits=num_splits)
+
+
+def latent_decode(q_lat: torch.Tensor, q_rot: torch.Tensor, pages: torch.Tensor, kv_lens: torch.Tensor,
+                  page_table: torch.Tensor, *, scale: float, window: int = 0, sinks=None,
+                  num_splits: int = 1) -> torch.Tensor:
+    """One absorbed query token per sequence over pages of latent rows: ``q_lat [B, H, L]`` (folded through the key
+    up-projection), ``q_rot [B, H, R]`` (rotated), pages ``[P, 128, 1, L + R]``; the views may be strided. ``window``: a
+    query sees its latest ``window`` keys; ``sinks [H]`` join the denominators. Returns ``[B, H, L]``."""
+    B, H, L = q_lat.shape
+    R = q_rot.shape[-1]
+    assert pages.shape[-1] == L + R and pages.shape[1] == PAGE_SIZE and pages.is_contiguous()
+    assert q_lat.stride(2) == 1 and q_rot.stride(2) == 1
     S_ = max(1, int(num_splits))
-    out = torch.empty((S_, B, H, 512), dtype=q.dtype, device=q.device)
-    lse = torch.empty((S_, H, B), dtype=torch.float32, device=q.device) if S_ > 1 else None
-    _lib.call("edl_attn_mla_decode", q.data_ptr(), pages.data_ptr(), out.data_ptr(), _lib.ptr(lse), H * 576, H * 512,
-              kv_lens.data_ptr(), page_table.data_ptr(), page_table.stride(0), B, pages.shape[0], H, float(scale), S_,
-              _lib.status_word(q.device).data_ptr(), _lib.stream_ptr())
-    if S_ == 1:
-        return out[0]
-    return attn_combine(out, lse)
+    out = torch.empty((S_, B, H, L), dtype=q_lat.dtype, device=q_lat.device)
+    lse = torch.empty((S_, H, B), dtype=torch.float32, device=q_lat.device) if S_ > 1 else None
+    _lib.call("edl_attn_mla_decode", q_lat.data_ptr(), q_lat.stride(0), q_lat.stride(1), q_rot.data_ptr(), q_rot.stride(0),
+              q_rot.stride(1), pages.data_ptr(), out.data_ptr(), _lib.ptr(lse), H * L, kv_lens.data_ptr(),
+              page_table.data_ptr(), page_table.stride(0), B, pages.shape[0], H, L, R, float(scale), int(window or 0),
+              _lib.ptr(sinks) if S_ == 1 else None, S_, _lib.status_word(q_lat.device).data_ptr(), _lib.stream_ptr())
+    return out[0] if S_ == 1 else attn_combine(out, lse, sinks=sinks)
 
 
 def mla_decode_kernel_supports(q: torch.Tensor, pages: torch.Tensor) -> bool:

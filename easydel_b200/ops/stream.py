@@ -16,9 +16,11 @@ from . import _lib, kernels as K
 vp, i32, i64, f32 = _lib.vp, _lib.i32, _lib.i64, _lib.f32
 _lib.register("edl_embed_stream", i32, [vp, i32, vp, vp, vp, i64, i32, i32, i32, vp, vp])
 _lib.register("edl_cast_rows", i32, [vp, vp, i32, i64, i32, i32, vp])
-_lib.register("edl_norm_shift", i32, [vp, vp, vp, f32, i32, i32, vp, i32, vp, vp, i64, vp, i32, vp])
+_lib.register("edl_norm_shift", i32, [vp, vp, vp, f32, i32, i32, vp, i32, vp, vp, i64, f32, vp, i32, vp])
 _lib.register("edl_head_norm", i32, [vp, vp, f32, i64, i32, vp, i32, vp])
 _lib.register("edl_xielu", i32, [vp, vp, vp, i32, i64, vp])
+_lib.register("edl_gelu_erf", i32, [vp, vp, i32, i64, vp])
+_lib.register("edl_post_norm", i32, [vp, vp, vp, vp, vp, i32, f32, vp, f32, f32, vp, i32, i32, i32, vp])
 _lib.register("edl_qkv_prologue", i32, [vp, i32, i64, vp, vp, vp, vp, f32, f32, f32, i32, i32, i32, i32, i32, vp, vp, vp,
                                         i64, i64, i64, vp, vp])
 
@@ -79,6 +81,16 @@ def linear_add_(stream: torch.Tensor, x: torch.Tensor, w: torch.Tensor) -> torch
     return stream + tF.linear(x, w).float()
 
 
+def bmm(a: torch.Tensor, b: torch.Tensor) -> torch.Tensor:
+    """Batched product in the operand type, true 32-bit for fp32 (vendor library)."""
+    allow = torch.backends.cuda.matmul.allow_tf32
+    torch.backends.cuda.matmul.allow_tf32 = False
+    try:
+        return torch.bmm(a, b)
+    finally:
+        torch.backends.cuda.matmul.allow_tf32 = allow
+
+
 # ---------------------------------------------------------------------------------------------- rows of the stream
 def embed(table: torch.Tensor, ids: torch.Tensor, right: torch.Tensor | None = None) -> torch.Tensor:
     """fp32 rows ``table[ids]`` ``[T, W]``; ``right`` (a view ``[T, W]`` of the right half of a ``[x ; x0]`` operand)
@@ -129,8 +141,8 @@ def norm_shift_reference(x, w, eps, out_dtype, mu=None, cu=None, slots=None, sta
 
 def norm_shift(x: torch.Tensor, w: torch.Tensor, eps: float, out_dtype: torch.dtype, mu: torch.Tensor | None = None,
                cu: torch.Tensor | None = None, slots: torch.Tensor | None = None,
-               state: torch.Tensor | None = None) -> torch.Tensor:
-    """RMS norm of the fp32 stream ``x [T, W]`` times ``w`` (fp32), in 32 bits, cast once to ``out_dtype``.
+               state: torch.Tensor | None = None, offset: float = 0.0) -> torch.Tensor:
+    """RMS norm of the fp32 stream ``x [T, W]`` times ``w + offset`` (fp32), in 32 bits, cast once to ``out_dtype``.
 
     ``mu`` (fp32 ``[W]``): token shift. Row t becomes ``h_t + (h_{t-1} - h_t) * mu`` inside the sequences bounded by
     ``cu`` (int32 ``[B + 1]``); the row before a sequence's first one comes from ``state[slots[b]]`` (fp32
@@ -140,9 +152,9 @@ def norm_shift(x: torch.Tensor, w: torch.Tensor, eps: float, out_dtype: torch.dt
         nseq = cu.numel() - 1 if cu is not None else 0
         _lib.call("edl_norm_shift", x.data_ptr(), w.data_ptr(), _lib.ptr(mu), float(eps), x.shape[0], x.shape[1],
                   _lib.ptr(cu), nseq, _lib.ptr(slots), _lib.ptr(state), state.stride(0) if state is not None else 0,
-                  out.data_ptr(), _f32flag(out_dtype), _lib.stream_ptr())
+                  float(offset), out.data_ptr(), _f32flag(out_dtype), _lib.stream_ptr())
         return out
-    return norm_shift_reference(x, w.float(), eps, out_dtype, None if mu is None else mu.float(), cu, slots, state)
+    return norm_shift_reference(x, w.float() + offset, eps, out_dtype, None if mu is None else mu.float(), cu, slots, state)
 
 
 def head_norm(o: torch.Tensor, w: torch.Tensor, eps: float, out_dtype: torch.dtype) -> torch.Tensor:
@@ -168,6 +180,39 @@ def xielu(z: torch.Tensor, act: torch.Tensor) -> torch.Tensor:
     ap, an = tF.softplus(a[0]), 0.5 + tF.softplus(a[1])
     neg = zf.clamp(max=0.0)
     return torch.where(zf > 0, ap * zf * zf + 0.5 * zf, an * (torch.expm1(neg) - neg) + 0.5 * neg).to(z.dtype)
+
+
+def gelu_erf(z: torch.Tensor) -> torch.Tensor:
+    """Exact GELU, ``z / 2 (1 + erf(z / sqrt 2))``."""
+    if on_kernels(z):
+        z = z if z.is_contiguous() else z.contiguous()
+        y = torch.empty_like(z)
+        _lib.call("edl_gelu_erf", z.data_ptr(), y.data_ptr(), _f32flag(z.dtype), z.numel(), _lib.stream_ptr())
+        return y
+    return tF.gelu(z)
+
+
+# ---------------------------------------------------------------------------------------------- norm after the sum
+def post_norm(x: torch.Tensor, branch, alpha: float, w: torch.Tensor, eps: float, out_dtype: torch.dtype,
+              offset: float = 0.0) -> tuple[torch.Tensor, torch.Tensor]:
+    """``rms_norm(alpha x + branch) * (w + offset)`` over the fp32 stream ``x [T, W]`` in 32 bits: the new stream (in place
+    on the kernels) and the same rows as the operand of the next product. ``branch``: fp32 rows ``[T, W]``, or an
+    :class:`..ops.moe_kernels.ExpertRows`, whose weighted sum over each token's experts happens in the same pass."""
+    rows = None if isinstance(branch, torch.Tensor) else branch
+    if on_kernels(x):
+        h = torch.empty(x.shape, dtype=out_dtype, device=x.device)
+        y = branch if rows is None else None
+        if y is not None and (y.dtype != torch.float32 or not y.is_contiguous()):
+            y = y.float().contiguous()
+        assert x.is_contiguous() and (rows is None or rows.ys.dtype == out_dtype)
+        _lib.call("edl_post_norm", x.data_ptr(), _lib.ptr(y), _lib.ptr(rows.ys) if rows else None,
+                  _lib.ptr(rows.weights) if rows else None, _lib.ptr(rows.pos) if rows else None, rows.k if rows else 0,
+                  float(alpha), w.data_ptr(), float(offset), float(eps), h.data_ptr(), _f32flag(out_dtype), x.shape[0],
+                  x.shape[1], _lib.stream_ptr())
+        return x, h
+    v = x * alpha + (branch.float() if rows is None else rows.combine())
+    v = v * torch.rsqrt(v.pow(2).mean(-1, keepdim=True) + eps) * (w.float() + offset)
+    return v, v.to(out_dtype)
 
 
 # ---------------------------------------------------------------------------------------------- attention prologue

@@ -22,6 +22,9 @@ FUSED_SPLITS: dict[str, tuple[str, ...]] = {
     "qkv_proj": ("q_proj", "k_proj", "v_proj"),
     "gate_up_proj": ("gate_proj", "up_proj"),
     "qfv_proj": ("q_proj", "f_proj", "v_proj"),
+    "qdg_proj": ("q_proj", "dkv_proj", "g_proj"),
+    "qd_proj": ("q_proj", "dkv_proj"),
+    "ukv_proj": ("uk_proj", "uv_proj"),
 }
 
 _EXPERT_RE = re.compile(r"^(.*\.)experts\.(\d+)\.(gate_proj|up_proj|down_proj|w1|w2|w3)\.weight$")
