@@ -1,8 +1,8 @@
 // Flash-attention forward on tcgen05 tensor cores (tiles of 64 or 128 columns per head, bf16, GQA,
 // causal, variable-length batches, sliding window, logit soft-cap, attention sinks).
 //
-// The query / key size and the value size of a head are separate and may be any multiple of 8 up to 128: a tile is
-// DQ (or DV) columns wide, 64 or 128, and the tensor maps carry the real sizes, so the columns past a head's end
+// The query / key size and the value size of a head are separate and may be any multiple of 8 up to 192 (keys) and 128
+// (values): a tile is DQ (or DV) columns wide, 64, 128 or 192, and the tensor maps carry the real sizes, so the columns past a head's end
 // arrive as zeros and only the real value columns are stored. Memory holds no padding.
 //
 // One CTA per (block of 256 query rows = two tiles A and B, query head, sequence):
@@ -22,6 +22,9 @@
 //               bf16 over the same tensor-memory columns (the A operand of the PV product). O is
 //               rescaled in tensor memory only when the running maximum moved by more than 2^8.
 // Tensor memory map (512 columns): S_A/P_A [0,128)  S_B/P_B [128,256)  O_A [256,384)  O_B [384,512).
+//
+// Tiles 192 columns wide (expanded latent attention) leave shared memory for one stage of 128-wide values, and none for the
+// exchange between the halves of a row: that goes through two spare tensor-memory columns of the row's own scores.
 //
 // Queries, keys and values are read straight out of the packed projection output
 // through 3-D tensor maps (head_dim, heads, tokens), so no transposes are needed.
@@ -86,11 +89,14 @@ struct ACfg {
   static constexpr int Q_BYTES = BQ * DQ * 2;     // one query tile
   static constexpr int K_BYTES = BKV * DQ * 2;
   static constexpr int V_BYTES = BKV * DV * 2;
+  static constexpr bool WIDE = DQ > 128;
+  static constexpr int VS = WIDE && DV > 64 ? 1 : 2;      // value stages
   static constexpr int OFF_K = 2 * Q_BYTES;
   static constexpr int OFF_V = OFF_K + 2 * K_BYTES;
-  static constexpr int OFF_BAR = OFF_V + 2 * V_BYTES;
+  static constexpr int OFF_BAR = OFF_V + VS * V_BYTES;
   static constexpr int OFF_XCH = OFF_BAR + 256;   // float [tile][parity][half][row]: row maxima / sums of a half
-  static constexpr int SMEM = OFF_XCH + 2 * 2 * 2 * BQ * 4 + 1024;
+  static constexpr int SMEM = OFF_XCH + (WIDE ? 0 : 2 * 2 * 2 * BQ * 4) + 1024;
+  static_assert(SMEM <= 232448, "shared memory of one CTA");
 };
 
 struct TileRange {
@@ -207,24 +213,35 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
 #pragma unroll
         for (int c = 0; c < C::QCH; ++c)
           tma_load_3d(sQ + t * C::Q_BYTES + c * (BQ * 128), &tq, b_qfull, c * 64, h_first, q_start + qblock0 + t * TQ);
-      for (int j = jmin; j < jmax; ++j) {
-        const int it = j - jmin;
-        const int s = it & 1;
-        const int krow = pt ? pt[j] * BKV : k_start + j * BKV;
+      auto row_of = [&](int j) { return pt ? pt[j] * BKV : k_start + j * BKV; };
+      auto load_k = [&](int j) -> bool {
+        const int it = j - jmin, s = it & 1, row = row_of(j);
         if (it >= 2 &&
             !mbar_wait(b_kempty + 8 * s, ((it >> 1) - 1) & 1, abort_flag, p.status, EDL_TIMEOUT_PRODUCER))
-          break;
+          return false;
         mbar_expect_tx(b_kfull + 8 * s, C::K_BYTES);
 #pragma unroll
         for (int c = 0; c < C::QCH; ++c)
-          tma_load_3d(sK0 + s * C::K_BYTES + c * (BKV * 128), &tk, b_kfull + 8 * s, c * 64, hk, krow);
-        if (it >= 2 &&
-            !mbar_wait(b_vempty + 8 * s, ((it >> 1) - 1) & 1, abort_flag, p.status, EDL_TIMEOUT_PRODUCER))
-          break;
+          tma_load_3d(sK0 + s * C::K_BYTES + c * (BKV * 128), &tk, b_kfull + 8 * s, c * 64, hk, row);
+        return true;
+      };
+      auto load_v = [&](int j) -> bool {
+        const int it = j - jmin, s = it % C::VS, row = row_of(j);
+        if (it >= C::VS &&
+            !mbar_wait(b_vempty + 8 * s, (it / C::VS - 1) & 1, abort_flag, p.status, EDL_TIMEOUT_PRODUCER))
+          return false;
         mbar_expect_tx(b_vfull + 8 * s, C::V_BYTES);
 #pragma unroll
         for (int c = 0; c < C::VCH; ++c)
-          tma_load_3d(sV0 + s * C::V_BYTES + c * (BKV * 128), &tv, b_vfull + 8 * s, c * 64, hk, krow);
+          tma_load_3d(sV0 + s * C::V_BYTES + c * (BKV * 128), &tv, b_vfull + 8 * s, c * 64, hk, row);
+        return true;
+      };
+      if constexpr (C::VS == 2) {
+        for (int j = jmin; j < jmax; ++j)
+          if (!load_k(j) || !load_v(j)) break;
+      } else {   // the only value stage is free late: keys stay one tile ahead of it
+        bool ok = load_k(jmin);
+        for (int j = jmin; j < jmax && ok; ++j) ok = (j + 1 >= jmax || load_k(j + 1)) && load_v(j);
       }
     }
   } else if (warp == 1) {
@@ -254,7 +271,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
         if (leader) tc_commit(b_sfull + 8 * t);
       };
       auto issue_pv = [&](int t, int j) -> bool {
-        const int s = (j - jmin) & 1;
+        const int s = (j - jmin) % C::VS;
         if (!mbar_wait(b_pfull + 8 * t, pv_cnt[t] & 1, abort_flag, p.status, EDL_TIMEOUT_MMA)) return false;
         tc_fence_after();
         const uint32_t vb = sV0 + s * C::V_BYTES;
@@ -287,7 +304,8 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
         const int s = it & 1;
         const bool more = j + 1 < jmax;
         TRACE(2, it, 0);
-        if (!mbar_wait(b_vfull + 8 * s, (it >> 1) & 1, abort_flag, p.status, EDL_TIMEOUT_MMA)) break;
+        const int vs = it % C::VS;
+        if (!mbar_wait(b_vfull + 8 * vs, (it / C::VS) & 1, abort_flag, p.status, EDL_TIMEOUT_MMA)) break;
         if (more && !mbar_wait(b_kfull + 8 * (s ^ 1), ((it + 1) >> 1) & 1, abort_flag, p.status, EDL_TIMEOUT_MMA))
           break;
         tc_fence_after();
@@ -298,7 +316,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
         TRACE(2, it, 3);
         if (valid(1, j) && !issue_pv(1, j)) break;
         TRACE(2, it, 4);
-        if (leader) tc_commit(b_vempty + 8 * s);
+        if (leader) tc_commit(b_vempty + 8 * vs);
         if (more) {
           if (valid(1, j + 1)) issue_qk(1, j + 1);
           if (leader) tc_commit(b_kempty + 8 * (s ^ 1));
@@ -331,9 +349,27 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
     const float mul = capped ? 1.f : p.scale_log2;
     bool alive = true;
     int n = 0;
-    // One value per thread to the other half of the row and back (shared memory, 64-thread barrier, bounded).
-    auto exchange = [&](float mine, float& other) -> bool {
+    // One value per thread to the other half of the row and back (64-thread barrier, bounded). Wide tiles pass it through
+    // tensor memory: the left half's value lies in a score column that the left half has read and that only the right
+    // half overwrites (with its P, after reading it); the right half's in its own first column, which P never reaches.
+    // At the end (`last`) P may still be an operand, so both use columns behind it, whose scores everyone has read
+    // (not those of the step before, which the other half may still be reading).
+    auto exchange = [&](float mine, float& other, bool last) -> bool {
       const int par = n & 1;
+      if constexpr (C::WIDE) {
+        const uint32_t left = tS + (last ? 65 : 63), right = tS + (last ? 66 : 64);
+        tmem_st_32x32b_x1(half ? right : left, __float_as_uint(mine));
+        tc_wait_st();
+        tc_fence_before();
+        mbar_arrive(bx);
+        if (!mbar_wait(bx, par, abort_flag, p.status, EDL_TIMEOUT_SOFTMAX)) return false;
+        tc_fence_after();
+        uint32_t got;
+        tmem_ld_32x32b_x1(half ? left : right, got);
+        tc_wait_ld();
+        other = __uint_as_float(got);
+        return true;
+      }
       xch[(par * 2 + half) * BQ + r] = mine;
       mbar_arrive(bx);
       if (!mbar_wait(bx, par, abort_flag, p.status, EDL_TIMEOUT_SOFTMAX)) return false;
@@ -383,7 +419,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
       }
       float mx_other;
       TRACE(t, n, 2);
-      if (!exchange(mx, mx_other)) {
+      if (!exchange(mx, mx_other, false)) {
         alive = false;
         break;
       }
@@ -442,7 +478,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
     const bool any = rg.hi > rg.lo;
     if (any && alive) {
       float l_other;
-      if (!exchange(l, l_other)) alive = false;
+      if (!exchange(l, l_other, true)) alive = false;
       l += l_other;
     }
     if (any && alive) {
@@ -523,6 +559,9 @@ int launch_fwd(const void* q, const void* k, const void* v, long long ldq, long 
 // Tile widths from the real head sizes.
 int dispatch_fwd(const void* q, const void* k, const void* v, long long ldq, long long ldk, long long ldv,
                  long long total_q, long long total_k, const AttnFwdParams& p, cudaStream_t s) {
+  if (p.dq > 128)
+    return p.dv > 64 ? launch_fwd<192, 128>(q, k, v, ldq, ldk, ldv, total_q, total_k, p, s)
+                     : launch_fwd<192, 64>(q, k, v, ldq, ldk, ldv, total_q, total_k, p, s);
   if (p.dq > 64)
     return p.dv > 64 ? launch_fwd<128, 128>(q, k, v, ldq, ldk, ldv, total_q, total_k, p, s)
                      : launch_fwd<128, 64>(q, k, v, ldq, ldk, ldv, total_q, total_k, p, s);
@@ -598,7 +637,7 @@ EDL_HOST_API int edl_attn_fwd(const void* q, const void* k, const void* v, void*
 //   max_q:    largest number of new tokens of any sequence (sizes the grid)
 // All query heads of a KV head share one tile (rows = token x head), so one pass over a page
 // serves the whole GQA group; a group whose size is not a power of two is cut into equal power-of-two parts.
-// Head sizes D (queries, keys) and Dv (values): multiples of 8 up to 128.
+// Head sizes: multiples of 8, D (queries, keys) up to 192 and Dv (values) up to 128.
 static int attn_paged_impl(const void* q, const void* k_pages, const void* v_pages, void* o, float* lse,
                            long long ldq, long long ld_kpage, long long ld_vpage, long long ldo, const int* cu_q, const int* kv_lens,
                            const int* page_table, int pt_stride, int B, int max_q, long long total_q,
@@ -606,7 +645,7 @@ static int attn_paged_impl(const void* q, const void* k_pages, const void* v_pag
                            float softcap, const float* sinks, int* status, void* stream) {
   using namespace edl;
   if (B <= 0 || max_q <= 0 || total_q <= 0) return 0;
-  if (D < 8 || D > 128 || (D & 7) || Dv < 8 || Dv > 128 || (Dv & 7) || Hkv < 1 || Hq % Hkv) {
+  if (D < 8 || D > 192 || (D & 7) || Dv < 8 || Dv > 128 || (Dv & 7) || Hkv < 1 || Hq % Hkv) {
     set_last_error("edl_attn_paged: unsupported head layout (D=%d, Dv=%d, Hq=%d, Hkv=%d)", D, Dv, Hq, Hkv);
     return -1;
   }

@@ -81,8 +81,8 @@ struct PrologueParams {
   int* status;
 };
 
-// One CTA per token. Angles are p * f with the product's rounding error and the frequency's own carried along as a first
-// order correction, so that they are as exact as 32-bit results can be at any position.
+// One CTA per token. Angles are p * f with the product's rounding error and the frequency's own carried along as a small
+// second rotation, so that they are as exact as 32-bit results can be at any position.
 template <typename T>
 __global__ void __launch_bounds__(LP_THREADS)
 latent_prologue_kernel(T* __restrict__ proj, T* __restrict__ pages, const PrologueParams p) {
@@ -97,7 +97,8 @@ latent_prologue_kernel(T* __restrict__ proj, T* __restrict__ pages, const Prolog
     const float e = fmaf(fp, f, -a) + fp * p.freq[p.pairs + i];
     float s, c;
     sincosf(a, &s, &c);
-    cs[i] = make_float2(c - e * s, s + e * c);
+    const float ce = 1.f - 0.5f * e * e, se = e - e * e * e * (1.f / 6.f);      // e is small: half an ulp of the angle
+    cs[i] = make_float2(c * ce - s * se, s * ce + c * se);
   }
   float ss = 0.f;
   for (int c = tid; c < p.L; c += LP_THREADS) {

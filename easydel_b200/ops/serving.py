@@ -26,7 +26,7 @@ _lib.register("edl_attn_mla_decode", i32, [vp, i64, i64, vp, i64, i64, vp, vp, v
                                             f32, i32, vp, i32, vp, vp])
 
 PAGE_SIZE = 128
-MAX_QK_DIM = 128      # widest query / key head of the tensor-core prefill kernel
+MAX_QK_DIM = 192      # widest query / key head of the tensor-core prefill kernel
 
 
 def kv_append(k: torch.Tensor, v: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor,

@@ -66,7 +66,9 @@ def latent_heads(q, c, kr, uk, uv, dim, scale, window, sink, mutate=None):
     """q [T, H, dim + rot] and the shared key part kr [T, rot] (both rotated), latents c [T, L], per-head up-projections
     uk [H, dim, L] and uv [H, V, L] -> [T, H, V]."""
     T, H, _ = q.shape
-    if mutate == "window_plus":
+    if window is None:
+        pass
+    elif mutate == "window_plus":
         window = window + 1
     elif mutate == "window_minus":
         window = window - 1
