@@ -172,16 +172,27 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap, const MlaParams p) {
     if (alive) alive = mbar_wait(bar0 + 8 * st, (i / ML_STAGES) & 1, abort_flag, p.status, EDL_TIMEOUT_SOFTMAX);
     const uint32_t tile = sbase + st * C::TILE_BYTES;
     // ---- scores of rows 8w .. 8w+7 of the tile
-    float s[4] = {0.f, 0.f, 0.f, 0.f};
-    if (alive) {
+    float s[4] = {0.f, 0.f, 0.f, 0.f}, s2[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+    if (alive) {                      // three independent chains of products
       const int row = warp * 8 + (lane & 7);
 #pragma unroll
       for (int ks = 0; ks < C::NKS; ks += 2) {
         uint32_t kb[4];
         ml_ldmatrix_x4(tile + ml_tile_off(row, ks * 2 + (lane >> 3)), kb);
-        ml_mma(s, qa[ks], kb[0], kb[1]);
-        ml_mma(s, qa[ks + 1], kb[2], kb[3]);
+        const int chain = (ks >> 1) % 3;
+        if (chain == 0) {
+          ml_mma(s, qa[ks], kb[0], kb[1]);
+          ml_mma(s2[0], qa[ks + 1], kb[2], kb[3]);
+        } else if (chain == 1) {
+          ml_mma(s2[1], qa[ks], kb[0], kb[1]);
+          ml_mma(s, qa[ks + 1], kb[2], kb[3]);
+        } else {
+          ml_mma(s2[0], qa[ks], kb[0], kb[1]);
+          ml_mma(s2[1], qa[ks + 1], kb[2], kb[3]);
+        }
       }
+#pragma unroll
+      for (int e = 0; e < 4; ++e) s[e] += s2[0][e] + s2[1][e];
     }
     const int key0 = (t0 + i) * ML_TK + warp * 8 + (lane & 3) * 2;
     float mx[2];
@@ -276,6 +287,11 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap, const MlaParams p) {
     if (p.lse && warp == 0 && (lane & 3) == 0)
       p.lse[((long long)split * p.H + hg * 16 + r) * p.B + b] =
           l > 0.f ? (m_run[h] + log2f(l)) * 0.6931471805599453f : -INFINITY;
+  }
+  if (s_abort) {   // a wait ran out: give copies still in flight time to land before shared memory is released
+    long long t0c = clock64();
+    while (clock64() - t0c < 400000) {
+    }
   }
 }
 

@@ -280,14 +280,23 @@ __global__ void __launch_bounds__(NT) post_norm_kernel(const PostNormParams<TO> 
       float m[VEC];
 #pragma unroll
       for (int j = 0; j < VEC; ++j) m[j] = 0.f;
-      for (int s = 0; s < p.k; ++s) {
-        const int at = p.pos[(long long)r * p.k + s];
-        if (at < 0) continue;
-        const float ws = p.wts[(long long)r * p.k + s];
-        float b[VEC];
-        ldv<VEC>(p.ys + (long long)at * p.W + c, b);
+      for (int s0 = 0; s0 < p.k; s0 += 4) {       // four rows in flight
+        float b[4][VEC], ws[4];
 #pragma unroll
-        for (int j = 0; j < VEC; ++j) m[j] = fmaf(ws, b[j], m[j]);
+        for (int u = 0; u < 4; ++u) {
+          const int at = s0 + u < p.k ? p.pos[(long long)r * p.k + s0 + u] : -1;
+          ws[u] = 0.f;
+#pragma unroll
+          for (int j = 0; j < VEC; ++j) b[u][j] = 0.f;
+          if (at >= 0) {
+            ws[u] = p.wts[(long long)r * p.k + s0 + u];
+            ldv<VEC>(p.ys + (long long)at * p.W + c, b[u]);
+          }
+        }
+#pragma unroll
+        for (int u = 0; u < 4; ++u)
+#pragma unroll
+          for (int j = 0; j < VEC; ++j) m[j] = fmaf(ws[u], b[u][j], m[j]);
       }
 #pragma unroll
       for (int j = 0; j < VEC; ++j) a[j] += m[j];

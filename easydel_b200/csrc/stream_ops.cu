@@ -612,8 +612,8 @@ EDL_HOST_API int edl_cast_rows(const float* x, void* out, int f32, long long ld_
   return check_cuda(cudaGetLastError(), "cast_rows launch");
 }
 
-// out [rows, W] = rms_norm(x) * (w + offset), blended with the previous row's norm by mu when mu is given. cu [nseq + 1] bounds the
-// sequences on the row axis; state [*, ld_state] fp32 holds, per slot, the normalised row before the step's first one
+// out [rows, W] = rms_norm(x) * (w + offset), blended with the previous row's norm by mu when mu is given. cu [nseq + 1]
+// bounds the sequences on the row axis; state [*, ld_state] fp32 holds, per slot, the normalised row before the step's first one
 // (null: sequences start here) and is updated to the step's last row.
 EDL_HOST_API int edl_norm_shift(const float* x, const float* w, const float* mu, float eps, int rows, int W,
                                 const int* cu, int nseq, const int* slots, float* state, long long ld_state, float offset,
