@@ -22,7 +22,7 @@ def _default_layers(width: int) -> list[dict]:
              "rot": {"base": 10000.0, "dims": 32}, "mask": {"size": 1024}}
     return [{"type": "latent_attention", "mixer": mixer, "mlp": {"kind": "dense", "ff": 4 * width}},
             {"type": "latent_attention", "mixer": mixer,
-             "mlp": {"kind": "moe", "router": {"experts": 16, "top": 2}, "expert": {"ff": width, "limit": 7.0}}}]
+             "mlp": {"kind": "moe", "router": {"experts": 32, "top": 4}, "expert": {"ff": width, "limit": 7.0}}}]
 
 
 @register_config("disunex", architecture="Disunex")
