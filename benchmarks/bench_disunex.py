@@ -26,7 +26,7 @@ SIZES = ((2048, 16, 128, 64, 128, 512, 64, 6, 1408, 8192, 1024),
 
 # ------------------------------------------------------------------------------------------------ kernels
 def bench_rows(t: Table, T: int, size) -> None:
-    from easydel_b200.ops import kernels as K, latent, stream
+    from easydel_b200.ops import kernels as K, latent, rotation, stream
     from easydel_b200.ops.moe_kernels import ExpertRows
 
     W, H, D, R, V, L, E, k, F, ff, _ = size
@@ -48,7 +48,7 @@ def bench_rows(t: Table, T: int, size) -> None:
     proj = _rand(T, H * (D + R) + L + R + H * V)
     pages = torch.zeros(T // 128 + 2, 128, 1, L + R, dtype=BF, device="cuda")
     sl, p = torch.arange(T, device="cuda", dtype=torch.int32) + 128, torch.arange(T, dtype=torch.int32, device="cuda")
-    nw, freq = torch.ones(L, device="cuda"), latent.pair_frequencies(1e4, R, "cuda")
+    nw, freq = torch.ones(L, device="cuda"), rotation.pair_frequencies(1e4, R, "cuda")
     packed = _rand(T, (H + 1) * R)
     cos, moved = torch.rand(T, R // 2, device="cuda"), torch.empty_like(packed)
     t.add("latent prologue (rotate, norm, append)", f"{name}, {H} heads",
@@ -103,8 +103,8 @@ def bench_experts(t: Table, T: int, size) -> None:
     from easydel_b200.ops import _lib
 
     t.add("clamped unit", f"rows {T * k} of {r.max_rows}, ff {F}",
-          (lambda: _lib.call("edl_moe_clamped_glu", x2.data_ptr(), 0, r.row_token.data_ptr(), r.meta.data_ptr(),
-                             act.data_ptr(), F, r.max_rows, 7.0, 1.702, _lib.stream_ptr()), 6 * T * k * F),
+          (lambda: _lib.call("edl_moe_glu", x2.data_ptr(), 0, r.row_token.data_ptr(), r.meta.data_ptr(), act.data_ptr(), F,
+                             r.max_rows, 7.0, 1.702, _lib.stream_ptr()), 6 * T * k * F),
           "gated silu over all rows", (lambda: K.gated_act_fwd(x2, "silu"), 6 * T * k * F))
 
 

@@ -260,10 +260,11 @@ class PagedLayerView:
         """Attention of ``q3 [T, Hq, D]`` over the pages, which already hold this step's keys and values."""
         table = meta.table_of(self.group)
         if meta.max_q == 1 and q3.shape[0] == meta.num_seqs and S.decode_kernel_supports(
-                q3, self.k_pages, attn.softcap, self.v_pages.shape[-1]):
+                q3, self.k_pages, self.v_pages.shape[-1]):
             # a pure decode step: the streaming kernel (one CTA per sequence, KV head and key split)
             o = S.decode_attention(q3, self.k_pages, self.v_pages, meta.kv_lens, table, scale=attn.scale,
-                                   window=attn.sliding_window or 0, sinks=attn.sinks, num_splits=meta.num_splits)
+                                   window=attn.sliding_window or 0, sinks=attn.sinks, softcap=attn.softcap,
+                                   num_splits=S.decode_splits(meta.num_splits, attn.sliding_window))
             return o
         if meta.num_splits > 1 and meta.max_q == 1 and not attn.sliding_window and q3.is_cuda and \
                 q3.dtype == torch.bfloat16 and self.v_pages.shape[-1] == q3.shape[-1] and q3.shape[-1] in (64, 128):

@@ -47,6 +47,7 @@ struct DecodeParams {
   int pt_stride, B, Hq, Hkv, splits, window;
   int dq, dv;               // real query / key and value sizes of a head
   float scale_log2;
+  float cap_k2, cap2;       // soft-cap (see soft_cap), cap2 = 0: none
   int* status;
 };
 
@@ -219,7 +220,8 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tk, const __grid_constant
       for (int e = 0; e < 4; ++e) {
         const int key = cbase + j * 8 + (e & 1);
         const bool ok = key < kv_len && key >= lo;
-        s[j][e] = ok ? s[j][e] * p.scale_log2 : -INFINITY;
+        const float z = p.cap2 > 0.f ? soft_cap(s[j][e], p.cap_k2, p.cap2) : s[j][e] * p.scale_log2;
+        s[j][e] = ok ? z : -INFINITY;
         mx[e >> 1] = fmaxf(mx[e >> 1], s[j][e]);
       }
     }
@@ -384,12 +386,13 @@ int launch_decode(const void* k_pages, const void* v_pages, long long ld_kpage, 
 // pages [num_pages * 128, ld_kpage / ld_vpage] with the KV heads packed in a row, page_table [B, pt_stride], kv_lens [B]
 // (keys per sequence, the new token included). o [splits, B, ldo]; with splits > 1 part s holds the result over
 // the s-th part of every sequence's keys and lse [splits, Hq, B] its log-sum-exp, for edl_attn_combine.
-// Hq / Hkv <= 16; D (queries, keys) and Dv (values) are multiples of 8 up to 128; window = 0 or the sliding-window length.
+// Hq / Hkv <= 16; D (queries, keys) and Dv (values) are multiples of 8 up to 128; window = 0 or the sliding-window length;
+// softcap > 0: scores become softcap * tanh(scale * dot / softcap).
 EDL_HOST_API int edl_attn_decode(const void* q, const void* k_pages, const void* v_pages, void* o, float* lse,
                                  long long ldq, long long ld_kpage, long long ld_vpage, long long ldo, const int* kv_lens,
                                  const int* page_table, int pt_stride, int B, long long num_pages, int Hq, int Hkv,
-                                 int D, int Dv, float scale, int window, int splits, const float* sinks, int* status,
-                                 void* stream) {
+                                 int D, int Dv, float scale, int window, int splits, float softcap,
+                                 const float* sinks, int* status, void* stream) {
   using namespace edl;
   if (B <= 0) return 0;
   if (D < 8 || D > 128 || (D & 7) || Dv < 8 || Dv > 128 || (Dv & 7) || Hkv < 1 || Hq % Hkv || Hq / Hkv > 16 ||
@@ -418,6 +421,8 @@ EDL_HOST_API int edl_attn_decode(const void* q, const void* k_pages, const void*
   p.splits = splits;
   p.window = window;
   p.scale_log2 = scale * 1.4426950408889634f;
+  p.cap2 = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
+  p.cap_k2 = softcap > 0.f ? 2.f * p.scale_log2 / softcap : 0.f;
   p.status = status;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   p.dq = D;

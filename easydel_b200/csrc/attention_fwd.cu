@@ -118,7 +118,8 @@ __device__ __forceinline__ TileRange tile_range(int q0, int tq, int len_q, int l
   return r;
 }
 
-template <int DQ, int DV>
+// CAP: soft-capped scores (a form of its own: the other one must not carry its registers).
+template <int DQ, int DV, bool CAP>
 __global__ void __launch_bounds__(ATT_THREADS, 1)
 attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CUtensorMap tk,
                 const __grid_constant__ CUtensorMap tv, const AttnFwdParams p) {
@@ -343,10 +344,9 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
     float m_used = -1e30f;
     float l = 0.f;                          // sum over this thread's columns only
     const float cap2 = p.softcap * LOG2E;   // soft-cap in log2 units
-    const float inv_cap = p.softcap > 0.f ? 1.f / p.softcap : 0.f;
-    const float scale_nat = p.scale_log2 * LN2;
-    const bool capped = p.softcap > 0.f;
-    const float mul = capped ? 1.f : p.scale_log2;
+    const float cap_k2 = CAP ? 2.f * p.scale_log2 / p.softcap : 0.f;
+    const float cap_k = cap_k2 * (0.5f * LN2);      // scale / cap
+    const float mul = CAP ? 1.f : p.scale_log2;
     bool alive = true;
     int n = 0;
     // One value per thread to the other half of the row and back (64-thread barrier, bounded). Wide tiles pass it through
@@ -394,9 +394,25 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
       const bool tile_mask = (kv0 + BKV > len_k) || (p.causal && kv0 + BKV - 1 > q0 + off) ||
                              (p.window > 0 && kv0 < q0 + TQ - 1 + off - p.window + 1);
       tc_wait_ld();
-      if (capped) {
+      if constexpr (CAP) {
+        float m0 = 0.f, m1 = 0.f;
 #pragma unroll
-        for (int i = 0; i < 64; ++i) a[i] = __float_as_uint(cap2 * tanhf(__uint_as_float(a[i]) * scale_nat * inv_cap));
+        for (int i = 0; i < 64; i += 4) {
+          m0 = fmax3(m0, fabsf(__uint_as_float(a[i])), fabsf(__uint_as_float(a[i + 1])));
+          m1 = fmax3(m1, fabsf(__uint_as_float(a[i + 2])), fabsf(__uint_as_float(a[i + 3])));
+        }
+        if (__all_sync(0xffffffffu, fmaxf(m0, m1) * cap_k <= SOFT_CAP_POLY_MAX)) {   // well below the cap: no MUFU
+#pragma unroll
+          for (int i = 0; i < 64; i += 2) {
+            float s0 = __uint_as_float(a[i]), s1 = __uint_as_float(a[i + 1]);
+            soft_cap_poly2(s0, s1, cap_k, cap2);
+            a[i] = __float_as_uint(s0);
+            a[i + 1] = __float_as_uint(s1);
+          }
+        } else {
+#pragma unroll
+          for (int i = 0; i < 64; ++i) a[i] = __float_as_uint(soft_cap(__uint_as_float(a[i]), cap_k2, cap2));
+        }
       }
       if (tile_mask) {
 #pragma unroll
@@ -528,15 +544,15 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
   if (warp == 1) tmem_dealloc(tmem_base, 512);
 }
 
-template <int DQ, int DV>
-int launch_fwd(const void* q, const void* k, const void* v, long long ldq, long long ldk, long long ldv,
-               long long total_q, long long total_k, const AttnFwdParams& p, cudaStream_t stream) {
+template <int DQ, int DV, bool CAP>
+int launch_fwd_as(const void* q, const void* k, const void* v, long long ldq, long long ldk, long long ldv,
+                  long long total_q, long long total_k, const AttnFwdParams& p, cudaStream_t stream) {
   using C = ACfg<DQ, DV>;
   CUtensorMap tq, tk, tv;
   if (make_tmap_3d_16b(&tq, q, p.dq, p.Hq, total_q, p.dq, ldq, 64, p.pack, BQ / p.pack, 3)) return -1;
   if (make_tmap_3d_16b(&tk, k, p.dq, p.Hkv, total_k, p.dq, ldk, 64, 1, BKV, 3)) return -1;
   if (make_tmap_3d_16b(&tv, v, p.dv, p.Hkv, total_k, p.dv, ldv, 64, 1, BKV, 3)) return -1;
-  auto kern = attn_fwd_kernel<DQ, DV>;
+  auto kern = attn_fwd_kernel<DQ, DV, CAP>;
   static bool attr_set[64] = {false};  // per device
   int dev = 0;
   cudaGetDevice(&dev);
@@ -554,6 +570,13 @@ int launch_fwd(const void* q, const void* k, const void* v, long long ldq, long 
   const long long blocks = (long long)pl.nx * pl.ny * p.B;
   kern<<<(unsigned)blocks, ATT_THREADS, C::SMEM, stream>>>(tq, tk, tv, pl);
   return check_cuda(cudaGetLastError(), "attn_fwd launch");
+}
+
+template <int DQ, int DV>
+int launch_fwd(const void* q, const void* k, const void* v, long long ldq, long long ldk, long long ldv,
+               long long total_q, long long total_k, const AttnFwdParams& p, cudaStream_t s) {
+  return p.softcap > 0.f ? launch_fwd_as<DQ, DV, true>(q, k, v, ldq, ldk, ldv, total_q, total_k, p, s)
+                         : launch_fwd_as<DQ, DV, false>(q, k, v, ldq, ldk, ldv, total_q, total_k, p, s);
 }
 
 // Tile widths from the real head sizes.

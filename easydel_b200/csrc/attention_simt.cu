@@ -50,7 +50,7 @@ __global__ void __launch_bounds__(ST)
 attn_simt_kernel(const T* __restrict__ q, const T* __restrict__ k_pages, const T* __restrict__ v_pages,
                  T* __restrict__ o, long long ldq, long long ld_kpage, long long ld_vpage, const int* __restrict__ cu,
                  const int* __restrict__ kv_lens, const int* __restrict__ page_table, int pt_stride, int B,
-                 long long num_pages, int Hq, int Hkv, int D, int Dv, float scale, int window,
+                 long long num_pages, int Hq, int Hkv, int D, int Dv, float scale, int window, float softcap,
                  const float* __restrict__ sinks, bool vec, int* status) {
   __shared__ float sq[MAX_D];
   __shared__ float sp[ST];
@@ -83,6 +83,7 @@ attn_simt_kernel(const T* __restrict__ q, const T* __restrict__ k_pages, const T
     const bool ok = key >= k_lo && key <= qpos;
     float s = -INFINITY;
     if (ok) s = dot_row(k_pages + (page * ST + tid) * ld_kpage + (long long)hk * D, sq, D, vec) * scale;
+    if (ok && softcap > 0.f) s = softcap * tanhf(s / softcap);
     const float m_new = fmaxf(m, block_max(s, red));
     const float alpha = m == -INFINITY ? 0.f : expf(m - m_new);
     const float p = ok ? expf(s - m_new) : 0.f;
@@ -124,12 +125,12 @@ attn_simt_kernel(const T* __restrict__ q, const T* __restrict__ k_pages, const T
 template <typename T>
 int launch_simt(const void* q, const void* k, const void* v, void* o, long long ldq, long long ldk, long long ldv,
                 const int* cu, const int* kv_lens, const int* pt, int pt_stride, int B, int T_rows,
-                long long num_pages, int Hq, int Hkv, int D, int Dv, float scale, int window, const float* sinks,
-                int* status, cudaStream_t s) {
+                long long num_pages, int Hq, int Hkv, int D, int Dv, float scale, int window, float softcap,
+                const float* sinks, int* status, cudaStream_t s) {
   const bool vec = D % 4 == 0 && ldk % 4 == 0 && (reinterpret_cast<uintptr_t>(k) & 15) == 0;
   attn_simt_kernel<T><<<dim3(T_rows, Hq), ST, 0, s>>>((const T*)q, (const T*)k, (const T*)v, (T*)o, ldq, ldk, ldv, cu,
                                                       kv_lens, pt, pt_stride, B, num_pages, Hq, Hkv, D, Dv, scale,
-                                                      window, sinks, vec, status);
+                                                      window, softcap, sinks, vec, status);
   return check_cuda(cudaGetLastError(), "attn_simt launch");
 }
 
@@ -137,12 +138,13 @@ int launch_simt(const void* q, const void* k, const void* v, void* o, long long 
 }  // namespace edl
 
 // q [T, ldq] (head h at columns h * D), key / value pages [num_pages * 128, ld] with the heads packed in a row,
-// o [T, Hq * Dv]; cu [B + 1], kv_lens [B], page_table [B, pt_stride] as in edl_attn_paged; f32: storage type.
+// o [T, Hq * Dv]; cu [B + 1], kv_lens [B], page_table [B, pt_stride] as in edl_attn_paged; f32: storage type; softcap > 0:
+// scores become softcap * tanh(score / softcap).
 EDL_HOST_API int edl_attn_simt(const void* q, const void* k_pages, const void* v_pages, void* o, int f32,
                                long long ldq, long long ld_kpage, long long ld_vpage, const int* cu,
                                const int* kv_lens, const int* page_table, int pt_stride, int B, int T,
                                long long num_pages, int Hq, int Hkv, int D, int Dv, float scale, int window,
-                               const float* sinks, int* status, void* stream) {
+                             float softcap, const float* sinks, int* status, void* stream) {
   using namespace edl;
   if (B <= 0 || T <= 0) return 0;
   if (D < 1 || D > MAX_D || Dv < 1 || Dv > MAX_VC * ST || Hkv < 1 || Hq % Hkv || Hq > 65535) {
@@ -151,7 +153,8 @@ EDL_HOST_API int edl_attn_simt(const void* q, const void* k_pages, const void* v
   }
   cudaStream_t s = (cudaStream_t)stream;
   return f32 ? launch_simt<float>(q, k_pages, v_pages, o, ldq, ld_kpage, ld_vpage, cu, kv_lens, page_table, pt_stride,
-                                  B, T, num_pages, Hq, Hkv, D, Dv, scale, window, sinks, status, s)
+                                  B, T, num_pages, Hq, Hkv, D, Dv, scale, window, softcap, sinks, status, s)
              : launch_simt<__nv_bfloat16>(q, k_pages, v_pages, o, ldq, ld_kpage, ld_vpage, cu, kv_lens, page_table,
-                                          pt_stride, B, T, num_pages, Hq, Hkv, D, Dv, scale, window, sinks, status, s);
+                                          pt_stride, B, T, num_pages, Hq, Hkv, D, Dv, scale, window, softcap, sinks,
+                                          status, s);
 }

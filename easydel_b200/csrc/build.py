@@ -55,6 +55,8 @@ SERVING_PARTS = {
                 "host_native", "stream_ops", "hgrn2"),
     "disunex": ("common", "gemm", "attention_fwd", "attention_mla_decode", "attn_combine", "attention_simt", "serving",
                 "host_native", "stream_ops", "latent_ops", "moe", "moe_serving"),
+    "gasetar": ("common", "gemm", "attention_fwd", "attention_decode", "attention_mla_decode", "attn_combine",
+                "attention_simt", "serving", "host_native", "stream_ops", "latent_ops", "moe", "moe_serving", "norm_act"),
 }
 MANIFEST_SUFFIX = ".sources.json"      # beside a linked library: the digest of every source it was built from
 

@@ -353,6 +353,28 @@ __device__ __forceinline__ float exp2_poly(float x) {
   return __int_as_float(__float_as_int(p) + (__float_as_int(t) << 23));
 }
 
+// Soft-cap of attention scores in 32-bit accuracy: cap2 tanh(y) with y = s * scale / cap, from
+// tanh(y) = 1 - 2 / (1 + e^(2y)); two_k = 2 log2(e) * scale / cap turns a raw score s into 2y log2(e).
+__device__ __forceinline__ float soft_cap(float s, float two_k, float cap2) {
+  return cap2 - __fdividef(2.f * cap2, 1.f + exp2f(s * two_k));
+}
+
+// The same on the FMA pipe alone for |y| <= SOFT_CAP_POLY_MAX, two scores at a time: tanh(y) / y as a polynomial in y^2,
+// fitted at the Chebyshev nodes of [0, SOFT_CAP_POLY_MAX^2] (relative error 2.0e-7 with the fp32 coefficients). k = scale / cap.
+constexpr float SOFT_CAP_POLY_MAX = 0.75f;
+__device__ __forceinline__ void soft_cap_poly2(float& s0, float& s1, float k, float cap2) {
+  float y0, y1, u0, u1, p0, p1;
+  mul2(y0, y1, s0, s1, k, k);
+  mul2(u0, u1, y0, y1, y0, y1);
+  fma2(p0, p1, u0, u1, -0.004723952151834965f, -0.004723952151834965f, 0.01959378644824028f, 0.01959378644824028f);
+  fma2(p0, p1, p0, p1, u0, u1, -0.053349819034338f, -0.053349819034338f);
+  fma2(p0, p1, p0, p1, u0, u1, 0.13325515389442444f, 0.13325515389442444f);
+  fma2(p0, p1, p0, p1, u0, u1, -0.3333296775817871f, -0.3333296775817871f);
+  fma2(p0, p1, p0, p1, u0, u1, 1.f, 1.f);
+  mul2(y0, y1, y0, y1, cap2, cap2);
+  mul2(s0, s1, y0, y1, p0, p1);
+}
+
 // Epilogue helper: a warp holds a 32-row block one row per lane, each row 128 bytes as eight 16-byte chunks
 // (64 bf16 or 32 fp32 values). Writing it straight out would make every store instruction touch 32 different rows
 // with 16 bytes each; instead the block goes through a swizzled 4 KB shared-memory stage and leaves as four whole

@@ -5,9 +5,9 @@
 //   * spans: the pages a step's multi-token portions can still see are numbered densely (a compact page table) and
 //     gathered, so that their keys and values can be expanded by one product;
 //   * head gate: attention output times sigmoid(gate);
-//   * norm after the sum: x <- rms_norm(alpha x + branch), where the branch is a projection's fp32 rows or the weighted sum
-//     of expert rows (the combine step of a mixture of experts); x is updated in place and also written as the operand of
-//     the next product;
+//   * sum and norm: s = alpha x + beta branch, where the branch is a projection's fp32 rows, the weighted sum of expert
+//     rows (the combine step of a mixture of experts) or both; the norm of s is the operand of the next product, and x
+//     becomes that norm (layers that normalise after the sum) or s itself (layers that normalise before a branch);
 //   * exact (erf) GELU.
 //
 // Compiled without fast-math: these are the parts of such a model that are computed in 32 bits.
@@ -77,6 +77,7 @@ struct PrologueParams {
   const float* freq;         // [pairs] leading parts of the frequencies, then [pairs] the parts below their last bit
   float eps;
   int H, D, R, L, pairs;     // heads, unrotated and rotary size of a head, latent size, rotated pairs (2 * pairs <= R)
+  int halves;                // pair j is (j, j + pairs) of the rotary part instead of its neighbours (2j, 2j + 1)
   long long ld_page, num_slots;
   int* status;
 };
@@ -116,7 +117,19 @@ latent_prologue_kernel(T* __restrict__ proj, T* __restrict__ pages, const Prolog
     const float rs = 1.f / sqrtf(ss / (float)p.L + p.eps);
     for (int c = tid; c < p.L; c += LP_THREADS) st1(dst + c, ld1(lat + c) * rs * p.norm_w[c]);
     const T* kr = lat + p.L;
-    for (int i = tid; i < (p.R + 1) / 2; i += LP_THREADS) {
+    if (p.halves) {
+      for (int i = tid; i < p.R - p.pairs; i += LP_THREADS) {
+        if (i < p.pairs) {
+          const float u = ld1(kr + i), v = ld1(kr + i + p.pairs);
+          const float2 a = cs[i];
+          st1(dst + p.L + i, u * a.x - v * a.y);
+          st1(dst + p.L + i + p.pairs, v * a.x + u * a.y);
+        } else {
+          dst[p.L + i + p.pairs] = kr[i + p.pairs];
+        }
+      }
+    }
+    for (int i = p.halves ? p.R : tid; i < (p.R + 1) / 2; i += LP_THREADS) {
       if (i < p.pairs) {
         const float u = ld1(kr + 2 * i), v = ld1(kr + 2 * i + 1);
         const float2 a = cs[i];
@@ -127,6 +140,30 @@ latent_prologue_kernel(T* __restrict__ proj, T* __restrict__ pages, const Prolog
         if (2 * i + 1 < p.R) dst[p.L + 2 * i + 1] = kr[2 * i + 1];
       }
     }
+  }
+  if (p.halves) {
+    // two pairs at a time where the elements come as aligned bf16 pairs
+    const bool two = sizeof(T) == 2 && p.pairs % 2 == 0 && (p.D + p.R) % 2 == 0 &&
+                     (reinterpret_cast<uintptr_t>(row + p.D) & 3) == 0;
+    const int step = two ? 2 : 1, per = p.pairs / step;
+    for (int i = tid; i < p.H * per; i += LP_THREADS) {
+      const int h = i / per, j = (i - h * per) * step;
+      T* q = row + (long long)h * (p.D + p.R) + p.D + j;
+      const float2 a = cs[j];
+      if constexpr (sizeof(T) == 2) {
+        if (two) {
+          uint32_t *pu = reinterpret_cast<uint32_t*>(q), *pv = reinterpret_cast<uint32_t*>(q + p.pairs);
+          const float2 u = unpack_bf16x2(*pu), v = unpack_bf16x2(*pv), b = cs[j + 1];
+          *pu = pack_bf16x2(u.x * a.x - v.x * a.y, u.y * b.x - v.y * b.y);
+          *pv = pack_bf16x2(v.x * a.x + u.x * a.y, v.y * b.x + u.y * b.y);
+          continue;
+        }
+      }
+      const float u = ld1(q), v = ld1(q + p.pairs);
+      st1(q, u * a.x - v * a.y);
+      st1(q + p.pairs, v * a.x + u * a.y);
+    }
+    return;
   }
   const int total = p.H * p.pairs;
   for (int i = tid; i < total; i += LP_THREADS) {
@@ -241,7 +278,7 @@ __global__ void __launch_bounds__(NT) gelu_erf_kernel(const T* __restrict__ z, T
   }
 }
 
-// ---- norm after the sum ---------------------------------------------------------------------------------------------
+// ---- sum and norm ---------------------------------------------------------------------------------------------------
 template <typename TO>
 struct PostNormParams {
   float* x;                 // [rows, W] in and out
@@ -250,7 +287,8 @@ struct PostNormParams {
   const float* wts;         // [rows, k] weights of the expert rows
   const int* pos;           // [rows, k] their row numbers (< 0: none)
   int k;
-  float alpha;
+  float alpha, beta;
+  int keep;                 // x receives the sum, not its norm
   const float* w;           // [W]
   float offset, eps;
   TO* h;                    // [rows, W] operand of the next product
@@ -267,19 +305,12 @@ __global__ void __launch_bounds__(NT) post_norm_kernel(const PostNormParams<TO> 
   float* xr = p.x + (long long)r * p.W;
   float v[KEEP][VEC];
   auto sum_at = [&](int c, float (&a)[VEC]) {
+    float m[VEC];
     ldv<VEC>(xr + c, a);
 #pragma unroll
-    for (int j = 0; j < VEC; ++j) a[j] *= p.alpha;
-    if (p.y) {
-      float b[VEC];
-      ldv<VEC>(p.y + (long long)r * p.W + c, b);
-#pragma unroll
-      for (int j = 0; j < VEC; ++j) a[j] += b[j];
-    }
+    for (int j = 0; j < VEC; ++j) m[j] = 0.f;
+    if (p.y) ldv<VEC>(p.y + (long long)r * p.W + c, m);
     if (p.ys) {
-      float m[VEC];
-#pragma unroll
-      for (int j = 0; j < VEC; ++j) m[j] = 0.f;
       for (int s0 = 0; s0 < p.k; s0 += 4) {       // four rows in flight
         float b[4][VEC], ws[4];
 #pragma unroll
@@ -298,9 +329,9 @@ __global__ void __launch_bounds__(NT) post_norm_kernel(const PostNormParams<TO> 
 #pragma unroll
           for (int j = 0; j < VEC; ++j) m[j] = fmaf(ws[u], b[u][j], m[j]);
       }
-#pragma unroll
-      for (int j = 0; j < VEC; ++j) a[j] += m[j];
     }
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) a[j] = fmaf(p.beta, m[j], p.alpha * a[j]);
   };
   float ss = 0.f;
   if constexpr (NV > 0) {
@@ -325,9 +356,10 @@ __global__ void __launch_bounds__(NT) post_norm_kernel(const PostNormParams<TO> 
   auto emit = [&](int c, float (&a)[VEC]) {
     float wv[VEC];
     ldv<VEC>(p.w + c, wv);
+    if (p.keep && NV > 0) stv<VEC>(xr + c, a);
 #pragma unroll
     for (int j = 0; j < VEC; ++j) a[j] = a[j] * rs * (wv[j] + p.offset);
-    stv<VEC>(xr + c, a);
+    if (!p.keep) stv<VEC>(xr + c, a);
     stv<VEC>(p.h + (long long)r * p.W + c, a);
   };
   if constexpr (NV > 0) {
@@ -366,8 +398,8 @@ int launch_post_norm(const PostNormParams<TO>& p, cudaStream_t s) {
 
 template <typename TO>
 int post_norm(float* x, const float* y, const void* ys, const float* wts, const int* pos, int k, float alpha,
-              const float* w, float offset, float eps, void* h, int rows, int W, cudaStream_t s) {
-  PostNormParams<TO> p{x, y, (const TO*)ys, wts, pos, k, alpha, w, offset, eps, (TO*)h, rows, W};
+              float beta, int keep, const float* w, float offset, float eps, void* h, int rows, int W, cudaStream_t s) {
+  PostNormParams<TO> p{x, y, (const TO*)ys, wts, pos, k, alpha, beta, keep, w, offset, eps, (TO*)h, rows, W};
   const size_t a = sizeof(TO) == 4 ? 16 : 8;
   const bool v4 = W % 4 == 0 && al(x, 16) && (!y || al(y, 16)) && (!ys || al(ys, a)) && al(w, 16) && al(h, a);
   return v4 ? launch_post_norm<TO, 4>(p, s) : launch_post_norm<TO, 1>(p, s);
@@ -379,18 +411,18 @@ int post_norm(float* x, const float* y, const void* ys, const float* wts, const 
 using namespace edl;
 
 // proj [T, ld]: per token H query heads of (D + R), the latent (L), the rotary key (R). The first 2 * pairs of every head's
-// R rotary elements are rotated in place (neighbours form a pair); slots[t] of the page pool [num_slots, ld_page]
+// R rotary elements are rotated in place (neighbours form a pair, or with `halves` elements j and j + pairs); slots[t] of the page pool [num_slots, ld_page]
 // receives [rms_norm(latent) * norm_w | rotated key]. freq: 2 * pairs floats (leading and trailing parts).
 EDL_HOST_API int edl_latent_prologue(void* proj, int f32, long long ld, const int* pos, const int* slots,
                                      const float* norm_w, const float* freq, float eps, int T, int H, int D, int R, int L,
-                                     int pairs, void* pages, long long ld_page, long long num_slots, int* status,
+                                     int pairs, int halves, void* pages, long long ld_page, long long num_slots, int* status,
                                      void* stream) {
   if (T <= 0) return 0;
   if (H <= 0 || D < 0 || R < 0 || L <= 0 || pairs < 0 || 2 * pairs > R || pairs > LP_MAX_PAIRS || !slots || !pos) {
     set_last_error("edl_latent_prologue: bad arguments (H=%d, D=%d, R=%d, L=%d, pairs=%d)", H, D, R, L, pairs);
     return -1;
   }
-  PrologueParams p{ld, pos, slots, norm_w, freq, eps, H, D, R, L, pairs, ld_page, num_slots, status};
+  PrologueParams p{ld, pos, slots, norm_w, freq, eps, H, D, R, L, pairs, halves, ld_page, num_slots, status};
   cudaStream_t s = (cudaStream_t)stream;
   if (f32) latent_prologue_kernel<float><<<T, LP_THREADS, 0, s>>>((float*)proj, (float*)pages, p);
   else latent_prologue_kernel<__nv_bfloat16><<<T, LP_THREADS, 0, s>>>((__nv_bfloat16*)proj, (__nv_bfloat16*)pages, p);
@@ -456,17 +488,17 @@ EDL_HOST_API int edl_gelu_erf(const void* z, void* y, int f32, long long n, void
   return check_cuda(cudaGetLastError(), "gelu_erf launch");
 }
 
-// x [rows, W] fp32 <- rms_norm(alpha x + branch) * (w + offset), also written to h (fp32 or bf16). The branch is y (fp32
-// rows), or sum_s wts[r, s] * ys[pos[r, s]] over expert rows in h's type, or both.
+// x [rows, W] fp32: s = alpha x + beta branch; h (fp32 or bf16) = rms_norm(s) * (w + offset), and x becomes the same (keep =
+// 0) or s (keep = 1). The branch is y (fp32 rows), or sum_s wts[r, s] * ys[pos[r, s]] over expert rows in h's type, or both.
 EDL_HOST_API int edl_post_norm(float* x, const float* y, const void* ys, const float* wts, const int* pos, int k,
-                               float alpha, const float* w, float offset, float eps, void* h, int f32, int rows, int W,
-                               void* stream) {
+                               float alpha, float beta, int keep, const float* w, float offset, float eps, void* h,
+                               int f32, int rows, int W, void* stream) {
   if (rows <= 0) return 0;
   if (ys && (!wts || !pos || k <= 0)) {
     set_last_error("edl_post_norm: expert rows need weights and positions");
     return -1;
   }
   cudaStream_t s = (cudaStream_t)stream;
-  return f32 ? post_norm<float>(x, y, ys, wts, pos, k, alpha, w, offset, eps, h, rows, W, s)
-             : post_norm<__nv_bfloat16>(x, y, ys, wts, pos, k, alpha, w, offset, eps, h, rows, W, s);
+  return f32 ? post_norm<float>(x, y, ys, wts, pos, k, alpha, beta, keep, w, offset, eps, h, rows, W, s)
+             : post_norm<__nv_bfloat16>(x, y, ys, wts, pos, k, alpha, beta, keep, w, offset, eps, h, rows, W, s);
 }

@@ -1,9 +1,10 @@
 // Routing and expert products of a mixture of experts in inference, around the grouped tcgen05 products of gemm.cu.
 //
-//   * route: sigmoid scores of the router's fp32 logits, choice by score + correction, weights = the chosen scores over
-//     their sum. For the few tokens of a decode step the same launch also buckets the (token, choice) pairs by expert
+//   * route, from the router's fp32 logits: either sigmoid scores, choice by score + correction, weights = the chosen
+//     scores over their sum; or choice by logit, weights = the softmax over the chosen logits. For the few tokens of a decode step the same launch also buckets the (token, choice) pairs by expert
 //     (the tables that edl_moe_route builds in several launches);
-//   * clamped gated unit: g' sigmoid(alpha g') (u' + 1) with g' = min(g, limit), u' = clamp(u, +-limit), over used rows;
+//   * gated unit over used rows: silu(g) u, or clamped: g' sigmoid(alpha g') (u' + 1) with g' = min(g, limit), u' =
+//     clamp(u, +-limit);
 //   * grouped product on the general-purpose cores for models in 32 bits and sizes outside the tensor-core tiles.
 //
 // Compiled without fast-math.
@@ -25,13 +26,13 @@ __device__ __forceinline__ void put(__nv_bfloat16* p, float v) { *p = __float2bf
 
 // One warp routes one token over at most 32 * NE experts. Lane s < top returns the s-th choice and its weight.
 template <int NE>
-__device__ __forceinline__ void route_token(const float* __restrict__ logits, const float* __restrict__ corr, int E,
-                                            int top, int lane, int& mine, float& weight) {
+__device__ __forceinline__ void route_token(const float* __restrict__ logits, const float* __restrict__ corr,
+                                            bool sigmoid, int E, int top, int lane, int& mine, float& weight) {
   float score[NE], choice[NE];
 #pragma unroll
   for (int i = 0; i < NE; ++i) {
     const int e = i * 32 + lane;
-    score[i] = e < E ? 1.f / (1.f + expf(-logits[e])) : 0.f;
+    score[i] = e < E ? (sigmoid ? 1.f / (1.f + expf(-logits[e])) : logits[e]) : 0.f;
     choice[i] = e < E ? score[i] + (corr ? corr[e] : 0.f) : -INFINITY;
   }
   mine = 0;
@@ -66,18 +67,22 @@ __device__ __forceinline__ void route_token(const float* __restrict__ logits, co
       got = bs;
     }
   }
+  if (!sigmoid) {                 // lane 0 has the largest logit
+    const float top_logit = __shfl_sync(0xffffffffu, got, 0);
+    got = lane < top ? expf(got - top_logit) : 0.f;
+  }
   weight = got / (warp_sum(got) + 1e-20f);
 }
 
 template <int NE>
 __global__ void __launch_bounds__(256)
-route_kernel(const float* __restrict__ logits, const float* __restrict__ corr, int T, int E, int top,
+route_kernel(const float* __restrict__ logits, const float* __restrict__ corr, bool sigmoid, int T, int E, int top,
              long long* __restrict__ idx, float* __restrict__ wts) {
   const int lane = threadIdx.x & 31;
   for (int t = blockIdx.x * 8 + (threadIdx.x >> 5); t < T; t += gridDim.x * 8) {
     int e;
     float w;
-    route_token<NE>(logits + (long long)t * E, corr, E, top, lane, e, w);
+    route_token<NE>(logits + (long long)t * E, corr, sigmoid, E, top, lane, e, w);
     if (lane < top) {
       idx[(long long)t * top + lane] = e;
       wts[(long long)t * top + lane] = w;
@@ -88,7 +93,7 @@ route_kernel(const float* __restrict__ logits, const float* __restrict__ corr, i
 // One CTA: routing and the bucket tables of a small step.
 template <int NE>
 __global__ void __launch_bounds__(SMALL_THREADS)
-route_small_kernel(const float* __restrict__ logits, const float* __restrict__ corr, int T, int E, int top,
+route_small_kernel(const float* __restrict__ logits, const float* __restrict__ corr, bool sigmoid, int T, int E, int top,
                    float* __restrict__ wts, int* __restrict__ tile_expert, int max_tiles, int* __restrict__ meta,
                    int* __restrict__ slot_pos, int* __restrict__ row_token) {
   __shared__ int count[MAX_E], offset[MAX_E + 1];
@@ -99,7 +104,7 @@ route_small_kernel(const float* __restrict__ logits, const float* __restrict__ c
   for (int t = warp; t < T; t += SMALL_THREADS / 32) {
     int e;
     float w;
-    route_token<NE>(logits + (long long)t * E, corr, E, top, lane, e, w);
+    route_token<NE>(logits + (long long)t * E, corr, sigmoid, E, top, lane, e, w);
     if (lane < top) {
       const int i = t * top + lane;
       wts[i] = w;
@@ -143,13 +148,15 @@ route_small_kernel(const float* __restrict__ logits, const float* __restrict__ c
 
 template <typename T, int VEC>
 __global__ void __launch_bounds__(256)
-clamped_glu_kernel(const T* __restrict__ gu, const int* __restrict__ row_token, const int* __restrict__ meta,
-                   T* __restrict__ out, int F, float limit, float alpha) {
+glu_kernel(const T* __restrict__ gu, const int* __restrict__ row_token, const int* __restrict__ meta,
+           T* __restrict__ out, int F, long long rows, float limit, float alpha) {
   const int per = F / VEC;
-  const long long total = (long long)meta[1] * per;
+  const bool clamped = limit > 0.f;
+  const float k = clamped ? alpha : 1.f;
+  const long long total = (meta ? (long long)meta[1] : rows) * per;
   for (long long i = blockIdx.x * 256LL + threadIdx.x; i < total; i += gridDim.x * 256LL) {
     const long long r = i / per;
-    if (row_token[r] < 0) continue;
+    if (row_token && row_token[r] < 0) continue;
     const int c = (int)(i - r * per) * VEC;
     const T* gp = gu + r * 2 * F + c;
     alignas(16) T g_[VEC], u_[VEC], o_[VEC];
@@ -165,11 +172,14 @@ clamped_glu_kernel(const T* __restrict__ gu, const int* __restrict__ row_token, 
     }
 #pragma unroll
     for (int j = 0; j < VEC; ++j) {
-      const float g = fminf(f_of(g_[j]), limit), u = fminf(fmaxf(f_of(u_[j]), -limit), limit);
-      float s;
-      if constexpr (sizeof(T) == 4) s = g / (1.f + expf(-alpha * g));
-      else s = __fdividef(g, 1.f + __expf(-alpha * g));
-      put(&o_[j], s * (u + 1.f));
+      float g = f_of(g_[j]), u = f_of(u_[j]), s;
+      if (clamped) {
+        g = fminf(g, limit);
+        u = fminf(fmaxf(u, -limit), limit) + 1.f;
+      }
+      if constexpr (sizeof(T) == 4) s = g / (1.f + expf(-k * g));
+      else s = __fdividef(g, 1.f + __expf(-k * g));
+      put(&o_[j], s * u);
     }
     T* dst = out + r * F + c;
     if constexpr (VEC * sizeof(T) == 16) {
@@ -256,54 +266,55 @@ static int check_route(const char* who, int E, int top) {
   return 0;
 }
 
-// logits [T, E] fp32; corr [E] fp32 or null -> idx [T, top] (best first), wts [T, top].
-EDL_HOST_API int edl_moe_sigmoid_route(const float* logits, const float* corr, int T, int E, int top, long long* idx,
-                                       float* wts, void* stream) {
+// logits [T, E] fp32; corr [E] fp32 or null -> idx [T, top] (best first), wts [T, top]. sigmoid: see the top of the file.
+EDL_HOST_API int edl_moe_logit_route(const float* logits, const float* corr, int sigmoid, int T, int E, int top,
+                                     long long* idx, float* wts, void* stream) {
   if (T <= 0) return 0;
-  if (check_route("edl_moe_sigmoid_route", E, top)) return -1;
+  if (check_route("edl_moe_logit_route", E, top)) return -1;
   const int cap = 8 * sm_count(), nb = (T + 7) / 8 < cap ? (T + 7) / 8 : cap;
-#define EDL_R(NE) route_kernel<NE><<<nb, 256, 0, (cudaStream_t)stream>>>(logits, corr, T, E, top, idx, wts)
+#define EDL_R(NE) route_kernel<NE><<<nb, 256, 0, (cudaStream_t)stream>>>(logits, corr, sigmoid != 0, T, E, top, idx, wts)
   EDL_BY_EXPERTS(E, EDL_R);
 #undef EDL_R
-  return check_cuda(cudaGetLastError(), "moe_sigmoid_route launch");
+  return check_cuda(cudaGetLastError(), "moe_logit_route launch");
 }
 
 // Routing plus the bucket tables (tile_expert [max_tiles], meta [2], slot_pos [T * top], row_token [max_tiles * 128]; the
 // layout of edl_moe_route) in one launch; T * top <= 4096.
-EDL_HOST_API int edl_moe_sigmoid_route_small(const float* logits, const float* corr, int T, int E, int top, float* wts,
-                                             int* tile_expert, int max_tiles, int* meta, int* slot_pos, int* row_token,
-                                             void* stream) {
+EDL_HOST_API int edl_moe_logit_route_small(const float* logits, const float* corr, int sigmoid, int T, int E, int top,
+                                           float* wts, int* tile_expert, int max_tiles, int* meta, int* slot_pos,
+                                           int* row_token, void* stream) {
   if (T <= 0) return 0;
-  if (check_route("edl_moe_sigmoid_route_small", E, top)) return -1;
+  if (check_route("edl_moe_logit_route_small", E, top)) return -1;
   if ((long long)T * top > SMALL_PAIRS || max_tiles < (T * top + SEG - 1) / SEG + (E < T * top ? E : T * top)) {
-    set_last_error("edl_moe_sigmoid_route_small: at most %d pairs, and tables for every expert's ragged tile", SMALL_PAIRS);
+    set_last_error("edl_moe_logit_route_small: at most %d pairs, and tables for every expert's ragged tile", SMALL_PAIRS);
     return -1;
   }
 #define EDL_R(NE)                                                                                                  \
-  route_small_kernel<NE><<<1, SMALL_THREADS, 0, (cudaStream_t)stream>>>(logits, corr, T, E, top, wts, tile_expert, \
-                                                                        max_tiles, meta, slot_pos, row_token)
+  route_small_kernel<NE><<<1, SMALL_THREADS, 0, (cudaStream_t)stream>>>(logits, corr, sigmoid != 0, T, E, top, wts, \
+                                                                        tile_expert, max_tiles, meta, slot_pos, row_token)
   EDL_BY_EXPERTS(E, EDL_R);
 #undef EDL_R
-  return check_cuda(cudaGetLastError(), "moe_sigmoid_route_small launch");
+  return check_cuda(cudaGetLastError(), "moe_logit_route_small launch");
 }
 
-// gu [max_rows, 2F] (gate | up) -> out [max_rows, F], rows in use only.
-EDL_HOST_API int edl_moe_clamped_glu(const void* gu, int f32, const int* row_token, const int* meta, void* out, int F,
-                                     long long max_rows, float limit, float alpha, void* stream) {
+// gu [max_rows, 2F] (gate | up) -> out [max_rows, F], rows in use only (without tables: all rows). limit > 0: clamped unit.
+EDL_HOST_API int edl_moe_glu(const void* gu, int f32, const int* row_token, const int* meta, void* out, int F,
+                             long long max_rows, float limit, float alpha, void* stream) {
   if (max_rows <= 0 || F <= 0) return 0;
   cudaStream_t s = (cudaStream_t)stream;
   const int m = f32 ? 4 : 8;
   const bool vec = F % m == 0 && ((reinterpret_cast<uintptr_t>(gu) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
   const long long work = (max_rows * (F / (vec ? m : 1)) + 255) / 256;
   const int cap = 16 * sm_count(), nb = (int)(work < cap ? work : cap);
-#define EDL_C(T, V) clamped_glu_kernel<T, V><<<nb, 256, 0, s>>>((const T*)gu, row_token, meta, (T*)out, F, limit, alpha)
+#define EDL_C(T, V) \
+  glu_kernel<T, V><<<nb, 256, 0, s>>>((const T*)gu, row_token, meta, (T*)out, F, max_rows, limit, alpha)
   if (f32) {
     if (vec) EDL_C(float, 4); else EDL_C(float, 1);
   } else {
     if (vec) EDL_C(__nv_bfloat16, 8); else EDL_C(__nv_bfloat16, 1);
   }
 #undef EDL_C
-  return check_cuda(cudaGetLastError(), "moe_clamped_glu launch");
+  return check_cuda(cudaGetLastError(), "moe_glu launch");
 }
 
 // out [max_rows, N] = rows of a times W[e]^T, W [E, N, K]; gather != 0: row r reads a[row_token[r]].

@@ -10,7 +10,9 @@
 //   * the left half of a pass's [x ; x0] operand;
 //   * xIELU, a two-branch activation with two learned numbers;
 //   * the attention prologue: per-head RMS norm of q and k, position-dependent query temperature and the page append,
-//     in one pass over the packed projection.
+//     in one pass over the packed projection;
+//   * the same with norms over all query heads (all key heads) at once and rotated halves;
+//   * scaled and soft-capped logits.
 //
 // Compiled without fast-math: these are the parts of such a model that are computed in 32 bits.
 #include "common.cuh"
@@ -77,7 +79,7 @@ __device__ __forceinline__ int seq_of_row(const int* cu, int nseq, int r) {
 
 // ---- embedding -------------------------------------------------------------------------------------------------
 template <typename T, int VEC>
-__global__ void embed_stream_kernel(const T* __restrict__ table, const long long* __restrict__ ids,
+__global__ void embed_stream_kernel(const T* __restrict__ table, const long long* __restrict__ ids, float scale,
                                     float* __restrict__ x, T* __restrict__ right, long long ld_right, int rows, int W,
                                     int V, int* status) {
   const int per = W / VEC;
@@ -93,6 +95,8 @@ __global__ void embed_stream_kernel(const T* __restrict__ table, const long long
       for (int j = 0; j < VEC; ++j) v[j] = 0.f;
     } else {
       ldv<VEC>(table + id * W + c, v);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) v[j] *= scale;
     }
     stv<VEC>(x + (long long)r * W + c, v);
     if (right) stv<VEC>(right + r * ld_right + c, v);
@@ -538,6 +542,139 @@ qkv_prologue_small_kernel(const T* __restrict__ qkv, long long ld, const int* __
   }
 }
 
+// ---- attention prologue with full-width norms and rotation -----------------------------------------------------------------
+constexpr int RP_MAX_PAIRS = 512;     // rotated pairs of a head
+
+struct RotaryPrologueParams {
+  long long ld;
+  const int* pos;
+  const int* slots;
+  const float *qw, *kw;      // [Hq * D], [Hkv * D], or null: no norm
+  float eps;
+  const float* freq;         // [pairs] leading parts of the frequencies, then [pairs] the parts below their last bit
+  int pairs, Hq, Hkv, D, Dv;
+  long long ld_kpage, ld_vpage, num_slots;
+  int* status;
+};
+
+template <int VEC>
+__device__ __forceinline__ void ldw(const float* w, float (&v)[VEC]) {
+  if constexpr (VEC % 4 == 0) {
+#pragma unroll
+    for (int i = 0; i < VEC; i += 4) {
+      const float4 a = *reinterpret_cast<const float4*>(w + i);
+      v[i] = a.x; v[i + 1] = a.y; v[i + 2] = a.z; v[i + 3] = a.w;
+    }
+  } else {
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) v[i] = w[i];
+  }
+}
+
+// One CTA per token: qkv [T, ld] as above. Queries and keys are RMS-normed over all their heads at once, then elements j and
+// j + pairs of every head turn by position * frequency j (angles as exact as in the latent prologue: the product's rounding
+// error and the frequency's own are a small second rotation). A thread handles VEC elements and their partners.
+template <typename T, int VEC>
+__global__ void __launch_bounds__(NT)
+qkv_rotary_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, T* __restrict__ k_pages, T* __restrict__ v_pages,
+                  const RotaryPrologueParams p) {
+  __shared__ float2 cs[RP_MAX_PAIRS];
+  __shared__ float2 red[NT / 32];
+  const int t = blockIdx.x, tid = threadIdx.x;
+  const T* row = qkv + t * p.ld;
+  const int nq = p.Hq * p.D, nk = p.Hkv * p.D;
+  const float fp = p.pairs ? (float)p.pos[t] : 0.f;
+  for (int i = tid; i < p.pairs; i += NT) {
+    const float f = p.freq[i], a = fp * f;
+    const float e = fmaf(fp, f, -a) + fp * p.freq[p.pairs + i];
+    float s, c;
+    sincosf(a, &s, &c);
+    const float ce = 1.f - 0.5f * e * e, se = e - e * e * e * (1.f / 6.f);
+    cs[i] = make_float2(c * ce - s * se, s * ce + c * se);
+  }
+  float sq = 0.f, sk = 0.f;
+  if (p.qw)
+    for (int c = tid * VEC; c < nq; c += NT * VEC) {
+      float v[VEC];
+      ldv<VEC>(row + c, v);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) sq += v[j] * v[j];
+    }
+  if (p.kw)
+    for (int c = tid * VEC; c < nk; c += NT * VEC) {
+      float v[VEC];
+      ldv<VEC>(row + nq + c, v);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) sk += v[j] * v[j];
+    }
+  const float2 sums = block_sum2(sq, sk, red);       // its barriers also publish cs
+  const float rq = p.qw ? 1.f / sqrtf(sums.x / (float)nq + p.eps) : 1.f;
+  const float rk = p.kw ? 1.f / sqrtf(sums.y / (float)nk + p.eps) : 1.f;
+  long long slot = p.slots[t];
+  if (slot >= p.num_slots) {
+    if (p.status && tid == 0) atomicCAS(p.status, 0, EDL_BAD_INDEX);
+    slot = -1;
+  }
+  const int turned = p.pairs / VEC, per = turned + (p.D - 2 * p.pairs) / VEC;   // units of a head: pairs, then the rest
+  const int units = (p.Hq + (slot >= 0 ? p.Hkv : 0)) * per;
+  for (int i = tid; i < units; i += NT) {
+    const int h = i / per, u = i - h * per;
+    const bool is_q = h < p.Hq;
+    const T* src = row + h * p.D;                    // key heads follow the query heads
+    const float* w = is_q ? (p.qw ? p.qw + h * p.D : nullptr) : (p.kw ? p.kw + (h - p.Hq) * p.D : nullptr);
+    T* dst = is_q ? q_out + ((long long)t * p.Hq + h) * p.D : k_pages + slot * p.ld_kpage + (h - p.Hq) * p.D;
+    const float r = is_q ? rq : rk;
+    auto load = [&](int c, float (&v)[VEC]) {
+      ldv<VEC>(src + c, v);
+      if (w) {
+        float wv[VEC];
+        ldw<VEC>(w + c, wv);
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) v[j] *= r * wv[j];
+      }
+    };
+    float a[VEC];
+    if (u < turned) {
+      const int c = u * VEC;
+      float b[VEC];
+      load(c, a);
+      load(c + p.pairs, b);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) {
+        const float2 g = cs[c + j];
+        const float x = a[j], y = b[j];
+        a[j] = x * g.x - y * g.y;
+        b[j] = y * g.x + x * g.y;
+      }
+      stv<VEC>(dst + c, a);
+      stv<VEC>(dst + c + p.pairs, b);
+    } else {
+      const int c = 2 * p.pairs + (u - turned) * VEC;
+      load(c, a);
+      stv<VEC>(dst + c, a);
+    }
+  }
+  if (slot >= 0)
+    for (int c = tid * VEC; c < p.Hkv * p.Dv; c += NT * VEC) {
+      float v[VEC];
+      ldv<VEC>(row + nq + nk + c, v);
+      stv<VEC>(v_pages + slot * p.ld_vpage + c, v);
+    }
+}
+
+// ---- logits ------------------------------------------------------------------------------------------------------------------
+template <int VEC>
+__global__ void __launch_bounds__(NT) scale_cap_kernel(float* __restrict__ z, long long n_vec, float scale, float cap) {
+  const float k = cap > 0.f ? scale / cap : scale;
+  for (long long i = blockIdx.x * (long long)NT + threadIdx.x; i < n_vec; i += (long long)gridDim.x * NT) {
+    float v[VEC];
+    ldv<VEC>(z + i * VEC, v);
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) v[j] = cap > 0.f ? cap * tanhf(v[j] * k) : v[j] * k;
+    stv<VEC>(z + i * VEC, v);
+  }
+}
+
 int blocks_for(long long work, int per_block, int waves) {
   long long b = (work + per_block - 1) / per_block, cap = (long long)sm_count() * waves;
   return (int)(b < 1 ? 1 : (b > cap ? cap : b));
@@ -577,8 +714,8 @@ bool al(const void* p, size_t n) { return (reinterpret_cast<uintptr_t>(p) & (n -
 
 using namespace edl;
 
-// x [rows, W] fp32 = table[ids]; right (may be null): the same rows in the table's type at pitch ld_right.
-EDL_HOST_API int edl_embed_stream(const void* table, int f32, const long long* ids, float* x, void* right,
+// x [rows, W] fp32 = table[ids] * scale; right (may be null): the same rows in the table's type at pitch ld_right.
+EDL_HOST_API int edl_embed_stream(const void* table, int f32, const long long* ids, float scale, float* x, void* right,
                                   long long ld_right, int rows, int W, int V, int* status, void* stream) {
   if (rows <= 0) return 0;
   cudaStream_t s = (cudaStream_t)stream;
@@ -586,7 +723,7 @@ EDL_HOST_API int edl_embed_stream(const void* table, int f32, const long long* i
   const int vec = v4 ? 4 : 1;
   const int blocks = blocks_for((long long)rows * (W / vec), 256, 8);
 #define EDL_E(T, V_)                                                                                               \
-  embed_stream_kernel<T, V_><<<blocks, 256, 0, s>>>((const T*)table, ids, x, (T*)right, ld_right, rows, W, V, status)
+  embed_stream_kernel<T, V_><<<blocks, 256, 0, s>>>((const T*)table, ids, scale, x, (T*)right, ld_right, rows, W, V, status)
   if (f32) {
     if (v4 && (!right || al(right, 16))) EDL_E(float, 4); else EDL_E(float, 1);
   } else {
@@ -704,4 +841,47 @@ EDL_HOST_API int edl_qkv_prologue(const void* qkv, int f32, long long ld, const 
   }
 #undef EDL_P
   return check_cuda(cudaGetLastError(), "qkv_prologue launch");
+}
+
+// The prologue for queries and keys that are normed over all heads at once (qw [Hq * D], kw [Hkv * D], null: no norm) and
+// rotated by halves (freq: 2 * pairs floats, leading and trailing parts; pairs = 0: no rotation).
+EDL_HOST_API int edl_qkv_rotary_prologue(const void* qkv, int f32, long long ld, const int* pos, const int* slots,
+                                         const float* qw, const float* kw, float eps, const float* freq, int pairs, int T,
+                                         int Hq, int Hkv, int D, int Dv, void* q_out, void* k_pages, void* v_pages,
+                                         long long ld_kpage, long long ld_vpage, long long num_slots, int* status,
+                                         void* stream) {
+  if (T <= 0) return 0;
+  if (Hq <= 0 || Hkv <= 0 || D <= 0 || Dv <= 0 || !slots || pairs < 0 || 2 * pairs > D || pairs > RP_MAX_PAIRS ||
+      (pairs > 0 && (!pos || !freq))) {
+    set_last_error("edl_qkv_rotary_prologue: bad arguments (Hq=%d, Hkv=%d, D=%d, Dv=%d, pairs=%d)", Hq, Hkv, D, Dv, pairs);
+    return -1;
+  }
+  const RotaryPrologueParams p{ld, pos, slots, qw, kw, eps, freq, pairs, Hq, Hkv, D, Dv, ld_kpage, ld_vpage, num_slots, status};
+  cudaStream_t s = (cudaStream_t)stream;
+  auto fits = [&](int m, size_t a) {
+    return D % m == 0 && pairs % m == 0 && Dv % m == 0 && ld % m == 0 && ld_kpage % m == 0 && ld_vpage % m == 0 &&
+           al(qkv, a) && al(q_out, a) && al(k_pages, a) && al(v_pages, a) && (!qw || al(qw, 16)) && (!kw || al(kw, 16));
+  };
+#define EDL_RP(TT, V_) \
+  qkv_rotary_kernel<TT, V_><<<T, NT, 0, s>>>((const TT*)qkv, (TT*)q_out, (TT*)k_pages, (TT*)v_pages, p)
+  if (f32) {
+    if (fits(4, 16)) EDL_RP(float, 4); else EDL_RP(float, 1);
+  } else {
+    if (fits(8, 16)) EDL_RP(__nv_bfloat16, 8);
+    else if (fits(4, 8)) EDL_RP(__nv_bfloat16, 4);
+    else EDL_RP(__nv_bfloat16, 1);
+  }
+#undef EDL_RP
+  return check_cuda(cudaGetLastError(), "qkv_rotary_prologue launch");
+}
+
+// z <- cap * tanh(scale * z / cap), n elements in place (cap <= 0: scale * z).
+EDL_HOST_API int edl_scale_cap(float* z, long long n, float scale, float cap, void* stream) {
+  if (n <= 0) return 0;
+  cudaStream_t s = (cudaStream_t)stream;
+  const bool v4 = n % 4 == 0 && al(z, 16);
+  const int blocks = blocks_for(n / (v4 ? 4 : 1), NT, 8);
+  if (v4) scale_cap_kernel<4><<<blocks, NT, 0, s>>>(z, n / 4, scale, cap);
+  else scale_cap_kernel<1><<<blocks, NT, 0, s>>>(z, n, scale, cap);
+  return check_cuda(cudaGetLastError(), "scale_cap launch");
 }

@@ -20,7 +20,7 @@ import typing as tp
 import torch
 from torch import nn
 
-from ..ops import functional as F, stream
+from ..ops import functional as F, rotation, stream
 from .linears import ColumnParallelLinear, RowParallelLinear
 from .norms import LayerNorm, RMSNorm
 from .rotary import get_rope
@@ -61,7 +61,8 @@ class Attention(nn.Module):
                  tp_size: int = 1, tp_rank: int = 0, tp_group=None, qk_norm_offset: float = 0.0,
                  output_gate: bool = False, chunk_size: int | None = None,
                  temp_tuning: tuple[float, float] | None = None, head_scale_init: float | None = None,
-                 v_head_dim: int | None = None, norm_dtype: torch.dtype | None = None):
+                 v_head_dim: int | None = None, norm_dtype: torch.dtype | None = None,
+                 stream_rope: dict | None = None):
         super().__init__()
         # GIDD: one learned multiplier per query head on top of ``scale`` (with L2-normalised q / k it is the whole
         # temperature of the head)
@@ -105,8 +106,8 @@ class Attention(nn.Module):
             self.q_norm = RMSNorm(head_dim, qk_norm_eps, norm_dtype or dtype, offset=qk_norm_offset)
             self.k_norm = RMSNorm(head_dim, qk_norm_eps, norm_dtype or dtype, offset=qk_norm_offset)
         elif qk_norm == "rms_full":    # RMSNorm over the whole projection (OLMo2, Cohere-style full width)
-            self.q_norm = RMSNorm(self.num_heads * head_dim, qk_norm_eps, dtype)
-            self.k_norm = RMSNorm(self.num_kv_heads * head_dim, qk_norm_eps, dtype)
+            self.q_norm = RMSNorm(self.num_heads * head_dim, qk_norm_eps, norm_dtype or dtype)
+            self.k_norm = RMSNorm(self.num_kv_heads * head_dim, qk_norm_eps, norm_dtype or dtype)
         elif qk_norm == "layer_head":  # per-head LayerNorm without bias (Cohere, StableLM per-head)
             self.q_norm = LayerNorm(head_dim, qk_norm_eps, bias=False, dtype=dtype)
             self.k_norm = LayerNorm(head_dim, qk_norm_eps, bias=False, dtype=dtype)
@@ -117,6 +118,11 @@ class Attention(nn.Module):
         self.rotary = None
         if rope is not None:
             self.rotary = get_rope(head_size=head_dim, **rope)
+        # fp32-stream layers: base / dims / scaling of angles that are computed in place instead of read from a table
+        self.stream_rope = stream_rope
+        self._freq: torch.Tensor | None = None
+        if stream_rope is not None:
+            rotation.check_rotation(stream_rope["dims"], head_dim, "halves")
         self.sinks = nn.Parameter(torch.zeros(self.num_heads, dtype=torch.float32)) if use_sinks else None
         if use_alibi:
             sl = alibi_slopes(num_heads)[tp_rank * self.num_heads:(tp_rank + 1) * self.num_heads]
@@ -219,16 +225,24 @@ class Attention(nn.Module):
 
     def mix_stream(self, h: torch.Tensor, step, cache_view=None) -> torch.Tensor:
         """Form for layers over an fp32 residual stream: h ``[T, hidden]`` (all sequences on one axis) ->
-        ``[T, heads * v_head_dim]`` before the output projection, which the layer accumulates into the stream. Per-head
-        q / k norms, the query temperature and the page append are one kernel over the packed projection. ``step``:
-        :class:`..modules._base.decoder.StreamStep`."""
+        ``[T, heads * v_head_dim]`` before the output projection, which the layer accumulates into the stream. One kernel
+        over the packed projection does per-head q / k norms, the query temperature and the page append, or norms over the
+        whole projection, the rotation and the page append. ``step``: :class:`..modules._base.decoder.StreamStep`."""
+        turned = self.stream_rope is not None or self.qk_norm == "rms_full"
         if self.rotary is not None or self.alibi is not None or self.output_gate or self.clip_qkv is not None or \
-                self.head_scale is not None or self.chunk_size or self.qk_norm not in (None, "rms_head"):
-            raise NotImplementedError("fp32-stream attention covers plain, per-head-normed and tempered heads")
+                self.head_scale is not None or self.chunk_size or self.qk_norm not in (None, "rms_head", "rms_full") or \
+                (turned and (self.qk_norm == "rms_head" or self.temp_tuning is not None)):
+            raise NotImplementedError("fp32-stream attention covers plain, per-head-normed and tempered heads, or heads "
+                                      "rotated after a norm over the whole projection")
         qkv = stream.linear(h, self.qkv_proj.weight, self.qkv_proj.bias)
         T = h.shape[0]
         Hq, Hkv, D, Dv = self.num_heads, self.num_kv_heads, self.head_dim, self.v_head_dim
         qw, kw = (self.q_norm.weight, self.k_norm.weight) if self.qk_norm else (None, None)
+        freq = self._frequencies(qkv.device) if turned else None
+        if cache_view is not None and turned:
+            q = stream.qkv_rotary_prologue(qkv, (Hq, Hkv, D, Dv), qw, kw, self.qk_norm_eps, step.positions, freq,
+                                           step.meta.slots_of(cache_view.group), cache_view.k_pages, cache_view.v_pages)
+            return cache_view.attend_pages(self, q, step.meta).reshape(T, Hq * Dv)
         if cache_view is not None:
             q = stream.qkv_prologue(qkv, (Hq, Hkv, D, Dv), qw, kw, self.qk_norm_eps, step.positions, self.temp_tuning,
                                     step.meta.slots_of(cache_view.group), cache_view.k_pages, cache_view.v_pages)
@@ -237,13 +251,22 @@ class Attention(nn.Module):
         from ..ops import reference as R
 
         q, k, v = torch.split(qkv, [Hq * D, Hkv * D, Hkv * Dv], -1)
-        q, k = stream.qk_norm_temper(q.reshape(T, Hq, D), k.reshape(T, Hkv, D), qw, kw, self.qk_norm_eps,
-                                     step.positions, self.temp_tuning)
+        if turned:
+            q, k = stream.qk_norm_rotate(q, k, D, qw, kw, self.qk_norm_eps, step.positions, freq)
+        else:
+            q, k = stream.qk_norm_temper(q.reshape(T, Hq, D), k.reshape(T, Hkv, D), qw, kw, self.qk_norm_eps,
+                                         step.positions, self.temp_tuning)
         B = step.batch
         o = R.attention(q.view(B, T // B, Hq, D), k.view(B, T // B, Hkv, D), v.reshape(B, T // B, Hkv, Dv),
                         causal=self.causal, scale=self.scale, segment_ids=step.segment_ids,
                         sliding_window=self.sliding_window, softcap=self.softcap, sinks=self.sinks)
         return o.reshape(T, Hq * Dv)
+
+    def _frequencies(self, device) -> torch.Tensor | None:
+        r = self.stream_rope
+        if r is not None and (self._freq is None or self._freq.device != device):
+            self._freq = rotation.pair_frequencies(r["base"], r["dims"], device, r.get("scaling"))
+        return self._freq
 
     def _alibi_attention(self, q, k, v, segment_ids):
         # ALiBi families (Falcon-RW, MPT, BLOOM-style) are served by the dense oracle path: a

@@ -13,7 +13,7 @@ from __future__ import annotations
 import torch
 from torch import nn
 
-from ..ops import functional as F, latent, stream
+from ..ops import functional as F, latent, rotation, stream
 from ..ops import reference as R
 from .linears import ColumnParallelLinear, RowParallelLinear
 from .norms import RMSNorm
@@ -199,8 +199,8 @@ class MLAttention(nn.Module):
 
 
 class LatentStreamAttention(nn.Module):
-    """Latent attention of layers over an fp32 residual stream, with a sliding window, a sink per head, rotary pairs on
-    neighbouring channels of the rotary part and an output gate (each optional).
+    """Latent attention of layers over an fp32 residual stream, with a sliding window, a sink per head, rotary pairs
+    (neighbouring channels of the rotary part, or its halves) and an output gate (each optional).
 
     One packed product gives the queries of every head, the latent, the shared rotary key and the gate; the two
     up-projections (unrotated keys, values) are stacked. The cache holds rows ``[normalised latent | rotated key]``;
@@ -209,7 +209,8 @@ class LatentStreamAttention(nn.Module):
     def __init__(self, hidden_size: int, heads: int, *, dim: int, rot_dim: int, vdim: int, kv_rank: int, scale: float,
                  rope_base: float = 10000.0, rope_dims: int | None = None, sliding_window: int | None = None,
                  use_sinks: bool = False, output_gate: bool = False, norm_eps: float = 1e-6, layer_idx: int = 0,
-                 dtype=torch.bfloat16, init_std: float = 0.02):
+                 dtype=torch.bfloat16, init_std: float = 0.02, rope_layout: str = "neighbours",
+                 rope_scaling: dict | None = None):
         super().__init__()
         self.heads, self.dim, self.rot_dim, self.vdim, self.kv_rank = heads, dim, rot_dim, vdim, kv_rank
         self.scale, self.sliding_window, self.output_gate = scale, sliding_window, output_gate
@@ -226,16 +227,16 @@ class LatentStreamAttention(nn.Module):
         self.o_proj = RowParallelLinear(heads * vdim, hidden_size, bias=False, **kw)
         self.sinks = nn.Parameter(torch.zeros(heads, dtype=torch.float32)) if use_sinks else None
         dims = rot_dim if rope_dims is None else rope_dims
-        if dims % 2 or dims > rot_dim:
-            raise ValueError(f"{dims} rotated channels of a rotary part of {rot_dim}")
+        rotation.check_rotation(dims, rot_dim, rope_layout)
         self.rope_base, self.rope_dims = float(rope_base), dims
+        self.rope_layout, self.rope_scaling = rope_layout, rope_scaling
         self.tiles = latent.tiles_support(self)
         self._freq: torch.Tensor | None = None
         self._expansion: tuple | None = None
 
     def frequencies(self, device) -> torch.Tensor:
         if self._freq is None or self._freq.device != device:
-            self._freq = latent.pair_frequencies(self.rope_base, self.rope_dims, device)
+            self._freq = rotation.pair_frequencies(self.rope_base, self.rope_dims, device, self.rope_scaling)
         return self._freq
 
     def expansion(self) -> torch.Tensor:
@@ -256,13 +257,13 @@ class LatentStreamAttention(nn.Module):
         if cache_view is not None:
             meta, pages = step.meta, cache_view.pages
             latent.prologue(proj, (H, D, R, L), self.kv_norm.weight, self.eps, freq, step.positions,
-                            meta.slots_of(cache_view.group), pages)
+                            meta.slots_of(cache_view.group), pages, self.rope_layout)
             return latent.attend(self, proj, pages, meta, meta.table_of(cache_view.group), cache_view.group)
         # no cache (autograd): the batch's rows are equally long
         q, c, kr, gate = latent.split_packed(proj, H, D, R, L)
         pos = step.positions
-        q = torch.cat([q[..., :D], latent.rotate_pairs(q[..., D:], pos, freq)], -1)
-        c, kr = latent.latent_norm(c, self.kv_norm.weight, self.eps), latent.rotate_pairs(kr, pos, freq)
+        q = torch.cat([q[..., :D], rotation.rotate(q[..., D:], pos, freq, self.rope_layout)], -1)
+        c, kr = latent.latent_norm(c, self.kv_norm.weight, self.eps), rotation.rotate(kr, pos, freq, self.rope_layout)
         B = step.batch
         fold = lambda t: t.reshape(B, t.shape[0] // B, *t.shape[1:])  # noqa: E731
         up = self.ukv_proj.weight

@@ -38,6 +38,13 @@ class GatedMLP(nn.Module):
         y = self.down_proj(F.gated_act(gu, self.act))
         return y if self.down_multiplier == 1.0 else y * self.down_multiplier
 
+    def stream_rows(self, h: torch.Tensor, base: torch.Tensor | None = None) -> torch.Tensor:
+        """Branch of a layer over an fp32 residual stream as fp32 rows, added to the rows ``base`` if there are any."""
+        if self.gate_multiplier != 1.0 or self.down_multiplier != 1.0 or self.down_proj.bias is not None:
+            raise NotImplementedError("fp32-stream feed-forwards: no multipliers, no bias on the way down")
+        gu = stream.linear(h, self.gate_up_proj.weight, self.gate_up_proj.bias)
+        return stream.branch_product(stream.gated_unit(gu, self.act), self.down_proj.weight, base)
+
 
 class PlainMLP(nn.Module):
     """``fc2(act(fc1(x)))`` (GPT-2, OPT, Falcon, GPT-NeoX, Phi, StarCoder...)."""
@@ -62,9 +69,9 @@ class PlainMLP(nn.Module):
             return stream.xielu(z, self.act_params)
         return stream.gelu_erf(z) if self.act == "gelu" and stream.on_kernels(z) else ACT2FN[self.act](z)
 
-    def stream_rows(self, h: torch.Tensor) -> torch.Tensor:
-        """Branch of a layer over an fp32 residual stream: fp32 rows for :func:`..ops.stream.post_norm`."""
-        return stream.linear(self.hidden(h), self.fc2.weight, self.fc2.bias, torch.float32)
+    def stream_rows(self, h: torch.Tensor, base: torch.Tensor | None = None) -> torch.Tensor:
+        """Branch of a layer over an fp32 residual stream as fp32 rows, added to the rows ``base`` if there are any."""
+        return stream.branch_product(self.hidden(h), self.fc2.weight, base, self.fc2.bias)
 
     def forward(self, x: torch.Tensor) -> torch.Tensor:
         return self.fc2(self.hidden(x))

@@ -337,19 +337,25 @@ class MoEBlock(nn.Module):
         return y.view(shape), logits
 
     # ------------------------------------------------------------------ fp32-stream layers
-    def stream_rows(self, h: torch.Tensor):
-        """Branch of a layer over an fp32 residual stream: h ``[T, H]`` -> what :func:`..ops.stream.post_norm` adds to the
-        stream, either expert rows with their weights (kernels) or fp32 rows. Router logits and scores are fp32."""
+    def stream_rows(self, h: torch.Tensor, base: torch.Tensor | None = None):
+        """Branch of a layer over an fp32 residual stream: h ``[T, H]`` -> what :func:`..ops.stream.post_norm` or
+        ``add_norm`` adds to the stream, either expert rows with their weights (kernels) or fp32 rows. ``base``: fp32 rows
+        of other parts of the branch; shared experts add theirs. Router logits and scores are fp32."""
+        sigmoid = self.scoring == "sigmoid"
+        plain = (sigmoid or self.scoring == "softmax" and self.e_score_correction_bias is None) and self.norm_topk_prob and \
+            self.routing_strategy is None and self.n_group == 1 and self.capacity_factor is None and \
+            self.routed_scaling_factor == 1.0 and self.shared_expert_gate is None and not self.scale_input
+        if not plain or self.ep_size > 1 or self.gate_up_proj.bias is not None or \
+                (self.act_limit is None and self.act != "silu"):
+            raise NotImplementedError("fp32-stream experts: sigmoid or softmax scores, renormalised; silu or clamped units")
         logits = stream.linear(h, self.gate.weight, self.gate.bias, torch.float32)
-        plain = self.scoring == "sigmoid" and self.norm_topk_prob and self.routing_strategy is None and \
-            self.n_group == 1 and self.capacity_factor is None and self.routed_scaling_factor == 1.0
-        if self.act_limit is None or not plain or self.shared_experts is not None or self.ep_size > 1 or \
-                self.gate_up_proj.bias is not None:
-            raise NotImplementedError("fp32-stream experts: sigmoid scores, renormalised, clamped gated units")
+        if self.shared_experts is not None:
+            base = self.shared_experts.stream_rows(h, base)
         if stream.on_kernels(h):
             from ..ops import moe_kernels as MK
 
-            r = MK.SigmoidRouting(logits, self.e_score_correction_bias, self.top_k)
-            return MK.clamped_experts(h, r, self.gate_up_proj.weight, self.down_proj.weight, self.act_limit)
+            r = MK.LogitRouting(logits, self.top_k, sigmoid, self.e_score_correction_bias)
+            return MK.stream_experts(h, r, self.gate_up_proj.weight, self.down_proj.weight, self.act_limit, base=base)
         w, idx, _ = self.route(logits)
-        return G.moe_ffn(h, self.gate_up_proj.weight, self.down_proj.weight, w, idx, self.act).float()
+        rows = G.moe_ffn(h, self.gate_up_proj.weight, self.down_proj.weight, w, idx, self.act).float()
+        return rows if base is None else base + rows

@@ -15,6 +15,8 @@ from dataclasses import dataclass, field
 
 import torch
 
+from ..ops.rotation import llama3_scaling
+
 
 def _base_inv_freq(base: float, rotary_dim: int) -> torch.Tensor:
     return 1.0 / (base ** (torch.arange(0, rotary_dim, 2, dtype=torch.float32) / rotary_dim))
@@ -106,17 +108,9 @@ def get_inv_frequencies(rope: RopeConfig, base: float, rotary_dim: int, max_posi
         nb = base * ((factor * sl / orig) - (factor - 1)) ** (rotary_dim / (rotary_dim - 2))
         inv = _base_inv_freq(nb, rotary_dim)
     elif t == "llama3":
-        factor = float(rope.factor or 8.0)
-        lo = float(rope.low_freq_factor or 1.0)
-        hi = float(rope.high_freq_factor or 4.0)
-        old = float(rope.original_max_position_embeddings or 8192)
-        low_wl, high_wl = old / lo, old / hi
-        wl = 2 * math.pi / inv
-        scaled = torch.where(wl > low_wl, inv / factor, inv)
-        smooth = (old / wl - lo) / (hi - lo)
-        smoothed = (1 - smooth) * inv / factor + smooth * inv
-        mid = (wl >= high_wl) & (wl <= low_wl)
-        inv = torch.where(mid, smoothed, scaled)
+        inv = llama3_scaling(inv, float(rope.factor or 8.0), float(rope.low_freq_factor or 1.0),
+                             float(rope.high_freq_factor or 4.0),
+                             float(rope.original_max_position_embeddings or 8192))
     elif t in ("yarn", "deepseek_yarn"):
         factor = float(rope.factor or 1.0)
         orig = rope.original_max_position_embeddings or max_position

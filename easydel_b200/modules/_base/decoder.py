@@ -99,7 +99,8 @@ class ArchSpec:
     attn_scale: float | None = None
     sliding_window: int | None = None
     layer_types: tuple[str, ...] | None = None  # per layer: "full" | "sliding" | "nope" (full, no rope)
-    residual: str = "pre"             # pre | parallel | post (norm applied to the branch output, OLMo2) | post_sum
+    residual: str = "pre"             # pre | parallel (x + mixer(h) + mlp(h), h = norm(x); fp32-stream models too) |
+                                      # post (norm applied to the branch output, OLMo2) | post_sum
                                       # (x <- norm(residual_alpha x + branch), branches read x; fp32-stream models)
     sandwich_norm: bool = False       # extra norms after attention / MLP outputs (Gemma2/3)
     shared_parallel_norm: bool = True  # parallel residual with one norm (GPT-J, Phi) vs two (NeoX)
@@ -132,6 +133,7 @@ class ArchSpec:
     branch_multipliers: tuple[float, float, float] = (1.0, 1.0, 1.0)  # attention input, attention output, SSM output
     mlp_multipliers: tuple[float, float] = (1.0, 1.0)                  # gate pre-activation, MLP output
     residual_f32: bool = False        # the residual stream is fp32 [tokens, hidden]; branches accumulate into it
+    stream_rope: dict | None = None   # base / dims / scaling of rotated halves in fp32-stream attention layers, see ops.rotation
     token_shift: bool = False         # every mixer reads h + (h of the previous token - h) * shift (fp32-stream models)
     v_head_dim: int | None = None     # width of a value head when it differs from head_dim (fp32-stream models)
     hgrn2: dict | None = None         # heads / dim / vdim of layers.hgrn2.HGRN2Mixer for layers of type "hgrn2"
@@ -175,6 +177,10 @@ def _norm(spec: ArchSpec, dtype) -> nn.Module:
         return LayerNorm(spec.hidden_size, spec.norm_eps if spec.norm_eps > 1e-6 else 1e-5, dtype=dtype,
                          elementwise_affine=False)
     return LayerNorm(spec.hidden_size, spec.norm_eps, bias=spec.norm_bias, dtype=dtype)
+
+
+def _residual_multiplier(spec: ArchSpec) -> float:
+    return 1.0 if spec.residual_multiplier is None else float(spec.residual_multiplier)
 
 
 def _resolve(x):
@@ -281,7 +287,7 @@ class DecoderLayer(nn.Module):
             use_alibi=spec.pos_emb == "alibi", clip_qkv=spec.clip_qkv, dtype=dtype, init_std=spec.init_std,
             tp_size=tp_size, tp_rank=tp_rank, tp_group=tp_group, qk_norm_offset=spec.norm_offset,
             output_gate=spec.attn_output_gate, v_head_dim=spec.v_head_dim,
-            norm_dtype=torch.float32 if spec.residual_f32 else None)
+            norm_dtype=torch.float32 if spec.residual_f32 else None, stream_rope=spec.stream_rope)
 
     def _build_mlp(self, config, spec, layer_idx, dtype, tp_size, tp_rank, tp_group):
         moe = spec.moe
@@ -369,20 +375,27 @@ class DecoderLayer(nn.Module):
         return LayerSlotState(zeros(spec.hidden_size) if self.shift is not None else None,
                               zeros(m.heads, m.dim, m.vdim) if m is not None else None)
 
+    @property
+    def _stream_mixer(self) -> nn.Module:
+        return self.linear_attn if self.ltype == "hgrn2" else self.self_attn
+
+    def _mix_stream(self, h: torch.Tensor, step: StreamStep, view) -> torch.Tensor:
+        """The mixer's output before its output projection."""
+        if self.ltype == "hgrn2":
+            state = view.linear_state if view is not None else None
+            return self.linear_attn(h, step, None if state is None else state.recurrent)
+        return self.self_attn.mix_stream(h, step, view)
+
     def _forward_stream(self, x: torch.Tensor, step: StreamStep, view):
         """One layer on the fp32 stream ``x [T, hidden]``: norm (+ token shift) -> mixer -> the output projection
         accumulates into the stream; then norm -> MLP likewise."""
         spec = self.spec
-        mixer = self.linear_attn if self.ltype == "hgrn2" else self.self_attn
+        mixer = self._stream_mixer
         dt = mixer.o_proj.weight.dtype
         state = view.linear_state if view is not None else None
         h = stream.norm_shift(x, self.input_layernorm.weight, spec.norm_eps, dt, mu=self.shift, cu=step.cu,
                               slots=step.slots, state=None if state is None else state.shift)
-        if self.ltype == "hgrn2":
-            o = mixer(h, step, None if state is None else state.recurrent)
-        else:
-            o = mixer.mix_stream(h, step, view)
-        x = stream.linear_add_(x, o, mixer.o_proj.weight)
+        x = stream.linear_add_(x, self._mix_stream(h, step, view), mixer.o_proj.weight)
         if self.mlp is not None:
             h = stream.norm_shift(x, self.post_attention_layernorm.weight, spec.norm_eps, dt)
             x = stream.linear_add_(x, self.mlp.hidden(h), self.mlp.fc2.weight)
@@ -402,8 +415,20 @@ class DecoderLayer(nn.Module):
             x, h = stream.post_norm(x, branch, spec.residual_alpha, n2.weight, spec.norm_eps, h.dtype, n2.offset)
         return x, h
 
+    def _forward_parallel_stream(self, x: torch.Tensor, pending, step: StreamStep, view):
+        """One layer on the fp32 stream ``x [T, hidden]`` whose branches both read one norm of it. ``pending`` is what the
+        layer before adds to the stream (None: nothing), times the residual multiplier: that sum and this layer's norm are
+        one pass. Returns the stream and this layer's own pending sum."""
+        spec, n, mixer = self.spec, self.input_layernorm, self._stream_mixer
+        x, h = stream.add_norm(x, pending, _residual_multiplier(spec), n.weight, spec.norm_eps, mixer.o_proj.weight.dtype,
+                               n.offset)
+        branch = stream.branch_product(self._mix_stream(h, step, view), mixer.o_proj.weight)
+        return x, branch if self.mlp is None else self.mlp.stream_rows(h, branch)
+
     def forward(self, x, pending, positions, segment_ids=None, cache_view=None, attn_meta=None):
         spec = self.spec
+        if spec.residual_f32 and spec.residual == "parallel":
+            return *self._forward_parallel_stream(x, pending, attn_meta, cache_view), None
         if spec.residual == "post_sum":
             return *self._forward_post_sum(x, pending, attn_meta, cache_view), None
         if spec.residual_f32:
@@ -713,17 +738,20 @@ def _forward_stream(self, input_ids, inputs_embeds, attention_mask, position_ids
         flat = flat[index]
     n = flat.numel() if flat is not None else (index.numel() if index is not None else B * T)
     operand = right = None
-    h = None                              # "post_sum" layers: the stream's rows in the operand type
+    # "post_sum" layers: the stream's rows in the operand type; "parallel" layers: what the last one adds to the stream
+    h = None
+    parallel, mult = spec.residual == "parallel", _residual_multiplier(spec)
     if spec.residual == "post_sum":
         right = h = torch.empty(n, W, dtype=self.embed_tokens.weight.dtype, device=self.device)
     if spec.loop is not None:             # [x ; x0]: x0 is written once, x before every pass
         operand = torch.empty(n, 2 * W, dtype=self.loop_in.weight.dtype, device=self.device)
         right = operand[:, W:]
+    scale = 1.0 if spec.embed_scale is None else float(spec.embed_scale)
     if inputs_embeds is None:
-        x = stream.embed(self.embed_tokens.weight, flat, right)
+        x = stream.embed(self.embed_tokens.weight, flat, right, scale)
     else:
         x = inputs_embeds.reshape(B * T, W)
-        x = (x if index is None else x[index]).float()
+        x = (x if index is None else x[index]).float() * scale
         if right is not None:
             stream.cast_rows(x, right)
         x = x.clone()
@@ -740,10 +768,10 @@ def _forward_stream(self, input_ids, inputs_embeds, attention_mask, position_ids
                 x = stream.linear(operand, self.loop_in.weight, bias, torch.float32)
             done += 1
         if hidden is not None:
-            hidden.append(x.clone())
+            hidden.append(x + mult * stream.branch_rows(h) if parallel and h is not None else x.clone())
         view = cache.view(run) if cache is not None else None
         x, h, _ = self.layers[i](x, h, step.positions, None, view, step)
-    x = stream.norm_shift(x, self.norm.weight, spec.norm_eps, dt, offset=self.norm.offset)
+    x = stream.add_norm(x, h if parallel else None, mult, self.norm.weight, spec.norm_eps, dt, self.norm.offset)[1]
 
     def unflatten(t):
         if index is not None:
@@ -806,6 +834,8 @@ class DecoderForCausalLM(EasyDeLBaseModule):
         if spec.residual_f32:      # the head's accumulators are the logits: no 16-bit rounding of them
             out = stream.linear(hidden.reshape(-1, hidden.shape[-1]), self.lm_head_weight(), self.lm_head_bias(),
                                 torch.float32)
+            if spec.logit_scale is not None or spec.logit_softcap:
+                out = stream.scale_cap(out, 1.0 if spec.logit_scale is None else spec.logit_scale, spec.logit_softcap)
             return out.view(*hidden.shape[:-1], out.shape[-1])
         logits = F.linear(hidden, self.lm_head_weight(), self.lm_head_bias())
         if spec.logit_scale is not None:

@@ -18,32 +18,14 @@ from __future__ import annotations
 import torch
 
 from . import _lib, kernels as K, serving as S, stream
+from .rotation import rotate
 
 vp, i32, i64, f32 = _lib.vp, _lib.i32, _lib.i64, _lib.f32
-_lib.register("edl_latent_prologue", i32, [vp, i32, i64, vp, vp, vp, vp, f32, i32, i32, i32, i32, i32, i32, vp, i64, i64, vp,
-                                           vp])
+_lib.register("edl_latent_prologue", i32, [vp, i32, i64, vp, vp, vp, vp, f32, i32, i32, i32, i32, i32, i32, i32, vp, i64, i64,
+                                           vp, vp])
 _lib.register("edl_latent_spans", i32, [vp, vp, vp, i32, i32, i32, i32, i32, i32, vp, vp, vp, vp])
 _lib.register("edl_gather_pages", i32, [vp, vp, vp, i32, i64, vp])
 _lib.register("edl_head_gate", i32, [vp, i32, i64, i64, vp, i64, vp, i64, i32, i32, i32, vp])
-
-
-def pair_frequencies(base: float, dims: int, device=None) -> torch.Tensor:
-    """``base^(-2i / dims)`` for i < dims / 2 as fp32 leading parts followed by the fp32 remainders."""
-    f = float(base) ** (-torch.arange(0, dims, 2, dtype=torch.float64) / dims)
-    hi = f.float()
-    return torch.cat([hi, (f - hi.double()).float()]).to(device)
-
-
-def rotate_pairs(x: torch.Tensor, positions: torch.Tensor, freq: torch.Tensor) -> torch.Tensor:
-    """Tensor form: neighbours (2i, 2i + 1) of the first ``2 * pairs`` elements of ``x [T, ..., R]`` turned by
-    ``position * frequency``; computed in fp32, cast back."""
-    n = freq.numel() // 2
-    a = positions.double()[:, None] * (freq[:n].double() + freq[n:].double())
-    c, s = torch.cos(a).float(), torch.sin(a).float()
-    c, s = (t.view(t.shape[0], *[1] * (x.dim() - 2), n) for t in (c, s))
-    u, v = x[..., 0:2 * n:2].float(), x[..., 1:2 * n:2].float()
-    r = torch.stack([u * c - v * s, v * c + u * s], -1).flatten(-2).to(x.dtype)
-    return torch.cat([r, x[..., 2 * n:]], -1)
 
 
 def split_packed(proj: torch.Tensor, H: int, D: int, R: int, L: int):
@@ -58,21 +40,21 @@ def latent_norm(c: torch.Tensor, w: torch.Tensor, eps: float) -> torch.Tensor:
 
 
 def prologue(proj: torch.Tensor, heads: tuple[int, int, int, int], norm_w: torch.Tensor, eps: float, freq: torch.Tensor,
-             positions: torch.Tensor, slot_mapping: torch.Tensor, pages: torch.Tensor) -> None:
+             positions: torch.Tensor, slot_mapping: torch.Tensor, pages: torch.Tensor, layout: str = "neighbours") -> None:
     """Rotates the queries inside ``proj [T, ld]`` and writes the cache rows to ``pages [P, page, 1, L + R]``.
-    ``heads = (H, D, R, L)``."""
+    ``heads = (H, D, R, L)``; ``layout``: see :mod:`.rotation`."""
     H, D, R, L = heads
     T = proj.shape[0]
     if stream.on_kernels(proj):
         pos = positions.reshape(-1).to(torch.int32)
         _lib.call("edl_latent_prologue", proj.data_ptr(), stream._f32flag(proj.dtype), proj.stride(0), pos.data_ptr(),
                   slot_mapping.data_ptr(), norm_w.data_ptr(), freq.data_ptr(), float(eps), T, H, D, R, L, freq.numel() // 2,
-                  pages.data_ptr(), pages.stride(1), pages.shape[0] * pages.shape[1],
+                  int(layout == "halves"), pages.data_ptr(), pages.stride(1), pages.shape[0] * pages.shape[1],
                   _lib.status_word(proj.device).data_ptr(), _lib.stream_ptr())
         return
     q, c, kr, _ = split_packed(proj, H, D, R, L)
-    q[..., D:] = rotate_pairs(q[..., D:], positions, freq)
-    row = torch.cat([latent_norm(c, norm_w, eps), rotate_pairs(kr, positions, freq)], -1)
+    q[..., D:] = rotate(q[..., D:], positions, freq, layout)
+    row = torch.cat([latent_norm(c, norm_w, eps), rotate(kr, positions, freq, layout)], -1)
     S.kv_append(row[:, None], row[:, None], pages, pages, slot_mapping)
 
 

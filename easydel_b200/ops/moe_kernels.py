@@ -237,9 +237,9 @@ def grouped_linear(x_sorted, w, group_sizes):
 
 
 # ------------------------------------------------------------------------------------------------ fp32-stream inference
-_lib.register("edl_moe_sigmoid_route", i32, [vp, vp, i32, i32, i32, vp, vp, vp])
-_lib.register("edl_moe_sigmoid_route_small", i32, [vp, vp, i32, i32, i32, vp, vp, i32, vp, vp, vp, vp])
-_lib.register("edl_moe_clamped_glu", i32, [vp, i32, vp, vp, vp, i32, i64, _lib.f32, _lib.f32, vp])
+_lib.register("edl_moe_logit_route", i32, [vp, vp, i32, i32, i32, i32, vp, vp, vp])
+_lib.register("edl_moe_logit_route_small", i32, [vp, vp, i32, i32, i32, i32, vp, vp, i32, vp, vp, vp, vp])
+_lib.register("edl_moe_glu", i32, [vp, i32, vp, vp, vp, i32, i64, _lib.f32, _lib.f32, vp])
 _lib.register("edl_moe_grouped_simt", i32, [vp, i32, i64, vp, i32, vp, vp, vp, vp, i32, i32, i32, vp])
 
 SMALL_ROUTE_PAIRS = 4096      # (token, choice) pairs that one launch routes and buckets
@@ -247,30 +247,33 @@ SMALL_ROUTE_PAIRS = 4096      # (token, choice) pairs that one launch routes and
 
 class ExpertRows:
     """Outputs of the routed experts before they are combined: token t's branch is ``sum_s weights[t, s] *
-    ys[pos[t, s]]``. The norm that follows an fp32-stream layer's branch takes them in this form
-    (:func:`.stream.post_norm`)."""
+    ys[pos[t, s]]``, plus the fp32 rows ``base`` where there are some (other parts of the same branch). The norm that
+    follows an fp32-stream layer's branch takes them in this form (:func:`.stream.post_norm`, :func:`.stream.add_norm`)."""
 
-    def __init__(self, ys: torch.Tensor, weights: torch.Tensor, pos: torch.Tensor):
-        self.ys, self.weights, self.pos = ys, weights, pos
+    def __init__(self, ys: torch.Tensor, weights: torch.Tensor, pos: torch.Tensor, base: torch.Tensor | None = None):
+        self.ys, self.weights, self.pos, self.base = ys, weights, pos, base
         self.k = weights.shape[1]
 
     def combine(self) -> torch.Tensor:
         p = self.pos.view(self.weights.shape).long()
-        return (self.ys[p.clamp_min(0)].float() * (self.weights * (p >= 0))[..., None]).sum(1)
+        out = (self.ys[p.clamp_min(0)].float() * (self.weights * (p >= 0))[..., None]).sum(1)
+        return out if self.base is None else out + self.base
 
 
-class SigmoidRouting(Routing):
-    """Routing tables straight from fp32 router logits ``[T, E]``: sigmoid scores, choice by score + ``correction``,
-    weights = the chosen scores over their sum. A decode step's few tokens take one launch."""
+class LogitRouting(Routing):
+    """Routing tables straight from fp32 router logits ``[T, E]``. ``sigmoid``: sigmoid scores, choice by score +
+    ``correction``, weights = the chosen scores over their sum; otherwise choice by logit, weights = the softmax over the
+    chosen logits. A decode step's few tokens take one launch."""
 
-    def __init__(self, logits: torch.Tensor, correction: torch.Tensor | None, top_k: int):
+    def __init__(self, logits: torch.Tensor, top_k: int, sigmoid: bool, correction: torch.Tensor | None = None):
+        sig = int(sigmoid)
         T, E = logits.shape
         dev = logits.device
         self.weights = torch.empty(T, top_k, dtype=torch.float32, device=dev)
         corr = _lib.ptr(correction)
         if T * top_k > SMALL_ROUTE_PAIRS:
             idx = torch.empty(T, top_k, dtype=torch.int64, device=dev)
-            _lib.call("edl_moe_sigmoid_route", logits.data_ptr(), corr, T, E, top_k, idx.data_ptr(),
+            _lib.call("edl_moe_logit_route", logits.data_ptr(), corr, sig, T, E, top_k, idx.data_ptr(),
                       self.weights.data_ptr(), _lib.stream_ptr())
             super().__init__(idx, E)
             return
@@ -282,15 +285,41 @@ class SigmoidRouting(Routing):
         self.tile_expert, self.meta, self.slot_pos, self.row_token = torch.split(
             ints, [self.max_tiles, 2, T * top_k, self.max_rows])
         self.offsets = self.meta         # only the weight-gradient product reads segment offsets
-        _lib.call("edl_moe_sigmoid_route_small", logits.data_ptr(), corr, T, E, top_k, self.weights.data_ptr(),
+        _lib.call("edl_moe_logit_route_small", logits.data_ptr(), corr, sig, T, E, top_k, self.weights.data_ptr(),
                   self.tile_expert.data_ptr(), self.max_tiles, self.meta.data_ptr(), self.slot_pos.data_ptr(),
                   self.row_token.data_ptr(), _lib.stream_ptr())
 
 
-def clamped_experts(x: torch.Tensor, r: SigmoidRouting, w_gate_up: torch.Tensor, w_down: torch.Tensor, limit: float,
+class SigmoidRouting(LogitRouting):
+    def __init__(self, logits: torch.Tensor, correction: torch.Tensor | None, top_k: int):
+        super().__init__(logits, top_k, True, correction)
+
+
+class SoftmaxRouting(LogitRouting):
+    def __init__(self, logits: torch.Tensor, top_k: int):
+        super().__init__(logits, top_k, False)
+
+
+def expert_unit(gu: torch.Tensor, r: Routing | None = None, limit: float | None = None, alpha: float = 1.702) -> torch.Tensor:
+    """Gated unit of rows ``[gate | up]``, of the rows in use when ``r`` has tables: ``silu(gate) * up``, or with a
+    ``limit`` the clamped unit."""
+    F = gu.shape[1] // 2
+    a = torch.empty(gu.shape[0], F, dtype=gu.dtype, device=gu.device)
+    _lib.call("edl_moe_glu", gu.data_ptr(), int(gu.dtype == torch.float32), r.row_token.data_ptr() if r else None,
+              r.meta.data_ptr() if r else None, a.data_ptr(), F, gu.shape[0], float(limit or 0.0), float(alpha),
+              _lib.stream_ptr())
+    return a
+
+
+def clamped_experts(x: torch.Tensor, r: LogitRouting, w_gate_up: torch.Tensor, w_down: torch.Tensor, limit: float,
                     alpha: float = 1.702) -> ExpertRows:
-    """Routed experts with the clamped gated unit, inference only: rows in use are computed, padding rows of the
-    segments stay undefined and are never read back."""
+    return stream_experts(x, r, w_gate_up, w_down, limit, alpha)
+
+
+def stream_experts(x: torch.Tensor, r: LogitRouting, w_gate_up: torch.Tensor, w_down: torch.Tensor,
+                   limit: float | None = None, alpha: float = 1.702, base: torch.Tensor | None = None) -> ExpertRows:
+    """Routed experts with the silu gated unit (with a ``limit``: the clamped one), inference only: rows in use are
+    computed, padding rows of the segments stay undefined and are never read back."""
     F2, H = w_gate_up.shape[1:]
     f32_ = int(x.dtype == torch.float32)
     tiles = not f32_ and F2 % 16 == 0 and H % 8 == 0 and x.stride(0) % 8 == 0
@@ -304,8 +333,5 @@ def clamped_experts(x: torch.Tensor, r: SigmoidRouting, w_gate_up: torch.Tensor,
                   w.shape[2], _lib.stream_ptr())
         return out
 
-    gu = product(x, w_gate_up, True)
-    a = torch.empty(r.max_rows, F2 // 2, dtype=x.dtype, device=x.device)
-    _lib.call("edl_moe_clamped_glu", gu.data_ptr(), f32_, r.row_token.data_ptr(), r.meta.data_ptr(), a.data_ptr(), F2 // 2,
-              r.max_rows, float(limit), float(alpha), _lib.stream_ptr())
-    return ExpertRows(product(a, w_down, False), r.weights, r.slot_pos)
+    a = expert_unit(product(x, w_gate_up, True), r, limit, alpha)
+    return ExpertRows(product(a, w_down, False), r.weights, r.slot_pos, base)

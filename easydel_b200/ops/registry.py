@@ -318,9 +318,10 @@ class AutoRegressiveDecodeAttn(OperationImpl):
         from . import serving as S
 
         c = self._opts(kw)
-        if S.decode_kernel_supports(query, k_pages, c["softcap"]):
+        if S.decode_kernel_supports(query, k_pages):
             o = S.decode_attention(query, k_pages, v_pages, kv_lens, page_table, scale=c["scale"],
-                                   window=int(c["sliding_window"] or 0), sinks=sinks, num_splits=num_splits)
+                                   window=int(c["sliding_window"] or 0), sinks=sinks, num_splits=num_splits,
+                                   softcap=c["softcap"])
         else:
             cu = torch.arange(query.shape[0] + 1, dtype=torch.int32, device=query.device)
             o = S.paged_attention(query, k_pages, v_pages, cu, kv_lens, page_table, 1, scale=c["scale"],

@@ -20,7 +20,7 @@ _lib.register("edl_count_update", i32, [vp, i64, vp, vp, i32, i32, vp])
 _lib.register("edl_gather_rows", i32, [vp, vp, vp, i32, i32, i64, vp])
 _lib.register("edl_attn_decode", i32, [vp, vp, vp, vp, vp, i64, i64, i64, i64, vp, vp, i32, i32, i64, i32, i32, i32, i32,
                                        f32,
-                                       i32, i32, vp, vp, vp])
+                                       i32, i32, f32, vp, vp, vp])
 
 _lib.register("edl_attn_mla_decode", i32, [vp, i64, i64, vp, i64, i64, vp, vp, vp, i64, vp, vp, i32, i32, i64, i32, i32, i32,
                                             f32, i32, vp, i32, vp, vp])
@@ -66,10 +66,10 @@ def paged_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tenso
     B = kv_lens.numel()
     scale = scale if scale is not None else 1.0 / math.sqrt(D)
     if q.is_cuda and not paged_kernel_supports(q, k_pages, v_pages):
-        if not causal or softcap:
-            raise NotImplementedError("the SIMT attention kernel is causal and has no soft-cap")
+        if not causal:
+            raise NotImplementedError("the SIMT attention kernel is causal")
         return simt_attention(q, k_pages, v_pages, cu_q, kv_lens, page_table, scale=scale, window=window, sinks=sinks,
-                              out=out)
+                              out=out, softcap=softcap)
     if q.is_cuda:
         assert k_pages.shape[1] == PAGE_SIZE, "the paged kernels use pages of 128 tokens"
         assert q.stride(-1) == 1 and q.stride(-2) == D
@@ -86,12 +86,12 @@ def paged_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tenso
 
 
 _lib.register("edl_attn_simt", i32, [vp, vp, vp, vp, i32, i64, i64, i64, vp, vp, vp, i32, i32, i32, i64, i32, i32, i32, i32,
-                                     f32, i32, vp, vp, vp])
+                                     f32, i32, f32, vp, vp, vp])
 
 
 def simt_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, cu_q: torch.Tensor,
                    kv_lens: torch.Tensor, page_table: torch.Tensor, *, scale: float, window: int = 0, sinks=None,
-                   out: torch.Tensor | None = None, v_dim: int | None = None) -> torch.Tensor:
+                   out: torch.Tensor | None = None, v_dim: int | None = None, softcap: float = 0.0) -> torch.Tensor:
     """Causal paged attention in fp32 arithmetic (``csrc/attention_simt.cu``): fp32 models, and head sizes outside the
     tensor-core kernels'. Arguments as :func:`paged_attention`; ``v_dim``: only the first elements of a value row count
     (latent rows, which are keys and values at once; one KV head)."""
@@ -107,18 +107,19 @@ def simt_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor
     _lib.call("edl_attn_simt", q.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), out.data_ptr(),
               int(q.dtype == torch.float32), q.stride(0), k_pages.stride(1), v_pages.stride(1), cu_q.data_ptr(),
               kv_lens.data_ptr(), page_table.data_ptr(), page_table.stride(0), kv_lens.numel(), T, k_pages.shape[0], Hq,
-              Hkv, D, Dv, float(scale), int(window or 0), _lib.ptr(sinks), _lib.status_word(q.device).data_ptr(),
-              _lib.stream_ptr())
+              Hkv, D, Dv, float(scale), int(window or 0), float(softcap or 0.0), _lib.ptr(sinks),
+              _lib.status_word(q.device).data_ptr(), _lib.stream_ptr())
     return out
 
 
 def decode_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, kv_lens: torch.Tensor,
                      page_table: torch.Tensor, *, scale: float | None = None, window: int = 0, sinks=None,
-                     num_splits: int = 1) -> torch.Tensor:
+                     num_splits: int = 1, softcap: float = 0.0) -> torch.Tensor:
     """Decode-step attention (one query token per sequence) with the streaming kernel of
     ``csrc/attention_decode.cu``. q ``[B, Hq, D]``; pages ``[P, 128, Hkv, D]`` (values may have another width than
     keys); ``num_splits`` cuts every
-    sequence's keys into that many parts that run as separate CTAs and are merged by :func:`attn_combine`."""
+    sequence's keys into that many parts that run as separate CTAs and are merged by :func:`attn_combine`; ``softcap``:
+    scores become ``softcap * tanh(score / softcap)``."""
     B, Hq, D = q.shape
     Hkv, Dv = k_pages.shape[2], v_pages.shape[-1]
     scale = scale if scale is not None else 1.0 / math.sqrt(D)
@@ -128,7 +129,7 @@ def decode_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tens
     _lib.call("edl_attn_decode", q.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), out.data_ptr(), _lib.ptr(lse),
               q.stride(0), k_pages.stride(1), v_pages.stride(1), Hq * Dv, kv_lens.data_ptr(), page_table.data_ptr(),
               page_table.stride(0), B, k_pages.shape[0], Hq, Hkv, D, Dv, float(scale), int(window or 0), S_,
-              _lib.ptr(sinks) if S_ == 1 else None, _lib.status_word(q.device).data_ptr(), _lib.stream_ptr())
+              float(softcap or 0.0), _lib.ptr(sinks) if S_ == 1 else None, _lib.status_word(q.device).data_ptr(), _lib.stream_ptr())
     if S_ == 1:
         return out[0]
     return attn_combine(out, lse, sinks=sinks)
@@ -181,11 +182,17 @@ def paged_kernel_supports(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch
             and _tile_width(q.shape[-1]) and _tile_width(v_pages.shape[-1]) and q.stride(0) % 8 == 0)
 
 
-def decode_kernel_supports(q: torch.Tensor, k_pages: torch.Tensor, softcap: float, v_dim: int | None = None) -> bool:
+def decode_splits(splits: int, window: int | None) -> int:
+    """Key splits of a layer's decode step: as many as planned for the whole context, but under a sliding window no more
+    than leave every split some tiles of 32 keys."""
+    return splits if not window else int(max(1, min(splits, (window + 31) // 32 // 4)))
+
+
+def decode_kernel_supports(q: torch.Tensor, k_pages: torch.Tensor, v_dim: int | None = None) -> bool:
     Hq, D = q.shape[-2], q.shape[-1]
     Hkv = k_pages.shape[2]
     return (q.is_cuda and q.dtype == torch.bfloat16 and _tile_width(D) and _tile_width(v_dim or D) and Hq % Hkv == 0
-            and Hq // Hkv <= 16 and not softcap and k_pages.shape[1] == PAGE_SIZE and q.stride(-1) == 1 and q.stride(-2) == D)
+            and Hq // Hkv <= 16 and k_pages.shape[1] == PAGE_SIZE and q.stride(-1) == 1 and q.stride(-2) == D)
 
 
 def attn_combine(o_parts: torch.Tensor, lse_parts: torch.Tensor, sinks=None, want_lse: bool = False):

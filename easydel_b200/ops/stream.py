@@ -11,18 +11,21 @@ from __future__ import annotations
 import torch
 import torch.nn.functional as tF
 
-from . import _lib, kernels as K
+from . import _lib, kernels as K, reference as R, rotation
 
 vp, i32, i64, f32 = _lib.vp, _lib.i32, _lib.i64, _lib.f32
-_lib.register("edl_embed_stream", i32, [vp, i32, vp, vp, vp, i64, i32, i32, i32, vp, vp])
+_lib.register("edl_embed_stream", i32, [vp, i32, vp, f32, vp, vp, i64, i32, i32, i32, vp, vp])
 _lib.register("edl_cast_rows", i32, [vp, vp, i32, i64, i32, i32, vp])
 _lib.register("edl_norm_shift", i32, [vp, vp, vp, f32, i32, i32, vp, i32, vp, vp, i64, f32, vp, i32, vp])
 _lib.register("edl_head_norm", i32, [vp, vp, f32, i64, i32, vp, i32, vp])
 _lib.register("edl_xielu", i32, [vp, vp, vp, i32, i64, vp])
 _lib.register("edl_gelu_erf", i32, [vp, vp, i32, i64, vp])
-_lib.register("edl_post_norm", i32, [vp, vp, vp, vp, vp, i32, f32, vp, f32, f32, vp, i32, i32, i32, vp])
+_lib.register("edl_post_norm", i32, [vp, vp, vp, vp, vp, i32, f32, f32, i32, vp, f32, f32, vp, i32, i32, i32, vp])
+_lib.register("edl_scale_cap", i32, [vp, i64, f32, f32, vp])
 _lib.register("edl_qkv_prologue", i32, [vp, i32, i64, vp, vp, vp, vp, f32, f32, f32, i32, i32, i32, i32, i32, vp, vp, vp,
                                         i64, i64, i64, vp, vp])
+_lib.register("edl_qkv_rotary_prologue", i32, [vp, i32, i64, vp, vp, vp, vp, f32, vp, i32, i32, i32, i32, i32, i32, vp, vp, vp,
+                                               i64, i64, i64, vp, vp])
 
 
 def on_kernels(t: torch.Tensor) -> bool:
@@ -81,6 +84,15 @@ def linear_add_(stream: torch.Tensor, x: torch.Tensor, w: torch.Tensor) -> torch
     return stream + tF.linear(x, w).float()
 
 
+def branch_product(x: torch.Tensor, w: torch.Tensor, base: torch.Tensor | None = None,
+                   bias: torch.Tensor | None = None) -> torch.Tensor:
+    """``x @ w.T (+ bias)`` as fp32 rows, added to the fp32 rows ``base`` (in place on the kernels) if there are any."""
+    if base is None:
+        return linear(x, w, bias, torch.float32)
+    out = linear_add_(base, x, w)
+    return out if bias is None else out + bias.float()
+
+
 def bmm(a: torch.Tensor, b: torch.Tensor) -> torch.Tensor:
     """Batched product in the operand type, true 32-bit for fp32 (vendor library)."""
     allow = torch.backends.cuda.matmul.allow_tf32
@@ -92,22 +104,22 @@ def bmm(a: torch.Tensor, b: torch.Tensor) -> torch.Tensor:
 
 
 # ---------------------------------------------------------------------------------------------- rows of the stream
-def embed(table: torch.Tensor, ids: torch.Tensor, right: torch.Tensor | None = None) -> torch.Tensor:
-    """fp32 rows ``table[ids]`` ``[T, W]``; ``right`` (a view ``[T, W]`` of the right half of a ``[x ; x0]`` operand)
-    receives the same rows in the table's type."""
+def embed(table: torch.Tensor, ids: torch.Tensor, right: torch.Tensor | None = None, scale: float = 1.0) -> torch.Tensor:
+    """fp32 rows ``table[ids] * scale`` ``[T, W]``; ``right`` (a view ``[T, W]`` of the right half of a ``[x ; x0]``
+    operand) receives the same rows in the table's type."""
     ids = ids.reshape(-1)
     W = table.shape[1]
     if on_kernels(table):
         ids = ids.to(torch.int64).contiguous()
         x = torch.empty(ids.numel(), W, dtype=torch.float32, device=table.device)
-        _lib.call("edl_embed_stream", table.data_ptr(), _f32flag(table.dtype), ids.data_ptr(), x.data_ptr(),
+        _lib.call("edl_embed_stream", table.data_ptr(), _f32flag(table.dtype), ids.data_ptr(), float(scale), x.data_ptr(),
                   _lib.ptr(right), right.stride(0) if right is not None else 0, ids.numel(), W, table.shape[0],
                   _lib.status_word(table.device).data_ptr(), _lib.stream_ptr())
         return x
-    rows = table[ids.long()]
+    rows = table[ids.long()].float() * scale
     if right is not None:
         right.copy_(rows)
-    return rows.float()
+    return rows
 
 
 def cast_rows(x: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
@@ -192,27 +204,68 @@ def gelu_erf(z: torch.Tensor) -> torch.Tensor:
     return tF.gelu(z)
 
 
+def gated_unit(gu: torch.Tensor, act: str = "silu") -> torch.Tensor:
+    """``act(gate) * up`` for rows ``gu [T, 2 F] = [gate | up]``."""
+    if on_kernels(gu):
+        F = gu.shape[1] // 2
+        if gu.dtype == torch.bfloat16 and F % 8 == 0 and gu.stride(0) % 8 == 0 and act in K.ACT_IDS:
+            return K.gated_act_fwd(gu, act)
+        if act == "silu":
+            from .moe_kernels import expert_unit
+
+            return expert_unit(gu if gu.is_contiguous() else gu.contiguous())
+    return R.gated_act(gu, act)
+
+
+def scale_cap(z: torch.Tensor, scale: float = 1.0, cap: float = 0.0) -> torch.Tensor:
+    """``cap tanh(scale z / cap)`` for fp32 ``z`` (``scale z`` without a cap), in place on the kernels."""
+    if on_kernels(z):
+        assert z.dtype == torch.float32 and z.is_contiguous()
+        _lib.call("edl_scale_cap", z.data_ptr(), z.numel(), float(scale), float(cap), _lib.stream_ptr())
+        return z
+    z = z * scale
+    return torch.tanh(z / cap) * cap if cap else z
+
+
 # ---------------------------------------------------------------------------------------------- norm after the sum
-def post_norm(x: torch.Tensor, branch, alpha: float, w: torch.Tensor, eps: float, out_dtype: torch.dtype,
-              offset: float = 0.0) -> tuple[torch.Tensor, torch.Tensor]:
-    """``rms_norm(alpha x + branch) * (w + offset)`` over the fp32 stream ``x [T, W]`` in 32 bits: the new stream (in place
-    on the kernels) and the same rows as the operand of the next product. ``branch``: fp32 rows ``[T, W]``, or an
-    :class:`..ops.moe_kernels.ExpertRows`, whose weighted sum over each token's experts happens in the same pass."""
+def _sum_and_norm(x, branch, alpha, beta, keep_sum, w, eps, out_dtype, offset):
     rows = None if isinstance(branch, torch.Tensor) else branch
     if on_kernels(x):
         h = torch.empty(x.shape, dtype=out_dtype, device=x.device)
-        y = branch if rows is None else None
+        y = branch if rows is None else rows.base
         if y is not None and (y.dtype != torch.float32 or not y.is_contiguous()):
             y = y.float().contiguous()
         assert x.is_contiguous() and (rows is None or rows.ys.dtype == out_dtype)
         _lib.call("edl_post_norm", x.data_ptr(), _lib.ptr(y), _lib.ptr(rows.ys) if rows else None,
                   _lib.ptr(rows.weights) if rows else None, _lib.ptr(rows.pos) if rows else None, rows.k if rows else 0,
-                  float(alpha), w.data_ptr(), float(offset), float(eps), h.data_ptr(), _f32flag(out_dtype), x.shape[0],
-                  x.shape[1], _lib.stream_ptr())
+                  float(alpha), float(beta), int(keep_sum), w.data_ptr(), float(offset), float(eps), h.data_ptr(),
+                  _f32flag(out_dtype), x.shape[0], x.shape[1], _lib.stream_ptr())
         return x, h
-    v = x * alpha + (branch.float() if rows is None else rows.combine())
-    v = v * torch.rsqrt(v.pow(2).mean(-1, keepdim=True) + eps) * (w.float() + offset)
-    return v, v.to(out_dtype)
+    s = x * alpha + branch_rows(branch) * beta
+    v = s * torch.rsqrt(s.pow(2).mean(-1, keepdim=True) + eps) * (w.float() + offset)
+    return s if keep_sum else v, v.to(out_dtype)
+
+
+def branch_rows(branch) -> torch.Tensor:
+    """A branch (fp32 rows or expert rows) as fp32 rows."""
+    return branch.float() if isinstance(branch, torch.Tensor) else branch.combine()
+
+
+def post_norm(x: torch.Tensor, branch, alpha: float, w: torch.Tensor, eps: float, out_dtype: torch.dtype,
+              offset: float = 0.0) -> tuple[torch.Tensor, torch.Tensor]:
+    """``rms_norm(alpha x + branch) * (w + offset)`` over the fp32 stream ``x [T, W]`` in 32 bits: the new stream (in place
+    on the kernels) and the same rows as the operand of the next product. ``branch``: fp32 rows ``[T, W]``, or an
+    :class:`..ops.moe_kernels.ExpertRows`, whose weighted sum over each token's experts happens in the same pass."""
+    return _sum_and_norm(x, branch, alpha, 1.0, False, w, eps, out_dtype, offset)
+
+
+def add_norm(x: torch.Tensor, branch, mult: float, w: torch.Tensor, eps: float, out_dtype: torch.dtype,
+             offset: float = 0.0) -> tuple[torch.Tensor, torch.Tensor]:
+    """``x + mult branch`` (in place on the kernels; ``branch`` as in :func:`post_norm`, or None) and the RMS norm of the
+    sum, ``* (w + offset)``, as the operand of the next products."""
+    if branch is None:
+        return x, norm_shift(x, w, eps, out_dtype, offset=offset)
+    return _sum_and_norm(x, branch, 1.0, mult, True, w, eps, out_dtype, offset)
 
 
 # ---------------------------------------------------------------------------------------------- attention prologue
@@ -257,3 +310,40 @@ def qkv_prologue(qkv: torch.Tensor, heads: tuple[int, int, int, int], qw, kw, ep
     q, k = qk_norm_temper(q.reshape(T, Hq, D), k.reshape(T, Hkv, D), qw, kw, eps, positions, temp)
     S.kv_append(k, v.reshape(T, Hkv, Dv), k_pages, v_pages, slot_mapping)
     return q
+
+
+def qkv_rotary_prologue(qkv: torch.Tensor, heads: tuple[int, int, int, int], qw, kw, eps: float, positions: torch.Tensor,
+                        freq: torch.Tensor | None, slot_mapping: torch.Tensor, k_pages: torch.Tensor,
+                        v_pages: torch.Tensor) -> torch.Tensor:
+    """:func:`qkv_prologue` for queries and keys that are normed over the whole projection (all heads at once; weights
+    ``qw [Hq D]``, ``kw [Hkv D]``, None: no norm) and then rotated: elements ``i`` and ``i + pairs`` of every head by the
+    position times frequency i (``freq``: see :mod:`.rotation`; None: no rotation)."""
+    Hq, Hkv, D, Dv = heads
+    T = qkv.shape[0]
+    if on_kernels(qkv):
+        q = torch.empty(T, Hq, D, dtype=qkv.dtype, device=qkv.device)
+        pos = positions.reshape(-1).to(torch.int32)
+        _lib.call("edl_qkv_rotary_prologue", qkv.data_ptr(), _f32flag(qkv.dtype), qkv.stride(0), pos.data_ptr(),
+                  slot_mapping.data_ptr(), _lib.ptr(qw), _lib.ptr(kw), float(eps), _lib.ptr(freq),
+                  freq.numel() // 2 if freq is not None else 0, T, Hq, Hkv, D, Dv, q.data_ptr(), k_pages.data_ptr(),
+                  v_pages.data_ptr(), k_pages.stride(1), v_pages.stride(1), k_pages.shape[0] * k_pages.shape[1],
+                  _lib.status_word(qkv.device).data_ptr(), _lib.stream_ptr())
+        return q
+    from . import serving as S
+
+    q, k, v = torch.split(qkv, [Hq * D, Hkv * D, Hkv * Dv], -1)
+    q, k = qk_norm_rotate(q, k, D, qw, kw, eps, positions, freq)
+    S.kv_append(k, v.reshape(T, Hkv, Dv), k_pages, v_pages, slot_mapping)
+    return q
+
+
+def qk_norm_rotate(q, k, D: int, qw, kw, eps: float, positions, freq):
+    """Tensor form of the q / k half of :func:`qkv_rotary_prologue`: flat rows -> ``[T, H, D]`` and ``[T, G, D]``."""
+    def one(x, w):
+        xf = x.float()
+        if w is not None:
+            xf = xf * torch.rsqrt(xf.pow(2).mean(-1, keepdim=True) + eps) * w.float()
+        xf = xf.reshape(x.shape[0], -1, D)
+        return (xf if freq is None else rotation.rotate(xf, positions.reshape(-1), freq, "halves")).to(x.dtype)
+
+    return one(q, qw), one(k, kw)

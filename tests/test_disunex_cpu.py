@@ -5,7 +5,7 @@ import oracle_disunex as O
 import pytest
 import torch
 
-from easydel_b200.ops import latent, stream
+from easydel_b200.ops import latent, rotation, stream
 
 TOL = 2e-5
 
@@ -27,14 +27,14 @@ def test_rotation_of_neighbouring_pairs():
     x = _r(7, 3, 10)
     pos = torch.tensor([0, 1, 2, 50, 999, 70001, 5])
     for dims in (10, 4):
-        got = latent.rotate_pairs(x, pos, latent.pair_frequencies(300.0, dims))
+        got = rotation.rotate(x, pos, rotation.pair_frequencies(300.0, dims))
         assert torch.allclose(got, O.rotate_pairs(x, pos, 300.0, dims), atol=1e-6)
         assert torch.equal(got[..., dims:], x[..., dims:]) and torch.equal(got[0], x[0])
     # scores depend on the distance only
     q, k = _r(1, 1, 8).expand(6, 1, 8), _r(1, 1, 8, seed=1).expand(6, 1, 8)
-    f = latent.pair_frequencies(50.0, 8)
+    f = rotation.pair_frequencies(50.0, 8)
     p = torch.arange(6) * 3
-    a, b = latent.rotate_pairs(q, p + 4, f), latent.rotate_pairs(k, p, f)
+    a, b = rotation.rotate(q, p + 4, f), rotation.rotate(k, p, f)
     assert torch.allclose((a * b).sum(-1), (a * b).sum(-1)[:1].expand(6, 1), atol=1e-5)
 
 

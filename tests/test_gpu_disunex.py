@@ -85,7 +85,7 @@ def test_gelu_and_head_gate(dtype):
 @pytest.mark.parametrize("dtype", DT)
 def test_prologue(heads, dims, dtype):
     """Rotated queries in place, cache rows on their pages; at positions far beyond any table too."""
-    from easydel_b200.ops import latent
+    from easydel_b200.ops import latent, rotation
 
     H, D, R, L = heads
     T, ld = 21, H * (D + R) + L + R + 5
@@ -93,7 +93,7 @@ def test_prologue(heads, dims, dtype):
     before = proj.clone()
     w = 1 + 0.2 * _r(L, seed=1)
     pos = torch.tensor([*range(11), *range(1000, 1005), 30001, 99999, 100000, 100001, 250000], dtype=torch.int32)
-    freq = latent.pair_frequencies(700.0, dims, "cuda")
+    freq = rotation.pair_frequencies(700.0, dims, "cuda")
     pages = torch.zeros(3, 128, 1, L + R, dtype=dtype, device="cuda")
     slots = torch.randperm(384, generator=torch.Generator().manual_seed(2))[:T].to(torch.int32).cuda()
     slots[3] = -1

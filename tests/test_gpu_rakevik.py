@@ -214,7 +214,7 @@ def test_decode_attention_with_its_own_value_size(layout, splits):
     kv = [1, 127, 128, 129, 640]
     ks, vs, kp, vp, table = _paged(kv, Hkv, D, Dv, torch.bfloat16, 1)
     q, sink = _r(5, Hq, D, dtype=torch.bfloat16), _r(Hq, seed=6) + 1
-    assert S.decode_kernel_supports(q, kp, 0.0, Dv)
+    assert S.decode_kernel_supports(q, kp, Dv)
     got = S.decode_attention(q, kp, vp, _i32(*kv), table, scale=0.3, sinks=sink, num_splits=splits)
     want = torch.cat([_expect(q[b:b + 1].cpu(), ks[b], vs[b], 0.3, sink.cpu()) for b in range(5)])
     _close(got.cpu(), want, torch.bfloat16, 2)
