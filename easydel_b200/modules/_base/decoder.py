@@ -622,7 +622,7 @@ class DecoderModel(EasyDeLBaseModule):
         if x.dtype != self.dtype and x.is_floating_point():
             x = x.to(self.dtype)
         if spec.embed_scale is not None:
-            x = x * torch.tensor(spec.embed_scale, dtype=x.dtype, device=x.device)
+            x = x * float(torch.tensor(spec.embed_scale, dtype=x.dtype))      # the factor in the embedding's own type
         if spec.embedding_multiplier is not None:
             x = x * spec.embedding_multiplier
         if position_ids is None:
