@@ -142,7 +142,7 @@ def bench_prefill(t: Table, T: int, size) -> None:
     for win in (window, 0):
         s = min(T, win or T)
         fl = 4 * H * (s * (s + 1) / 2 + (T - s) * s) * 128
-        for what, size_ in (("scores below 3/4 of the cap", 1.0), ("scores up to the cap", 6.0)):
+        for what, size_ in (("scores far below the cap", 1.0), ("scores up to the cap", 6.0)):
             q = _rand(T, H, 128, scale=size_)
 
             def case(cap):

@@ -346,6 +346,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
     const float cap2 = p.softcap * LOG2E;   // soft-cap in log2 units
     const float cap_k2 = CAP ? 2.f * p.scale_log2 / p.softcap : 0.f;
     const float cap_k = cap_k2 * (0.5f * LN2);      // scale / cap
+    const SoftCapNear near_cap(cap_k, cap2);
     const float mul = CAP ? 1.f : p.scale_log2;
     bool alive = true;
     int n = 0;
@@ -394,6 +395,9 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
       const bool tile_mask = (kv0 + BKV > len_k) || (p.causal && kv0 + BKV - 1 > q0 + off) ||
                              (p.window > 0 && kv0 < q0 + TQ - 1 + off - p.window + 1);
       tc_wait_ld();
+      // Scores far below the cap in tiles without a mask stay raw: the cap is monotone, so the maximum is taken first, and
+      // the polynomial goes into the exponents below. Elsewhere scores are capped here. Warp-uniform.
+      bool raw = false;
       if constexpr (CAP) {
         float m0 = 0.f, m1 = 0.f;
 #pragma unroll
@@ -401,7 +405,10 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
           m0 = fmax3(m0, fabsf(__uint_as_float(a[i])), fabsf(__uint_as_float(a[i + 1])));
           m1 = fmax3(m1, fabsf(__uint_as_float(a[i + 2])), fabsf(__uint_as_float(a[i + 3])));
         }
-        if (__all_sync(0xffffffffu, fmaxf(m0, m1) * cap_k <= SOFT_CAP_POLY_MAX)) {   // well below the cap: no MUFU
+        const float y = fmaxf(m0, m1) * cap_k;
+        raw = __all_sync(0xffffffffu, y <= SOFT_CAP_NEAR_MAX) && !tile_mask;
+        if (raw) {
+        } else if (__all_sync(0xffffffffu, y <= SOFT_CAP_POLY_MAX)) {   // no MUFU
 #pragma unroll
           for (int i = 0; i < 64; i += 2) {
             float s0 = __uint_as_float(a[i]), s1 = __uint_as_float(a[i + 1]);
@@ -433,6 +440,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
         }
         mx = fmax3(m0, m1, fmaxf(__uint_as_float(a[62]), __uint_as_float(a[63])));
       }
+      if (CAP && raw) mx = near_cap.at(mx);
       float mx_other;
       TRACE(t, n, 2);
       if (!exchange(mx, mx_other, false)) {
@@ -466,18 +474,24 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
       // Four scores per step: packed FMAs form x = s * mul - m, three exponentials go to the MUFU and one to the
       // polynomial on the FMA pipe, the row sum is accumulated with packed adds.
       uint32_t pk[32];
+      auto exponentials = [&](auto argument) {
 #pragma unroll
-      for (int i = 0; i < 64; i += 4) {
-        float x0, x1, x2, x3;
-        fma2(x0, x1, __uint_as_float(a[i]), __uint_as_float(a[i + 1]), mul, mul, neg_m, neg_m);
-        fma2(x2, x3, __uint_as_float(a[i + 2]), __uint_as_float(a[i + 3]), mul, mul, neg_m, neg_m);
-        const float e0 = exp2f(x0), e1 = exp2f(x1), e2 = exp2f(x2);
-        const float e3 = exp2_poly(x3);
-        add2(l0, l1, e0, e1);
-        add2(l2, l3, e2, e3);
-        pk[i >> 1] = pack_bf16x2(e0, e1);
-        pk[(i >> 1) + 1] = pack_bf16x2(e2, e3);
-      }
+        for (int i = 0; i < 64; i += 4) {
+          float x0, x1, x2, x3;
+          argument(x0, x1, __uint_as_float(a[i]), __uint_as_float(a[i + 1]));
+          argument(x2, x3, __uint_as_float(a[i + 2]), __uint_as_float(a[i + 3]));
+          const float e0 = exp2f(x0), e1 = exp2f(x1), e2 = exp2f(x2);
+          const float e3 = exp2_poly(x3);
+          add2(l0, l1, e0, e1);
+          add2(l2, l3, e2, e3);
+          pk[i >> 1] = pack_bf16x2(e0, e1);
+          pk[(i >> 1) + 1] = pack_bf16x2(e2, e3);
+        }
+      };
+      if (CAP && raw)
+        exponentials([&](float& x0, float& x1, float s0, float s1) { near_cap.add2(x0, x1, s0, s1, neg_m); });
+      else
+        exponentials([&](float& x0, float& x1, float s0, float s1) { fma2(x0, x1, s0, s1, mul, mul, neg_m, neg_m); });
       tmem_st_32x32b_x32(tS + half * 32, pk);
       l0 += l2;
       l1 += l3;

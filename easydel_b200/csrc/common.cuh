@@ -375,6 +375,34 @@ __device__ __forceinline__ void soft_cap_poly2(float& s0, float& s1, float k, fl
   mul2(s0, s1, y0, y1, p0, p1);
 }
 
+// The same for |y| <= SOFT_CAP_NEAR_MAX as s * (c0 + c1 s^2 + c2 s^4 + c3 s^6), with scale and cap folded into c (relative
+// error 1.6e-7 of the polynomial, fitted likewise).
+constexpr float SOFT_CAP_NEAR_MAX = 0.4f;
+struct SoftCapNear {
+  float c0, c1, c2, c3;
+  __device__ __forceinline__ SoftCapNear(float k, float cap2) {
+    const float k2 = k * k;
+    c0 = cap2 * k;
+    c1 = c0 * k2 * -0.3333137333393097f;
+    c2 = c0 * k2 * k2 * 0.13271155953407288f;
+    c3 = c0 * k2 * k2 * k2 * -0.047561075538396835f;
+    c0 *= 0.9999998807907104f;
+  }
+  __device__ __forceinline__ float at(float s) const {
+    const float u = s * s;
+    return s * fmaf(fmaf(fmaf(c3, u, c2), u, c1), u, c0);
+  }
+  // (x0, x1) = at(s0, s1) + (add, add)
+  __device__ __forceinline__ void add2(float& x0, float& x1, float s0, float s1, float add) const {
+    float u0, u1, p0, p1;
+    mul2(u0, u1, s0, s1, s0, s1);
+    fma2(p0, p1, u0, u1, c3, c3, c2, c2);
+    fma2(p0, p1, p0, p1, u0, u1, c1, c1);
+    fma2(p0, p1, p0, p1, u0, u1, c0, c0);
+    fma2(x0, x1, s0, s1, p0, p1, add, add);
+  }
+};
+
 // Epilogue helper: a warp holds a 32-row block one row per lane, each row 128 bytes as eight 16-byte chunks
 // (64 bf16 or 32 fp32 values). Writing it straight out would make every store instruction touch 32 different rows
 // with 16 bytes each; instead the block goes through a swizzled 4 KB shared-memory stage and leaves as four whole

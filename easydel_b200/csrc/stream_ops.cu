@@ -17,6 +17,8 @@
 // Compiled without fast-math: these are the parts of such a model that are computed in 32 bits.
 #include "common.cuh"
 
+#include <type_traits>
+
 namespace edl {
 namespace {
 
@@ -662,6 +664,138 @@ qkv_rotary_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, T* __restric
     }
 }
 
+// The same for rows whose units (a piece of VEC elements and its partner) fit KEEP to a thread: a CTA walks the tokens
+// blockIdx.x, blockIdx.x + gridDim.x, ...; norm weights stay in registers, each row is read once, the next one while the
+// current one is normed, and cosines and partial sums have two buffers, so that a token costs one barrier.
+constexpr int RW_THREADS = 512;
+
+template <typename T, int VEC, int KEEP>
+__global__ void __launch_bounds__(RW_THREADS)
+qkv_rotary_walk_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, T* __restrict__ k_pages, T* __restrict__ v_pages,
+                       const RotaryPrologueParams p, int rows) {
+  using Raw = typename std::conditional<sizeof(T) * VEC == 16, uint4, uint2>::type;
+  __shared__ float2 cs[2][RP_MAX_PAIRS];
+  __shared__ float2 red[2][RW_THREADS / 32];
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, warps = (blockDim.x + 31) >> 5;
+  const int nq = p.Hq * p.D, nk = p.Hkv * p.D, nv = p.Hkv * p.Dv;
+  const int turned = p.pairs / VEC, per = turned + (p.D - 2 * p.pairs) / VEC, units = (p.Hq + p.Hkv) * per;
+  int col[KEEP];             // first element within the row (< 0: no unit); partner `pairs` further
+  bool pair[KEEP];
+  float wa[KEEP][VEC], wb[KEEP][VEC];
+#pragma unroll
+  for (int i = 0; i < KEEP; ++i) {
+    const int u = tid + i * blockDim.x;
+    const int h = u / per, r = u - h * per;
+    pair[i] = r < turned;
+    col[i] = u < units ? h * p.D + (pair[i] ? r * VEC : 2 * p.pairs + (r - turned) * VEC) : -1;
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) wa[i][j] = wb[i][j] = 1.f;
+    if (col[i] >= 0) {
+      const bool is_q = col[i] < nq;
+      const float* w = is_q ? p.qw : p.kw;
+      if (w) {
+        const int c = is_q ? col[i] : col[i] - nq;
+        ldw<VEC>(w + c, wa[i]);
+        if (pair[i]) ldw<VEC>(w + c + p.pairs, wb[i]);
+      }
+    }
+  }
+  Raw a[KEEP], b[KEEP];
+  auto load = [&](int t) {
+    const T* row = qkv + t * p.ld;
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i)
+      if (col[i] >= 0) {
+        a[i] = *reinterpret_cast<const Raw*>(row + col[i]);
+        if (pair[i]) b[i] = *reinterpret_cast<const Raw*>(row + col[i] + p.pairs);
+      }
+  };
+  int t = blockIdx.x, buf = 0;
+  if (t < rows) load(t);
+  for (; t < rows; t += gridDim.x, buf ^= 1) {
+    long long slot = p.slots[t];
+    if (slot >= p.num_slots) {
+      if (p.status && tid == 0) atomicCAS(p.status, 0, EDL_BAD_INDEX);
+      slot = -1;
+    }
+    if (slot >= 0)
+      for (int c = tid * VEC; c < nv; c += blockDim.x * VEC)
+        *reinterpret_cast<Raw*>(v_pages + slot * p.ld_vpage + c) =
+            *reinterpret_cast<const Raw*>(qkv + t * p.ld + nq + nk + c);
+    const float fp = p.pairs ? (float)p.pos[t] : 0.f;
+    for (int i = tid; i < p.pairs; i += blockDim.x) {
+      const float f = p.freq[i], x = fp * f;
+      const float e = fmaf(fp, f, -x) + fp * p.freq[p.pairs + i];
+      float s, c;
+      sincosf(x, &s, &c);
+      const float ce = 1.f - 0.5f * e * e, se = e - e * e * e * (1.f / 6.f);
+      cs[buf][i] = make_float2(c * ce - s * se, s * ce + c * se);
+    }
+    float va[KEEP][VEC], vb[KEEP][VEC], sq = 0.f, sk = 0.f;
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i) {
+      if (col[i] < 0) continue;
+      ldv<VEC>(reinterpret_cast<const T*>(&a[i]), va[i]);
+      float s = 0.f;
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) s += va[i][j] * va[i][j];
+      if (pair[i]) {
+        ldv<VEC>(reinterpret_cast<const T*>(&b[i]), vb[i]);
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) s += vb[i][j] * vb[i][j];
+      }
+      if (col[i] < nq) sq += s; else sk += s;
+    }
+    if (t + (int)gridDim.x < rows) load(t + gridDim.x);
+    sq = warp_sum(sq);
+    sk = warp_sum(sk);
+    if (lane == 0) red[buf][warp] = make_float2(sq, sk);
+    __syncthreads();
+    float2 sums = lane < warps ? red[buf][lane] : make_float2(0.f, 0.f);
+    sums.x = warp_sum(sums.x);
+    sums.y = warp_sum(sums.y);
+    const float rq = p.qw ? 1.f / sqrtf(sums.x / (float)nq + p.eps) : 1.f;
+    const float rk = p.kw ? 1.f / sqrtf(sums.y / (float)nk + p.eps) : 1.f;
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i) {
+      if (col[i] < 0) continue;
+      const bool is_q = col[i] < nq;
+      if (!is_q && slot < 0) continue;
+      const float r = is_q ? rq : rk;
+      T* dst = is_q ? q_out + (long long)t * nq + col[i] : k_pages + slot * p.ld_kpage + (col[i] - nq);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) va[i][j] *= r * wa[i][j];
+      if (pair[i]) {
+        const int c0 = col[i] % p.D;
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) {
+          const float2 g = cs[buf][c0 + j];
+          const float x = va[i][j], y = vb[i][j] * (r * wb[i][j]);
+          va[i][j] = x * g.x - y * g.y;
+          vb[i][j] = y * g.x + x * g.y;
+        }
+        stv<VEC>(dst + p.pairs, vb[i]);
+      }
+      stv<VEC>(dst, va[i]);
+    }
+  }
+}
+
+template <typename T, int VEC>
+bool launch_rotary_walk(const void* qkv, void* q_out, void* k_pages, void* v_pages, const RotaryPrologueParams& p, int rows,
+                        cudaStream_t s) {
+  const int units = (p.Hq + p.Hkv) * (p.pairs / VEC + (p.D - 2 * p.pairs) / VEC);
+  const int keep = units <= RW_THREADS ? 1 : 2;
+  if (units > 2 * RW_THREADS) return false;
+  const int threads = ((units + keep - 1) / keep + 31) / 32 * 32;
+  const int grid = min(rows, sm_count() * max(1, 1024 / threads));
+#define EDL_RW(K) \
+  qkv_rotary_walk_kernel<T, VEC, K><<<grid, threads, 0, s>>>((const T*)qkv, (T*)q_out, (T*)k_pages, (T*)v_pages, p, rows)
+  if (keep == 1) EDL_RW(1); else EDL_RW(2);
+#undef EDL_RW
+  return true;
+}
+
 // ---- logits ------------------------------------------------------------------------------------------------------------------
 template <int VEC>
 __global__ void __launch_bounds__(NT) scale_cap_kernel(float* __restrict__ z, long long n_vec, float scale, float cap) {
@@ -862,6 +996,9 @@ EDL_HOST_API int edl_qkv_rotary_prologue(const void* qkv, int f32, long long ld,
     return D % m == 0 && pairs % m == 0 && Dv % m == 0 && ld % m == 0 && ld_kpage % m == 0 && ld_vpage % m == 0 &&
            al(qkv, a) && al(q_out, a) && al(k_pages, a) && al(v_pages, a) && (!qw || al(qw, 16)) && (!kw || al(kw, 16));
   };
+  const bool walked = f32 ? fits(4, 16) && launch_rotary_walk<float, 4>(qkv, q_out, k_pages, v_pages, p, T, s)
+                          : fits(8, 16) && launch_rotary_walk<__nv_bfloat16, 8>(qkv, q_out, k_pages, v_pages, p, T, s);
+  if (walked) return check_cuda(cudaGetLastError(), "qkv_rotary_prologue launch");
 #define EDL_RP(TT, V_) \
   qkv_rotary_kernel<TT, V_><<<T, NT, 0, s>>>((const TT*)qkv, (TT*)q_out, (TT*)k_pages, (TT*)v_pages, p)
   if (f32) {

@@ -89,7 +89,8 @@ POSITIONS = torch.tensor([*range(11), *range(1000, 1005), 30001, 99999, 100000, 
 
 
 @pytest.mark.parametrize("heads,dims", [((4, 2, 48, 24), 32), ((3, 1, 20, 12), 6), ((16, 2, 128, 64), 128), ((2, 2, 7, 3), 2),
-                                        ((12, 4, 64, 128), 0), ((2, 1, 24, 8), 8)])
+                                        ((12, 4, 64, 128), 0), ((2, 1, 24, 8), 8), ((32, 8, 128, 64), 32),
+                                        ((64, 8, 128, 128), 16), ((96, 8, 128, 16), 0)])
 @pytest.mark.parametrize("dtype", DT)
 def test_attention_prologue(heads, dims, dtype):
     """Full-width norms, rotated halves, keys and values on their pages; at positions far beyond any table too."""
@@ -118,6 +119,16 @@ def test_attention_prologue(heads, dims, dtype):
     _close(kp.view(384, G, D).cpu()[at], want_k[ok], dtype)
     assert torch.equal(vp.view(384, -1).cpu()[at], qkv.cpu()[ok][:, (H + G) * D:])
     assert int((kp.view(384, -1).abs().sum(1) > 0).sum()) == T - 1
+    # many tokens (a block walks several), the same rows over and over
+    n = 90
+    kp2, vp2 = (torch.zeros(T * n // 128 + 1, *p.shape[1:], dtype=dtype, device="cuda") for p in (kp, vp))
+    many = stream.qkv_rotary_prologue(qkv.repeat(n, 1), heads, qw, kw, 1e-4, POSITIONS.cuda().repeat(n), freq,
+                                      torch.arange(T * n, dtype=torch.int32, device="cuda"), kp2, vp2)
+    many, k = many.view(n, T, H, D), kp2.view(-1, G, D)[:T * n].view(n, T, G, D)
+    assert torch.equal(many, many[:1].expand_as(many)) and torch.equal(k, k[:1].expand_as(k))
+    _close(many[0], q, dtype)          # rows of another pitch may take another form of the kernel
+    _close(k[0].cpu()[ok], want_k[ok], dtype)
+    assert torch.equal(vp2.view(-1, G * V)[T * (n - 1):T * n], qkv[:, (H + G) * D:])
     # without norms, without rotation
     q = stream.qkv_rotary_prologue(qkv, heads, None, None, 1e-4, POSITIONS.cuda(), None, slots, kp, vp)
     assert torch.equal(q.view(T, -1), qkv[:, :H * D])
@@ -273,7 +284,7 @@ def test_windowed_attention_portions_beside_single_tokens(shape, window, cap, dt
     _close(got, want, dtype, 2.5)
 
 
-@pytest.mark.parametrize("size,cap", [(1.0, 10.0), (6.0, 10.0), (30.0, 200.0), (90.0, 200.0)])
+@pytest.mark.parametrize("size,cap", [(1.0, 10.0), (6.0, 10.0), (8.0, 60.0), (14.0, 60.0), (30.0, 200.0), (90.0, 200.0)])
 @pytest.mark.parametrize("new", [1, 200])
 def test_cap_of_16_bit_heads_is_computed_in_32_bits(size, cap, new):
     """Scores from well below the cap to far above it; under the large cap a score's last 16-bit digit would be a tenth."""
