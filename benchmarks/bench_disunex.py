@@ -170,7 +170,7 @@ def bench_prefill(t: Table, T: int, size) -> None:
         out = torch.empty(T, H, v, dtype=BF, device="cuda")
         return (lambda: _lib.call("edl_attn_paged", q.data_ptr(), k.data_ptr(), vv.data_ptr(), out.data_ptr(), q.stride(0),
                                   k.stride(1), vv.stride(1), H * v, cu.data_ptr(), lens.data_ptr(), table.data_ptr(),
-                                  table.stride(0), 1, T, T, k.shape[0], H, H, d, v, float(d ** -0.5), 1, win, 0.0,
+                                  table.stride(0), 1, T, T, k.shape[0], H, H, d, v, float(d ** -0.5), 1, win, 0, 0.0,
                                   _lib.ptr(sink), _lib.status_word(q.device).data_ptr(), _lib.stream_ptr()), nb,
                 2 * pairs * (d + v))
 

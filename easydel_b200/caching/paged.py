@@ -256,24 +256,28 @@ class PagedLayerView:
             return self._attend_gathered(attn, q3, meta)[None]
         return self.attend_pages(attn, q3, meta)[None]
 
-    def attend_pages(self, attn, q3, meta: PagedBatchMeta):
-        """Attention of ``q3 [T, Hq, D]`` over the pages, which already hold this step's keys and values."""
+    def attend_pages(self, attn, q3, meta: PagedBatchMeta, sigmoid: "S.SigmoidWeights | None" = None,
+                     out: torch.Tensor | None = None):
+        """Attention of ``q3 [T, Hq, D]`` over the pages, which already hold this step's keys and values. ``sigmoid``: weights
+        without a softmax; ``out [T, Hq, Dv]``: where to write."""
         table = meta.table_of(self.group)
+        keep = getattr(attn, "keep_first", 0)
         if meta.max_q == 1 and q3.shape[0] == meta.num_seqs and S.decode_kernel_supports(
                 q3, self.k_pages, self.v_pages.shape[-1]):
             # a pure decode step: the streaming kernel (one CTA per sequence, KV head and key split)
             o = S.decode_attention(q3, self.k_pages, self.v_pages, meta.kv_lens, table, scale=attn.scale,
                                    window=attn.sliding_window or 0, sinks=attn.sinks, softcap=attn.softcap,
-                                   num_splits=S.decode_splits(meta.num_splits, attn.sliding_window))
+                                   num_splits=S.decode_splits(meta.num_splits, attn.sliding_window, keep), keep_first=keep,
+                                   sigmoid=sigmoid, out=out)
             return o
-        if meta.num_splits > 1 and meta.max_q == 1 and not attn.sliding_window and q3.is_cuda and \
+        if meta.num_splits > 1 and sigmoid is None and out is None and meta.max_q == 1 and not attn.sliding_window and q3.is_cuda and \
                 q3.dtype == torch.bfloat16 and self.v_pages.shape[-1] == q3.shape[-1] and q3.shape[-1] in (64, 128):
             o = S.paged_attention_splitkv(q3, self.k_pages, self.v_pages, meta.kv_lens, table,
                                           meta.num_splits, scale=attn.scale, softcap=attn.softcap, sinks=attn.sinks)
             return o
         return S.paged_attention(q3, self.k_pages, self.v_pages, meta.cu_q, meta.kv_lens, table, meta.max_q,
-                              scale=attn.scale, causal=True, window=attn.sliding_window or 0, softcap=attn.softcap,
-                                 sinks=attn.sinks)
+                                 scale=attn.scale, causal=True, window=attn.sliding_window or 0, softcap=attn.softcap,
+                                 sinks=attn.sinks, keep_first=keep, sigmoid=sigmoid, out=out)
 
 
 class PagedBatchCache(PagedKVCache):

@@ -48,7 +48,13 @@ class KVCacheSpec:
         return context
 
     def first_useful_token(self, num_computed_tokens: int) -> int:
-        """Keys before this position are never read again once ``num_computed_tokens`` tokens are in the cache."""
+        """Keys before this position (but :attr:`first_kept` ones) are never read again once ``num_computed_tokens`` tokens
+        are in the cache."""
+        return 0
+
+    @property
+    def first_kept(self) -> int:
+        """Keys from the start of a sequence that stay readable whatever :meth:`first_useful_token` says."""
         return 0
 
     def pages_per_sequence(self, max_model_len: int, max_step_tokens: int = 1) -> int:
@@ -72,9 +78,14 @@ class FullAttentionSpec(KVCacheSpec):
 class SlidingWindowSpec(KVCacheSpec):
     sliding_window: int = 4096
     kind: str = "sliding"
+    keep_first: int = 0          # the first tokens of a sequence stay visible when the window has moved past them
+
+    @property
+    def first_kept(self) -> int:
+        return self.keep_first
 
     def tokens_kept(self, context: int) -> int:
-        return min(context, self.sliding_window)
+        return min(context, self.sliding_window + self.keep_first)
 
     def first_useful_token(self, num_computed_tokens: int) -> int:
         # the next query sits at position num_computed_tokens and sees keys > position - window
@@ -82,10 +93,12 @@ class SlidingWindowSpec(KVCacheSpec):
 
     def pages_per_sequence(self, max_model_len: int, max_step_tokens: int = 1) -> int:
         span = min(max_model_len, self.sliding_window - 1 + max_step_tokens)
-        return min(cdiv(max_model_len, self.page_size), cdiv(span, self.page_size) + 1)
+        pages = cdiv(span, self.page_size) + 1 + cdiv(self.keep_first, self.page_size)
+        return min(cdiv(max_model_len, self.page_size), pages)
 
     def group_key(self) -> tuple:
-        return (self.kind, self.sliding_window, self.num_kv_heads, self.head_dim, self.value_dim, self.element_size)
+        return (self.kind, self.sliding_window, self.num_kv_heads, self.head_dim, self.value_dim, self.element_size,
+                self.keep_first)
 
 
 @dataclass(frozen=True)
@@ -175,7 +188,7 @@ def layer_spec(info, element_size: int = 2, tp_size: int = 1, page_size: int = P
             return SlidingLatentSpec(sliding_window=int(info.sliding_window), **common)
         return MLAAttentionSpec(**common)
     if info.sliding_window:
-        return SlidingWindowSpec(sliding_window=int(info.sliding_window), **common)
+        return SlidingWindowSpec(sliding_window=int(info.sliding_window), keep_first=int(info.keep_first), **common)
     if info.chunk_size:
         return ChunkedLocalAttentionSpec(attention_chunk_size=int(info.chunk_size), **common)
     return FullAttentionSpec(**common)

@@ -49,6 +49,12 @@ struct DecodeParams {
   float scale_log2;
   float cap_k2, cap2;       // soft-cap (see soft_cap), cap2 = 0: none
   int* status;
+  int keep_first;           // with a window: keys before this position stay visible
+  const float* score_bias;  // [Hq]: no softmax, weights are sigmoid(score + bias) (SIG)
+  const __nv_bfloat16* gate;   // [B, ld_gate] or null: output rows times sigmoid(gate[b][head]) (SIG)
+  long long ld_gate;
+  float out_scale;          // SIG
+  float* parts;             // SIG with splits > 1: fp32 [splits, B, Hq, dv], the parts of a plain sum
 };
 
 __device__ __forceinline__ void ldmatrix_x4(uint32_t addr, uint32_t (&r)[4]) {
@@ -88,7 +94,7 @@ struct DCfg {
   static constexpr int SMEM = OFF_RED + DEC_WARPS * 2 * 16 * 4 + 1024;
 };
 
-template <int DQ, int DV>
+template <int DQ, int DV, bool SIG>
 __global__ void __launch_bounds__(DEC_THREADS)
 attn_decode_kernel(const __grid_constant__ CUtensorMap tk, const __grid_constant__ CUtensorMap tv,
                    const DecodeParams p) {
@@ -112,12 +118,15 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tk, const __grid_constant
   int lo = 0;
   if (p.window > 0) lo = max(0, kv_len - p.window);
   const int t_first = lo / TK, t_end = (kv_len + TK - 1) / TK;
-  const int n_all = max(0, t_end - t_first);
+  // kept tiles in front of the window come first: place v of the list is tile tile_at(v)
+  const int front = p.window > 0 ? min((p.keep_first + TK - 1) / TK, t_first) : 0;
+  auto tile_at = [&](int v) { return v < front ? v : t_first + v - front; };
+  const int n_all = max(0, front + t_end - t_first);
   const int per_split = (n_all + p.splits - 1) / p.splits;
-  const int t0 = t_first + split * per_split;
-  const int t1 = min(t_end, t0 + per_split);
+  const int t0 = split * per_split;
+  const int t1 = min(n_all, t0 + per_split);
   const int n_tiles = max(0, t1 - t0);
-  // tiles of this warp: t0 + warp, t0 + warp + 4, ...
+  // places of this warp: t0 + warp, t0 + warp + 4, ...
   const int my_n = n_tiles > warp ? (n_tiles - warp + DEC_WARPS - 1) / DEC_WARPS : 0;
 
   uint64_t* bars = reinterpret_cast<uint64_t*>(smem + C::OFF_BAR);
@@ -145,7 +154,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tk, const __grid_constant
   volatile int* abort_flag = &s_abort;
 
   auto issue = [&](int i) {   // lane 0 only: tile i of this warp into stage i % DEC_STAGES
-    const int tile = t0 + warp + i * DEC_WARPS;
+    const int tile = tile_at(t0 + warp + i * DEC_WARPS);
     const int page = pt[tile / (PAGE / TK)];
     const int row = page * PAGE + (tile % (PAGE / TK)) * TK;
     const int st = i % DEC_STAGES;
@@ -182,6 +191,12 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tk, const __grid_constant
   float m_run[2] = {-1e30f, -1e30f};   // rows lane/4 and lane/4 + 8
   float l_run[2] = {0.f, 0.f};
   bool alive = true;
+  float bias2[2] = {0.f, 0.f};         // score bias of rows lane/4 and lane/4 + 8, in log2 units
+  if constexpr (SIG) {
+#pragma unroll
+    for (int h = 0; h < 2; ++h)
+      if ((lane >> 2) + h * 8 < G) bias2[h] = p.score_bias[hk * G + (lane >> 2) + h * 8] * LOG2E_F;
+  }
 
   for (int i = 0; i < my_n && alive; ++i) {
     const int st = i % DEC_STAGES;
@@ -192,7 +207,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tk, const __grid_constant
     }
     const uint32_t kt = my_ring + st * C::STAGE_BYTES;
     const uint32_t vt = kt + C::K_BYTES;
-    const int tile = t0 + warp + i * DEC_WARPS;
+    const int tile = tile_at(t0 + warp + i * DEC_WARPS);
     const int key0 = tile * TK;
 
     // ---- S = Q K^T for 32 keys: four 8-key blocks
@@ -213,52 +228,67 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tk, const __grid_constant
     }
     // ---- mask the ragged end / the window start, online softmax (log2 domain)
     const int cbase = key0 + (lane & 3) * 2;
-    float mx[2] = {-INFINITY, -INFINITY};
-#pragma unroll
-    for (int j = 0; j < TK / 8; ++j) {
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int key = cbase + j * 8 + (e & 1);
-        const bool ok = key < kv_len && key >= lo;
-        const float z = p.cap2 > 0.f ? soft_cap(s[j][e], p.cap_k2, p.cap2) : s[j][e] * p.scale_log2;
-        s[j][e] = ok ? z : -INFINITY;
-        mx[e >> 1] = fmaxf(mx[e >> 1], s[j][e]);
-      }
-    }
-#pragma unroll
-    for (int h = 0; h < 2; ++h) {
-      mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 1));
-      mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 2));
-    }
-    float alpha[2];
-#pragma unroll
-    for (int h = 0; h < 2; ++h) {
-      const float m_new = fmaxf(m_run[h], mx[h]);
-      alpha[h] = exp2f(m_run[h] - m_new);
-      m_run[h] = m_new;
-      l_run[h] *= alpha[h];
-    }
     uint32_t pa[TK / 16][4];
-    float rs[2] = {0.f, 0.f};
+    if constexpr (SIG) {
 #pragma unroll
-    for (int j = 0; j < TK / 8; ++j) {
-      const float e0 = exp2f(s[j][0] - m_run[0]), e1 = exp2f(s[j][1] - m_run[0]);
-      const float e2 = exp2f(s[j][2] - m_run[1]), e3 = exp2f(s[j][3] - m_run[1]);
-      rs[0] += e0 + e1;
-      rs[1] += e2 + e3;
-      // S accumulator layout = A operand layout of the next product: blocks 2t, 2t+1 form k-step t
-      pa[j >> 1][(j & 1) * 2] = pack_bf16x2(e0, e1);
-      pa[j >> 1][(j & 1) * 2 + 1] = pack_bf16x2(e2, e3);
-    }
-    l_run[0] += rs[0];
-    l_run[1] += rs[1];
-    // ---- O = O * alpha + P V
+      for (int j = 0; j < TK / 8; ++j) {
 #pragma unroll
-    for (int j = 0; j < NDB; ++j) {
-      o_acc[j][0] *= alpha[0];
-      o_acc[j][1] *= alpha[0];
-      o_acc[j][2] *= alpha[1];
-      o_acc[j][3] *= alpha[1];
+        for (int e = 0; e < 4; ++e) {
+          const int key = cbase + j * 8 + (e & 1);
+          const bool ok = key < kv_len && (key >= lo || key < p.keep_first);
+          const float y = fminf(-fmaf(s[j][e], p.scale_log2, bias2[e >> 1]), 120.f);
+          s[j][e] = ok ? __fdividef(1.f, 1.f + exp2f(y)) : 0.f;
+        }
+        pa[j >> 1][(j & 1) * 2] = pack_bf16x2(s[j][0], s[j][1]);
+        pa[j >> 1][(j & 1) * 2 + 1] = pack_bf16x2(s[j][2], s[j][3]);
+      }
+    } else {
+      float mx[2] = {-INFINITY, -INFINITY};
+#pragma unroll
+      for (int j = 0; j < TK / 8; ++j) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int key = cbase + j * 8 + (e & 1);
+          const bool ok = key < kv_len && (key >= lo || key < p.keep_first);
+          const float z = p.cap2 > 0.f ? soft_cap(s[j][e], p.cap_k2, p.cap2) : s[j][e] * p.scale_log2;
+          s[j][e] = ok ? z : -INFINITY;
+          mx[e >> 1] = fmaxf(mx[e >> 1], s[j][e]);
+        }
+      }
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 1));
+        mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 2));
+      }
+      float alpha[2];
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        const float m_new = fmaxf(m_run[h], mx[h]);
+        alpha[h] = exp2f(m_run[h] - m_new);
+        m_run[h] = m_new;
+        l_run[h] *= alpha[h];
+      }
+      float rs[2] = {0.f, 0.f};
+#pragma unroll
+      for (int j = 0; j < TK / 8; ++j) {
+        const float e0 = exp2f(s[j][0] - m_run[0]), e1 = exp2f(s[j][1] - m_run[0]);
+        const float e2 = exp2f(s[j][2] - m_run[1]), e3 = exp2f(s[j][3] - m_run[1]);
+        rs[0] += e0 + e1;
+        rs[1] += e2 + e3;
+        // S accumulator layout = A operand layout of the next product: blocks 2t, 2t+1 form k-step t
+        pa[j >> 1][(j & 1) * 2] = pack_bf16x2(e0, e1);
+        pa[j >> 1][(j & 1) * 2 + 1] = pack_bf16x2(e2, e3);
+      }
+      l_run[0] += rs[0];
+      l_run[1] += rs[1];
+      // ---- O = O * alpha + P V
+#pragma unroll
+      for (int j = 0; j < NDB; ++j) {
+        o_acc[j][0] *= alpha[0];
+        o_acc[j][1] *= alpha[0];
+        o_acc[j][2] *= alpha[1];
+        o_acc[j][3] *= alpha[1];
+      }
     }
 #pragma unroll
     for (int t = 0; t < TK / 16; ++t) {
@@ -302,7 +332,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tk, const __grid_constant
     for (int w = 0; w < DEC_WARPS; ++w) l += red[w * 32 + 16 + r] * exp2f(red[w * 32 + r] - m);
     m_all[h] = m;
     l_all[h] = l;
-    w_mine[h] = exp2f(m_run[h] - m);
+    w_mine[h] = SIG ? 1.f : exp2f(m_run[h] - m);
   }
   // each warp scales its O by its weight and adds it into a shared fp32 [16 x DV] accumulator, one warp after another
   float* o_sh = reinterpret_cast<float*>(smem);   // 16 * DV * 4 bytes <= one warp's ring
@@ -334,6 +364,27 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tk, const __grid_constant
     for (int w = 0; w < DEC_WARPS; ++w) m = fmaxf(m, red[w * 32 + r]);
     for (int w = 0; w < DEC_WARPS; ++w) l += red[w * 32 + 16 + r] * exp2f(red[w * 32 + r] - m);
     const int head = hk * G + r;
+    if constexpr (SIG) {
+      float f = p.out_scale;
+      if (p.gate) {
+        const float g = __bfloat162float(p.gate[(long long)b * p.ld_gate + head]);
+        f = __fdividef(f, 1.f + exp2f(fminf(-g * LOG2E_F, 120.f)));
+      }
+      const float* src = o_sh + r * DV + c * 8;
+      if (p.splits > 1) {
+        float4* dst = reinterpret_cast<float4*>(p.parts + (orow * p.Hq + head) * p.dv + c * 8);
+        dst[0] = make_float4(src[0] * f, src[1] * f, src[2] * f, src[3] * f);
+        dst[1] = make_float4(src[4] * f, src[5] * f, src[6] * f, src[7] * f);
+      } else {
+        uint4 v;
+        v.x = pack_bf16x2(src[0] * f, src[1] * f);
+        v.y = pack_bf16x2(src[2] * f, src[3] * f);
+        v.z = pack_bf16x2(src[4] * f, src[5] * f);
+        v.w = pack_bf16x2(src[6] * f, src[7] * f);
+        *reinterpret_cast<uint4*>(p.o + orow * p.ldo + (long long)head * p.dv + c * 8) = v;
+      }
+      continue;
+    }
     if (p.sinks && p.splits == 1) l += exp2f(p.sinks[head] * LOG2E_F - m);
     const float inv = l > 0.f ? 1.f / l : 0.f;
     const float* src = o_sh + r * DV + c * 8;
@@ -355,7 +406,25 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tk, const __grid_constant
   }
 }
 
-template <int DQ, int DV>
+// out [B, width] (pitch ldo) = sum of the fp32 parts [splits, B, width]; width is a multiple of 8.
+__global__ void sum_parts_kernel(const float* __restrict__ parts, int splits, int B, int width, __nv_bfloat16* __restrict__ out,
+                                 long long ldo) {
+  const long long total = (long long)B * (width / 4);
+  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
+    const int b = (int)(i / (width / 4)), c = (int)(i - (long long)b * (width / 4)) * 4;
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int s = 0; s < splits; ++s) {
+      const float4 v = *reinterpret_cast<const float4*>(parts + ((long long)s * B + b) * width + c);
+      a.x += v.x;
+      a.y += v.y;
+      a.z += v.z;
+      a.w += v.w;
+    }
+    *reinterpret_cast<uint2*>(out + b * ldo + c) = make_uint2(pack_bf16x2(a.x, a.y), pack_bf16x2(a.z, a.w));
+  }
+}
+
+template <int DQ, int DV, bool SIG>
 int launch_decode(const void* k_pages, const void* v_pages, long long ld_kpage, long long ld_vpage,
                   long long num_pages, const DecodeParams& p, cudaStream_t stream) {
   using C = DCfg<DQ, DV>;
@@ -363,7 +432,7 @@ int launch_decode(const void* k_pages, const void* v_pages, long long ld_kpage, 
   const long long total_k = num_pages * PAGE;
   if (make_tmap_3d_16b(&tk, k_pages, p.dq, p.Hkv, total_k, p.dq, ld_kpage, 64, 1, TK, 3)) return -1;
   if (make_tmap_3d_16b(&tv, v_pages, p.dv, p.Hkv, total_k, p.dv, ld_vpage, 64, 1, TK, 3)) return -1;
-  auto kern = attn_decode_kernel<DQ, DV>;
+  auto kern = attn_decode_kernel<DQ, DV, SIG>;
   static bool attr_set[64] = {false};
   int dev = 0;
   cudaGetDevice(&dev);
@@ -376,7 +445,22 @@ int launch_decode(const void* k_pages, const void* v_pages, long long ld_kpage, 
   }
   const long long blocks = (long long)p.B * p.Hkv * p.splits;
   kern<<<(unsigned)blocks, DEC_THREADS, C::SMEM, stream>>>(tk, tv, p);
+  if (SIG && p.splits > 1) {
+    const int width = p.Hq * p.dv;
+    const long long n = (long long)p.B * (width / 4);
+    sum_parts_kernel<<<(int)((n + 255) / 256), 256, 0, stream>>>(p.parts, p.splits, p.B, width, p.o, p.ldo);
+  }
   return check_cuda(cudaGetLastError(), "attn_decode launch");
+}
+
+template <bool SIG>
+int dispatch_decode(const void* k_pages, const void* v_pages, long long ld_kpage, long long ld_vpage, long long num_pages,
+                    const DecodeParams& p, cudaStream_t s) {
+  if (p.dq > 64)
+    return p.dv > 64 ? launch_decode<128, 128, SIG>(k_pages, v_pages, ld_kpage, ld_vpage, num_pages, p, s)
+                     : launch_decode<128, 64, SIG>(k_pages, v_pages, ld_kpage, ld_vpage, num_pages, p, s);
+  return p.dv > 64 ? launch_decode<64, 128, SIG>(k_pages, v_pages, ld_kpage, ld_vpage, num_pages, p, s)
+                   : launch_decode<64, 64, SIG>(k_pages, v_pages, ld_kpage, ld_vpage, num_pages, p, s);
 }
 
 }  // namespace
@@ -386,13 +470,14 @@ int launch_decode(const void* k_pages, const void* v_pages, long long ld_kpage, 
 // pages [num_pages * 128, ld_kpage / ld_vpage] with the KV heads packed in a row, page_table [B, pt_stride], kv_lens [B]
 // (keys per sequence, the new token included). o [splits, B, ldo]; with splits > 1 part s holds the result over
 // the s-th part of every sequence's keys and lse [splits, Hq, B] its log-sum-exp, for edl_attn_combine.
-// Hq / Hkv <= 16; D (queries, keys) and Dv (values) are multiples of 8 up to 128; window = 0 or the sliding-window length;
-// softcap > 0: scores become softcap * tanh(scale * dot / softcap).
-EDL_HOST_API int edl_attn_decode(const void* q, const void* k_pages, const void* v_pages, void* o, float* lse,
-                                 long long ldq, long long ld_kpage, long long ld_vpage, long long ldo, const int* kv_lens,
-                                 const int* page_table, int pt_stride, int B, long long num_pages, int Hq, int Hkv,
-                                 int D, int Dv, float scale, int window, int splits, float softcap,
-                                 const float* sinks, int* status, void* stream) {
+// Hq / Hkv <= 16; D (queries, keys) and Dv (values) are multiples of 8 up to 128; window = 0 or the sliding-window length,
+// under which the first keep_first keys stay visible; softcap > 0: scores become softcap * tanh(scale * dot / softcap).
+static int decode_impl(const void* q, const void* k_pages, const void* v_pages, void* o, float* lse,
+                       long long ldq, long long ld_kpage, long long ld_vpage, long long ldo, const int* kv_lens,
+                       const int* page_table, int pt_stride, int B, long long num_pages, int Hq, int Hkv,
+                       int D, int Dv, float scale, int window, int keep_first, int splits, float softcap,
+                       const float* sinks, const float* score_bias, const void* gate, long long ld_gate, float out_scale,
+                       float* parts, int* status, void* stream) {
   using namespace edl;
   if (B <= 0) return 0;
   if (D < 8 || D > 128 || (D & 7) || Dv < 8 || Dv > 128 || (Dv & 7) || Hkv < 1 || Hq % Hkv || Hq / Hkv > 16 ||
@@ -427,9 +512,40 @@ EDL_HOST_API int edl_attn_decode(const void* q, const void* k_pages, const void*
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   p.dq = D;
   p.dv = Dv;
-  if (D > 64)
-    return Dv > 64 ? launch_decode<128, 128>(k_pages, v_pages, ld_kpage, ld_vpage, num_pages, p, s)
-                   : launch_decode<128, 64>(k_pages, v_pages, ld_kpage, ld_vpage, num_pages, p, s);
-  return Dv > 64 ? launch_decode<64, 128>(k_pages, v_pages, ld_kpage, ld_vpage, num_pages, p, s)
-                 : launch_decode<64, 64>(k_pages, v_pages, ld_kpage, ld_vpage, num_pages, p, s);
+  p.keep_first = keep_first;
+  p.score_bias = score_bias;
+  p.gate = reinterpret_cast<const __nv_bfloat16*>(gate);
+  p.ld_gate = ld_gate;
+  p.out_scale = out_scale;
+  p.parts = parts;
+  return score_bias ? dispatch_decode<true>(k_pages, v_pages, ld_kpage, ld_vpage, num_pages, p, s)
+                    : dispatch_decode<false>(k_pages, v_pages, ld_kpage, ld_vpage, num_pages, p, s);
+}
+
+EDL_HOST_API int edl_attn_decode(const void* q, const void* k_pages, const void* v_pages, void* o, float* lse,
+                                 long long ldq, long long ld_kpage, long long ld_vpage, long long ldo, const int* kv_lens,
+                                 const int* page_table, int pt_stride, int B, long long num_pages, int Hq, int Hkv,
+                                 int D, int Dv, float scale, int window, int keep_first, int splits, float softcap,
+                                 const float* sinks, int* status, void* stream) {
+  return decode_impl(q, k_pages, v_pages, o, lse, ldq, ld_kpage, ld_vpage, ldo, kv_lens, page_table, pt_stride, B, num_pages,
+                     Hq, Hkv, D, Dv, scale, window, keep_first, splits, softcap, sinks, nullptr, nullptr, 0, 1.f, nullptr,
+                     status, stream);
+}
+
+// The same without a softmax: a visible key's weight is sigmoid(score + score_bias[head]); the output o [B, ldo] is multiplied by
+// out_scale and, with a gate [B, ld_gate] (bf16), by sigmoid(gate[b][head]). parts: workspace fp32 [splits, B, Hq * Dv] when
+// splits > 1 (the parts of a plain sum need no log-sum-exp).
+EDL_HOST_API int edl_attn_decode_sigmoid(const void* q, const void* k_pages, const void* v_pages, void* o, float* parts,
+                                         long long ldq, long long ld_kpage, long long ld_vpage, long long ldo,
+                                         const int* kv_lens, const int* page_table, int pt_stride, int B,
+                                         long long num_pages, int Hq, int Hkv, int D, int Dv, float scale, int window,
+                                         int keep_first, int splits, const float* score_bias, const void* gate,
+                                         long long ld_gate, float out_scale, int* status, void* stream) {
+  if (!score_bias || (splits > 1 && !parts)) {
+    edl::set_last_error("edl_attn_decode_sigmoid: needs a bias per head, and a workspace for key splits");
+    return -1;
+  }
+  return decode_impl(q, k_pages, v_pages, o, nullptr, ldq, ld_kpage, ld_vpage, ldo, kv_lens, page_table, pt_stride, B,
+                     num_pages, Hq, Hkv, D, Dv, scale, window, keep_first, splits, 0.f, nullptr, score_bias, gate, ld_gate,
+                     out_scale, parts, status, stream);
 }

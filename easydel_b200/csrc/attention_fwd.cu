@@ -21,6 +21,9 @@
 //               maxima through shared memory, exponentiate in registers and write P back as packed
 //               bf16 over the same tensor-memory columns (the A operand of the PV product). O is
 //               rescaled in tensor memory only when the running maximum moved by more than 2^8.
+// Weights without a softmax (ATT_SIGMOID: the sigmoid of score + a number per head, not normalised over keys) need neither
+// maxima nor sums: the halves of a row never meet, and the output leaves times a gate per row.
+// A window may keep the first tokens of a sequence: their key tiles come before the window's.
 // Tensor memory map (512 columns): S_A/P_A [0,128)  S_B/P_B [128,256)  O_A [256,384)  O_B [384,512).
 //
 // Tiles 192 columns wide (expanded latent attention) leave shared memory for one stage of 128-wide values, and none for the
@@ -38,6 +41,8 @@
 #include "tmem_ops.cuh"
 
 #include <stdlib.h>
+
+#include <type_traits>
 
 namespace edl {
 namespace {
@@ -79,6 +84,11 @@ struct AttnFwdParams {
   int pt_stride;
   int pack;              // query heads per tile row group (1 = one head per CTA)
   int dq, dv;            // real query / key and value sizes of a head (<= the tile widths)
+  int keep_first;        // with a window: keys before this position stay visible
+  const float* score_bias;      // [Hq], ATT_SIGMOID
+  const __nv_bfloat16* gate;    // [total_q, ld_gate] or null: output rows times sigmoid(gate[token][head])
+  long long ld_gate;
+  float out_scale;       // ATT_SIGMOID: factor of the output
   int nx, ny;            // launch geometry: query blocks and heads (the grid itself is one-dimensional)
 };
 
@@ -91,6 +101,9 @@ struct ACfg {
   static constexpr int V_BYTES = BKV * DV * 2;
   static constexpr bool WIDE = DQ > 128;
   static constexpr int VS = WIDE && DV > 64 ? 1 : 2;      // value stages
+  // Without the exchange of maxima nothing tells one half of a row that the other has read its scores, so each half's P
+  // stays over its own scores (columns of a score tile where the right half's P starts).
+  static constexpr int P_RIGHT_SIG = 64;
   static constexpr int OFF_K = 2 * Q_BYTES;
   static constexpr int OFF_V = OFF_K + 2 * K_BYTES;
   static constexpr int OFF_BAR = OFF_V + VS * V_BYTES;
@@ -118,12 +131,15 @@ __device__ __forceinline__ TileRange tile_range(int q0, int tq, int len_q, int l
   return r;
 }
 
-// CAP: soft-capped scores (a form of its own: the other one must not carry its registers).
-template <int DQ, int DV, bool CAP>
+// What becomes of the scores; forms of their own, so that none carries another's registers.
+enum { ATT_SOFTMAX = 0, ATT_CAPPED = 1, ATT_SIGMOID = 2 };
+
+template <int DQ, int DV, int MODE>
 __global__ void __launch_bounds__(ATT_THREADS, 1)
 attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CUtensorMap tk,
                 const __grid_constant__ CUtensorMap tv, const AttnFwdParams p) {
   using C = ACfg<DQ, DV>;
+  constexpr bool CAP = MODE == ATT_CAPPED, SIG = MODE == ATT_SIGMOID;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   const uint32_t sQ = smem_u32(smem);
@@ -178,6 +194,12 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
     jmin = rgB.lo;
     jmax = rgB.hi;
   }
+  // Steps of the key loop: the kept tiles in front of the windows first (every query of this block sees them), then
+  // [jmin, jmax). Step i works on tile tile_at(i); a tile between the windows' starts may be one of the kept ones.
+  const int kept_tiles = p.window > 0 ? (p.keep_first + BKV - 1) / BKV : 0;
+  const int front = min(kept_tiles, jmin);
+  const int steps = jmax > jmin ? front + jmax - jmin : 0;
+  auto tile_at = [&](int i) { return i < front ? i : jmin + i - front; };
 
   if (threadIdx.x == 0) {
     mbar_init(b_qfull, 1);
@@ -215,8 +237,8 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
         for (int c = 0; c < C::QCH; ++c)
           tma_load_3d(sQ + t * C::Q_BYTES + c * (BQ * 128), &tq, b_qfull, c * 64, h_first, q_start + qblock0 + t * TQ);
       auto row_of = [&](int j) { return pt ? pt[j] * BKV : k_start + j * BKV; };
-      auto load_k = [&](int j) -> bool {
-        const int it = j - jmin, s = it & 1, row = row_of(j);
+      auto load_k = [&](int it) -> bool {
+        const int s = it & 1, row = row_of(tile_at(it));
         if (it >= 2 &&
             !mbar_wait(b_kempty + 8 * s, ((it >> 1) - 1) & 1, abort_flag, p.status, EDL_TIMEOUT_PRODUCER))
           return false;
@@ -226,8 +248,8 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
           tma_load_3d(sK0 + s * C::K_BYTES + c * (BKV * 128), &tk, b_kfull + 8 * s, c * 64, hk, row);
         return true;
       };
-      auto load_v = [&](int j) -> bool {
-        const int it = j - jmin, s = it % C::VS, row = row_of(j);
+      auto load_v = [&](int it) -> bool {
+        const int s = it % C::VS, row = row_of(tile_at(it));
         if (it >= C::VS &&
             !mbar_wait(b_vempty + 8 * s, (it / C::VS - 1) & 1, abort_flag, p.status, EDL_TIMEOUT_PRODUCER))
           return false;
@@ -238,11 +260,11 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
         return true;
       };
       if constexpr (C::VS == 2) {
-        for (int j = jmin; j < jmax; ++j)
-          if (!load_k(j) || !load_v(j)) break;
+        for (int i = 0; i < steps; ++i)
+          if (!load_k(i) || !load_v(i)) break;
       } else {   // the only value stage is free late: keys stay one tile ahead of it
-        bool ok = load_k(jmin);
-        for (int j = jmin; j < jmax && ok; ++j) ok = (j + 1 >= jmax || load_k(j + 1)) && load_v(j);
+        bool ok = load_k(0);
+        for (int i = 0; i < steps && ok; ++i) ok = (i + 1 >= steps || load_k(i + 1)) && load_v(i);
       }
     }
   } else if (warp == 1) {
@@ -256,9 +278,13 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
       constexpr uint32_t idesc_pv = umma_idesc_bf16(BQ, DV, 0, 1);
       bool ok = mbar_wait(b_qfull, 0, abort_flag, p.status, EDL_TIMEOUT_MMA);
       int pv_cnt[2] = {0, 0};
-      auto valid = [&](int t, int j) { return t == 0 ? (j >= rgA.lo && j < rgA.hi) : (j >= rgB.lo && j < rgB.hi); };
-      auto issue_qk = [&](int t, int j) {
-        const int s = (j - jmin) & 1;
+      auto valid = [&](int t, int i) {
+        const int j = tile_at(i);
+        return t == 0 ? anyA && (j >= rgA.lo || j < kept_tiles) && j < rgA.hi
+                      : anyB && (j >= rgB.lo || j < kept_tiles) && j < rgB.hi;
+      };
+      auto issue_qk = [&](int t, int i) {
+        const int s = i & 1;
         const uint32_t kb = sK0 + s * C::K_BYTES;
         const uint32_t qbase = sQ + t * C::Q_BYTES;
 #pragma unroll
@@ -271,16 +297,17 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
           }
         if (leader) tc_commit(b_sfull + 8 * t);
       };
-      auto issue_pv = [&](int t, int j) -> bool {
-        const int s = (j - jmin) % C::VS;
+      auto issue_pv = [&](int t, int i) -> bool {
+        const int j = tile_at(i), s = i % C::VS;
         if (!mbar_wait(b_pfull + 8 * t, pv_cnt[t] & 1, abort_flag, p.status, EDL_TIMEOUT_MMA)) return false;
         tc_fence_after();
         const uint32_t vb = sV0 + s * C::V_BYTES;
 #pragma unroll
         for (int k = 0; k < BKV / 16; ++k) {
+          const int pc = SIG && k >= 4 ? C::P_RIGHT_SIG + (k - 4) * 8 : k * 8;
           uint64_t bd = umma_smem_desc_sw128(vb + k * 2048, BKV * 128, 1024);
           if (leader)
-            umma_f16_ts(tmem_base + 256 + t * 128, tmem_base + t * 128 + k * 8, bd, idesc_pv,
+            umma_f16_ts(tmem_base + 256 + t * 128, tmem_base + t * 128 + pc, bd, idesc_pv,
                         (pv_cnt[t] | k) != 0 ? 1u : 0u);
         }
         ++pv_cnt[t];
@@ -293,17 +320,16 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
         if (ok) {
           tc_fence_after();
           TRACE(3, 0, 0);
-          if (valid(0, jmin)) issue_qk(0, jmin);
+          if (valid(0, 0)) issue_qk(0, 0);
           TRACE(3, 0, 1);
-          if (valid(1, jmin)) issue_qk(1, jmin);
+          if (valid(1, 0)) issue_qk(1, 0);
           TRACE(3, 0, 2);
           if (leader) tc_commit(b_kempty);
         }
       }
-      for (int j = jmin; j < jmax && ok; ++j) {
-        const int it = j - jmin;
+      for (int it = 0; it < steps && ok; ++it) {
         const int s = it & 1;
-        const bool more = j + 1 < jmax;
+        const bool more = it + 1 < steps;
         TRACE(2, it, 0);
         const int vs = it % C::VS;
         if (!mbar_wait(b_vfull + 8 * vs, (it / C::VS) & 1, abort_flag, p.status, EDL_TIMEOUT_MMA)) break;
@@ -311,15 +337,15 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
           break;
         tc_fence_after();
         TRACE(2, it, 1);
-        if (valid(0, j) && !issue_pv(0, j)) break;
+        if (valid(0, it) && !issue_pv(0, it)) break;
         TRACE(2, it, 2);
-        if (more && valid(0, j + 1)) issue_qk(0, j + 1);
+        if (more && valid(0, it + 1)) issue_qk(0, it + 1);
         TRACE(2, it, 3);
-        if (valid(1, j) && !issue_pv(1, j)) break;
+        if (valid(1, it) && !issue_pv(1, it)) break;
         TRACE(2, it, 4);
         if (leader) tc_commit(b_vempty + 8 * vs);
         if (more) {
-          if (valid(1, j + 1)) issue_qk(1, j + 1);
+          if (valid(1, it + 1)) issue_qk(1, it + 1);
           if (leader) tc_commit(b_kempty + 8 * (s ^ 1));
         }
         TRACE(2, it, 5);
@@ -348,6 +374,8 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
     const float cap_k = cap_k2 * (0.5f * LN2);      // scale / cap
     const SoftCapNear near_cap(cap_k, cap2);
     const float mul = CAP ? 1.f : p.scale_log2;
+    // sigmoid(score + bias) = 1 / (1 + 2^y), y = -(score + bias) log2 e
+    const float sig_mul = SIG ? -p.scale_log2 : 0.f, sig_add = SIG ? -p.score_bias[qhead] * LOG2E : 0.f;
     bool alive = true;
     int n = 0;
     // One value per thread to the other half of the row and back (64-thread barrier, bounded). Wide tiles pass it through
@@ -380,7 +408,10 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
 #ifdef EDL_ATTN_TRACE
     const bool trace_on = blockIdx.x == 0 && q == 0 && lane == 0 && half == 0;
 #endif
-    for (int j = rg.lo; j < rg.hi && alive; ++j, ++n) {
+    const bool any = rg.hi > rg.lo;
+    for (int it = 0; it < steps && alive; ++it) {
+      const int j = tile_at(it);
+      if (!any || j >= rg.hi || (j < rg.lo && j >= kept_tiles)) continue;      // not a tile of this group's
       const int kv0 = j * BKV;
       const int kbase = kv0 + half * 64;
       TRACE(t, n, 0);
@@ -425,9 +456,42 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
 #pragma unroll
         for (int i = 0; i < 64; ++i) {
           const int k0 = kbase + i;
-          const bool ok0 = (k0 < len_k) && (!p.causal || k0 <= qpos) && (p.window <= 0 || k0 > qpos - p.window);
+          const bool ok0 = (k0 < len_k) && (!p.causal || k0 <= qpos) &&
+                           (p.window <= 0 || k0 > qpos - p.window || k0 < p.keep_first);
           if (!ok0) a[i] = 0xff800000u;  // -inf
         }
+      }
+      if constexpr (SIG) {
+        // Four weights per step: two exponentials on the MUFU, two polynomials, and two reciprocals for the four of them
+        // (1/x = y / (x y); y is bounded so that no product overflows, the weights it cuts off are below 2^-60).
+        uint32_t pk[32];
+        auto weights = [&](auto masked) {
+#pragma unroll
+          for (int i = 0; i < 64; i += 4) {
+            float y0, y1, y2, y3;
+            fma2(y0, y1, __uint_as_float(a[i]), __uint_as_float(a[i + 1]), sig_mul, sig_mul, sig_add, sig_add);
+            fma2(y2, y3, __uint_as_float(a[i + 2]), __uint_as_float(a[i + 3]), sig_mul, sig_mul, sig_add, sig_add);
+            const float d0 = 1.f + exp2f(fminf(y0, 60.f)), d1 = 1.f + exp2f(fminf(y1, 60.f));
+            const float d2 = 1.f + exp2_poly(fminf(y2, 60.f)), d3 = 1.f + exp2_poly(fminf(y3, 60.f));
+            const float r01 = __fdividef(1.f, d0 * d1), r23 = __fdividef(1.f, d2 * d3);
+            float w0 = r01 * d1, w1 = r01 * d0, w2 = r23 * d3, w3 = r23 * d2;
+            if constexpr (decltype(masked)::value) {
+              if (a[i] == 0xff800000u) w0 = 0.f;
+              if (a[i + 1] == 0xff800000u) w1 = 0.f;
+              if (a[i + 2] == 0xff800000u) w2 = 0.f;
+              if (a[i + 3] == 0xff800000u) w3 = 0.f;
+            }
+            pk[i >> 1] = pack_bf16x2(w0, w1);
+            pk[(i >> 1) + 1] = pack_bf16x2(w2, w3);
+          }
+        };
+        if (tile_mask) weights(std::true_type{}); else weights(std::false_type{});
+        tmem_st_32x32b_x32(tS + half * C::P_RIGHT_SIG, pk);
+        tc_wait_st();
+        tc_fence_before();
+        mbar_arrive(bp);
+        ++n;
+        continue;
       }
       float mx;
       {
@@ -502,11 +566,11 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
       tc_fence_before();
       mbar_arrive(bp);
       TRACE(t, n, 6);
+      ++n;
     }
 
     // epilogue: O / l -> bf16, plus LSE. Each half writes its own DV / 2 columns; the row sum is the two halves'.
-    const bool any = rg.hi > rg.lo;
-    if (any && alive) {
+    if (!SIG && any && alive) {
       float l_other;
       if (!exchange(l, l_other, true)) alive = false;
       l += l_other;
@@ -516,9 +580,18 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
       tc_fence_after();
     }
     if (alive && q0 < len_q) {
-      if (p.sinks) l += exp2f(p.sinks[qhead] * LOG2E - m_used);
-      const float inv_l = l > 0.f ? 1.f / l : 0.f;
       const bool row_ok = qrow < len_q;
+      float inv_l;
+      if constexpr (SIG) {
+        inv_l = p.out_scale;
+        if (p.gate && row_ok) {
+          const float g = __bfloat162float(p.gate[(long long)(q_start + qrow) * p.ld_gate + qhead]);
+          inv_l = __fdividef(p.out_scale, 1.f + exp2f(fminf(-g * LOG2E, 60.f)));
+        }
+      } else {
+        if (p.sinks) l += exp2f(p.sinks[qhead] * LOG2E - m_used);
+        inv_l = l > 0.f ? 1.f / l : 0.f;
+      }
       __nv_bfloat16* op = p.o + (long long)(q_start + qrow) * p.ldo + (long long)qhead * p.dv + half * (DV / 2);
 #pragma unroll 1
       for (int c = 0; c < DV / 64; ++c) {
@@ -558,7 +631,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
   if (warp == 1) tmem_dealloc(tmem_base, 512);
 }
 
-template <int DQ, int DV, bool CAP>
+template <int DQ, int DV, int MODE>
 int launch_fwd_as(const void* q, const void* k, const void* v, long long ldq, long long ldk, long long ldv,
                   long long total_q, long long total_k, const AttnFwdParams& p, cudaStream_t stream) {
   using C = ACfg<DQ, DV>;
@@ -566,7 +639,7 @@ int launch_fwd_as(const void* q, const void* k, const void* v, long long ldq, lo
   if (make_tmap_3d_16b(&tq, q, p.dq, p.Hq, total_q, p.dq, ldq, 64, p.pack, BQ / p.pack, 3)) return -1;
   if (make_tmap_3d_16b(&tk, k, p.dq, p.Hkv, total_k, p.dq, ldk, 64, 1, BKV, 3)) return -1;
   if (make_tmap_3d_16b(&tv, v, p.dv, p.Hkv, total_k, p.dv, ldv, 64, 1, BKV, 3)) return -1;
-  auto kern = attn_fwd_kernel<DQ, DV, CAP>;
+  auto kern = attn_fwd_kernel<DQ, DV, MODE>;
   static bool attr_set[64] = {false};  // per device
   int dev = 0;
   cudaGetDevice(&dev);
@@ -589,8 +662,10 @@ int launch_fwd_as(const void* q, const void* k, const void* v, long long ldq, lo
 template <int DQ, int DV>
 int launch_fwd(const void* q, const void* k, const void* v, long long ldq, long long ldk, long long ldv,
                long long total_q, long long total_k, const AttnFwdParams& p, cudaStream_t s) {
-  return p.softcap > 0.f ? launch_fwd_as<DQ, DV, true>(q, k, v, ldq, ldk, ldv, total_q, total_k, p, s)
-                         : launch_fwd_as<DQ, DV, false>(q, k, v, ldq, ldk, ldv, total_q, total_k, p, s);
+  if constexpr (DQ <= 128)
+    if (p.score_bias) return launch_fwd_as<DQ, DV, ATT_SIGMOID>(q, k, v, ldq, ldk, ldv, total_q, total_k, p, s);
+  return p.softcap > 0.f ? launch_fwd_as<DQ, DV, ATT_CAPPED>(q, k, v, ldq, ldk, ldv, total_q, total_k, p, s)
+                         : launch_fwd_as<DQ, DV, ATT_SOFTMAX>(q, k, v, ldq, ldk, ldv, total_q, total_k, p, s);
 }
 
 // Tile widths from the real head sizes.
@@ -662,6 +737,11 @@ EDL_HOST_API int edl_attn_fwd(const void* q, const void* k, const void* v, void*
   p.pt_stride = 0;
   p.pack = 1;
   p.dq = p.dv = D;
+  p.keep_first = 0;
+  p.score_bias = nullptr;
+  p.gate = nullptr;
+  p.ld_gate = 0;
+  p.out_scale = 1.f;
   return dispatch_fwd(q, k, v, ldq, ldk, ldv, total_q, total_k, p, reinterpret_cast<cudaStream_t>(stream));
 }
 
@@ -679,9 +759,15 @@ static int attn_paged_impl(const void* q, const void* k_pages, const void* v_pag
                            long long ldq, long long ld_kpage, long long ld_vpage, long long ldo, const int* cu_q, const int* kv_lens,
                            const int* page_table, int pt_stride, int B, int max_q, long long total_q,
                            long long num_pages, int Hq, int Hkv, int D, int Dv, float scale, int causal, int window,
-                           float softcap, const float* sinks, int* status, void* stream) {
+                           float softcap, const float* sinks, int* status, void* stream, int keep_first = 0,
+                           const float* score_bias = nullptr, const void* gate = nullptr, long long ld_gate = 0,
+                           float out_scale = 1.f) {
   using namespace edl;
   if (B <= 0 || max_q <= 0 || total_q <= 0) return 0;
+  if (score_bias && (D > 128 || softcap > 0.f || sinks || lse)) {
+    set_last_error("edl_attn_paged: sigmoid weights go with heads up to 128 wide and without cap, sinks and log-sum-exp");
+    return -1;
+  }
   if (D < 8 || D > 192 || (D & 7) || Dv < 8 || Dv > 128 || (Dv & 7) || Hkv < 1 || Hq % Hkv) {
     set_last_error("edl_attn_paged: unsupported head layout (D=%d, Dv=%d, Hq=%d, Hkv=%d)", D, Dv, Hq, Hkv);
     return -1;
@@ -717,6 +803,11 @@ static int attn_paged_impl(const void* q, const void* k_pages, const void* v_pag
   p.pack = G;
   p.dq = D;
   p.dv = Dv;
+  p.keep_first = keep_first;
+  p.score_bias = score_bias;
+  p.gate = reinterpret_cast<const __nv_bfloat16*>(gate);
+  p.ld_gate = ld_gate;
+  p.out_scale = out_scale;
   return dispatch_fwd(q, k_pages, v_pages, ldq, ld_kpage, ld_vpage, total_q, num_pages * 128, p,
                       reinterpret_cast<cudaStream_t>(stream));
 }
@@ -725,9 +816,23 @@ EDL_HOST_API int edl_attn_paged(const void* q, const void* k_pages, const void* 
                                 long long ld_kpage, long long ld_vpage, long long ldo, const int* cu_q,
                                 const int* kv_lens, const int* page_table, int pt_stride, int B, int max_q, long long total_q,
                                 long long num_pages, int Hq, int Hkv, int D, int Dv, float scale, int causal, int window,
-                                float softcap, const float* sinks, int* status, void* stream) {
+                                int keep_first, float softcap, const float* sinks, int* status, void* stream) {
   return attn_paged_impl(q, k_pages, v_pages, o, nullptr, ldq, ld_kpage, ld_vpage, ldo, cu_q, kv_lens, page_table, pt_stride, B,
-                         max_q, total_q, num_pages, Hq, Hkv, D, Dv, scale, causal, window, softcap, sinks, status, stream);
+                         max_q, total_q, num_pages, Hq, Hkv, D, Dv, scale, causal, window, softcap, sinks, status, stream,
+                         keep_first);
+}
+
+// The same without a softmax: a visible key's weight is sigmoid(score + score_bias[head]); the output is multiplied by
+// out_scale and, with a gate [total_q, ld_gate] (bf16), by sigmoid(gate[token][head]). D up to 128.
+EDL_HOST_API int edl_attn_paged_sigmoid(const void* q, const void* k_pages, const void* v_pages, void* o, long long ldq,
+                                        long long ld_kpage, long long ld_vpage, long long ldo, const int* cu_q,
+                                        const int* kv_lens, const int* page_table, int pt_stride, int B, int max_q,
+                                        long long total_q, long long num_pages, int Hq, int Hkv, int D, int Dv, float scale,
+                                        int window, int keep_first, const float* score_bias, const void* gate,
+                                        long long ld_gate, float out_scale, int* status, void* stream) {
+  return attn_paged_impl(q, k_pages, v_pages, o, nullptr, ldq, ld_kpage, ld_vpage, ldo, cu_q, kv_lens, page_table, pt_stride, B,
+                         max_q, total_q, num_pages, Hq, Hkv, D, Dv, scale, 1, window, 0.f, nullptr, status, stream, keep_first,
+                         score_bias, gate, ld_gate, out_scale);
 }
 
 // Same, also writing lse [Hq, total_q] (natural log of the softmax denominator; -inf for a row without keys):

@@ -3,8 +3,8 @@
 // and head sizes outside the tensor-core kernels' tiles.
 //
 // One CTA per (query token, query head) walks the keys a page at a time: one key per thread for the scores, then one
-// value column per thread for the weighted sum, with an online softmax between them. The sink logit of a head joins the
-// denominator once at the end. Compiled without fast-math.
+// value column per thread for the weighted sum, with an online softmax between them (or weights that are sigmoids and need
+// no normalisation). The sink logit of a head joins the denominator once at the end. Compiled without fast-math.
 #include "common.cuh"
 
 namespace edl {
@@ -50,8 +50,9 @@ __global__ void __launch_bounds__(ST)
 attn_simt_kernel(const T* __restrict__ q, const T* __restrict__ k_pages, const T* __restrict__ v_pages,
                  T* __restrict__ o, long long ldq, long long ld_kpage, long long ld_vpage, const int* __restrict__ cu,
                  const int* __restrict__ kv_lens, const int* __restrict__ page_table, int pt_stride, int B,
-                 long long num_pages, int Hq, int Hkv, int D, int Dv, float scale, int window, float softcap,
-                 const float* __restrict__ sinks, bool vec, int* status) {
+                 long long num_pages, int Hq, int Hkv, int D, int Dv, float scale, int window, int keep_first,
+                 float softcap, const float* __restrict__ sinks, const float* __restrict__ score_bias,
+                 const T* __restrict__ gate, long long ld_gate, float out_scale, long long ldo, bool vec, int* status) {
   __shared__ float sq[MAX_D];
   __shared__ float sp[ST];
   __shared__ float red[32];
@@ -73,23 +74,30 @@ attn_simt_kernel(const T* __restrict__ q, const T* __restrict__ k_pages, const T
   float acc[MAX_VC];
 #pragma unroll
   for (int i = 0; i < MAX_VC; ++i) acc[i] = 0.f;
-  for (int tile = k_lo / ST; tile * ST <= qpos; ++tile) {
+  const int first_tile = k_lo / ST, front = window > 0 ? min((keep_first + ST - 1) / ST, first_tile) : 0;
+  for (int tile = front > 0 ? 0 : first_tile; tile * ST <= qpos; tile = tile + 1 == front ? first_tile : tile + 1) {
     const long long page = pt[tile];
     if (page < 0 || page >= num_pages) {               // uniform over the CTA
       if (status && tid == 0) atomicCAS(status, 0, EDL_BAD_INDEX);
       continue;
     }
     const int key = tile * ST + tid;
-    const bool ok = key >= k_lo && key <= qpos;
+    const bool ok = (key >= k_lo || key < keep_first) && key <= qpos;
     float s = -INFINITY;
     if (ok) s = dot_row(k_pages + (page * ST + tid) * ld_kpage + (long long)hk * D, sq, D, vec) * scale;
     if (ok && softcap > 0.f) s = softcap * tanhf(s / softcap);
-    const float m_new = fmaxf(m, block_max(s, red));
-    const float alpha = m == -INFINITY ? 0.f : expf(m - m_new);
-    const float p = ok ? expf(s - m_new) : 0.f;
-    sp[tid] = p;
-    l = l * alpha + block_sum(p, red);                 // its barriers also publish sp
-    m = m_new;
+    float alpha = 1.f;
+    if (score_bias) {                                  // no softmax: weights stand alone
+      sp[tid] = ok ? 1.f / (1.f + expf(-(s + score_bias[h]))) : 0.f;
+      __syncthreads();
+    } else {
+      const float m_new = fmaxf(m, block_max(s, red));
+      alpha = m == -INFINITY ? 0.f : expf(m - m_new);
+      const float p = ok ? expf(s - m_new) : 0.f;
+      sp[tid] = p;
+      l = l * alpha + block_sum(p, red);               // its barriers also publish sp
+      m = m_new;
+    }
     const int n = min(ST, qpos - tile * ST + 1);
     const T* vb = v_pages + page * ST * ld_vpage + (long long)hk * Dv;
 #pragma unroll
@@ -97,7 +105,7 @@ attn_simt_kernel(const T* __restrict__ q, const T* __restrict__ k_pages, const T
       const int c = tid + i * ST;
       if (c < Dv) {
         float a0 = acc[i] * alpha, a1 = 0.f;
-        int j = max(0, k_lo - tile * ST);
+        int j = tile * ST < keep_first ? 0 : max(0, k_lo - tile * ST);      // weights of unseen keys are zero
         for (; j + 1 < n; j += 2) {
           a0 = fmaf(sp[j], f_of(vb[j * ld_vpage + c]), a0);
           a1 = fmaf(sp[j + 1], f_of(vb[(j + 1) * ld_vpage + c]), a1);
@@ -114,23 +122,26 @@ attn_simt_kernel(const T* __restrict__ q, const T* __restrict__ k_pages, const T
     w = m == -INFINITY ? 0.f : expf(m - m_new);
     l = l * w + expf(sinks[h] - m_new);
   }
-  const float inv = l > 0.f ? w / l : 0.f;
+  float inv = l > 0.f ? w / l : 0.f;
+  if (score_bias) inv = out_scale / (gate ? 1.f + expf(-f_of(gate[t * ld_gate + h])) : 1.f);
 #pragma unroll
   for (int i = 0; i < MAX_VC; ++i) {
     const int c = tid + i * ST;
-    if (c < Dv) put(o + ((long long)t * Hq + h) * Dv + c, acc[i] * inv);
+    if (c < Dv) put(o + t * ldo + (long long)h * Dv + c, acc[i] * inv);
   }
 }
 
 template <typename T>
 int launch_simt(const void* q, const void* k, const void* v, void* o, long long ldq, long long ldk, long long ldv,
                 const int* cu, const int* kv_lens, const int* pt, int pt_stride, int B, int T_rows,
-                long long num_pages, int Hq, int Hkv, int D, int Dv, float scale, int window, float softcap,
-                const float* sinks, int* status, cudaStream_t s) {
+                long long num_pages, int Hq, int Hkv, int D, int Dv, float scale, int window, int keep_first, float softcap,
+                const float* sinks, const float* score_bias, const void* gate, long long ld_gate, float out_scale,
+                long long ldo, int* status, cudaStream_t s) {
   const bool vec = D % 4 == 0 && ldk % 4 == 0 && (reinterpret_cast<uintptr_t>(k) & 15) == 0;
   attn_simt_kernel<T><<<dim3(T_rows, Hq), ST, 0, s>>>((const T*)q, (const T*)k, (const T*)v, (T*)o, ldq, ldk, ldv, cu,
                                                       kv_lens, pt, pt_stride, B, num_pages, Hq, Hkv, D, Dv, scale,
-                                                      window, softcap, sinks, vec, status);
+                                                      window, keep_first, softcap, sinks, score_bias, (const T*)gate,
+                                                      ld_gate, out_scale, ldo, vec, status);
   return check_cuda(cudaGetLastError(), "attn_simt launch");
 }
 
@@ -138,13 +149,16 @@ int launch_simt(const void* q, const void* k, const void* v, void* o, long long 
 }  // namespace edl
 
 // q [T, ldq] (head h at columns h * D), key / value pages [num_pages * 128, ld] with the heads packed in a row,
-// o [T, Hq * Dv]; cu [B + 1], kv_lens [B], page_table [B, pt_stride] as in edl_attn_paged; f32: storage type; softcap > 0:
-// scores become softcap * tanh(score / softcap).
+// o [T, ldo] (head h at columns h * Dv); cu [B + 1], kv_lens [B], page_table [B, pt_stride] as in edl_attn_paged; f32: storage
+// type; softcap > 0: scores become softcap * tanh(score / softcap); keep_first: keys that stay visible under a window.
+// score_bias [Hq] (may be null): no softmax, weights are sigmoid(score + bias), the output is multiplied by out_scale and, with a
+// gate [T, ld_gate] in the storage type, by sigmoid(gate[t][h]).
 EDL_HOST_API int edl_attn_simt(const void* q, const void* k_pages, const void* v_pages, void* o, int f32,
-                               long long ldq, long long ld_kpage, long long ld_vpage, const int* cu,
+                               long long ldq, long long ld_kpage, long long ld_vpage, long long ldo, const int* cu,
                                const int* kv_lens, const int* page_table, int pt_stride, int B, int T,
-                               long long num_pages, int Hq, int Hkv, int D, int Dv, float scale, int window,
-                             float softcap, const float* sinks, int* status, void* stream) {
+                               long long num_pages, int Hq, int Hkv, int D, int Dv, float scale, int window, int keep_first,
+                               float softcap, const float* sinks, const float* score_bias, const void* gate,
+                               long long ld_gate, float out_scale, int* status, void* stream) {
   using namespace edl;
   if (B <= 0 || T <= 0) return 0;
   if (D < 1 || D > MAX_D || Dv < 1 || Dv > MAX_VC * ST || Hkv < 1 || Hq % Hkv || Hq > 65535) {
@@ -153,8 +167,9 @@ EDL_HOST_API int edl_attn_simt(const void* q, const void* k_pages, const void* v
   }
   cudaStream_t s = (cudaStream_t)stream;
   return f32 ? launch_simt<float>(q, k_pages, v_pages, o, ldq, ld_kpage, ld_vpage, cu, kv_lens, page_table, pt_stride,
-                                  B, T, num_pages, Hq, Hkv, D, Dv, scale, window, softcap, sinks, status, s)
+                                  B, T, num_pages, Hq, Hkv, D, Dv, scale, window, keep_first, softcap, sinks, score_bias,
+                                  gate, ld_gate, out_scale, ldo, status, s)
              : launch_simt<__nv_bfloat16>(q, k_pages, v_pages, o, ldq, ld_kpage, ld_vpage, cu, kv_lens, page_table,
-                                          pt_stride, B, T, num_pages, Hq, Hkv, D, Dv, scale, window, softcap, sinks,
-                                          status, s);
+                                          pt_stride, B, T, num_pages, Hq, Hkv, D, Dv, scale, window, keep_first, softcap,
+                                          sinks, score_bias, gate, ld_gate, out_scale, ldo, status, s);
 }

@@ -47,7 +47,7 @@ NVCC_FLAGS = [
 
 # Kernels whose job is 32-bit arithmetic (fp32 residual stream, gates and recurrences, attention of fp32 models) are
 # compiled without fast-math.
-PRECISE = frozenset({"stream_ops", "hgrn2", "attention_simt", "latent_ops", "moe_serving"})
+PRECISE = frozenset({"stream_ops", "hgrn2", "gdelta", "attention_simt", "latent_ops", "moe_serving"})
 
 # What serving a model family needs, by model type, for a first call on a machine without a built library.
 SERVING_PARTS = {
@@ -57,6 +57,8 @@ SERVING_PARTS = {
                 "host_native", "stream_ops", "latent_ops", "moe", "moe_serving"),
     "gasetar": ("common", "gemm", "attention_fwd", "attention_decode", "attention_mla_decode", "attn_combine",
                 "attention_simt", "serving", "host_native", "stream_ops", "latent_ops", "moe", "moe_serving", "norm_act"),
+    "ninisun": ("common", "gemm", "attention_fwd", "attention_decode", "attn_combine", "attention_simt", "serving",
+                "host_native", "stream_ops", "gdelta", "norm_act"),
 }
 MANIFEST_SUFFIX = ".sources.json"      # beside a linked library: the digest of every source it was built from
 

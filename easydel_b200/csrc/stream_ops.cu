@@ -11,8 +11,10 @@
 //   * xIELU, a two-branch activation with two learned numbers;
 //   * the attention prologue: per-head RMS norm of q and k, position-dependent query temperature and the page append,
 //     in one pass over the packed projection;
-//   * the same with norms over all query heads (all key heads) at once and rotated halves;
-//   * scaled and soft-capped logits.
+//   * the same with biases, norms over all query heads (all key heads) at once, rotated halves or neighbours, and values that
+//     blend with another layer's;
+//   * a branch that is normed (and scaled per channel) before it joins the stream, with the norm that reads the sum;
+//   * gated units in 32 bits or at odd sizes, and scaled and soft-capped logits.
 //
 // Compiled without fast-math: these are the parts of such a model that are computed in 32 bits.
 #include "common.cuh"
@@ -557,7 +559,45 @@ struct RotaryPrologueParams {
   int pairs, Hq, Hkv, D, Dv;
   long long ld_kpage, ld_vpage, num_slots;
   int* status;
+  int neighbours;            // elements 2j and 2j + 1 form a pair (else j and j + pairs)
+  float mag;                 // factor of cosines and sines
+  const float* bias;         // [Hq * D + Hkv * (D + Dv)] added to the row first, or null
+  const void* v_first;       // values [T, Hkv * Dv] at pitch ld_first to blend in by *lam, or null
+  long long ld_first;
+  const float* lam;
 };
+
+// cos and sin of position * frequency i, times mag. Angles are as exact as in the latent prologue: the product's rounding
+// error and the frequency's own are a small second rotation.
+__device__ __forceinline__ float2 turn_of(const RotaryPrologueParams& p, float fp, int i) {
+  const float f = p.freq[i], a = fp * f;
+  const float e = fmaf(fp, f, -a) + fp * p.freq[p.pairs + i];
+  float s, c;
+  sincosf(a, &s, &c);
+  const float ce = 1.f - 0.5f * e * e, se = e - e * e * e * (1.f / 6.f);
+  return make_float2((c * ce - s * se) * p.mag, (s * ce + c * se) * p.mag);
+}
+
+// v[j] += bias[at + j]
+template <int VEC>
+__device__ __forceinline__ void add_bias(const float* bias, int at, float (&v)[VEC]) {
+  if (!bias) return;
+#pragma unroll
+  for (int j = 0; j < VEC; ++j) v[j] += bias[at + j];
+}
+
+// Values of token t from column c on: bias, blend with the first layer's.
+template <typename T, int VEC>
+__device__ __forceinline__ void finish_values(const RotaryPrologueParams& p, int t, int c, int at, float (&v)[VEC]) {
+  add_bias<VEC>(p.bias, at, v);
+  if (p.lam) {
+    const float l = *p.lam;
+    float f[VEC];
+    ldv<VEC>(reinterpret_cast<const T*>(p.v_first) + t * p.ld_first + c, f);
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) v[j] = (1.f - l) * v[j] + l * f[j];
+  }
+}
 
 template <int VEC>
 __device__ __forceinline__ void ldw(const float* w, float (&v)[VEC]) {
@@ -573,9 +613,9 @@ __device__ __forceinline__ void ldw(const float* w, float (&v)[VEC]) {
   }
 }
 
-// One CTA per token: qkv [T, ld] as above. Queries and keys are RMS-normed over all their heads at once, then elements j and
-// j + pairs of every head turn by position * frequency j (angles as exact as in the latent prologue: the product's rounding
-// error and the frequency's own are a small second rotation). A thread handles VEC elements and their partners.
+// One CTA per token: qkv [T, ld] as above. Queries and keys are RMS-normed over all their heads at once, then the pairs of
+// every head turn by position * frequency. A thread handles VEC elements and their partners (neighbours, unless VEC is 1, are
+// each other's partners within the piece).
 template <typename T, int VEC>
 __global__ void __launch_bounds__(NT)
 qkv_rotary_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, T* __restrict__ k_pages, T* __restrict__ v_pages,
@@ -586,19 +626,13 @@ qkv_rotary_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, T* __restric
   const T* row = qkv + t * p.ld;
   const int nq = p.Hq * p.D, nk = p.Hkv * p.D;
   const float fp = p.pairs ? (float)p.pos[t] : 0.f;
-  for (int i = tid; i < p.pairs; i += NT) {
-    const float f = p.freq[i], a = fp * f;
-    const float e = fmaf(fp, f, -a) + fp * p.freq[p.pairs + i];
-    float s, c;
-    sincosf(a, &s, &c);
-    const float ce = 1.f - 0.5f * e * e, se = e - e * e * e * (1.f / 6.f);
-    cs[i] = make_float2(c * ce - s * se, s * ce + c * se);
-  }
+  for (int i = tid; i < p.pairs; i += NT) cs[i] = turn_of(p, fp, i);
   float sq = 0.f, sk = 0.f;
   if (p.qw)
     for (int c = tid * VEC; c < nq; c += NT * VEC) {
       float v[VEC];
       ldv<VEC>(row + c, v);
+      add_bias<VEC>(p.bias, c, v);
 #pragma unroll
       for (int j = 0; j < VEC; ++j) sq += v[j] * v[j];
     }
@@ -606,6 +640,7 @@ qkv_rotary_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, T* __restric
     for (int c = tid * VEC; c < nk; c += NT * VEC) {
       float v[VEC];
       ldv<VEC>(row + nq + c, v);
+      add_bias<VEC>(p.bias, nq + c, v);
 #pragma unroll
       for (int j = 0; j < VEC; ++j) sk += v[j] * v[j];
     }
@@ -617,7 +652,9 @@ qkv_rotary_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, T* __restric
     if (p.status && tid == 0) atomicCAS(p.status, 0, EDL_BAD_INDEX);
     slot = -1;
   }
-  const int turned = p.pairs / VEC, per = turned + (p.D - 2 * p.pairs) / VEC;   // units of a head: pairs, then the rest
+  const bool inside = p.neighbours && VEC > 1;       // pairs lie within a piece
+  const int turned = (inside ? 2 : 1) * p.pairs / VEC;
+  const int per = turned + (p.D - 2 * p.pairs) / VEC;   // units of a head: pairs, then the rest
   const int units = (p.Hq + (slot >= 0 ? p.Hkv : 0)) * per;
   for (int i = tid; i < units; i += NT) {
     const int h = i / per, u = i - h * per;
@@ -628,6 +665,7 @@ qkv_rotary_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, T* __restric
     const float r = is_q ? rq : rk;
     auto load = [&](int c, float (&v)[VEC]) {
       ldv<VEC>(src + c, v);
+      add_bias<VEC>(p.bias, h * p.D + c, v);
       if (w) {
         float wv[VEC];
         ldw<VEC>(w + c, wv);
@@ -636,20 +674,31 @@ qkv_rotary_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, T* __restric
       }
     };
     float a[VEC];
-    if (u < turned) {
+    if (u < turned && inside) {
       const int c = u * VEC;
+      load(c, a);
+#pragma unroll
+      for (int j = 0; j + 1 < VEC; j += 2) {
+        const float2 g = cs[(c + j) >> 1];
+        const float x = a[j], y = a[j + 1];
+        a[j] = x * g.x - y * g.y;
+        a[j + 1] = y * g.x + x * g.y;
+      }
+      stv<VEC>(dst + c, a);
+    } else if (u < turned) {
+      const int c = p.neighbours ? 2 * u : u * VEC, partner = c + (p.neighbours ? 1 : p.pairs);
       float b[VEC];
       load(c, a);
-      load(c + p.pairs, b);
+      load(partner, b);
 #pragma unroll
       for (int j = 0; j < VEC; ++j) {
-        const float2 g = cs[c + j];
+        const float2 g = cs[u * VEC + j];
         const float x = a[j], y = b[j];
         a[j] = x * g.x - y * g.y;
         b[j] = y * g.x + x * g.y;
       }
       stv<VEC>(dst + c, a);
-      stv<VEC>(dst + c + p.pairs, b);
+      stv<VEC>(dst + partner, b);
     } else {
       const int c = 2 * p.pairs + (u - turned) * VEC;
       load(c, a);
@@ -660,6 +709,7 @@ qkv_rotary_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, T* __restric
     for (int c = tid * VEC; c < p.Hkv * p.Dv; c += NT * VEC) {
       float v[VEC];
       ldv<VEC>(row + nq + nk + c, v);
+      finish_values<T, VEC>(p, t, c, nq + nk + c, v);
       stv<VEC>(v_pages + slot * p.ld_vpage + c, v);
     }
 }
@@ -678,16 +728,18 @@ qkv_rotary_walk_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, T* __re
   __shared__ float2 red[2][RW_THREADS / 32];
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, warps = (blockDim.x + 31) >> 5;
   const int nq = p.Hq * p.D, nk = p.Hkv * p.D, nv = p.Hkv * p.Dv;
-  const int turned = p.pairs / VEC, per = turned + (p.D - 2 * p.pairs) / VEC, units = (p.Hq + p.Hkv) * per;
-  int col[KEEP];             // first element within the row (< 0: no unit); partner `pairs` further
-  bool pair[KEEP];
+  const int turned = (p.neighbours ? 2 : 1) * p.pairs / VEC, per = turned + (p.D - 2 * p.pairs) / VEC;
+  const int units = (p.Hq + p.Hkv) * per;
+  int col[KEEP];             // first element within the row (< 0: no unit); halves have a partner `pairs` further
+  bool pair[KEEP], inside[KEEP];
   float wa[KEEP][VEC], wb[KEEP][VEC];
 #pragma unroll
   for (int i = 0; i < KEEP; ++i) {
     const int u = tid + i * blockDim.x;
     const int h = u / per, r = u - h * per;
-    pair[i] = r < turned;
-    col[i] = u < units ? h * p.D + (pair[i] ? r * VEC : 2 * p.pairs + (r - turned) * VEC) : -1;
+    pair[i] = r < turned && !p.neighbours;
+    inside[i] = r < turned && p.neighbours;
+    col[i] = u < units ? h * p.D + (r < turned ? r * VEC : 2 * p.pairs + (r - turned) * VEC) : -1;
 #pragma unroll
     for (int j = 0; j < VEC; ++j) wa[i][j] = wb[i][j] = 1.f;
     if (col[i] >= 0) {
@@ -719,41 +771,51 @@ qkv_rotary_walk_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, T* __re
       slot = -1;
     }
     if (slot >= 0)
-      for (int c = tid * VEC; c < nv; c += blockDim.x * VEC)
-        *reinterpret_cast<Raw*>(v_pages + slot * p.ld_vpage + c) =
-            *reinterpret_cast<const Raw*>(qkv + t * p.ld + nq + nk + c);
+      for (int c = tid * VEC; c < nv; c += blockDim.x * VEC) {
+        const T* src = qkv + t * p.ld + nq + nk + c;
+        T* dst = v_pages + slot * p.ld_vpage + c;
+        if (p.lam || p.bias) {
+          float v[VEC];
+          ldv<VEC>(src, v);
+          finish_values<T, VEC>(p, t, c, nq + nk + c, v);
+          stv<VEC>(dst, v);
+        } else {
+          *reinterpret_cast<Raw*>(dst) = *reinterpret_cast<const Raw*>(src);
+        }
+      }
     const float fp = p.pairs ? (float)p.pos[t] : 0.f;
-    for (int i = tid; i < p.pairs; i += blockDim.x) {
-      const float f = p.freq[i], x = fp * f;
-      const float e = fmaf(fp, f, -x) + fp * p.freq[p.pairs + i];
-      float s, c;
-      sincosf(x, &s, &c);
-      const float ce = 1.f - 0.5f * e * e, se = e - e * e * e * (1.f / 6.f);
-      cs[buf][i] = make_float2(c * ce - s * se, s * ce + c * se);
-    }
+    for (int i = tid; i < p.pairs; i += blockDim.x) cs[buf][i] = turn_of(p, fp, i);
     float va[KEEP][VEC], vb[KEEP][VEC], sq = 0.f, sk = 0.f;
 #pragma unroll
     for (int i = 0; i < KEEP; ++i) {
       if (col[i] < 0) continue;
       ldv<VEC>(reinterpret_cast<const T*>(&a[i]), va[i]);
+      add_bias<VEC>(p.bias, col[i], va[i]);
       float s = 0.f;
 #pragma unroll
       for (int j = 0; j < VEC; ++j) s += va[i][j] * va[i][j];
       if (pair[i]) {
         ldv<VEC>(reinterpret_cast<const T*>(&b[i]), vb[i]);
+        add_bias<VEC>(p.bias, col[i] + p.pairs, vb[i]);
 #pragma unroll
         for (int j = 0; j < VEC; ++j) s += vb[i][j] * vb[i][j];
       }
       if (col[i] < nq) sq += s; else sk += s;
     }
     if (t + (int)gridDim.x < rows) load(t + gridDim.x);
-    sq = warp_sum(sq);
-    sk = warp_sum(sk);
-    if (lane == 0) red[buf][warp] = make_float2(sq, sk);
+    const bool normed = p.qw || p.kw;
+    if (normed) {
+      sq = warp_sum(sq);
+      sk = warp_sum(sk);
+      if (lane == 0) red[buf][warp] = make_float2(sq, sk);
+    }
     __syncthreads();
-    float2 sums = lane < warps ? red[buf][lane] : make_float2(0.f, 0.f);
-    sums.x = warp_sum(sums.x);
-    sums.y = warp_sum(sums.y);
+    float2 sums = make_float2(0.f, 0.f);
+    if (normed) {
+      if (lane < warps) sums = red[buf][lane];
+      sums.x = warp_sum(sums.x);
+      sums.y = warp_sum(sums.y);
+    }
     const float rq = p.qw ? 1.f / sqrtf(sums.x / (float)nq + p.eps) : 1.f;
     const float rk = p.kw ? 1.f / sqrtf(sums.y / (float)nk + p.eps) : 1.f;
 #pragma unroll
@@ -775,6 +837,15 @@ qkv_rotary_walk_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, T* __re
           vb[i][j] = y * g.x + x * g.y;
         }
         stv<VEC>(dst + p.pairs, vb[i]);
+      } else if (inside[i]) {
+        const int c0 = (col[i] % p.D) >> 1;
+#pragma unroll
+        for (int j = 0; j < VEC; j += 2) {
+          const float2 g = cs[buf][c0 + (j >> 1)];
+          const float x = va[i][j], y = va[i][j + 1];
+          va[i][j] = x * g.x - y * g.y;
+          va[i][j + 1] = y * g.x + x * g.y;
+        }
       }
       stv<VEC>(dst, va[i]);
     }
@@ -784,7 +855,7 @@ qkv_rotary_walk_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, T* __re
 template <typename T, int VEC>
 bool launch_rotary_walk(const void* qkv, void* q_out, void* k_pages, void* v_pages, const RotaryPrologueParams& p, int rows,
                         cudaStream_t s) {
-  const int units = (p.Hq + p.Hkv) * (p.pairs / VEC + (p.D - 2 * p.pairs) / VEC);
+  const int units = (p.Hq + p.Hkv) * ((p.neighbours ? 2 : 1) * p.pairs / VEC + (p.D - 2 * p.pairs) / VEC);
   const int keep = units <= RW_THREADS ? 1 : 2;
   if (units > 2 * RW_THREADS) return false;
   const int threads = ((units + keep - 1) / keep + 31) / 32 * 32;
@@ -794,6 +865,126 @@ bool launch_rotary_walk(const void* qkv, void* q_out, void* k_pages, void* v_pag
   if (keep == 1) EDL_RW(1); else EDL_RW(2);
 #undef EDL_RW
   return true;
+}
+
+// ---- a normed branch joins the stream ----------------------------------------------------------------------------------------
+// x <- x + rms_norm(y) * wb * ls, h = rms_norm(x) * w: one CTA per row. NV as above (0: wide rows are read again).
+template <typename TO, int VEC, int NV>
+__global__ void __launch_bounds__(NT)
+branch_norm_kernel(float* __restrict__ x, const float* __restrict__ y, const float* __restrict__ wb,
+                   const float* __restrict__ ls, float eps_b, const float* __restrict__ w, float eps, TO* __restrict__ h,
+                   int W) {
+  __shared__ float2 red[NT / 32];
+  constexpr int STEP = NT * VEC, KEEP = NV > 0 ? NV : 1;
+  const long long at = (long long)blockIdx.x * W;
+  float* xr = x + at;
+  const float* yr = y + at;
+  float a[KEEP][VEC], s[KEEP][VEC];
+  float sum = 0.f;
+  // branch rows and stream rows are fetched together, so that the two sums wait for memory once
+  auto fetch = [&](int c, float (&ya)[VEC], float (&xa)[VEC]) {
+    ldv<VEC>(yr + c, ya);
+    ldv<VEC>(xr + c, xa);
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) sum += ya[j] * ya[j];
+  };
+  if constexpr (NV > 0) {
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+      const int c = threadIdx.x * VEC + k * STEP;
+      if (c < W) fetch(c, a[k], s[k]);
+    }
+  } else {
+    for (int c = threadIdx.x * VEC; c < W; c += STEP) fetch(c, a[0], s[0]);
+  }
+  const float rb = 1.f / sqrtf(block_sum2(sum, 0.f, red).x / (float)W + eps_b);
+  sum = 0.f;
+  auto join = [&](int c, const float (&ya)[VEC], float (&xa)[VEC]) {
+    float wv[VEC], lv[VEC];
+    ldv<VEC>(wb + c, wv);
+    if (ls) ldv<VEC>(ls + c, lv);
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) {
+      float b = ya[j] * rb * wv[j];
+      if (ls) b *= lv[j];
+      xa[j] += b;
+      sum += xa[j] * xa[j];
+    }
+    stv<VEC>(xr + c, xa);
+  };
+  if constexpr (NV > 0) {
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+      const int c = threadIdx.x * VEC + k * STEP;
+      if (c < W) join(c, a[k], s[k]);
+    }
+  } else {
+    for (int c = threadIdx.x * VEC; c < W; c += STEP) {
+      ldv<VEC>(yr + c, a[0]);
+      ldv<VEC>(xr + c, s[0]);
+      join(c, a[0], s[0]);         // read back below by the thread that wrote it
+    }
+  }
+  const float rs = 1.f / sqrtf(block_sum2(sum, 0.f, red).x / (float)W + eps);
+  auto emit = [&](int c, const float (&xa)[VEC]) {
+    float wv[VEC], o[VEC];
+    ldv<VEC>(w + c, wv);
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) o[j] = xa[j] * rs * wv[j];
+    stv<VEC>(h + at + c, o);
+  };
+  if constexpr (NV > 0) {
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+      const int c = threadIdx.x * VEC + k * STEP;
+      if (c < W) emit(c, s[k]);
+    }
+  } else {
+    for (int c = threadIdx.x * VEC; c < W; c += STEP) {
+      ldv<VEC>(xr + c, s[0]);
+      emit(c, s[0]);
+    }
+  }
+}
+
+template <typename TO, int VEC>
+void launch_branch_norm(float* x, const float* y, const float* wb, const float* ls, float eps_b, const float* w, float eps,
+                        TO* h, int rows, int W, cudaStream_t s) {
+  const int nv = (W + NT * VEC - 1) / (NT * VEC);
+#define EDL_BN(N) branch_norm_kernel<TO, VEC, N><<<rows, NT, 0, s>>>(x, y, wb, ls, eps_b, w, eps, h, W)
+  if (nv <= 1) EDL_BN(1);
+  else if (nv <= 2) EDL_BN(2);
+  else if (nv <= 4) EDL_BN(4);
+  else if (nv <= 8) EDL_BN(8);
+  else EDL_BN(0);
+#undef EDL_BN
+}
+
+// ---- gated units of any size -------------------------------------------------------------------------------------------------
+enum { ACT_SILU = 0, ACT_GELU_TANH = 1, ACT_GELU_ERF = 2, ACT_RELU = 3 };
+
+__device__ __forceinline__ float act_of(float z, int act) {
+  if (act == ACT_SILU) return z / (1.f + expf(-z));
+  if (act == ACT_GELU_TANH) return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+  if (act == ACT_GELU_ERF) return 0.5f * z * (1.f + erff(z * 0.7071067811865476f));
+  return fmaxf(z, 0.f);
+}
+
+// out [T, F] = act(gu[:, :F]) * gu[:, F:]
+template <typename T, int VEC>
+__global__ void __launch_bounds__(NT)
+gated_unit_kernel(const T* __restrict__ gu, long long ld, T* __restrict__ out, int rows, int F, int act) {
+  const int per = F / VEC;
+  const long long total = (long long)rows * per;
+  for (long long i = blockIdx.x * (long long)NT + threadIdx.x; i < total; i += (long long)gridDim.x * NT) {
+    const int r = (int)(i / per), c = (int)(i - (long long)r * per) * VEC;
+    float g[VEC], u[VEC];
+    ldv<VEC>(gu + r * ld + c, g);
+    ldv<VEC>(gu + r * ld + F + c, u);
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) g[j] = act_of(g[j], act) * u[j];
+    stv<VEC>(out + (long long)r * F + c, g);
+  }
 }
 
 // ---- logits ------------------------------------------------------------------------------------------------------------------
@@ -978,22 +1169,27 @@ EDL_HOST_API int edl_qkv_prologue(const void* qkv, int f32, long long ld, const 
 }
 
 // The prologue for queries and keys that are normed over all heads at once (qw [Hq * D], kw [Hkv * D], null: no norm) and
-// rotated by halves (freq: 2 * pairs floats, leading and trailing parts; pairs = 0: no rotation).
+// rotated, by halves or by neighbours (freq: 2 * pairs floats, leading and trailing parts; pairs = 0: no rotation; mag: factor
+// of cosines and sines). bias [Hq * D + Hkv * (D + Dv)] (may be null) is added first; with lam the cached values are
+// (1 - *lam) v + *lam v_first, v_first [T, Hkv * Dv] at pitch ld_first.
 EDL_HOST_API int edl_qkv_rotary_prologue(const void* qkv, int f32, long long ld, const int* pos, const int* slots,
-                                         const float* qw, const float* kw, float eps, const float* freq, int pairs, int T,
-                                         int Hq, int Hkv, int D, int Dv, void* q_out, void* k_pages, void* v_pages,
-                                         long long ld_kpage, long long ld_vpage, long long num_slots, int* status,
-                                         void* stream) {
+                                         const float* qw, const float* kw, float eps, const float* freq, int pairs,
+                                         int neighbours, float mag, const float* bias, const void* v_first,
+                                         long long ld_first, const float* lam, int T, int Hq, int Hkv, int D, int Dv,
+                                         void* q_out, void* k_pages, void* v_pages, long long ld_kpage, long long ld_vpage,
+                                         long long num_slots, int* status, void* stream) {
   if (T <= 0) return 0;
   if (Hq <= 0 || Hkv <= 0 || D <= 0 || Dv <= 0 || !slots || pairs < 0 || 2 * pairs > D || pairs > RP_MAX_PAIRS ||
-      (pairs > 0 && (!pos || !freq))) {
+      (pairs > 0 && (!pos || !freq)) || (lam && !v_first)) {
     set_last_error("edl_qkv_rotary_prologue: bad arguments (Hq=%d, Hkv=%d, D=%d, Dv=%d, pairs=%d)", Hq, Hkv, D, Dv, pairs);
     return -1;
   }
-  const RotaryPrologueParams p{ld, pos, slots, qw, kw, eps, freq, pairs, Hq, Hkv, D, Dv, ld_kpage, ld_vpage, num_slots, status};
+  const RotaryPrologueParams p{ld,       pos,       slots,  qw,         kw,  eps,  freq,    pairs,    Hq,  Hkv, D, Dv,
+                               ld_kpage, ld_vpage, num_slots, status, neighbours, mag, bias, v_first, ld_first, lam};
   cudaStream_t s = (cudaStream_t)stream;
   auto fits = [&](int m, size_t a) {
-    return D % m == 0 && pairs % m == 0 && Dv % m == 0 && ld % m == 0 && ld_kpage % m == 0 && ld_vpage % m == 0 &&
+    return D % m == 0 && (neighbours ? 2 * pairs : pairs) % m == 0 && Dv % m == 0 && ld % m == 0 &&
+           (!lam || (ld_first % m == 0 && al(v_first, a))) && ld_kpage % m == 0 && ld_vpage % m == 0 &&
            al(qkv, a) && al(q_out, a) && al(k_pages, a) && al(v_pages, a) && (!qw || al(qw, 16)) && (!kw || al(kw, 16));
   };
   const bool walked = f32 ? fits(4, 16) && launch_rotary_walk<float, 4>(qkv, q_out, k_pages, v_pages, p, T, s)
@@ -1010,6 +1206,42 @@ EDL_HOST_API int edl_qkv_rotary_prologue(const void* qkv, int f32, long long ld,
   }
 #undef EDL_RP
   return check_cuda(cudaGetLastError(), "qkv_rotary_prologue launch");
+}
+
+// x [rows, W] <- x + rms_norm(y) * wb * ls (ls null: 1), h [rows, W] = rms_norm(x) * w in the operand type.
+EDL_HOST_API int edl_branch_norm(float* x, const float* y, const float* wb, const float* ls, float eps_b, const float* w,
+                                 float eps, void* h, int f32, int rows, int W, void* stream) {
+  if (rows <= 0) return 0;
+  cudaStream_t s = (cudaStream_t)stream;
+  const bool v4 = W % 4 == 0 && al(x, 16) && al(y, 16) && al(wb, 16) && (!ls || al(ls, 16)) && al(w, 16) && al(h, f32 ? 16 : 8);
+  if (f32) {
+    if (v4) launch_branch_norm<float, 4>(x, y, wb, ls, eps_b, w, eps, (float*)h, rows, W, s);
+    else launch_branch_norm<float, 1>(x, y, wb, ls, eps_b, w, eps, (float*)h, rows, W, s);
+  } else {
+    if (v4) launch_branch_norm<__nv_bfloat16, 4>(x, y, wb, ls, eps_b, w, eps, (__nv_bfloat16*)h, rows, W, s);
+    else launch_branch_norm<__nv_bfloat16, 1>(x, y, wb, ls, eps_b, w, eps, (__nv_bfloat16*)h, rows, W, s);
+  }
+  return check_cuda(cudaGetLastError(), "branch_norm launch");
+}
+
+// out [rows, F] = act(gu[:, :F]) * gu[:, F:], gu at pitch ld; act: 0 silu, 1 tanh form of gelu, 2 gelu, 3 relu.
+EDL_HOST_API int edl_gated_unit(const void* gu, int f32, long long ld, void* out, int rows, int F, int act, void* stream) {
+  if (rows <= 0) return 0;
+  if (act < ACT_SILU || act > ACT_RELU) {
+    set_last_error("edl_gated_unit: unknown activation %d", act);
+    return -1;
+  }
+  cudaStream_t s = (cudaStream_t)stream;
+  const bool v4 = F % 4 == 0 && ld % 4 == 0 && al(gu, f32 ? 16 : 8) && al(out, f32 ? 16 : 8);
+  const int blocks = blocks_for((long long)rows * (F / (v4 ? 4 : 1)), NT, 8);
+#define EDL_GU(TT, V_) gated_unit_kernel<TT, V_><<<blocks, NT, 0, s>>>((const TT*)gu, ld, (TT*)out, rows, F, act)
+  if (f32) {
+    if (v4) EDL_GU(float, 4); else EDL_GU(float, 1);
+  } else {
+    if (v4) EDL_GU(__nv_bfloat16, 4); else EDL_GU(__nv_bfloat16, 1);
+  }
+#undef EDL_GU
+  return check_cuda(cudaGetLastError(), "gated_unit launch");
 }
 
 // z <- cap * tanh(scale * z / cap), n elements in place (cap <= 0: scale * z).

@@ -38,12 +38,13 @@ class GroupManager:
         pages.clear()
 
     def remove_skipped(self, pages: list[int], num_computed_tokens: int) -> int:
-        """Gives back the pages that lie entirely in front of the first key any later query can read."""
+        """Gives back the pages that lie entirely in front of the first key any later query can read, but for those of kept
+        first tokens."""
         if not self.bounded:
             return 0
         upto = min(self.spec.first_useful_token(num_computed_tokens) // self.spec.page_size, len(pages))
         freed = []
-        for i in range(upto - 1, -1, -1):
+        for i in range(upto - 1, self.kept_pages - 1, -1):
             if pages[i] == NULL_PAGE:     # everything further left went in an earlier call
                 break
             freed.append(pages[i])
@@ -53,23 +54,36 @@ class GroupManager:
         return len(freed)
 
     # -- prefix cache
+    @property
+    def kept_pages(self) -> int:
+        """Pages at the start of a sequence that are never given back."""
+        return cdiv(self.spec.first_kept, self.spec.page_size)
+
     def window_start_page(self, num_pages_hit: int) -> int:
-        """First page a hit of ``num_pages_hit`` pages must still hold."""
+        """First page a hit of ``num_pages_hit`` pages must still hold (beside the kept ones)."""
         if not self.bounded:
             return 0
         return self.spec.first_useful_token(num_pages_hit * self.spec.page_size) // self.spec.page_size
 
+    def _needed(self, n: int) -> list[int]:
+        """Pages a hit of ``n`` pages must still hold."""
+        lo = self.window_start_page(n)
+        return [*range(min(lo, self.kept_pages)), *range(lo, n)]
+
     def holds(self, hashes: tp.Sequence[bytes], n: int) -> bool:
         cached = self.pool.cached
-        return all(hashes[i] in cached for i in range(self.window_start_page(n), n))
+        return all(hashes[i] in cached for i in self._needed(n))
 
     def take_cached(self, hashes: tp.Sequence[bytes], n: int) -> list[int]:
-        lo = self.window_start_page(n)
-        got = [self.pool.cached[hashes[i]] for i in range(lo, n)]
+        need = self._needed(n)
+        got = [self.pool.cached[hashes[i]] for i in need]
         self.pool.touch(got)
         self.pool.stats.queries += n
         self.pool.stats.hits += n
-        return [NULL_PAGE] * lo + got
+        pages = [NULL_PAGE] * n
+        for i, page in zip(need, got):
+            pages[i] = page
+        return pages
 
 
 class KVCacheCoordinator:

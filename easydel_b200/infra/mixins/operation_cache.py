@@ -47,6 +47,7 @@ class LayerOperationInfo:
     num_kv_heads: int = 0
     head_dim: int = 0
     v_head_dim: int = 0                   # 0 = values are as wide as keys
+    keep_first: int = 0                   # first tokens that stay visible under a sliding window
 
     @property
     def is_attention_layer(self) -> bool:
@@ -65,7 +66,7 @@ class LayerOperationInfo:
         if not self.requires_kv_cache:
             return 0
         if self.sliding_window:
-            return min(context, self.sliding_window)
+            return min(context, self.sliding_window + self.keep_first)
         if self.chunk_size:
             return min(context, self.chunk_size)
         return context
@@ -127,11 +128,11 @@ class OperationsCacheInfo:
             if not l.requires_kv_cache:
                 continue
             if l.sliding_window:
-                key = ("sliding", int(l.sliding_window))
+                key = ("sliding", int(l.sliding_window), int(l.keep_first))
             elif l.chunk_size:
-                key = ("chunked", int(l.chunk_size))
+                key = ("chunked", int(l.chunk_size), 0)
             else:
-                key = ("full", 0)
+                key = ("full", 0, 0)
             g = groups.setdefault(key, {"kind": key[0], "window": key[1], "layers": []})
             g["layers"].append(l.layer_index)
         return sorted(groups.values(), key=lambda g: (g["kind"] != "full", g["window"]))
@@ -218,15 +219,21 @@ def _describe_layer(i: int, layer) -> list[LayerOperationInfo]:
                                       CacheType.TRANSFORMER | CacheType.LATENT_PAGES | CacheType.HYBRID, True, False,
                                       getattr(attn, "sliding_window", None) or None, num_kv_heads=1, head_dim=width))
         return out
+    twin = getattr(layer, "mixer", None) if ltype == "twin" else None
+    if twin is not None:
+        attn = twin.left
     if attn is not None:
         window = getattr(attn, "sliding_window", None) or None
         chunk = getattr(attn, "chunk_size", None) or None
         kind = "sliding_attention" if window else ("chunked_attention" if chunk else "full_attention")
         out.append(LayerOperationInfo(i, kind, "flash_attention", "paged_decode_attention",
                                       0 if hasattr(layer, "mamba") or getattr(layer, "shift", None) is not None
-                                      else None, paged, True, False, window, chunk,
+                                      or twin is not None else None, paged, True, False, window, chunk,
                                       getattr(attn, "num_kv_heads", 0), getattr(attn, "head_dim", 0),
-                                      getattr(attn, "v_head_dim", 0)))
+                                      getattr(attn, "v_head_dim", 0), getattr(attn, "keep_first", 0)))
+    if twin is not None:
+        out.append(LayerOperationInfo(i, "linear_attention", "generalized_delta_rule", None, 1,
+                                      CacheType.RECURRENT | CacheType.HYBRID, False, True))
     if getattr(layer, "shift", None) is not None:         # the previous token's normalised row, per sequence
         out.append(LayerOperationInfo(i, "token_shift", "norm_shift", None, 1, CacheType.RECURRENT | CacheType.HYBRID,
                                       False, True))

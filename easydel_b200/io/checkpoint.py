@@ -236,6 +236,24 @@ def _read_safetensors(path: str) -> dict[str, torch.Tensor]:
     raise FileNotFoundError(f"no model weights found under {path}")
 
 
+def safetensors_shapes(path: str) -> dict[str, tuple[int, ...]]:
+    """Name -> shape of the tensors in a directory's safetensors files, from their headers alone (empty: none there)."""
+    names = [SAFETENSORS_NAME]
+    index = os.path.join(path, SAFETENSORS_INDEX_NAME)
+    if os.path.exists(index):
+        with open(index, encoding="utf-8") as f:
+            names = sorted(set(json.load(f)["weight_map"].values()))
+    out = {}
+    for fn in names:
+        full = os.path.join(path, fn)
+        if not os.path.exists(full):
+            continue
+        with open(full, "rb") as f:
+            head = json.loads(f.read(int.from_bytes(f.read(8), "little")))
+        out.update({k: tuple(v["shape"]) for k, v in head.items() if k != "__metadata__"})
+    return out
+
+
 def _resolve_dir(path: str) -> str:
     """A checkpoint directory, or a training directory whose newest ``run-*`` is used."""
     if os.path.exists(os.path.join(path, CONFIG_NAME)):
@@ -260,6 +278,8 @@ def load_config(path: str, config_kwargs: dict | None = None, **overrides):
         d.pop(k, None) if k != "architectures" else None
     arch = d.pop("architectures", None)
     cls = registry.get_config(mtype)
+    if hasattr(cls, "complete_from_shapes"):      # families whose configurations leave some sizes to the tensors
+        d = cls.complete_from_shapes(d, safetensors_shapes(path))
     cfg = cls(**d)
     cfg.architectures = arch
     kw = dict(config_kwargs or {})

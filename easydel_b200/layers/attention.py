@@ -62,8 +62,18 @@ class Attention(nn.Module):
                  output_gate: bool = False, chunk_size: int | None = None,
                  temp_tuning: tuple[float, float] | None = None, head_scale_init: float | None = None,
                  v_head_dim: int | None = None, norm_dtype: torch.dtype | None = None,
-                 stream_rope: dict | None = None):
+                 stream_rope: dict | None = None, keep_first: int = 0, score_bias: bool = False, head_gate: bool = False,
+                 value_mix: bool = False, projections: bool = True):
         super().__init__()
+        # forms of fp32-stream layers: the first keys stay visible under a window; no softmax but sigmoid(score + a number per
+        # head); a gate per head on the output; values blended with those of the first such layer; a layer whose projections
+        # belong to its owner (which hands rows to :meth:`mix_rows`)
+        self.keep_first = keep_first
+        self.score_bias = nn.Parameter(torch.zeros(num_heads, dtype=torch.float32)) if score_bias else None
+        self.head_gate = head_gate
+        self.value_mix = nn.Parameter(torch.zeros((), dtype=torch.float32)) if value_mix else None
+        if head_gate and (projections or not score_bias):
+            raise NotImplementedError("a gate per head goes with sigmoid weights and projections of the layer's owner")
         # GIDD: one learned multiplier per query head on top of ``scale`` (with L2-normalised q / k it is the whole
         # temperature of the head)
         self.head_scale = None if head_scale_init is None else nn.Parameter(
@@ -94,13 +104,12 @@ class Attention(nn.Module):
         self.clip_qkv = clip_qkv
         self.scale = scale if scale is not None else 1.0 / math.sqrt(head_dim)
         kv_heads = num_kv_heads if not self.kv_replicated else self.num_kv_heads * tp_size
-        self.qkv_proj = ColumnParallelLinear(hidden_size, (num_heads * head_dim * (2 if output_gate else 1),
-                                                           kv_heads * head_dim, kv_heads * self.v_head_dim), bias=bias,
-                                             dtype=dtype, init_std=init_std, tp_size=tp_size, tp_rank=tp_rank,
-                                             tp_group=tp_group)
-        self.o_proj = RowParallelLinear(num_heads * self.v_head_dim, hidden_size, bias=o_bias, dtype=dtype,
-                                        init_std=init_std, tp_size=tp_size, tp_rank=tp_rank, tp_group=tp_group)
-        self.qkv_proj.remat_name, self.o_proj.remat_name = "attn_qkv", "attn_output"
+        self.qkv_bias = None
+        if not projections:
+            if bias:
+                self.qkv_bias = nn.Parameter(torch.zeros(sum(self.in_splits[:3]), dtype=torch.float32))
+        else:
+            self._build_projections(hidden_size, kv_heads, bias, o_bias, dtype, init_std, tp_group)
         self.qk_norm, self.qk_norm_eps = qk_norm, qk_norm_eps
         if qk_norm == "rms_head":      # per-head RMSNorm over head_dim (Qwen3, Gemma3, OLMo... per-head flavour)
             self.q_norm = RMSNorm(head_dim, qk_norm_eps, norm_dtype or dtype, offset=qk_norm_offset)
@@ -122,13 +131,34 @@ class Attention(nn.Module):
         self.stream_rope = stream_rope
         self._freq: torch.Tensor | None = None
         if stream_rope is not None:
-            rotation.check_rotation(stream_rope["dims"], head_dim, "halves")
+            rotation.check_rotation(stream_rope["dims"], head_dim, stream_rope.get("layout", "halves"))
         self.sinks = nn.Parameter(torch.zeros(self.num_heads, dtype=torch.float32)) if use_sinks else None
         if use_alibi:
             sl = alibi_slopes(num_heads)[tp_rank * self.num_heads:(tp_rank + 1) * self.num_heads]
             self.register_buffer("alibi", sl, persistent=False)
         else:
             self.alibi = None
+
+    def _build_projections(self, hidden_size, kv_heads, bias, o_bias, dtype, init_std, tp_group):
+        num_heads, head_dim = self.num_heads_global, self.head_dim
+        tp_size, tp_rank = self.tp_size, self.tp_rank
+        self.qkv_proj = ColumnParallelLinear(hidden_size, (num_heads * head_dim * (2 if self.output_gate else 1),
+                                                           kv_heads * head_dim, kv_heads * self.v_head_dim), bias=bias,
+                                             dtype=dtype, init_std=init_std, tp_size=tp_size, tp_rank=tp_rank,
+                                             tp_group=tp_group)
+        self.o_proj = RowParallelLinear(num_heads * self.v_head_dim, hidden_size, bias=o_bias, dtype=dtype,
+                                        init_std=init_std, tp_size=tp_size, tp_rank=tp_rank, tp_group=tp_group)
+        self.qkv_proj.remat_name, self.o_proj.remat_name = "attn_qkv", "attn_output"
+
+    @property
+    def in_splits(self) -> tuple[int, ...]:
+        """Widths of queries, keys, values and the gates per head."""
+        return (self.num_heads * self.head_dim, self.num_kv_heads * self.head_dim, self.num_kv_heads * self.v_head_dim,
+                self.num_heads if self.head_gate else 0)
+
+    @property
+    def out_width(self) -> int:
+        return self.num_heads * self.v_head_dim
 
     # ------------------------------------------------------------------
     #: set by the decoder when the sequence is sharded over the ``sp`` mesh axis (``attn_mechanism="ring"``)
@@ -225,42 +255,73 @@ class Attention(nn.Module):
 
     def mix_stream(self, h: torch.Tensor, step, cache_view=None) -> torch.Tensor:
         """Form for layers over an fp32 residual stream: h ``[T, hidden]`` (all sequences on one axis) ->
-        ``[T, heads * v_head_dim]`` before the output projection, which the layer accumulates into the stream. One kernel
-        over the packed projection does per-head q / k norms, the query temperature and the page append, or norms over the
-        whole projection, the rotation and the page append. ``step``: :class:`..modules._base.decoder.StreamStep`."""
-        turned = self.stream_rope is not None or self.qk_norm == "rms_full"
+        ``[T, heads * v_head_dim]`` before the output projection, which the layer accumulates into the stream."""
+        return self.mix_rows(stream.linear(h, self.qkv_proj.weight, self.qkv_proj.bias), step, cache_view)
+
+    def mix_rows(self, qkv: torch.Tensor, step, cache_view=None, gate: torch.Tensor | None = None,
+                 out: torch.Tensor | None = None, out_scale: float = 1.0) -> torch.Tensor:
+        """:meth:`mix_stream` from the projected rows ``qkv [T, q | k | v]`` (which may be columns of wider rows). One kernel
+        does per-head q / k norms, the query temperature and the page append, or biases, norms over the whole projection, the
+        rotation, the blend of the values and the page append. ``step``: :class:`..modules._base.decoder.StreamStep`.
+        ``gate [T, heads]``, ``out_scale``: factors of the output (sigmoid weights); ``out``: where to write."""
+        turned = self.stream_rope is not None or self.qk_norm == "rms_full" or self.qkv_bias is not None or \
+            self.value_mix is not None
         if self.rotary is not None or self.alibi is not None or self.output_gate or self.clip_qkv is not None or \
                 self.head_scale is not None or self.chunk_size or self.qk_norm not in (None, "rms_head", "rms_full") or \
                 (turned and (self.qk_norm == "rms_head" or self.temp_tuning is not None)):
             raise NotImplementedError("fp32-stream attention covers plain, per-head-normed and tempered heads, or heads "
                                       "rotated after a norm over the whole projection")
-        qkv = stream.linear(h, self.qkv_proj.weight, self.qkv_proj.bias)
-        T = h.shape[0]
-        Hq, Hkv, D, Dv = self.num_heads, self.num_kv_heads, self.head_dim, self.v_head_dim
+        from ..ops import serving as S
+
+        sigmoid = None if self.score_bias is None else S.SigmoidWeights(self.score_bias, gate, out_scale)
+        if sigmoid is None and (gate is not None or out_scale != 1.0):
+            raise NotImplementedError("gates and factors of the output go with sigmoid weights")
+        T = qkv.shape[0]
+        Hq, Hkv, D, Dv = heads = self.num_heads, self.num_kv_heads, self.head_dim, self.v_head_dim
         qw, kw = (self.q_norm.weight, self.k_norm.weight) if self.qk_norm else (None, None)
-        freq = self._frequencies(qkv.device) if turned else None
-        if cache_view is not None and turned:
-            q = stream.qkv_rotary_prologue(qkv, (Hq, Hkv, D, Dv), qw, kw, self.qk_norm_eps, step.positions, freq,
-                                           step.meta.slots_of(cache_view.group), cache_view.k_pages, cache_view.v_pages)
-            return cache_view.attend_pages(self, q, step.meta).reshape(T, Hq * Dv)
+        if turned:
+            r = self.stream_rope or {}
+            kw_args = dict(layout=r.get("layout", "halves"), mag=rotation.magnitude(r.get("scaling")), bias=self.qkv_bias,
+                           **self._blend(qkv, step))
+            freq = self._frequencies(qkv.device)
         if cache_view is not None:
-            q = stream.qkv_prologue(qkv, (Hq, Hkv, D, Dv), qw, kw, self.qk_norm_eps, step.positions, self.temp_tuning,
-                                    step.meta.slots_of(cache_view.group), cache_view.k_pages, cache_view.v_pages)
-            return cache_view.attend_pages(self, q, step.meta).reshape(T, Hq * Dv)
+            pages = (step.meta.slots_of(cache_view.group), cache_view.k_pages, cache_view.v_pages)
+            if turned:
+                q = stream.qkv_rotary_prologue(qkv, heads, qw, kw, self.qk_norm_eps, step.positions, freq, *pages, **kw_args)
+            else:
+                q = stream.qkv_prologue(qkv, heads, qw, kw, self.qk_norm_eps, step.positions, self.temp_tuning, *pages)
+            o = None if out is None else out.unflatten(1, (Hq, Dv))
+            return cache_view.attend_pages(self, q, step.meta, sigmoid=sigmoid, out=o).reshape(T, Hq * Dv)
         # no cache (autograd): the batch's rows are equally long
         from ..ops import reference as R
 
-        q, k, v = torch.split(qkv, [Hq * D, Hkv * D, Hkv * Dv], -1)
         if turned:
-            q, k = stream.qk_norm_rotate(q, k, D, qw, kw, self.qk_norm_eps, step.positions, freq)
+            q, k, v = stream.rotary_rows(qkv, heads, qw, kw, self.qk_norm_eps, step.positions, freq, **kw_args)
         else:
+            q, k, v = torch.split(qkv, [Hq * D, Hkv * D, Hkv * Dv], -1)
             q, k = stream.qk_norm_temper(q.reshape(T, Hq, D), k.reshape(T, Hkv, D), qw, kw, self.qk_norm_eps,
                                          step.positions, self.temp_tuning)
         B = step.batch
         o = R.attention(q.view(B, T // B, Hq, D), k.view(B, T // B, Hkv, D), v.reshape(B, T // B, Hkv, Dv),
                         causal=self.causal, scale=self.scale, segment_ids=step.segment_ids,
-                        sliding_window=self.sliding_window, softcap=self.softcap, sinks=self.sinks)
-        return o.reshape(T, Hq * Dv)
+                        sliding_window=self.sliding_window, softcap=self.softcap, sinks=self.sinks,
+                        keep_first=self.keep_first, score_bias=self.score_bias).reshape(T, Hq, Dv)
+        return (o if sigmoid is None else sigmoid.finish(o)).reshape(T, Hq * Dv)
+
+    def _blend(self, qkv: torch.Tensor, step) -> dict:
+        """Blend of the values with the first such layer's of the same tokens; that layer leaves its values in ``step``."""
+        if self.value_mix is None:
+            return {}
+        if self.qkv_bias is not None:
+            raise NotImplementedError("blended values have no biases")
+        n = (self.num_heads + self.num_kv_heads) * self.head_dim
+        values = qkv[:, n:n + self.num_kv_heads * self.v_head_dim]
+        if step.first_values is None:
+            step.first_values = values
+            return {}
+        if step.first_values.shape != values.shape:
+            raise ValueError(f"values of width {values.shape[1]} cannot blend with the first layer's {step.first_values.shape[1]}")
+        return {"first": step.first_values, "lam": self.value_mix}
 
     def _frequencies(self, device) -> torch.Tensor | None:
         r = self.stream_rope

@@ -44,6 +44,8 @@ from . import disunex  # noqa: F401
 from .disunex import *  # noqa: F401,F403
 from . import gasetar  # noqa: F401
 from .gasetar import *  # noqa: F401,F403
+from . import ninisun  # noqa: F401
+from .ninisun import *  # noqa: F401,F403
 from . import rakevik  # noqa: F401
 from .rakevik import *  # noqa: F401,F403
 

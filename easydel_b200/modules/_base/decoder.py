@@ -102,7 +102,8 @@ class ArchSpec:
     residual: str = "pre"             # pre | parallel (x + mixer(h) + mlp(h), h = norm(x); fp32-stream models too) |
                                       # post (norm applied to the branch output, OLMo2) | post_sum
                                       # (x <- norm(residual_alpha x + branch), branches read x; fp32-stream models)
-    sandwich_norm: bool = False       # extra norms after attention / MLP outputs (Gemma2/3)
+    sandwich_norm: bool = False       # extra norms after attention / MLP outputs (Gemma2/3; fp32-stream models too)
+    layer_scale: bool = False         # a factor per channel on every normed branch (fp32-stream models with sandwich_norm)
     shared_parallel_norm: bool = True  # parallel residual with one norm (GPT-J, Phi) vs two (NeoX)
     use_sinks: bool = False
     moe: MoESpec | None = None
@@ -133,7 +134,13 @@ class ArchSpec:
     branch_multipliers: tuple[float, float, float] = (1.0, 1.0, 1.0)  # attention input, attention output, SSM output
     mlp_multipliers: tuple[float, float] = (1.0, 1.0)                  # gate pre-activation, MLP output
     residual_f32: bool = False        # the residual stream is fp32 [tokens, hidden]; branches accumulate into it
-    stream_rope: dict | None = None   # base / dims / scaling of rotated halves in fp32-stream attention layers, see ops.rotation
+    stream_rope: dict | None = None   # base / dims / scaling / layout of rotated pairs in fp32-stream attention layers, see
+                                      # ops.rotation
+    keep_first: int = 0               # keys that stay visible when a sliding window has moved past them (fp32-stream models)
+    value_mix: bool = False           # values blend with those of the first such layer (fp32-stream models)
+    attn_score_bias: bool = False     # no softmax: weights are sigmoid(score + a number per head) (fp32-stream models)
+    twin: dict | None = None          # layers of type "twin" (fp32-stream models): attention beside a generalised delta rule;
+                                      # "delta" (heads / dim / rank of layers.delta_rule), "scales" of the two sides
     token_shift: bool = False         # every mixer reads h + (h of the previous token - h) * shift (fp32-stream models)
     v_head_dim: int | None = None     # width of a value head when it differs from head_dim (fp32-stream models)
     hgrn2: dict | None = None         # heads / dim / vdim of layers.hgrn2.HGRN2Mixer for layers of type "hgrn2"
@@ -157,6 +164,7 @@ class StreamStep:
     slots: torch.Tensor | None = None     # int32 [B] state rows of the sequences
     meta: tp.Any = None                   # PagedBatchMeta, with a paged cache
     segment_ids: torch.Tensor | None = None
+    first_values: torch.Tensor | None = None   # values [T, heads * width] of the first layer that blends values
 
 
 @dataclass
@@ -164,7 +172,7 @@ class LayerSlotState:
     """Per-slot state of one layer run of an fp32-stream model, read and written in place by its kernels."""
 
     shift: torch.Tensor | None            # fp32 [slots, hidden]: the previous token's normalised row
-    recurrent: torch.Tensor | None        # fp32 [slots, heads, dim, vdim]: HGRN2
+    recurrent: torch.Tensor | None        # fp32 [slots, heads, dim, vdim]: HGRN2, generalised delta rule
     in_place: tp.ClassVar[bool] = True
 
 
@@ -240,6 +248,8 @@ class DecoderLayer(nn.Module):
 
             self.linear_attn = GatedDeltaNet(spec.hidden_size, layer_idx=layer_idx, dtype=dtype,
                                              init_std=spec.init_std, norm_eps=spec.norm_eps, **spec.linear_attn)
+        elif ltype == "twin":
+            self.mixer = self._twin(spec, layer_idx, dtype)
         elif spec.mla is not None and spec.residual_f32:
             from ...layers.mla import LatentStreamAttention
 
@@ -273,8 +283,17 @@ class DecoderLayer(nn.Module):
             if not self.is_moe:
                 (self.mlp.down_proj if hasattr(self.mlp, "down_proj") else self.mlp.fc2).defer_reduce = True
 
+    @classmethod
+    def _twin(cls, spec, layer_idx, dtype):
+        from ...layers.delta_rule import GeneralizedDeltaMixer
+        from ...layers.twin import TwinMixer
+
+        left = cls._mha(spec, layer_idx, dtype, None, None, 1, 0, None, head_gate=True, projections=False)
+        right = GeneralizedDeltaMixer(norm_eps=spec.norm_eps, dtype=dtype, init_std=spec.init_std, **spec.twin["delta"])
+        return TwinMixer(spec.hidden_size, left, right, spec.twin["scales"], dtype, spec.init_std)
+
     @staticmethod
-    def _mha(spec, layer_idx, dtype, rope, window, tp_size, tp_rank, tp_group):
+    def _mha(spec, layer_idx, dtype, rope, window, tp_size, tp_rank, tp_group, **kw):
         qk_norm = spec.qk_norm if (rope is not None or not spec.qk_norm_rope_only) else None
         return Attention(
             spec.hidden_size, spec.num_heads, spec.num_kv_heads, spec.head_dim, layer_idx=layer_idx,
@@ -287,7 +306,8 @@ class DecoderLayer(nn.Module):
             use_alibi=spec.pos_emb == "alibi", clip_qkv=spec.clip_qkv, dtype=dtype, init_std=spec.init_std,
             tp_size=tp_size, tp_rank=tp_rank, tp_group=tp_group, qk_norm_offset=spec.norm_offset,
             output_gate=spec.attn_output_gate, v_head_dim=spec.v_head_dim,
-            norm_dtype=torch.float32 if spec.residual_f32 else None, stream_rope=spec.stream_rope)
+            norm_dtype=torch.float32 if spec.residual_f32 else None, stream_rope=spec.stream_rope,
+            keep_first=spec.keep_first if window else 0, score_bias=spec.attn_score_bias, value_mix=spec.value_mix, **kw)
 
     def _build_mlp(self, config, spec, layer_idx, dtype, tp_size, tp_rank, tp_group):
         moe = spec.moe
@@ -333,13 +353,21 @@ class DecoderLayer(nn.Module):
             self.post_feedforward_layernorm = _norm(spec, dtype)
         else:
             self.input_layernorm = _norm(spec, dtype)
+            if spec.residual_f32 and spec.sandwich_norm:
+                if spec.norm_offset or spec.residual_multiplier is not None or spec.residual != "pre" or spec.token_shift:
+                    raise NotImplementedError("normed branches on an fp32 stream: plain pre-norm layers")
+                self.post_attn_out_layernorm = _norm(spec, dtype)
+                scale = lambda: nn.Parameter(torch.ones(spec.hidden_size, dtype=torch.float32))  # noqa: E731
+                self.mixer_scale = scale() if spec.layer_scale else None
+                self.mlp_scale = scale() if spec.layer_scale and self.mlp is not None else None
             if self.mlp is None:
                 return
             if (spec.residual == "pre" and not spec.sandwich_norm) or \
                     (spec.residual == "parallel" and not spec.shared_parallel_norm):
                 self.post_attention_layernorm = _norm(spec, dtype)
             if spec.sandwich_norm:
-                self.post_attn_out_layernorm = _norm(spec, dtype)
+                if not spec.residual_f32:
+                    self.post_attn_out_layernorm = _norm(spec, dtype)
                 self.pre_feedforward_layernorm = _norm(spec, dtype)
                 self.post_feedforward_layernorm = _norm(spec, dtype)
 
@@ -368,15 +396,17 @@ class DecoderLayer(nn.Module):
     def make_slot_state(self, num_slots: int, device) -> LayerSlotState | None:
         """State pool of this layer for ``num_slots`` sequences (fp32-stream models; None for the others)."""
         spec = self.spec
-        if not spec.residual_f32 or (self.shift is None and self.ltype != "hgrn2"):
+        if not spec.residual_f32 or (self.shift is None and self.ltype not in ("hgrn2", "twin")):
             return None
         zeros = lambda *s: torch.zeros(num_slots, *s, dtype=torch.float32, device=device)  # noqa: E731
-        m = self.linear_attn if self.ltype == "hgrn2" else None
+        m = self.linear_attn if self.ltype == "hgrn2" else self.mixer.right if self.ltype == "twin" else None
         return LayerSlotState(zeros(spec.hidden_size) if self.shift is not None else None,
                               zeros(m.heads, m.dim, m.vdim) if m is not None else None)
 
     @property
     def _stream_mixer(self) -> nn.Module:
+        if self.ltype == "twin":
+            return self.mixer
         return self.linear_attn if self.ltype == "hgrn2" else self.self_attn
 
     def _mix_stream(self, h: torch.Tensor, step: StreamStep, view) -> torch.Tensor:
@@ -384,6 +414,9 @@ class DecoderLayer(nn.Module):
         if self.ltype == "hgrn2":
             state = view.linear_state if view is not None else None
             return self.linear_attn(h, step, None if state is None else state.recurrent)
+        if self.ltype == "twin":
+            state = view.linear_state if view is not None else None
+            return self.mixer.mix_stream(h, step, view, None if state is None else state.recurrent)
         return self.self_attn.mix_stream(h, step, view)
 
     def _forward_stream(self, x: torch.Tensor, step: StreamStep, view):
@@ -415,6 +448,21 @@ class DecoderLayer(nn.Module):
             x, h = stream.post_norm(x, branch, spec.residual_alpha, n2.weight, spec.norm_eps, h.dtype, n2.offset)
         return x, h
 
+    def _forward_sandwich_stream(self, x: torch.Tensor, pending, step: StreamStep, view):
+        """One layer on the fp32 stream ``x [T, hidden]`` whose branches are normed (and scaled per channel) before they join
+        it. ``pending`` is the last branch of the layer before: norm, sum and the norm that reads the sum are one pass.
+        Returns the stream and this layer's own pending branch."""
+        spec, n1, mixer = self.spec, self.input_layernorm, self._stream_mixer
+        dt = mixer.o_proj.weight.dtype
+        x, h = stream.add_norm(x, pending, 1.0, n1.weight, spec.norm_eps, dt)
+        rows = stream.branch_product(self._mix_stream(h, step, view), mixer.o_proj.weight)
+        pending = stream.NormedBranch(rows, self.post_attn_out_layernorm.weight, spec.norm_eps, self.mixer_scale)
+        if self.mlp is not None:
+            x, h = stream.add_norm(x, pending, 1.0, self.pre_feedforward_layernorm.weight, spec.norm_eps, dt)
+            pending = stream.NormedBranch(self.mlp.stream_rows(h), self.post_feedforward_layernorm.weight, spec.norm_eps,
+                                          self.mlp_scale)
+        return x, pending
+
     def _forward_parallel_stream(self, x: torch.Tensor, pending, step: StreamStep, view):
         """One layer on the fp32 stream ``x [T, hidden]`` whose branches both read one norm of it. ``pending`` is what the
         layer before adds to the stream (None: nothing), times the residual multiplier: that sum and this layer's norm are
@@ -431,6 +479,8 @@ class DecoderLayer(nn.Module):
             return *self._forward_parallel_stream(x, pending, attn_meta, cache_view), None
         if spec.residual == "post_sum":
             return *self._forward_post_sum(x, pending, attn_meta, cache_view), None
+        if spec.residual_f32 and spec.sandwich_norm:
+            return *self._forward_sandwich_stream(x, pending, attn_meta, cache_view), None
         if spec.residual_f32:
             return self._forward_stream(x, attn_meta, cache_view), None, None
         rl = None
@@ -738,9 +788,10 @@ def _forward_stream(self, input_ids, inputs_embeds, attention_mask, position_ids
         flat = flat[index]
     n = flat.numel() if flat is not None else (index.numel() if index is not None else B * T)
     operand = right = None
-    # "post_sum" layers: the stream's rows in the operand type; "parallel" layers: what the last one adds to the stream
+    # "post_sum" layers: the stream's rows in the operand type; "parallel" layers and those with normed branches: what the last
+    # one adds to the stream
     h = None
-    parallel, mult = spec.residual == "parallel", _residual_multiplier(spec)
+    pends, mult = spec.residual == "parallel" or spec.sandwich_norm, _residual_multiplier(spec)
     if spec.residual == "post_sum":
         right = h = torch.empty(n, W, dtype=self.embed_tokens.weight.dtype, device=self.device)
     if spec.loop is not None:             # [x ; x0]: x0 is written once, x before every pass
@@ -768,10 +819,10 @@ def _forward_stream(self, input_ids, inputs_embeds, attention_mask, position_ids
                 x = stream.linear(operand, self.loop_in.weight, bias, torch.float32)
             done += 1
         if hidden is not None:
-            hidden.append(x + mult * stream.branch_rows(h) if parallel and h is not None else x.clone())
+            hidden.append(x + mult * stream.branch_rows(h) if pends and h is not None else x.clone())
         view = cache.view(run) if cache is not None else None
         x, h, _ = self.layers[i](x, h, step.positions, None, view, step)
-    x = stream.add_norm(x, h if parallel else None, mult, self.norm.weight, spec.norm_eps, dt, self.norm.offset)[1]
+    x = stream.add_norm(x, h if pends else None, mult, self.norm.weight, spec.norm_eps, dt, self.norm.offset)[1]
 
     def unflatten(t):
         if index is not None:

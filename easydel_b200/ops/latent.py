@@ -142,7 +142,7 @@ def attend(attn, proj: torch.Tensor, pages: torch.Tensor, meta, table: torch.Ten
         _lib.call("edl_attn_paged", proj.data_ptr(), kv.data_ptr(), kv.data_ptr() + 2 * k_width, o.data_ptr(),
                   proj.stride(0), kv.stride(0), kv.stride(0), H * V, meta.cu_q.data_ptr() + 4 * single,
                   meta.kv_lens.data_ptr() + 4 * single, compact.data_ptr(), compact.stride(0), B - single,
-                  int(meta.max_q), T, n_pages, H, H, D + R, V, float(attn.scale), 1, window, 0.0, _lib.ptr(attn.sinks),
+                  int(meta.max_q), T, n_pages, H, H, D + R, V, float(attn.scale), 1, window, 0, 0.0, _lib.ptr(attn.sinks),
                   _lib.status_word(proj.device).data_ptr(), _lib.stream_ptr())
         finish(o[rows], rows)
     return out

@@ -97,7 +97,7 @@ def apply_rope(x, pos, cos_table, sin_table, rot_dim=None, interleaved: bool = F
 
 def attention(q, k, v, *, causal: bool = True, scale: float | None = None, segment_ids=None, q_offset=None,
               sliding_window: int | None = None, softcap: float = 0.0, sinks=None, bias=None, kv_segment_ids=None,
-              return_lse: bool = False):
+              return_lse: bool = False, keep_first: int = 0, score_bias=None):
     """Dense softmax attention, the oracle for the flash kernels.
 
     q: [B, Tq, Hq, D]; k, v: [B, Tk, Hkv, D]. GQA by repeating KV heads.
@@ -105,6 +105,8 @@ def attention(q, k, v, *, causal: bool = True, scale: float | None = None, segme
     ``q_offset`` [B] or int: absolute position of q row 0 relative to k row 0
     (default Tk - Tq, i.e. the queries are the last Tq positions).
     ``sinks`` [Hq]: per-head extra logit that joins the softmax but carries no value.
+    ``keep_first``: the first keys stay visible when a sliding window has moved past them.
+    ``score_bias`` [Hq]: no softmax; a visible key's weight is ``sigmoid(score + score_bias)``, not normalised over keys.
     """
     B, Tq, Hq, D = q.shape
     Tk, Hkv = k.shape[1], k.shape[2]
@@ -127,11 +129,14 @@ def attention(q, k, v, *, causal: bool = True, scale: float | None = None, segme
     if causal:
         mask &= kpos[:, None, :] <= qpos[:, :, None]
     if sliding_window is not None and sliding_window > 0:
-        mask &= kpos[:, None, :] > (qpos[:, :, None] - sliding_window)
+        mask &= (kpos[:, None, :] > (qpos[:, :, None] - sliding_window)) | (kpos[:, None, :] < keep_first)
     if segment_ids is not None:
         ks = kv_segment_ids if kv_segment_ids is not None else segment_ids
         mask &= (segment_ids[:, :, None] == ks[:, None, :]) & (ks[:, None, :] != 0)
     s = s.masked_fill(~mask[:, None], float("-inf"))
+    if score_bias is not None:
+        p = torch.sigmoid(s + score_bias.float().view(1, Hq, 1, 1))      # masked scores are -inf: weight 0
+        return torch.matmul(p, vf).permute(0, 2, 1, 3).to(q.dtype)
     if sinks is not None:
         sk = sinks.float().view(1, Hq, 1, 1).expand(B, Hq, Tq, 1)
         s_all = torch.cat([s, sk], dim=-1)

@@ -24,22 +24,43 @@ def llama3_scaling(f: torch.Tensor, factor: float, low: float, high: float, orig
     return torch.where(between, (1 - s) * f / factor + s * f, out)
 
 
+def yarn_scaling(f: torch.Tensor, base: float, dims: int, factor: float, original: float, fast: float,
+                 slow: float) -> torch.Tensor:
+    """YaRN's frequency scaling: pairs that turn at least ``fast`` times within ``original`` positions stay, those that turn
+    at most ``slow`` times are slowed down by ``factor``, with a linear ramp over the pair index in between. In ``f``'s type."""
+    def index_of(turns):
+        return dims * math.log(original / (2 * math.pi * turns)) / (2 * math.log(base))
+
+    lo, hi = max(math.floor(index_of(fast)), 0), min(math.ceil(index_of(slow)), dims - 1)
+    ramp = ((torch.arange(f.numel(), dtype=f.dtype) - lo) / max(hi - lo, 0.001)).clamp(0, 1)
+    return f / factor * ramp + f * (1 - ramp)
+
+
+def magnitude(scaling: dict | None) -> float:
+    """Factor of cosines and sines: ``0.1 ln(factor) + 1`` under :func:`yarn_scaling`, else 1."""
+    return 0.1 * math.log(float(scaling["factor"])) + 1.0 if scaling and "fast" in scaling else 1.0
+
+
 def pair_frequencies(base: float, dims: int, device=None, scaling: dict | None = None) -> torch.Tensor:
     """``base^(-2i / dims)`` for i < dims / 2, as leading parts and remainders. ``scaling``: the ``factor``, ``low``,
-    ``high`` and ``original`` of :func:`llama3_scaling`."""
+    ``high`` and ``original`` of :func:`llama3_scaling`, or the ``factor``, ``original``, ``fast`` and ``slow`` of
+    :func:`yarn_scaling`."""
     f = float(base) ** (-torch.arange(0, dims, 2, dtype=torch.float64) / dims)
-    if scaling:
+    if scaling and "fast" in scaling:
+        f = yarn_scaling(f, float(base), dims, *(float(scaling[k]) for k in ("factor", "original", "fast", "slow")))
+    elif scaling:
         f = llama3_scaling(f, *(float(scaling[k]) for k in ("factor", "low", "high", "original")))
     hi = f.float()
     return torch.cat([hi, (f - hi.double()).float()]).to(device)
 
 
-def rotate(x: torch.Tensor, positions: torch.Tensor, freq: torch.Tensor, layout: str = "neighbours") -> torch.Tensor:
+def rotate(x: torch.Tensor, positions: torch.Tensor, freq: torch.Tensor, layout: str = "neighbours",
+           mag: float = 1.0) -> torch.Tensor:
     """Tensor form: the pairs of the first ``2 * pairs`` elements of ``x [T, ..., R]`` turned by ``position *
-    frequency``; computed in fp32, cast back."""
+    frequency`` and scaled by ``mag``; computed in fp32, cast back."""
     n = freq.numel() // 2
     a = positions.double()[:, None] * (freq[:n].double() + freq[n:].double())
-    c, s = torch.cos(a).float(), torch.sin(a).float()
+    c, s = (torch.cos(a) * mag).float(), (torch.sin(a) * mag).float()
     c, s = (t.view(t.shape[0], *[1] * (x.dim() - 2), n) for t in (c, s))
     if layout == "halves":
         u, v = x[..., :n].float(), x[..., n:2 * n].float()

@@ -3,6 +3,7 @@
 from __future__ import annotations
 
 import math
+from dataclasses import dataclass
 
 import torch
 
@@ -13,17 +14,40 @@ _lib.register("edl_attn_paged_lse", i32, [vp, vp, vp, vp, vp, i64, i64, i64, i64
                                           i32, i32, i32, i32, _lib.f32, i32, i32, _lib.f32, vp, vp, vp])
 _lib.register("edl_attn_combine", i32, [vp, i64, vp, i32, i32, i32, i32, vp, vp, vp, vp])
 _lib.register("edl_attn_paged", i32, [vp, vp, vp, vp, i64, i64, i64, i64, vp, vp, vp, i32, i32, i32, i64, i64, i32, i32,
-                                      i32, i32, f32, i32, i32, f32, vp, vp, vp])
+                                      i32, i32, f32, i32, i32, i32, f32, vp, vp, vp])
+_lib.register("edl_attn_paged_sigmoid", i32, [vp, vp, vp, vp, i64, i64, i64, i64, vp, vp, vp, i32, i32, i32, i64, i64, i32, i32,
+                                              i32, i32, f32, i32, i32, vp, vp, i64, f32, vp, vp])
 _lib.register("edl_paged_kv_append", i32, [vp, vp, vp, vp, vp, i32, i32, i64, i64, i64, i64, vp, vp])
 _lib.register("edl_sample", i32, [vp, i32, i64, i32, i32, vp, vp, vp, vp, vp, vp, vp, vp, i64, vp, vp, vp, vp, vp])
 _lib.register("edl_count_update", i32, [vp, i64, vp, vp, i32, i32, vp])
 _lib.register("edl_gather_rows", i32, [vp, vp, vp, i32, i32, i64, vp])
 _lib.register("edl_attn_decode", i32, [vp, vp, vp, vp, vp, i64, i64, i64, i64, vp, vp, i32, i32, i64, i32, i32, i32, i32,
                                        f32,
-                                       i32, i32, f32, vp, vp, vp])
-
+                                       i32, i32, i32, f32, vp, vp, vp])
+_lib.register("edl_attn_decode_sigmoid", i32, [vp, vp, vp, vp, vp, i64, i64, i64, i64, vp, vp, i32, i32, i64, i32, i32, i32, i32,
+                                               f32, i32, i32, i32, vp, vp, i64, f32, vp, vp])
 _lib.register("edl_attn_mla_decode", i32, [vp, i64, i64, vp, i64, i64, vp, vp, vp, i64, vp, vp, i32, i32, i64, i32, i32, i32,
                                             f32, i32, vp, i32, vp, vp])
+
+@dataclass
+class SigmoidWeights:
+    """Attention without a softmax: a visible key's weight is ``sigmoid(score + bias[h])``, not normalised over keys; head h's
+    output is multiplied by ``out_scale`` and, with a ``gate [T, H]`` (rows may be strided), by ``sigmoid(gate[t, h])``."""
+
+    bias: torch.Tensor                    # fp32 [H]
+    gate: torch.Tensor | None = None
+    out_scale: float = 1.0
+
+    def args(self) -> tuple:
+        g = self.gate
+        assert self.bias.dtype == torch.float32 and (g is None or g.stride(1) == 1)
+        return _lib.ptr(self.bias), _lib.ptr(g), g.stride(0) if g is not None else 0, float(self.out_scale)
+
+    def finish(self, o: torch.Tensor) -> torch.Tensor:
+        """Tensor form of the last step: ``o [T, H, Dv]`` scaled and gated."""
+        f = self.out_scale if self.gate is None else torch.sigmoid(self.gate.float())[..., None] * self.out_scale
+        return (o.float() * f).to(o.dtype)
+
 
 PAGE_SIZE = 128
 MAX_QK_DIM = 192      # widest query / key head of the tensor-core prefill kernel
@@ -53,13 +77,15 @@ def kv_append(k: torch.Tensor, v: torch.Tensor, k_pages: torch.Tensor, v_pages: 
 def paged_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, cu_q: torch.Tensor,
                     kv_lens: torch.Tensor, page_table: torch.Tensor, max_q: int, *, scale: float | None = None,
                     causal: bool = True, window: int = 0, softcap: float = 0.0, sinks=None,
-                    out: torch.Tensor | None = None) -> torch.Tensor:
+                    out: torch.Tensor | None = None, keep_first: int = 0,
+                    sigmoid: SigmoidWeights | None = None) -> torch.Tensor:
     """Mixed prefill/decode attention over a paged KV cache.
 
     q ``[T, Hq, D]`` (new tokens of all sequences, concatenated), key pages ``[P, 128, Hkv, D]``, value pages
     ``[P, 128, Hkv, Dv]`` (``Dv`` may differ from ``D``), ``cu_q`` int32 ``[B+1]``, ``kv_lens`` int32 ``[B]`` (cached +
     new keys), ``page_table`` int32 ``[B, maxP]``. Layouts outside :func:`paged_kernel_supports` (32-bit floats,
-    heads wider than 128) run the plain SIMT kernel.
+    heads wider than 128) run the plain SIMT kernel. ``keep_first``: keys that stay visible when ``window`` has moved past
+    them; ``sigmoid``: weights without a softmax; ``out [T, Hq, Dv]`` may have a row pitch of its own.
     """
     T, Hq, D = q.shape
     Hkv, Dv = k_pages.shape[2], v_pages.shape[-1]
@@ -69,29 +95,40 @@ def paged_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tenso
         if not causal:
             raise NotImplementedError("the SIMT attention kernel is causal")
         return simt_attention(q, k_pages, v_pages, cu_q, kv_lens, page_table, scale=scale, window=window, sinks=sinks,
-                              out=out, softcap=softcap)
+                              out=out, softcap=softcap, keep_first=keep_first, sigmoid=sigmoid)
     if q.is_cuda:
         assert k_pages.shape[1] == PAGE_SIZE, "the paged kernels use pages of 128 tokens"
         assert q.stride(-1) == 1 and q.stride(-2) == D
         if out is None:
             out = torch.empty((T, Hq, Dv), dtype=q.dtype, device=q.device)
+        if sigmoid is not None:
+            assert causal and not softcap and sinks is None
+            _lib.call("edl_attn_paged_sigmoid", q.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), out.data_ptr(),
+                      q.stride(0), k_pages.stride(1), v_pages.stride(1), out.stride(0), cu_q.data_ptr(),
+                      kv_lens.data_ptr(), page_table.data_ptr(), page_table.stride(0), B, int(max_q), T, k_pages.shape[0],
+                      Hq, Hkv, D, Dv, float(scale), int(window or 0), int(keep_first), *sigmoid.args(),
+                      _lib.status_word(q.device).data_ptr(), _lib.stream_ptr())
+            return out
         _lib.call("edl_attn_paged", q.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), out.data_ptr(),
                   q.stride(0), k_pages.stride(1), v_pages.stride(1), out.stride(0), cu_q.data_ptr(),
                   kv_lens.data_ptr(), page_table.data_ptr(), page_table.stride(0), B, int(max_q), T, k_pages.shape[0],
-                  Hq, Hkv, D, Dv, float(scale), int(causal), int(window or 0), float(softcap or 0.0), _lib.ptr(sinks),
+                  Hq, Hkv, D, Dv, float(scale), int(causal), int(window or 0), int(keep_first), float(softcap or 0.0),
+                  _lib.ptr(sinks),
                   _lib.status_word(q.device).data_ptr(), _lib.stream_ptr())
         return out
-    return paged_attention_reference(q, k_pages, v_pages, cu_q, kv_lens, page_table, scale=scale, causal=causal,
-                                     window=window, softcap=softcap, sinks=sinks)
+    o = paged_attention_reference(q, k_pages, v_pages, cu_q, kv_lens, page_table, scale=scale, causal=causal,
+                                  window=window, softcap=softcap, sinks=sinks, keep_first=keep_first, sigmoid=sigmoid)
+    return o if out is None else out.copy_(o)
 
 
-_lib.register("edl_attn_simt", i32, [vp, vp, vp, vp, i32, i64, i64, i64, vp, vp, vp, i32, i32, i32, i64, i32, i32, i32, i32,
-                                     f32, i32, f32, vp, vp, vp])
+_lib.register("edl_attn_simt", i32, [vp, vp, vp, vp, i32, i64, i64, i64, i64, vp, vp, vp, i32, i32, i32, i64, i32, i32, i32, i32,
+                                     f32, i32, i32, f32, vp, vp, vp, i64, f32, vp, vp])
 
 
 def simt_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, cu_q: torch.Tensor,
                    kv_lens: torch.Tensor, page_table: torch.Tensor, *, scale: float, window: int = 0, sinks=None,
-                   out: torch.Tensor | None = None, v_dim: int | None = None, softcap: float = 0.0) -> torch.Tensor:
+                   out: torch.Tensor | None = None, v_dim: int | None = None, softcap: float = 0.0, keep_first: int = 0,
+                   sigmoid: SigmoidWeights | None = None) -> torch.Tensor:
     """Causal paged attention in fp32 arithmetic (``csrc/attention_simt.cu``): fp32 models, and head sizes outside the
     tensor-core kernels'. Arguments as :func:`paged_attention`; ``v_dim``: only the first elements of a value row count
     (latent rows, which are keys and values at once; one KV head)."""
@@ -103,32 +140,49 @@ def simt_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor
     assert k_pages.shape[1] == PAGE_SIZE and q.stride(-1) == 1 and q.stride(-2) == D
     if out is None:
         out = torch.empty((T, Hq, Dv), dtype=q.dtype, device=q.device)
-    assert out.is_contiguous()
+    assert out.stride(2) == 1 and out.stride(1) == Dv
+    assert sigmoid is None or (sinks is None and (sigmoid.gate is None or sigmoid.gate.dtype == q.dtype))
     _lib.call("edl_attn_simt", q.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), out.data_ptr(),
-              int(q.dtype == torch.float32), q.stride(0), k_pages.stride(1), v_pages.stride(1), cu_q.data_ptr(),
+              int(q.dtype == torch.float32), q.stride(0), k_pages.stride(1), v_pages.stride(1), out.stride(0), cu_q.data_ptr(),
               kv_lens.data_ptr(), page_table.data_ptr(), page_table.stride(0), kv_lens.numel(), T, k_pages.shape[0], Hq,
-              Hkv, D, Dv, float(scale), int(window or 0), float(softcap or 0.0), _lib.ptr(sinks),
-              _lib.status_word(q.device).data_ptr(), _lib.stream_ptr())
+              Hkv, D, Dv, float(scale), int(window or 0), int(keep_first), float(softcap or 0.0), _lib.ptr(sinks),
+              *(sigmoid.args() if sigmoid is not None else (None, None, 0, 1.0)), _lib.status_word(q.device).data_ptr(), _lib.stream_ptr())
     return out
 
 
 def decode_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, kv_lens: torch.Tensor,
                      page_table: torch.Tensor, *, scale: float | None = None, window: int = 0, sinks=None,
-                     num_splits: int = 1, softcap: float = 0.0) -> torch.Tensor:
+                     num_splits: int = 1, softcap: float = 0.0, keep_first: int = 0,
+                     sigmoid: SigmoidWeights | None = None, out: torch.Tensor | None = None) -> torch.Tensor:
     """Decode-step attention (one query token per sequence) with the streaming kernel of
     ``csrc/attention_decode.cu``. q ``[B, Hq, D]``; pages ``[P, 128, Hkv, D]`` (values may have another width than
     keys); ``num_splits`` cuts every
     sequence's keys into that many parts that run as separate CTAs and are merged by :func:`attn_combine`; ``softcap``:
-    scores become ``softcap * tanh(score / softcap)``."""
+    scores become ``softcap * tanh(score / softcap)``; ``keep_first``, ``sigmoid``: as for :func:`paged_attention`.
+    ``out [B, Hq, Dv]`` may have a row pitch of its own (without a softmax, or without key splits)."""
     B, Hq, D = q.shape
     Hkv, Dv = k_pages.shape[2], v_pages.shape[-1]
     scale = scale if scale is not None else 1.0 / math.sqrt(D)
     S_ = max(1, int(num_splits))
+    if sigmoid is not None:
+        assert not softcap and sinks is None
+        if out is None:
+            out = torch.empty((B, Hq, Dv), dtype=q.dtype, device=q.device)
+        parts = torch.empty((S_, B, Hq, Dv), dtype=torch.float32, device=q.device) if S_ > 1 else None
+        _lib.call("edl_attn_decode_sigmoid", q.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), out.data_ptr(),
+                  _lib.ptr(parts), q.stride(0), k_pages.stride(1), v_pages.stride(1), out.stride(0), kv_lens.data_ptr(),
+                  page_table.data_ptr(), page_table.stride(0), B, k_pages.shape[0], Hq, Hkv, D, Dv, float(scale),
+                  int(window or 0), int(keep_first), S_, *sigmoid.args(), _lib.status_word(q.device).data_ptr(),
+                  _lib.stream_ptr())
+        return out
+    if out is not None:
+        return out.copy_(decode_attention(q, k_pages, v_pages, kv_lens, page_table, scale=scale, window=window, sinks=sinks,
+                                          num_splits=S_, softcap=softcap, keep_first=keep_first))
     out = torch.empty((S_, B, Hq, Dv), dtype=q.dtype, device=q.device)
     lse = torch.empty((S_, Hq, B), dtype=torch.float32, device=q.device) if S_ > 1 else None
     _lib.call("edl_attn_decode", q.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), out.data_ptr(), _lib.ptr(lse),
               q.stride(0), k_pages.stride(1), v_pages.stride(1), Hq * Dv, kv_lens.data_ptr(), page_table.data_ptr(),
-              page_table.stride(0), B, k_pages.shape[0], Hq, Hkv, D, Dv, float(scale), int(window or 0), S_,
+              page_table.stride(0), B, k_pages.shape[0], Hq, Hkv, D, Dv, float(scale), int(window or 0), int(keep_first), S_,
               float(softcap or 0.0), _lib.ptr(sinks) if S_ == 1 else None, _lib.status_word(q.device).data_ptr(), _lib.stream_ptr())
     if S_ == 1:
         return out[0]
@@ -182,10 +236,10 @@ def paged_kernel_supports(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch
             and _tile_width(q.shape[-1]) and _tile_width(v_pages.shape[-1]) and q.stride(0) % 8 == 0)
 
 
-def decode_splits(splits: int, window: int | None) -> int:
-    """Key splits of a layer's decode step: as many as planned for the whole context, but under a sliding window no more
-    than leave every split some tiles of 32 keys."""
-    return splits if not window else int(max(1, min(splits, (window + 31) // 32 // 4)))
+def decode_splits(splits: int, window: int | None, keep_first: int = 0) -> int:
+    """Key splits of a layer's decode step: as many as planned for the whole context, but under a sliding window (with
+    ``keep_first`` kept keys) no more than leave every split some tiles of 32 keys."""
+    return splits if not window else int(max(1, min(splits, (window + keep_first + 31) // 32 // 4)))
 
 
 def decode_kernel_supports(q: torch.Tensor, k_pages: torch.Tensor, v_dim: int | None = None) -> bool:
@@ -256,7 +310,7 @@ def paged_attention_splitkv(q: torch.Tensor, k_pages: torch.Tensor, v_pages: tor
 
 
 def paged_attention_reference(q, k_pages, v_pages, cu_q, kv_lens, page_table, *, scale=None, causal=True, window=0,
-                              softcap=0.0, sinks=None):
+                              softcap=0.0, sinks=None, keep_first=0, sigmoid=None):
     """Dense oracle: gathers each sequence's keys/values from its pages and runs reference attention."""
     from . import reference as R
 
@@ -272,9 +326,11 @@ def paged_attention_reference(q, k_pages, v_pages, cu_q, kv_lens, page_table, *,
         ks = k_pages[ids].reshape(-1, *k_pages.shape[2:])[:L]
         vs = v_pages[ids].reshape(-1, *v_pages.shape[2:])[:L]
         o = R.attention(qs[None], ks[None].to(qs.dtype), vs[None].to(qs.dtype), causal=causal, scale=scale,
-                        sliding_window=window or None, softcap=softcap, sinks=sinks)
+                        sliding_window=window or None, softcap=softcap, sinks=sinks, keep_first=keep_first,
+                        score_bias=None if sigmoid is None else sigmoid.bias)
         outs.append(o[0])
-    return torch.cat(outs, dim=0)
+    o = torch.cat(outs, dim=0)
+    return o if sigmoid is None else sigmoid.finish(o)
 
 
 def sample(logits: torch.Tensor, *, temperature=None, top_k=None, top_p=None, min_p=None, presence=None,

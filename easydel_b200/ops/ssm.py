@@ -1,5 +1,6 @@
 """State-space and linear-attention recurrences: Mamba-1 selective scan, Mamba-2 SSD, gated delta rule, KDA and
-the ragged causal conv1d in front of them (``csrc/ssm.cu``), HGRN2 (``csrc/hgrn2.cu``).
+the ragged causal conv1d in front of them (``csrc/ssm.cu``), HGRN2 (``csrc/hgrn2.cu``), the generalised delta rule
+(``csrc/gdelta.cu``).
 
 Every op has a PyTorch reference (also its autograd path: training differentiates the reference, chunk by chunk,
 while inference and evaluation call the CUDA recurrences). Sequences are packed on the token axis with
@@ -7,6 +8,8 @@ while inference and evaluation call the CUDA recurrences). Sequences are packed 
 """
 
 from __future__ import annotations
+
+from dataclasses import dataclass
 
 import torch
 import torch.nn.functional as tF
@@ -20,6 +23,12 @@ _lib.register("edl_delta_rule", i32, [vp, vp, vp, vp, vp, i32, vp, i32, i32, i32
 _lib.register("edl_ragged_conv1d", i32, [vp, vp, vp, vp, vp, i32, i32, i32, i32, vp, vp, vp])
 _lib.register("edl_hgrn2_scan", i32, [vp, i32, _lib.i64, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, vp, vp, vp])
 _lib.register("edl_hgrn2_decode", i32, [vp, i32, _lib.i64, vp, vp, vp, vp, vp, vp, f32, vp, i32, i32, i32, i32, vp])
+_lib.register("edl_gdelta_scan", i32, [vp, vp, vp, vp, i32, _lib.i64, vp, vp, vp, f32, f32, vp, vp, vp, vp, vp, i32, i32, i32,
+                                       i32, i32, vp])
+_lib.register("edl_gdelta_finish", i32, [vp, vp, i32, _lib.i64, vp, f32, f32, vp, _lib.i64, i32, i32, i32, vp])
+_lib.register("edl_gdelta_decode", i32, [vp, vp, vp, vp, vp, vp, i32, _lib.i64, vp, i32, vp, vp, f32, f32, vp, vp, vp, vp, f32,
+                                         f32, vp, _lib.i64, i32, i32, i32, i32, vp])
+_lib.register("edl_tanh_rows", i32, [vp, i32, _lib.i64, vp, i32, i32, vp])
 _lib.register("edl_wkv4", i32, [vp, vp, vp, vp, vp, i32, i32, vp, vp, vp])
 
 
@@ -576,3 +585,109 @@ def hgrn2(proj: torch.Tensor, heads: tuple[int, int, int], bias: torch.Tensor, l
               cu.data_ptr(), _lib.ptr(slots), _lib.ptr(state), o.data_ptr(), rows.data_ptr(), T, B, H, D, V, seg_len, n, _lib.ptr(ws),
               _lib.ptr(prod), sp)
     return ST.head_norm(o, norm, eps, proj.dtype).view(T, H * V)
+
+
+# ----------------------------------------------------------------------------------------- generalised delta rule
+@dataclass
+class DeltaColumns:
+    """Columns of a packed projection (views with one row pitch): receptance ``r``, key ``k`` and removal rate ``a`` ``[T, H
+    D]``, value ``v`` and output gate ``g`` ``[T, H V]``, and ``x [T, rank]``, the input of the low-rank decay."""
+
+    r: torch.Tensor
+    k: torch.Tensor
+    v: torch.Tensor
+    a: torch.Tensor
+    g: torch.Tensor
+    x: torch.Tensor
+
+
+@dataclass
+class DeltaWeights:
+    """``w2 [H D, rank]`` (operand type), ``w0`` and ``a0`` fp32 ``[H D]``, ``norm`` fp32 ``[H V]``. ``rate``: the strongest
+    decay of a token is ``e^-rate``; ``unit_eps`` is added to a key's squared length; ``eps`` belongs to the output norm."""
+
+    w2: torch.Tensor
+    w0: torch.Tensor
+    a0: torch.Tensor
+    norm: torch.Tensor
+    rate: float
+    unit_eps: float
+    eps: float
+
+
+def _low_rank(x: torch.Tensor, w2: torch.Tensor) -> torch.Tensor:
+    """fp32 ``W2 tanh(x)``."""
+    from . import stream as ST
+
+    if ST.on_kernels(x):
+        t = torch.empty(x.shape, dtype=x.dtype, device=x.device)
+        _lib.call("edl_tanh_rows", x.data_ptr(), int(x.dtype == torch.float32), x.stride(0), t.data_ptr(), x.shape[0],
+                  x.shape[1], _lib.stream_ptr())
+        return ST.linear(t, w2, out_dtype=torch.float32)
+    return torch.tanh(x.float()) @ w2.float().t()
+
+
+def generalized_delta_reference(cols: DeltaColumns, heads, wt: DeltaWeights, scale: float, cu, slots=None, state=None):
+    """Token by token, in tensors (also the form that is differentiated): ``[T, H V]`` in the projection's type. With the unit
+    key ``u``: ``S = diag(w) S - (a u) (u^T S) + k v^T`` on the old state, ``o = S^T r``, normed per head and gated."""
+    H, D, V = heads
+    T = cols.r.shape[0]
+    h3 = lambda t: t.float().reshape(T, H, -1)  # noqa: E731
+    r, k, v = h3(cols.r), h3(cols.k), h3(cols.v)
+    w = torch.exp(-wt.rate * torch.sigmoid(h3(_low_rank(cols.x, wt.w2) + wt.w0.float())))
+    u = k * torch.rsqrt(k.pow(2).sum(-1, keepdim=True) + wt.unit_eps)
+    au = torch.sigmoid(h3(cols.a.float() + wt.a0.float())) * u
+    bounds = cu.tolist()
+    rows = list(range(len(bounds) - 1)) if slots is None else slots.tolist()
+    outs = []
+    for b in range(len(bounds) - 1):
+        if bounds[b + 1] <= bounds[b]:
+            continue
+        s = state[rows[b]].clone() if state is not None else r.new_zeros(H, D, V)
+        for t in range(bounds[b], bounds[b + 1]):
+            seen = (u[t][:, :, None] * s).sum(1, keepdim=True)
+            s = w[t][:, :, None] * s - au[t][:, :, None] * seen + k[t][:, :, None] * v[t][:, None, :]
+            outs.append((s * r[t][:, :, None]).sum(1))
+        if state is not None:
+            with torch.no_grad():
+                state[rows[b]] = s
+    o = torch.stack(outs)
+    o = (o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + wt.eps)).reshape(T, H * V)
+    return (o * wt.norm.float() * torch.sigmoid(cols.g.float()) * scale).to(cols.r.dtype)
+
+
+def generalized_delta_rule(cols: DeltaColumns, heads: tuple[int, int, int], wt: DeltaWeights, cu: torch.Tensor, max_len: int,
+                           slots: torch.Tensor | None = None, state: torch.Tensor | None = None, scale: float = 1.0,
+                           out: torch.Tensor | None = None) -> torch.Tensor:
+    """The generalised delta rule over a packed projection, with output norm, gate and the factor ``scale``.
+
+    ``heads = (H, D, V)``; ``cu`` int32 ``[B + 1]``; ``state`` fp32 ``[*, H, D, V]``, rows ``slots`` (int32 ``[B]``) read and
+    updated in place; ``max_len``: longest sequence of the step; ``out [T, H V]``: where to write (may be a view)."""
+    from . import stream as ST
+
+    H, D, V = heads
+    T, B = cols.r.shape[0], cu.numel() - 1
+    if not ST.on_kernels(cols.r):
+        o = generalized_delta_reference(cols, heads, wt, scale, cu, slots, state)
+        return o if out is None else out.copy_(o)
+    f32_in, ld = int(cols.r.dtype == torch.float32), cols.r.stride(0)
+    assert all(t.stride(0) == ld and t.stride(1) == 1 for t in vars(cols).values()) or T == 1
+    assert wt.w2.is_contiguous() and wt.w2.dtype == cols.r.dtype
+    if out is None:
+        out = torch.empty(T, H * V, dtype=cols.r.dtype, device=cols.r.device)
+    sp = _lib.stream_ptr()
+    if max_len == 1 and state is not None:
+        _lib.call("edl_gdelta_decode", *(t.data_ptr() for t in (cols.r, cols.k, cols.v, cols.a, cols.g, cols.x)), f32_in, ld,
+                  wt.w2.data_ptr(), wt.w2.shape[1], wt.w0.data_ptr(), wt.a0.data_ptr(), float(wt.rate), float(wt.unit_eps),
+                  cu.data_ptr(), _lib.ptr(slots), state.data_ptr(), wt.norm.data_ptr(), float(wt.eps), float(scale),
+                  out.data_ptr(), out.stride(0), B, H, D, V, sp)
+        return out
+    z = _low_rank(cols.x, wt.w2)
+    o = torch.empty(T, H, V, dtype=torch.float32, device=cols.r.device)
+    rows = torch.empty(T * H * (4 * D + V), dtype=torch.float32, device=cols.r.device)
+    _lib.call("edl_gdelta_scan", *(t.data_ptr() for t in (cols.r, cols.k, cols.v, cols.a)), f32_in, ld, z.data_ptr(),
+              wt.w0.data_ptr(), wt.a0.data_ptr(), float(wt.rate), float(wt.unit_eps), cu.data_ptr(), _lib.ptr(slots),
+              _lib.ptr(state), o.data_ptr(), rows.data_ptr(), T, B, H, D, V, sp)
+    _lib.call("edl_gdelta_finish", o.data_ptr(), cols.g.data_ptr(), f32_in, ld, wt.norm.data_ptr(), float(wt.eps), float(scale),
+              out.data_ptr(), out.stride(0), T, H, V, sp)
+    return out

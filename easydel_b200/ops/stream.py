@@ -8,6 +8,8 @@ and calls under autograd run the tensor forms below, which return new tensors.
 
 from __future__ import annotations
 
+from dataclasses import dataclass
+
 import torch
 import torch.nn.functional as tF
 
@@ -24,8 +26,10 @@ _lib.register("edl_post_norm", i32, [vp, vp, vp, vp, vp, i32, f32, f32, i32, vp,
 _lib.register("edl_scale_cap", i32, [vp, i64, f32, f32, vp])
 _lib.register("edl_qkv_prologue", i32, [vp, i32, i64, vp, vp, vp, vp, f32, f32, f32, i32, i32, i32, i32, i32, vp, vp, vp,
                                         i64, i64, i64, vp, vp])
-_lib.register("edl_qkv_rotary_prologue", i32, [vp, i32, i64, vp, vp, vp, vp, f32, vp, i32, i32, i32, i32, i32, i32, vp, vp, vp,
-                                               i64, i64, i64, vp, vp])
+_lib.register("edl_qkv_rotary_prologue", i32, [vp, i32, i64, vp, vp, vp, vp, f32, vp, i32, i32, f32, vp, vp, i64, vp, i32, i32,
+                                               i32, i32, i32, vp, vp, vp, i64, i64, i64, vp, vp])
+_lib.register("edl_branch_norm", i32, [vp, vp, vp, vp, f32, vp, f32, vp, i32, i32, i32, vp])
+_lib.register("edl_gated_unit", i32, [vp, i32, i64, vp, i32, i32, i32, vp])
 
 
 def on_kernels(t: torch.Tensor) -> bool:
@@ -210,10 +214,11 @@ def gated_unit(gu: torch.Tensor, act: str = "silu") -> torch.Tensor:
         F = gu.shape[1] // 2
         if gu.dtype == torch.bfloat16 and F % 8 == 0 and gu.stride(0) % 8 == 0 and act in K.ACT_IDS:
             return K.gated_act_fwd(gu, act)
-        if act == "silu":
-            from .moe_kernels import expert_unit
-
-            return expert_unit(gu if gu.is_contiguous() else gu.contiguous())
+        if act in K.ACT_IDS and gu.stride(1) == 1:
+            out = torch.empty(gu.shape[0], F, dtype=gu.dtype, device=gu.device)
+            _lib.call("edl_gated_unit", gu.data_ptr(), _f32flag(gu.dtype), gu.stride(0), out.data_ptr(), gu.shape[0], F,
+                      K.ACT_IDS[act], _lib.stream_ptr())
+            return out
     return R.gated_act(gu, act)
 
 
@@ -246,8 +251,24 @@ def _sum_and_norm(x, branch, alpha, beta, keep_sum, w, eps, out_dtype, offset):
     return s if keep_sum else v, v.to(out_dtype)
 
 
+@dataclass
+class NormedBranch:
+    """A branch that is RMS-normed before it joins the stream: ``rms_norm(rows) * weight * scale`` (all fp32; ``scale [W]``:
+    one factor per channel, or None)."""
+
+    rows: torch.Tensor
+    weight: torch.Tensor
+    eps: float
+    scale: torch.Tensor | None = None
+
+    def combine(self) -> torch.Tensor:
+        f = self.rows.float()
+        y = f * torch.rsqrt(f.pow(2).mean(-1, keepdim=True) + self.eps) * self.weight.float()
+        return y if self.scale is None else y * self.scale.float()
+
+
 def branch_rows(branch) -> torch.Tensor:
-    """A branch (fp32 rows or expert rows) as fp32 rows."""
+    """A branch (fp32 rows, expert rows or a normed branch) as fp32 rows."""
     return branch.float() if isinstance(branch, torch.Tensor) else branch.combine()
 
 
@@ -261,10 +282,20 @@ def post_norm(x: torch.Tensor, branch, alpha: float, w: torch.Tensor, eps: float
 
 def add_norm(x: torch.Tensor, branch, mult: float, w: torch.Tensor, eps: float, out_dtype: torch.dtype,
              offset: float = 0.0) -> tuple[torch.Tensor, torch.Tensor]:
-    """``x + mult branch`` (in place on the kernels; ``branch`` as in :func:`post_norm`, or None) and the RMS norm of the
-    sum, ``* (w + offset)``, as the operand of the next products."""
+    """``x + mult branch`` (in place on the kernels; ``branch`` as in :func:`post_norm`, a :class:`NormedBranch`, or None) and
+    the RMS norm of the sum, ``* (w + offset)``, as the operand of the next products."""
     if branch is None:
         return x, norm_shift(x, w, eps, out_dtype, offset=offset)
+    if isinstance(branch, NormedBranch) and on_kernels(x) and mult == 1.0 and offset == 0.0:
+        y = branch.rows
+        assert x.is_contiguous() and y.is_contiguous() and y.dtype == torch.float32 and branch.weight.dtype == torch.float32
+        h = torch.empty(x.shape, dtype=out_dtype, device=x.device)
+        _lib.call("edl_branch_norm", x.data_ptr(), y.data_ptr(), branch.weight.data_ptr(), _lib.ptr(branch.scale),
+                  float(branch.eps), w.data_ptr(), float(eps), h.data_ptr(), _f32flag(out_dtype), x.shape[0], x.shape[1],
+                  _lib.stream_ptr())
+        return x, h
+    if isinstance(branch, NormedBranch):
+        branch = branch.combine()
     return _sum_and_norm(x, branch, 1.0, mult, True, w, eps, out_dtype, offset)
 
 
@@ -314,10 +345,13 @@ def qkv_prologue(qkv: torch.Tensor, heads: tuple[int, int, int, int], qw, kw, ep
 
 def qkv_rotary_prologue(qkv: torch.Tensor, heads: tuple[int, int, int, int], qw, kw, eps: float, positions: torch.Tensor,
                         freq: torch.Tensor | None, slot_mapping: torch.Tensor, k_pages: torch.Tensor,
-                        v_pages: torch.Tensor) -> torch.Tensor:
+                        v_pages: torch.Tensor, layout: str = "halves", mag: float = 1.0, bias: torch.Tensor | None = None,
+                        first: torch.Tensor | None = None, lam: torch.Tensor | None = None) -> torch.Tensor:
     """:func:`qkv_prologue` for queries and keys that are normed over the whole projection (all heads at once; weights
-    ``qw [Hq D]``, ``kw [Hkv D]``, None: no norm) and then rotated: elements ``i`` and ``i + pairs`` of every head by the
-    position times frequency i (``freq``: see :mod:`.rotation`; None: no rotation)."""
+    ``qw [Hq D]``, ``kw [Hkv D]``, None: no norm) and then rotated: the pairs of every head (``layout``, ``freq``: see
+    :mod:`.rotation`; None: no rotation) by the position times their frequency, cosines and sines times ``mag``.
+    ``bias`` fp32 ``[Hq D + Hkv (D + Dv)]`` is added first. ``lam`` (fp32 scalar): the cached values are ``(1 - lam) v + lam
+    first``, ``first [T, Hkv Dv]`` in the operand type."""
     Hq, Hkv, D, Dv = heads
     T = qkv.shape[0]
     if on_kernels(qkv):
@@ -325,25 +359,38 @@ def qkv_rotary_prologue(qkv: torch.Tensor, heads: tuple[int, int, int, int], qw,
         pos = positions.reshape(-1).to(torch.int32)
         _lib.call("edl_qkv_rotary_prologue", qkv.data_ptr(), _f32flag(qkv.dtype), qkv.stride(0), pos.data_ptr(),
                   slot_mapping.data_ptr(), _lib.ptr(qw), _lib.ptr(kw), float(eps), _lib.ptr(freq),
-                  freq.numel() // 2 if freq is not None else 0, T, Hq, Hkv, D, Dv, q.data_ptr(), k_pages.data_ptr(),
-                  v_pages.data_ptr(), k_pages.stride(1), v_pages.stride(1), k_pages.shape[0] * k_pages.shape[1],
-                  _lib.status_word(qkv.device).data_ptr(), _lib.stream_ptr())
+                  freq.numel() // 2 if freq is not None else 0, int(layout == "neighbours"), float(mag), _lib.ptr(bias),
+                  _lib.ptr(first), first.stride(0) if first is not None else 0, _lib.ptr(lam), T, Hq, Hkv, D, Dv,
+                  q.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), k_pages.stride(1), v_pages.stride(1),
+                  k_pages.shape[0] * k_pages.shape[1], _lib.status_word(qkv.device).data_ptr(), _lib.stream_ptr())
         return q
     from . import serving as S
 
-    q, k, v = torch.split(qkv, [Hq * D, Hkv * D, Hkv * Dv], -1)
-    q, k = qk_norm_rotate(q, k, D, qw, kw, eps, positions, freq)
-    S.kv_append(k, v.reshape(T, Hkv, Dv), k_pages, v_pages, slot_mapping)
+    q, k, v = rotary_rows(qkv, heads, qw, kw, eps, positions, freq, layout, mag, bias, first, lam)
+    S.kv_append(k, v, k_pages, v_pages, slot_mapping)
     return q
 
 
-def qk_norm_rotate(q, k, D: int, qw, kw, eps: float, positions, freq):
-    """Tensor form of the q / k half of :func:`qkv_rotary_prologue`: flat rows -> ``[T, H, D]`` and ``[T, G, D]``."""
+def rotary_rows(qkv, heads, qw, kw, eps: float, positions, freq, layout="halves", mag=1.0, bias=None, first=None, lam=None):
+    """Tensor form of :func:`qkv_rotary_prologue` without the pages: ``q [T, H, D]``, ``k [T, G, D]``, ``v [T, G, Dv]``."""
+    Hq, Hkv, D, Dv = heads
+    dt = qkv.dtype
+    if bias is not None:
+        qkv = qkv.float() + bias.float()
+    q, k, v = torch.split(qkv, [Hq * D, Hkv * D, Hkv * Dv], -1)
+    q, k = qk_norm_rotate(q, k, D, qw, kw, eps, positions, freq, layout, mag)
+    if lam is not None:
+        v = (1.0 - lam.float()) * v.float() + lam.float() * first.float()
+    return q.to(dt), k.to(dt), v.to(dt).reshape(-1, Hkv, Dv)
+
+
+def qk_norm_rotate(q, k, D: int, qw, kw, eps: float, positions, freq, layout: str = "halves", mag: float = 1.0):
+    """The q / k half of :func:`rotary_rows`: flat rows -> ``[T, H, D]`` and ``[T, G, D]``."""
     def one(x, w):
         xf = x.float()
         if w is not None:
             xf = xf * torch.rsqrt(xf.pow(2).mean(-1, keepdim=True) + eps) * w.float()
         xf = xf.reshape(x.shape[0], -1, D)
-        return (xf if freq is None else rotation.rotate(xf, positions.reshape(-1), freq, "halves")).to(x.dtype)
+        return (xf if freq is None else rotation.rotate(xf, positions.reshape(-1), freq, layout, mag)).to(x.dtype)
 
     return one(q, qw), one(k, kw)

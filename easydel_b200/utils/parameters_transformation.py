@@ -25,6 +25,8 @@ FUSED_SPLITS: dict[str, tuple[str, ...]] = {
     "qdg_proj": ("q_proj", "dkv_proj", "g_proj"),
     "qd_proj": ("q_proj", "dkv_proj"),
     "ukv_proj": ("uk_proj", "uv_proj"),
+    "twin_proj": ("left_q_proj", "left_k_proj", "left_v_proj", "right_r_proj", "right_k_proj", "right_v_proj", "right_a_proj",
+                  "right_g_proj", "right_x_proj", "left_g_proj"),
 }
 
 _EXPERT_RE = re.compile(r"^(.*\.)experts\.(\d+)\.(gate_proj|up_proj|down_proj|w1|w2|w3)\.weight$")
