@@ -315,12 +315,13 @@ class Attention(nn.Module):
         if self.qkv_bias is not None:
             raise NotImplementedError("blended values have no biases")
         n = (self.num_heads + self.num_kv_heads) * self.head_dim
-        values = qkv[:, n:n + self.num_kv_heads * self.v_head_dim]
+        values = qkv[:, n:n + self.num_kv_heads * self.v_head_dim].unflatten(1, (self.num_kv_heads, self.v_head_dim))
         if step.first_values is None:
             step.first_values = values
             return {}
         if step.first_values.shape != values.shape:
-            raise ValueError(f"values of width {values.shape[1]} cannot blend with the first layer's {step.first_values.shape[1]}")
+            raise ValueError(f"value heads {tuple(values.shape[1:])} cannot blend with the first layer's "
+                             f"{tuple(step.first_values.shape[1:])}")
         return {"first": step.first_values, "lam": self.value_mix}
 
     def _frequencies(self, device) -> torch.Tensor | None:

@@ -164,7 +164,7 @@ class StreamStep:
     slots: torch.Tensor | None = None     # int32 [B] state rows of the sequences
     meta: tp.Any = None                   # PagedBatchMeta, with a paged cache
     segment_ids: torch.Tensor | None = None
-    first_values: torch.Tensor | None = None   # values [T, heads * width] of the first layer that blends values
+    first_values: torch.Tensor | None = None   # values [T, heads, width] of the first layer that blends values
 
 
 @dataclass

@@ -351,7 +351,7 @@ def qkv_rotary_prologue(qkv: torch.Tensor, heads: tuple[int, int, int, int], qw,
     ``qw [Hq D]``, ``kw [Hkv D]``, None: no norm) and then rotated: the pairs of every head (``layout``, ``freq``: see
     :mod:`.rotation`; None: no rotation) by the position times their frequency, cosines and sines times ``mag``.
     ``bias`` fp32 ``[Hq D + Hkv (D + Dv)]`` is added first. ``lam`` (fp32 scalar): the cached values are ``(1 - lam) v + lam
-    first``, ``first [T, Hkv Dv]`` in the operand type."""
+    first``, ``first [T, Hkv, Dv]`` in the operand type (rows may be strided)."""
     Hq, Hkv, D, Dv = heads
     T = qkv.shape[0]
     if on_kernels(qkv):
@@ -380,7 +380,7 @@ def rotary_rows(qkv, heads, qw, kw, eps: float, positions, freq, layout="halves"
     q, k, v = torch.split(qkv, [Hq * D, Hkv * D, Hkv * Dv], -1)
     q, k = qk_norm_rotate(q, k, D, qw, kw, eps, positions, freq, layout, mag)
     if lam is not None:
-        v = (1.0 - lam.float()) * v.float() + lam.float() * first.float()
+        v = (1.0 - lam.float()) * v.float() + lam.float() * first.float().flatten(1)
     return q.to(dt), k.to(dt), v.to(dt).reshape(-1, Hkv, Dv)
 
 
