@@ -17,7 +17,7 @@ At 8 GPUs (``--serving auto``; ``on`` forces it at any N) the same JSON line car
 output tokens/s and TTFT / TPOT percentiles for Llama-3-70B at TP = N on the Poisson workload of the baseline
 (``easydel_b200/inference/esurge/bench_serving.py``), measured after the training state has been freed.
 
-``--model rakevik`` / ``disunex`` / ``gasetar`` measures that family instead (kernels and serving throughput beside the closest
+``--model rakevik`` / ``disunex`` / ``gasetar`` / ``ninisun`` measures that family instead (kernels and serving throughput beside the closest
 existing models).
 
 ``--impl reference`` reports whether the unmodified reference can run here.
@@ -251,7 +251,7 @@ def main() -> None:
     ap.add_argument("--serving-rate", type=float, default=8.0, help="Poisson arrival rate, requests/s")
     ap.add_argument("--serving-seconds", type=float, default=270.0,
                     help="requests stop being admitted after this long; the ones admitted are finished")
-    ap.add_argument("--model", default=None, choices=["rakevik", "disunex", "gasetar"],
+    ap.add_argument("--model", default=None, choices=["rakevik", "disunex", "gasetar", "ninisun"],
                     help="instead of the headline workload: kernels and serving throughput of this family beside the "
                          "closest existing models (benchmarks/bench_<model>.py), one JSON line per row")
     args = ap.parse_args()

@@ -233,11 +233,16 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tk, const __grid_constant
 #pragma unroll
       for (int j = 0; j < TK / 8; ++j) {
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const int key = cbase + j * 8 + (e & 1);
-          const bool ok = key < kv_len && (key >= lo || key < p.keep_first);
-          const float y = fminf(-fmaf(s[j][e], p.scale_log2, bias2[e >> 1]), 120.f);
-          s[j][e] = ok ? __fdividef(1.f, 1.f + exp2f(y)) : 0.f;
+        for (int e = 0; e < 4; e += 2) {
+          const int key = cbase + j * 8;
+          const bool ok0 = key < kv_len && (key >= lo || key < p.keep_first);
+          const bool ok1 = key + 1 < kv_len && (key + 1 >= lo || key + 1 < p.keep_first);
+          // one reciprocal for two weights; the bound keeps the product finite, what it cuts off is below 2^-60
+          const float d0 = 1.f + exp2f(fminf(-fmaf(s[j][e], p.scale_log2, bias2[e >> 1]), 60.f));
+          const float d1 = 1.f + exp2f(fminf(-fmaf(s[j][e + 1], p.scale_log2, bias2[e >> 1]), 60.f));
+          const float r = __fdividef(1.f, d0 * d1);
+          s[j][e] = ok0 ? r * d1 : 0.f;
+          s[j][e + 1] = ok1 ? r * d0 : 0.f;
         }
         pa[j >> 1][(j & 1) * 2] = pack_bf16x2(s[j][0], s[j][1]);
         pa[j >> 1][(j & 1) * 2 + 1] = pack_bf16x2(s[j][2], s[j][3]);

@@ -149,16 +149,16 @@ template <int DP, int RPT, int CPT, int NT>
 struct ScanCfg {
   static constexpr int SPLIT = DP / RPT;
   static constexpr int CT = (NT / SPLIT) * CPT;                 // columns of a CTA
-  static constexpr int TC = DP <= 128 ? 8 : 1024 / DP;          // tokens per stage
+  static constexpr int TC = DP <= 64 ? 16 : 1024 / DP;          // tokens per stage
   static constexpr int CTP = (CT + 3) / 4 * 4;
   static constexpr int STAGE = TC * (4 * DP + CTP);             // floats
 };
 
 template <int DP, int RPT, int CPT, int NT>
-__global__ void __launch_bounds__(NT) gdelta_scan_kernel(const DeltaParams p) {
+__global__ void __launch_bounds__(NT, 256 / NT) gdelta_scan_kernel(const DeltaParams p) {
   using C = ScanCfg<DP, RPT, CPT, NT>;
   constexpr int SPLIT = C::SPLIT, CT = C::CT, TC = C::TC, NK = RPT / 4;
-  static_assert(SPLIT >= CPT && SPLIT <= 32 && RPT % 4 == 0 && (CPT == 1 || CPT == 2), "");
+  static_assert(SPLIT >= CPT && SPLIT <= 32 && RPT % 4 == 0 && (CPT == 1 || CPT == 2 || CPT == 4), "");
   extern __shared__ __align__(16) float smem[];
   const int tid = threadIdx.x;
   const int part = tid % SPLIT, grp = tid / SPLIT;
@@ -217,9 +217,34 @@ __global__ void __launch_bounds__(NT) gdelta_scan_kernel(const DeltaParams p) {
 #pragma unroll
       for (int c = 0; c < CPT; ++c) S[i][j][c] = (pool && row < D && col + c < V) ? pool[(long long)row * V + col + c] : 0.f;
     }
-  const int mine = CPT == 2 ? (part & 1) : 0;                   // column whose output this lane writes
-  float* out = p.o + ((long long)t0 * p.H + h) * V + col + mine;
-  const bool writes = part < CPT && col + mine < V;
+  // column whose output this lane writes
+  const int mine = CPT == 4 ? (part & 1) * 2 + ((part >> 1) & 1) : CPT == 2 ? (part & 1) : 0;
+  const unsigned pitch = (unsigned)p.H * V;
+  float* out = p.o + ((long long)t0 * p.H + h) * V + col + mine;       // where the next `late` goes: the first one is no
+  const bool writes = part < CPT && col + mine < V;                    // token's and is written over
+  unsigned step = 0;
+  // The lanes' sums over a column are the longest wait of a token: those of the outputs are taken one token late, together
+  // with the next token's u^T S, and diag(w) S + u v^T is formed while both are on their way.
+  constexpr int STEPS = SPLIT == 4 ? 2 : SPLIT == 8 ? 3 : SPLIT == 16 ? 4 : 5;
+  float late[CPT];
+#pragma unroll
+  for (int c = 0; c < CPT; ++c) late[c] = 0.f;
+  // step q of the sum of the outputs; the first steps also spread the columns over lanes
+  auto late_step = [&](int q) {
+    if (CPT == 4 && q == 0) {
+      const bool hi = part & 1;
+      const float x0 = __shfl_xor_sync(0xffffffffu, hi ? late[0] : late[2 % CPT], 1);
+      const float x1 = __shfl_xor_sync(0xffffffffu, hi ? late[1 % CPT] : late[3 % CPT], 1);
+      late[0] = (hi ? late[2 % CPT] : late[0]) + x0;
+      late[1 % CPT] = (hi ? late[3 % CPT] : late[1 % CPT]) + x1;
+    } else if ((CPT == 4 && q == 1) || (CPT == 2 && q == 0)) {
+      const bool hi = part & (1 << q);
+      const float x = __shfl_xor_sync(0xffffffffu, hi ? late[0] : late[1 % CPT], 1 << q);
+      late[0] = (hi ? late[1 % CPT] : late[0]) + x;
+    } else {
+      late[0] += __shfl_xor_sync(0xffffffffu, late[0], 1 << q);
+    }
+  };
   int buf = 0;
   for (int tb = t0; tb < t1; tb += TC, buf ^= 1) {
     const int n = min(TC, t1 - tb);
@@ -231,77 +256,96 @@ __global__ void __launch_bounds__(NT) gdelta_scan_kernel(const DeltaParams p) {
     }
     __syncthreads();
     const float* st = smem + buf * C::STAGE;
+    const float* sw = st + 4 * part;
+    const float* sv = st + 4 * TC * DP + grp * CPT;
+    float4 u4[NK];
+#pragma unroll
+    for (int i = 0; i < NK; ++i) u4[i] = *reinterpret_cast<const float4*>(sw + TC * DP + 4 * SPLIT * i);
 #pragma unroll 2
-    for (int t = 0; t < n; ++t) {
-      const float* sw = st + t * DP + 4 * part;
-      float v[CPT];
+    for (int t = 0; t < n; ++t, sw += DP, sv += C::CTP) {
+      float v[CPT], d[CPT][4], seen[CPT];
+      float4 w4[NK], b4[NK], r4[NK];
 #pragma unroll
-      for (int c = 0; c < CPT; ++c) v[c] = st[4 * TC * DP + t * C::CTP + grp * CPT + c];
-      float4 u4[NK];
-      float d[CPT][4];
+      for (int c = 0; c < CPT; ++c) v[c] = sv[c];
 #pragma unroll
-      for (int c = 0; c < CPT; ++c) d[c][0] = d[c][1] = d[c][2] = d[c][3] = 0.f;
+      for (int i = 0; i < NK; ++i) w4[i] = *reinterpret_cast<const float4*>(sw + 4 * SPLIT * i);
 #pragma unroll
-      for (int i = 0; i < NK; ++i) {
-        u4[i] = *reinterpret_cast<const float4*>(sw + TC * DP + 4 * SPLIT * i);
+      for (int i = 0; i < NK; ++i)
 #pragma unroll
         for (int c = 0; c < CPT; ++c) {
-          fma2(d[c][0], d[c][1], u4[i].x, u4[i].y, S[i][0][c], S[i][1][c], d[c][0], d[c][1]);
-          fma2(d[c][2], d[c][3], u4[i].z, u4[i].w, S[i][2][c], S[i][3][c], d[c][2], d[c][3]);
+          if (i == 0) {
+            mul2(d[c][0], d[c][1], u4[i].x, u4[i].y, S[i][0][c], S[i][1][c]);
+            mul2(d[c][2], d[c][3], u4[i].z, u4[i].w, S[i][2][c], S[i][3][c]);
+          } else {
+            fma2(d[c][0], d[c][1], u4[i].x, u4[i].y, S[i][0][c], S[i][1][c], d[c][0], d[c][1]);
+            fma2(d[c][2], d[c][3], u4[i].z, u4[i].w, S[i][2][c], S[i][3][c], d[c][2], d[c][3]);
+          }
         }
+#pragma unroll
+      for (int i = 0; i < NK; ++i) {
+        b4[i] = *reinterpret_cast<const float4*>(sw + 2 * TC * DP + 4 * SPLIT * i);
+        r4[i] = *reinterpret_cast<const float4*>(sw + 3 * TC * DP + 4 * SPLIT * i);
       }
-      float seen[CPT];
 #pragma unroll
-      for (int c = 0; c < CPT; ++c) seen[c] = (d[c][0] + d[c][1]) + (d[c][2] + d[c][3]);
+      for (int c = 0; c < CPT; ++c) {
+        add2(d[c][0], d[c][1], d[c][2], d[c][3]);
+        seen[c] = d[c][0] + d[c][1];
+      }
+      // a share of diag(w) S + u v^T behind every exchange
+      constexpr int SHARE = (NK + STEPS - 1) / STEPS;
 #pragma unroll
-      for (int o = 1; o < SPLIT; o <<= 1)
+      for (int q = 0; q < STEPS; ++q) {
+        float more[CPT];
 #pragma unroll
-        for (int c = 0; c < CPT; ++c) seen[c] += __shfl_xor_sync(0xffffffffu, seen[c], o);
-      // diag(w) S + u v^T does not wait for the sum
+        for (int c = 0; c < CPT; ++c) more[c] = __shfl_xor_sync(0xffffffffu, seen[c], 1 << q);
+        late_step(q);
 #pragma unroll
-      for (int i = 0; i < NK; ++i) {
-        const float4 w4 = *reinterpret_cast<const float4*>(sw + 4 * SPLIT * i);
+        for (int i = q * SHARE; i < (q + 1) * SHARE && i < NK; ++i)
 #pragma unroll
-        for (int c = 0; c < CPT; ++c) {
-          float x0, x1, x2, x3;
-          mul2(x0, x1, u4[i].x, u4[i].y, v[c], v[c]);
-          mul2(x2, x3, u4[i].z, u4[i].w, v[c], v[c]);
-          fma2(S[i][0][c], S[i][1][c], w4.x, w4.y, S[i][0][c], S[i][1][c], x0, x1);
-          fma2(S[i][2][c], S[i][3][c], w4.z, w4.w, S[i][2][c], S[i][3][c], x2, x3);
-        }
+          for (int c = 0; c < CPT; ++c) {
+            float x0, x1, x2, x3;
+            mul2(x0, x1, u4[i].x, u4[i].y, v[c], v[c]);
+            mul2(x2, x3, u4[i].z, u4[i].w, v[c], v[c]);
+            fma2(S[i][0][c], S[i][1][c], w4[i].x, w4[i].y, S[i][0][c], S[i][1][c], x0, x1);
+            fma2(S[i][2][c], S[i][3][c], w4[i].z, w4[i].w, S[i][2][c], S[i][3][c], x2, x3);
+          }
+#pragma unroll
+        for (int c = 0; c < CPT; ++c) seen[c] += more[c];
+      }
+      if (writes) *out = late[0];
+      out += step;
+      step = pitch;
+      {
+        const float* next = sw + (t + 1 < n ? TC + 1 : TC) * DP;
+#pragma unroll
+        for (int i = 0; i < NK; ++i) u4[i] = *reinterpret_cast<const float4*>(next + 4 * SPLIT * i);
       }
       float a[CPT][4];
 #pragma unroll
-      for (int c = 0; c < CPT; ++c) a[c][0] = a[c][1] = a[c][2] = a[c][3] = 0.f;
-#pragma unroll
-      for (int i = 0; i < NK; ++i) {
-        const float4 b4 = *reinterpret_cast<const float4*>(sw + 2 * TC * DP + 4 * SPLIT * i);
-        const float4 r4 = *reinterpret_cast<const float4*>(sw + 3 * TC * DP + 4 * SPLIT * i);
+      for (int i = 0; i < NK; ++i)
 #pragma unroll
         for (int c = 0; c < CPT; ++c) {
-          fma2(S[i][0][c], S[i][1][c], b4.x, b4.y, -seen[c], -seen[c], S[i][0][c], S[i][1][c]);
-          fma2(S[i][2][c], S[i][3][c], b4.z, b4.w, -seen[c], -seen[c], S[i][2][c], S[i][3][c]);
-          fma2(a[c][0], a[c][1], r4.x, r4.y, S[i][0][c], S[i][1][c], a[c][0], a[c][1]);
-          fma2(a[c][2], a[c][3], r4.z, r4.w, S[i][2][c], S[i][3][c], a[c][2], a[c][3]);
+          fma2(S[i][0][c], S[i][1][c], b4[i].x, b4[i].y, -seen[c], -seen[c], S[i][0][c], S[i][1][c]);
+          fma2(S[i][2][c], S[i][3][c], b4[i].z, b4[i].w, -seen[c], -seen[c], S[i][2][c], S[i][3][c]);
+          if (i == 0) {
+            mul2(a[c][0], a[c][1], r4[i].x, r4[i].y, S[i][0][c], S[i][1][c]);
+            mul2(a[c][2], a[c][3], r4[i].z, r4[i].w, S[i][2][c], S[i][3][c]);
+          } else {
+            fma2(a[c][0], a[c][1], r4[i].x, r4[i].y, S[i][0][c], S[i][1][c], a[c][0], a[c][1]);
+            fma2(a[c][2], a[c][3], r4[i].z, r4[i].w, S[i][2][c], S[i][3][c], a[c][2], a[c][3]);
+          }
         }
-      }
-      float s[CPT];
 #pragma unroll
-      for (int c = 0; c < CPT; ++c) s[c] = (a[c][0] + a[c][1]) + (a[c][2] + a[c][3]);
-      float y = s[0];
-      int o = 1;
-      if constexpr (CPT == 2) {       // the first exchange also spreads the columns over two lanes
-        const float other = __shfl_xor_sync(0xffffffffu, mine ? s[0] : s[1], 1);
-        y = (mine ? s[1] : s[0]) + other;
-        o = 2;
+      for (int c = 0; c < CPT; ++c) {
+        add2(a[c][0], a[c][1], a[c][2], a[c][3]);
+        late[c] = a[c][0] + a[c][1];
       }
-#pragma unroll
-      for (; o < SPLIT; o <<= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
-      if (writes) *out = y;
-      out += (long long)p.H * V;
     }
     __syncthreads();
   }
+#pragma unroll
+  for (int q = 0; q < STEPS; ++q) late_step(q);        // the last token's output
+  if (writes) *out = late[0];
   if (pool) {
 #pragma unroll
     for (int i = 0; i < NK; ++i)
@@ -354,14 +398,13 @@ __global__ void __launch_bounds__(RT) gdelta_finish_kernel(const DeltaParams p, 
 
 // ---- decode ---------------------------------------------------------------------------------------------------------
 constexpr int DCT = 256;
-constexpr int DKEEP = 16;      // rows of the state a thread holds
 
-// One token per sequence; VEC columns per thread. HELD: the state stays in registers between its two uses.
-template <typename T, int VEC, bool HELD>
+// One token per sequence; VEC columns per thread. KEEP: rows of the state a thread holds between its two uses (0: read twice).
+template <typename T, int VEC, int KEEP>
 __global__ void __launch_bounds__(DCT) gdelta_decode_kernel(const DeltaParams p) {
   extern __shared__ __align__(16) float dsm[];   // w | u | a u | r [D each] | x [rank] | seen [V] | sums [groups][V]
   __shared__ float red[32];
-  const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x, lane = tid & 31;
+  const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x;
   const long long t = p.cu[b];
   if (p.cu[b + 1] <= t) return;
   const int D = p.D, V = p.V, HD = h * D, rank = p.rank;
@@ -371,11 +414,11 @@ __global__ void __launch_bounds__(DCT) gdelta_decode_kernel(const DeltaParams p)
 
   // the state is on its way while the gates are formed
   const int cg = tid % vcols, rg = tid / vcols;
-  const bool on = HELD && rg < groups;
-  float s[HELD ? DKEEP : 1][VEC];
-  if constexpr (HELD) {
+  const bool on = KEEP && rg < groups;
+  float s[KEEP ? KEEP : 1][VEC];
+  if constexpr (KEEP > 0) {
 #pragma unroll
-    for (int i = 0; i < DKEEP; ++i) {
+    for (int i = 0; i < KEEP; ++i) {
       const int d = rg + i * groups;
       if (on && d < D) d_load<VEC>(st + (long long)d * V + cg * VEC, s[i]);
     }
@@ -390,36 +433,31 @@ __global__ void __launch_bounds__(DCT) gdelta_decode_kernel(const DeltaParams p)
     ss += kv * kv;
   }
   const float len = sqrtf(block_sum(ss, red) + p.unit_eps), inv = 1.f / len;      // its barriers also publish sx and su
-  // a warp forms the low-rank products of a channel at a time, four of them in flight
+  // low-rank products: a few adjacent lanes share a channel
   const T* w2 = reinterpret_cast<const T*>(p.w2) + (long long)HD * rank;
   const bool vec2 = rank % 4 == 0 && (reinterpret_cast<uintptr_t>(p.w2) & 15) == 0;
-  for (int d0 = (tid >> 5) * 4; d0 < D; d0 += (DCT / 32) * 4) {
-    float z[4] = {0.f, 0.f, 0.f, 0.f};
-    if (vec2) {
-      for (int i = lane * 4; i < rank; i += 128) {
-#pragma unroll
-        for (int q = 0; q < 4; ++q)
-          if (d0 + q < D) {
-            float m[4];
-            d_load<4>(w2 + (long long)(d0 + q) * rank + i, m);
-            z[q] += m[0] * sx[i] + m[1] * sx[i + 1] + m[2] * sx[i + 2] + m[3] * sx[i + 3];
-          }
+  int share = 1;
+  while (share < 32 && 2 * share * D <= DCT) share <<= 1;
+  for (int d0 = 0; d0 < D; d0 += DCT / share) {      // the same rounds for every lane
+    const int d = d0 + tid / share, sub = tid % share;
+    float z = 0.f;
+    if (d < D) {
+      const T* m = w2 + (long long)d * rank;
+      if (vec2) {
+#pragma unroll 4
+        for (int i = sub * 4; i < rank; i += share * 4) {
+          float c[4];
+          d_load<4>(m + i, c);
+          z += (c[0] * sx[i] + c[1] * sx[i + 1]) + (c[2] * sx[i + 2] + c[3] * sx[i + 3]);
+        }
+      } else {
+        for (int i = sub; i < rank; i += share) z += d_of(m[i]) * sx[i];
       }
-    } else {
-      for (int i = lane; i < rank; i += 32)
-#pragma unroll
-        for (int q = 0; q < 4; ++q)
-          if (d0 + q < D) z[q] += d_of(w2[(long long)(d0 + q) * rank + i]) * sx[i];
     }
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1)
-#pragma unroll
-      for (int q = 0; q < 4; ++q) z[q] += __shfl_xor_sync(0xffffffffu, z[q], o);
-    if (lane < 4 && d0 + lane < D) {
-      const int d = d0 + lane;
-      const float zz = lane == 0 ? z[0] : lane == 1 ? z[1] : lane == 2 ? z[2] : z[3];
+    for (int o = share >> 1; o > 0; o >>= 1) z += __shfl_xor_sync(0xffffffffu, z, o);
+    if (d < D && sub == 0) {
       const float u = su[d] * inv;
-      sw[d] = expf(-p.rate * sigm(zz + p.w0[HD + d]));
+      sw[d] = expf(-p.rate * sigm(z + p.w0[HD + d]));
       su[d] = u;
       sb[d] = sigm(d_of(reinterpret_cast<const T*>(p.a)[t * p.ld + HD + d]) + p.a0[HD + d]) * u;
       sr[d] = d_of(reinterpret_cast<const T*>(p.r)[t * p.ld + HD + d]);
@@ -433,9 +471,9 @@ __global__ void __launch_bounds__(DCT) gdelta_decode_kernel(const DeltaParams p)
     float acc[VEC];
 #pragma unroll
     for (int j = 0; j < VEC; ++j) acc[j] = 0.f;
-    if constexpr (HELD) {
+    if constexpr (KEEP > 0) {
 #pragma unroll
-      for (int i = 0; i < DKEEP; ++i) {
+      for (int i = 0; i < KEEP; ++i) {
         const int d = g + i * groups;
         if (d < D)
 #pragma unroll
@@ -476,9 +514,9 @@ __global__ void __launch_bounds__(DCT) gdelta_decode_kernel(const DeltaParams p)
       }
       d_store<VEC>(st + (long long)d * V + c * VEC, a);
     };
-    if constexpr (HELD) {
+    if constexpr (KEEP > 0) {
 #pragma unroll
-      for (int i = 0; i < DKEEP; ++i)
+      for (int i = 0; i < KEEP; ++i)
         if (g + i * groups < D) update(g + i * groups, s[i]);
     } else {
       for (int d = g; d < D; d += groups) {
@@ -555,11 +593,18 @@ int run_scan(DeltaParams& p, cudaStream_t s) {
   if (p.vec) gdelta_rows_kernel<T, 4><<<blocks, RT, 0, s>>>(p, lanes);
   else gdelta_rows_kernel<T, 1><<<blocks, RT, 0, s>>>(p, lanes);
   if (check_cuda(cudaGetLastError(), "gdelta_rows launch")) return -1;
-  if (p.D <= 32) return launch_scan<32, 8, 2, 64>(p, s);
-  if (p.D <= 64) return launch_scan<64, 16, 2, 64>(p, s);
-  if (p.D <= 128) return launch_scan<128, 16, 2, 64>(p, s);
+  // one column per thread while the GPU is not full of warps (the shortest wait per token), else more
+  const long long warps = (long long)p.B * p.H * p.V * (p.D <= 64 ? 4 : p.D <= 128 ? 8 : 16) / 32;
+  const int cols = warps <= 4LL * sm_count() ? 1 : warps <= 8LL * sm_count() ? 2 : 4;
+#define EDL_GS(DP, RPT, NT_)                                        \
+  return cols == 1 ? launch_scan<DP, RPT, 1, NT_>(p, s) : cols == 2 \
+             ? launch_scan<DP, RPT, 2, NT_>(p, s) : launch_scan<DP, RPT, 4, NT_>(p, s)
+  if (p.D <= 32) EDL_GS(32, 8, 64);
+  if (p.D <= 64) EDL_GS(64, 16, 64);
+  if (p.D <= 128) EDL_GS(128, 16, 64);
   if (p.D <= 256) return launch_scan<256, 16, 2, 128>(p, s);
   return launch_scan<512, 16, 2, 128>(p, s);
+#undef EDL_GS
 }
 
 bool bad_sizes(const char* who, int B, int H, int D, int V) {
@@ -635,11 +680,15 @@ EDL_HOST_API int edl_gdelta_decode(const void* r, const void* k, const void* v, 
   const bool v4 = V % 4 == 0 && al(state, 16);
   const int vcols = v4 ? V / 4 : V;
   const int groups = vcols >= DCT ? 1 : DCT / vcols;
-  const bool held = vcols <= DCT && (D + groups - 1) / groups <= DKEEP;
+  const int rows = vcols <= DCT ? (D + groups - 1) / groups : 17;
   const size_t smem = (size_t)(4 * D + rank + V + groups * V) * sizeof(float);     // <= 2048 + 4096 + 1024 + 1024 floats
   const dim3 grid(H, B);
-#define EDL_GD(TT, V_, H_) gdelta_decode_kernel<TT, V_, H_><<<grid, DCT, smem, s>>>(p)
-#define EDL_GDH(TT, V_) if (held) EDL_GD(TT, V_, true); else EDL_GD(TT, V_, false)
+#define EDL_GD(TT, V_, K_) gdelta_decode_kernel<TT, V_, K_><<<grid, DCT, smem, s>>>(p)
+#define EDL_GDH(TT, V_)                \
+  if (rows <= 4) EDL_GD(TT, V_, 4);    \
+  else if (rows <= 8) EDL_GD(TT, V_, 8);  \
+  else if (rows <= 16) EDL_GD(TT, V_, 16); \
+  else EDL_GD(TT, V_, 0)
   if (f32) {
     if (v4) { EDL_GDH(float, 4); } else { EDL_GDH(float, 1); }
   } else {

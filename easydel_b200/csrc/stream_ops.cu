@@ -11,7 +11,7 @@
 //   * xIELU, a two-branch activation with two learned numbers;
 //   * the attention prologue: per-head RMS norm of q and k, position-dependent query temperature and the page append,
 //     in one pass over the packed projection;
-//   * the same with biases, norms over all query heads (all key heads) at once, rotated halves or neighbours, and values that
+//   * the same with biases, optional norms over all query heads (all key heads) at once, rotated halves or neighbours, and values that
 //     blend with another layer's;
 //   * a branch that is normed (and scaled per channel) before it joins the stream, with the norm that reads the sum;
 //   * gated units in 32 bits or at odd sizes, and scaled and soft-capped logits.
@@ -578,12 +578,28 @@ __device__ __forceinline__ float2 turn_of(const RotaryPrologueParams& p, float f
   return make_float2((c * ce - s * se) * p.mag, (s * ce + c * se) * p.mag);
 }
 
+template <int VEC>
+__device__ __forceinline__ void ldw(const float* w, float (&v)[VEC]) {
+  if constexpr (VEC % 4 == 0) {
+#pragma unroll
+    for (int i = 0; i < VEC; i += 4) {
+      const float4 a = *reinterpret_cast<const float4*>(w + i);
+      v[i] = a.x; v[i + 1] = a.y; v[i + 2] = a.z; v[i + 3] = a.w;
+    }
+  } else {
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) v[i] = w[i];
+  }
+}
+
 // v[j] += bias[at + j]
 template <int VEC>
 __device__ __forceinline__ void add_bias(const float* bias, int at, float (&v)[VEC]) {
   if (!bias) return;
+  float b[VEC];
+  ldw<VEC>(bias + at, b);
 #pragma unroll
-  for (int j = 0; j < VEC; ++j) v[j] += bias[at + j];
+  for (int j = 0; j < VEC; ++j) v[j] += b[j];
 }
 
 // Values of token t from column c on: bias, blend with the first layer's.
@@ -599,23 +615,57 @@ __device__ __forceinline__ void finish_values(const RotaryPrologueParams& p, int
   }
 }
 
-template <int VEC>
-__device__ __forceinline__ void ldw(const float* w, float (&v)[VEC]) {
-  if constexpr (VEC % 4 == 0) {
+// Piece u of a head: VEC elements and their partners (neighbours, unless VEC is 1, are each other's partners within the piece).
+// The first `turned` pieces rotate by the cosines cs of their pairs. at: the head's place in the row (for the bias); w, r: norm
+// weights of the head and the factor of its norm (w null: no norm).
+template <typename T, int VEC>
+__device__ __forceinline__ void turn_unit(const RotaryPrologueParams& p, const T* src, T* dst, int at, const float* w, float r,
+                                          int u, int turned, const float2* cs) {
+  auto load = [&](int c, float (&v)[VEC]) {
+    ldv<VEC>(src + c, v);
+    add_bias<VEC>(p.bias, at + c, v);
+    if (w) {
+      float wv[VEC];
+      ldw<VEC>(w + c, wv);
 #pragma unroll
-    for (int i = 0; i < VEC; i += 4) {
-      const float4 a = *reinterpret_cast<const float4*>(w + i);
-      v[i] = a.x; v[i + 1] = a.y; v[i + 2] = a.z; v[i + 3] = a.w;
+      for (int j = 0; j < VEC; ++j) v[j] *= r * wv[j];
     }
-  } else {
+  };
+  float a[VEC];
+  if (u >= turned) {
+    const int c = 2 * p.pairs + (u - turned) * VEC;
+    load(c, a);
+    stv<VEC>(dst + c, a);
+  } else if (p.neighbours && VEC > 1) {
+    const int c = u * VEC;
+    load(c, a);
 #pragma unroll
-    for (int i = 0; i < VEC; ++i) v[i] = w[i];
+    for (int j = 0; j + 1 < VEC; j += 2) {
+      const float2 g = cs[(c + j) >> 1];
+      const float x = a[j], y = a[j + 1];
+      a[j] = x * g.x - y * g.y;
+      a[j + 1] = y * g.x + x * g.y;
+    }
+    stv<VEC>(dst + c, a);
+  } else {
+    const int c = p.neighbours ? 2 * u : u * VEC, partner = c + (p.neighbours ? 1 : p.pairs);
+    float b[VEC];
+    load(c, a);
+    load(partner, b);
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) {
+      const float2 g = cs[u * VEC + j];
+      const float x = a[j], y = b[j];
+      a[j] = x * g.x - y * g.y;
+      b[j] = y * g.x + x * g.y;
+    }
+    stv<VEC>(dst + c, a);
+    stv<VEC>(dst + partner, b);
   }
 }
 
 // One CTA per token: qkv [T, ld] as above. Queries and keys are RMS-normed over all their heads at once, then the pairs of
-// every head turn by position * frequency. A thread handles VEC elements and their partners (neighbours, unless VEC is 1, are
-// each other's partners within the piece).
+// every head turn by position * frequency.
 template <typename T, int VEC>
 __global__ void __launch_bounds__(NT)
 qkv_rotary_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, T* __restrict__ k_pages, T* __restrict__ v_pages,
@@ -662,48 +712,7 @@ qkv_rotary_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, T* __restric
     const T* src = row + h * p.D;                    // key heads follow the query heads
     const float* w = is_q ? (p.qw ? p.qw + h * p.D : nullptr) : (p.kw ? p.kw + (h - p.Hq) * p.D : nullptr);
     T* dst = is_q ? q_out + ((long long)t * p.Hq + h) * p.D : k_pages + slot * p.ld_kpage + (h - p.Hq) * p.D;
-    const float r = is_q ? rq : rk;
-    auto load = [&](int c, float (&v)[VEC]) {
-      ldv<VEC>(src + c, v);
-      add_bias<VEC>(p.bias, h * p.D + c, v);
-      if (w) {
-        float wv[VEC];
-        ldw<VEC>(w + c, wv);
-#pragma unroll
-        for (int j = 0; j < VEC; ++j) v[j] *= r * wv[j];
-      }
-    };
-    float a[VEC];
-    if (u < turned && inside) {
-      const int c = u * VEC;
-      load(c, a);
-#pragma unroll
-      for (int j = 0; j + 1 < VEC; j += 2) {
-        const float2 g = cs[(c + j) >> 1];
-        const float x = a[j], y = a[j + 1];
-        a[j] = x * g.x - y * g.y;
-        a[j + 1] = y * g.x + x * g.y;
-      }
-      stv<VEC>(dst + c, a);
-    } else if (u < turned) {
-      const int c = p.neighbours ? 2 * u : u * VEC, partner = c + (p.neighbours ? 1 : p.pairs);
-      float b[VEC];
-      load(c, a);
-      load(partner, b);
-#pragma unroll
-      for (int j = 0; j < VEC; ++j) {
-        const float2 g = cs[u * VEC + j];
-        const float x = a[j], y = b[j];
-        a[j] = x * g.x - y * g.y;
-        b[j] = y * g.x + x * g.y;
-      }
-      stv<VEC>(dst + c, a);
-      stv<VEC>(dst + partner, b);
-    } else {
-      const int c = 2 * p.pairs + (u - turned) * VEC;
-      load(c, a);
-      stv<VEC>(dst + c, a);
-    }
+    turn_unit<T, VEC>(p, src, dst, h * p.D, w, is_q ? rq : rk, u, turned, cs);
   }
   if (slot >= 0)
     for (int c = tid * VEC; c < p.Hkv * p.Dv; c += NT * VEC) {
@@ -714,7 +723,7 @@ qkv_rotary_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, T* __restric
     }
 }
 
-// The same for rows whose units (a piece of VEC elements and its partner) fit KEEP to a thread: a CTA walks the tokens
+// The same for halves whose units (a piece of VEC elements and its partner) fit KEEP to a thread, without biases and blends: a CTA walks the tokens
 // blockIdx.x, blockIdx.x + gridDim.x, ...; norm weights stay in registers, each row is read once, the next one while the
 // current one is normed, and cosines and partial sums have two buffers, so that a token costs one barrier.
 constexpr int RW_THREADS = 512;
@@ -728,18 +737,16 @@ qkv_rotary_walk_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, T* __re
   __shared__ float2 red[2][RW_THREADS / 32];
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, warps = (blockDim.x + 31) >> 5;
   const int nq = p.Hq * p.D, nk = p.Hkv * p.D, nv = p.Hkv * p.Dv;
-  const int turned = (p.neighbours ? 2 : 1) * p.pairs / VEC, per = turned + (p.D - 2 * p.pairs) / VEC;
-  const int units = (p.Hq + p.Hkv) * per;
-  int col[KEEP];             // first element within the row (< 0: no unit); halves have a partner `pairs` further
-  bool pair[KEEP], inside[KEEP];
+  const int turned = p.pairs / VEC, per = turned + (p.D - 2 * p.pairs) / VEC, units = (p.Hq + p.Hkv) * per;
+  int col[KEEP];             // first element within the row (< 0: no unit); partner `pairs` further
+  bool pair[KEEP];
   float wa[KEEP][VEC], wb[KEEP][VEC];
 #pragma unroll
   for (int i = 0; i < KEEP; ++i) {
     const int u = tid + i * blockDim.x;
     const int h = u / per, r = u - h * per;
-    pair[i] = r < turned && !p.neighbours;
-    inside[i] = r < turned && p.neighbours;
-    col[i] = u < units ? h * p.D + (r < turned ? r * VEC : 2 * p.pairs + (r - turned) * VEC) : -1;
+    pair[i] = r < turned;
+    col[i] = u < units ? h * p.D + (pair[i] ? r * VEC : 2 * p.pairs + (r - turned) * VEC) : -1;
 #pragma unroll
     for (int j = 0; j < VEC; ++j) wa[i][j] = wb[i][j] = 1.f;
     if (col[i] >= 0) {
@@ -771,18 +778,9 @@ qkv_rotary_walk_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, T* __re
       slot = -1;
     }
     if (slot >= 0)
-      for (int c = tid * VEC; c < nv; c += blockDim.x * VEC) {
-        const T* src = qkv + t * p.ld + nq + nk + c;
-        T* dst = v_pages + slot * p.ld_vpage + c;
-        if (p.lam || p.bias) {
-          float v[VEC];
-          ldv<VEC>(src, v);
-          finish_values<T, VEC>(p, t, c, nq + nk + c, v);
-          stv<VEC>(dst, v);
-        } else {
-          *reinterpret_cast<Raw*>(dst) = *reinterpret_cast<const Raw*>(src);
-        }
-      }
+      for (int c = tid * VEC; c < nv; c += blockDim.x * VEC)
+        *reinterpret_cast<Raw*>(v_pages + slot * p.ld_vpage + c) =
+            *reinterpret_cast<const Raw*>(qkv + t * p.ld + nq + nk + c);
     const float fp = p.pairs ? (float)p.pos[t] : 0.f;
     for (int i = tid; i < p.pairs; i += blockDim.x) cs[buf][i] = turn_of(p, fp, i);
     float va[KEEP][VEC], vb[KEEP][VEC], sq = 0.f, sk = 0.f;
@@ -790,32 +788,24 @@ qkv_rotary_walk_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, T* __re
     for (int i = 0; i < KEEP; ++i) {
       if (col[i] < 0) continue;
       ldv<VEC>(reinterpret_cast<const T*>(&a[i]), va[i]);
-      add_bias<VEC>(p.bias, col[i], va[i]);
       float s = 0.f;
 #pragma unroll
       for (int j = 0; j < VEC; ++j) s += va[i][j] * va[i][j];
       if (pair[i]) {
         ldv<VEC>(reinterpret_cast<const T*>(&b[i]), vb[i]);
-        add_bias<VEC>(p.bias, col[i] + p.pairs, vb[i]);
 #pragma unroll
         for (int j = 0; j < VEC; ++j) s += vb[i][j] * vb[i][j];
       }
       if (col[i] < nq) sq += s; else sk += s;
     }
     if (t + (int)gridDim.x < rows) load(t + gridDim.x);
-    const bool normed = p.qw || p.kw;
-    if (normed) {
-      sq = warp_sum(sq);
-      sk = warp_sum(sk);
-      if (lane == 0) red[buf][warp] = make_float2(sq, sk);
-    }
+    sq = warp_sum(sq);
+    sk = warp_sum(sk);
+    if (lane == 0) red[buf][warp] = make_float2(sq, sk);
     __syncthreads();
-    float2 sums = make_float2(0.f, 0.f);
-    if (normed) {
-      if (lane < warps) sums = red[buf][lane];
-      sums.x = warp_sum(sums.x);
-      sums.y = warp_sum(sums.y);
-    }
+    float2 sums = lane < warps ? red[buf][lane] : make_float2(0.f, 0.f);
+    sums.x = warp_sum(sums.x);
+    sums.y = warp_sum(sums.y);
     const float rq = p.qw ? 1.f / sqrtf(sums.x / (float)nq + p.eps) : 1.f;
     const float rk = p.kw ? 1.f / sqrtf(sums.y / (float)nk + p.eps) : 1.f;
 #pragma unroll
@@ -837,15 +827,6 @@ qkv_rotary_walk_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, T* __re
           vb[i][j] = y * g.x + x * g.y;
         }
         stv<VEC>(dst + p.pairs, vb[i]);
-      } else if (inside[i]) {
-        const int c0 = (col[i] % p.D) >> 1;
-#pragma unroll
-        for (int j = 0; j < VEC; j += 2) {
-          const float2 g = cs[buf][c0 + (j >> 1)];
-          const float x = va[i][j], y = va[i][j + 1];
-          va[i][j] = x * g.x - y * g.y;
-          va[i][j + 1] = y * g.x + x * g.y;
-        }
       }
       stv<VEC>(dst, va[i]);
     }
@@ -855,7 +836,7 @@ qkv_rotary_walk_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, T* __re
 template <typename T, int VEC>
 bool launch_rotary_walk(const void* qkv, void* q_out, void* k_pages, void* v_pages, const RotaryPrologueParams& p, int rows,
                         cudaStream_t s) {
-  const int units = (p.Hq + p.Hkv) * ((p.neighbours ? 2 : 1) * p.pairs / VEC + (p.D - 2 * p.pairs) / VEC);
+  const int units = (p.Hq + p.Hkv) * (p.pairs / VEC + (p.D - 2 * p.pairs) / VEC);
   const int keep = units <= RW_THREADS ? 1 : 2;
   if (units > 2 * RW_THREADS) return false;
   const int threads = ((units + keep - 1) / keep + 31) / 32 * 32;
@@ -865,6 +846,69 @@ bool launch_rotary_walk(const void* qkv, void* q_out, void* k_pages, void* v_pag
   if (keep == 1) EDL_RW(1); else EDL_RW(2);
 #undef EDL_RW
   return true;
+}
+
+// Without norms nothing ties a token's heads together: a CTA takes a few tokens, forms their cosines, and then every warp
+// streams one token's pieces (q and k heads, then values).
+constexpr int TURN_WARPS = 8;
+constexpr int TURN_PAIRS = 2048;      // cosines of a CTA
+
+template <typename T, int VEC>
+__global__ void __launch_bounds__(TURN_WARPS * 32)
+qkv_turn_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, T* __restrict__ k_pages, T* __restrict__ v_pages,
+                const RotaryPrologueParams p, int rows, int tokens, int shift) {
+  __shared__ float2 cs[TURN_PAIRS];
+  const int t0 = blockIdx.x * tokens, n = min(tokens, rows - t0);
+  for (int i = threadIdx.x; i < n * p.pairs; i += TURN_WARPS * 32) {
+    const int t = i / p.pairs;
+    cs[i] = turn_of(p, (float)p.pos[t0 + t], i - t * p.pairs);
+  }
+  __syncthreads();
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, split = TURN_WARPS / tokens;    // warps of a token
+  const int mine = warp / split, sub = warp - mine * split;
+  if (mine >= n) return;
+  const int t = t0 + mine;
+  const bool inside = p.neighbours && VEC > 1;
+  const int turned = (inside ? 2 : 1) * p.pairs / VEC, per = turned + (p.D - 2 * p.pairs) / VEC;
+  const int nq = p.Hq * p.D, nk = p.Hkv * p.D, heads = p.Hq + p.Hkv, vunits = p.Hkv * p.Dv / VEC;
+  const float2* g = cs + mine * p.pairs;
+  const T* row = qkv + t * p.ld;
+  long long slot = p.slots[t];
+  if (slot >= p.num_slots) {
+    if (p.status && lane == 0) atomicCAS(p.status, 0, EDL_BAD_INDEX);
+    slot = -1;
+  }
+  const int units = slot >= 0 ? heads * per : p.Hq * per;
+  T* kdst = k_pages + slot * p.ld_kpage;
+#pragma unroll 4
+  for (int i = sub * 32 + lane; i < units; i += split * 32) {
+    const int h = shift >= 0 ? i >> shift : i / per;
+    const T* src = row + h * p.D;
+    T* dst = h < p.Hq ? q_out + (long long)t * nq + h * p.D : kdst + (h - p.Hq) * p.D;
+    turn_unit<T, VEC>(p, src, dst, h * p.D, nullptr, 1.f, i - h * per, turned, g);
+  }
+  if (slot >= 0)
+#pragma unroll 2
+    for (int i = sub * 32 + lane; i < vunits; i += split * 32) {
+      float v[VEC];
+      ldv<VEC>(row + nq + nk + i * VEC, v);
+      finish_values<T, VEC>(p, t, i * VEC, nq + nk + i * VEC, v);
+      stv<VEC>(v_pages + slot * p.ld_vpage + i * VEC, v);
+    }
+}
+
+template <typename T, int VEC>
+void launch_turn(const void* qkv, void* q_out, void* k_pages, void* v_pages, const RotaryPrologueParams& p, int rows,
+                 cudaStream_t s) {
+  int tokens = TURN_WARPS;                // of a CTA: a power of two, fewer when there are few of them
+  while (tokens > 1 && (rows < 2 * sm_count() * tokens || tokens * p.pairs > TURN_PAIRS)) tokens >>= 1;
+  const int per = ((p.neighbours && VEC > 1 ? 2 : 1) * p.pairs + p.D - 2 * p.pairs) / VEC;
+  int shift = -1;
+  if ((per & (per - 1)) == 0)
+    for (shift = 0; (1 << shift) < per; ++shift) {
+    }
+  qkv_turn_kernel<T, VEC><<<(rows + tokens - 1) / tokens, TURN_WARPS * 32, 0, s>>>(
+      (const T*)qkv, (T*)q_out, (T*)k_pages, (T*)v_pages, p, rows, tokens, shift);
 }
 
 // ---- a normed branch joins the stream ----------------------------------------------------------------------------------------
@@ -1190,9 +1234,23 @@ EDL_HOST_API int edl_qkv_rotary_prologue(const void* qkv, int f32, long long ld,
   auto fits = [&](int m, size_t a) {
     return D % m == 0 && (neighbours ? 2 * pairs : pairs) % m == 0 && Dv % m == 0 && ld % m == 0 &&
            (!lam || (ld_first % m == 0 && al(v_first, a))) && ld_kpage % m == 0 && ld_vpage % m == 0 &&
-           al(qkv, a) && al(q_out, a) && al(k_pages, a) && al(v_pages, a) && (!qw || al(qw, 16)) && (!kw || al(kw, 16));
+           al(qkv, a) && al(q_out, a) && al(k_pages, a) && al(v_pages, a) && (!qw || al(qw, 16)) && (!kw || al(kw, 16)) &&
+           (!bias || al(bias, 16));
   };
-  const bool walked = f32 ? fits(4, 16) && launch_rotary_walk<float, 4>(qkv, q_out, k_pages, v_pages, p, T, s)
+#define EDL_RT(TT, V_) launch_turn<TT, V_>(qkv, q_out, k_pages, v_pages, p, T, s)
+  if (!qw && !kw) {
+    if (f32) {
+      if (fits(4, 16)) EDL_RT(float, 4); else EDL_RT(float, 1);
+    } else {
+      if (fits(8, 16)) EDL_RT(__nv_bfloat16, 8);
+      else if (fits(4, 8)) EDL_RT(__nv_bfloat16, 4);
+      else EDL_RT(__nv_bfloat16, 1);
+    }
+    return check_cuda(cudaGetLastError(), "qkv_turn launch");
+  }
+#undef EDL_RT
+  const bool plain = !neighbours && !bias && !lam;
+  const bool walked = !plain ? false : f32 ? fits(4, 16) && launch_rotary_walk<float, 4>(qkv, q_out, k_pages, v_pages, p, T, s)
                           : fits(8, 16) && launch_rotary_walk<__nv_bfloat16, 8>(qkv, q_out, k_pages, v_pages, p, T, s);
   if (walked) return check_cuda(cudaGetLastError(), "qkv_rotary_prologue launch");
 #define EDL_RP(TT, V_) \
