@@ -41,6 +41,7 @@ def _entry(rank, fn, world, port, args):
         dist.barrier()      # nobody tears its sockets down while a peer still has transfers in flight
     finally:
         dist.destroy_process_group()
+    os._exit(0)             # the rank has passed: gloo's threads and the interpreter's teardown race on a loaded machine
 
 
 def _tiny(seed):
