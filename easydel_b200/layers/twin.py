@@ -39,7 +39,8 @@ class TwinMixer(nn.Module):
         cols = ssm.DeltaColumns(r, k, v, a, g, x)
         n, (ls, rs) = self.left.out_width, self.scales
         if stream.on_kernels(h):
-            out = torch.empty(h.shape[0], n + self.right.out_width, dtype=h.dtype, device=h.device)
+            width = n + self.right.out_width
+            out = torch.empty(h.shape[0], (width + 7) // 8 * 8, dtype=h.dtype, device=h.device)[:, :width]   # aligned rows
             self.left.mix_rows(qkv, step, view, gate=parts[9], out=out[:, :n], out_scale=ls)
             self.right.mix_rows(cols, step, state, out[:, n:], rs)
             return out

@@ -101,6 +101,10 @@ def paged_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tenso
         assert q.stride(-1) == 1 and q.stride(-2) == D
         if out is None:
             out = torch.empty((T, Hq, Dv), dtype=q.dtype, device=q.device)
+        elif not _aligned_rows(out):
+            return out.copy_(paged_attention(q, k_pages, v_pages, cu_q, kv_lens, page_table, max_q, scale=scale, causal=causal,
+                                             window=window, softcap=softcap, sinks=sinks, keep_first=keep_first,
+                                             sigmoid=sigmoid))
         if sigmoid is not None:
             assert causal and not softcap and sinks is None
             _lib.call("edl_attn_paged_sigmoid", q.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), out.data_ptr(),
@@ -164,7 +168,7 @@ def decode_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tens
     Hkv, Dv = k_pages.shape[2], v_pages.shape[-1]
     scale = scale if scale is not None else 1.0 / math.sqrt(D)
     S_ = max(1, int(num_splits))
-    if sigmoid is not None:
+    if sigmoid is not None and (out is None or _aligned_rows(out)):
         assert not softcap and sinks is None
         if out is None:
             out = torch.empty((B, Hq, Dv), dtype=q.dtype, device=q.device)
@@ -177,7 +181,7 @@ def decode_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tens
         return out
     if out is not None:
         return out.copy_(decode_attention(q, k_pages, v_pages, kv_lens, page_table, scale=scale, window=window, sinks=sinks,
-                                          num_splits=S_, softcap=softcap, keep_first=keep_first))
+                                          num_splits=S_, softcap=softcap, keep_first=keep_first, sigmoid=sigmoid))
     out = torch.empty((S_, B, Hq, Dv), dtype=q.dtype, device=q.device)
     lse = torch.empty((S_, Hq, B), dtype=torch.float32, device=q.device) if S_ > 1 else None
     _lib.call("edl_attn_decode", q.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), out.data_ptr(), _lib.ptr(lse),
@@ -224,6 +228,11 @@ def latent_decode(q_lat: torch.Tensor, q_rot: torch.Tensor, pages: torch.Tensor,
 def mla_decode_kernel_supports(q: torch.Tensor, pages: torch.Tensor) -> bool:
     return (q.is_cuda and q.dtype == torch.bfloat16 and pages.dtype == torch.bfloat16 and q.shape[-1] == 576
             and pages.shape[-1] == 576 and pages.shape[1] == PAGE_SIZE and pages.is_contiguous())
+
+
+def _aligned_rows(out: torch.Tensor) -> bool:
+    """The tensor-core kernels store 16 bytes at a time."""
+    return out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0
 
 
 def _tile_width(n: int) -> bool:

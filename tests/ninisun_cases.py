@@ -31,6 +31,11 @@ CONFIGS = {
          O.windowed(16, 2, 128, 64, 0.06, 260, 130, base=1e5, dims=64, mlp=O.dense(128)),
          O.parallel((8, 2, 64, 128, 0.09, 16, 1e4, YARN), (1, 128), (0.5, 0.8), O.dense(96)),
          O.windowed(34, 2, 64, 64, 0.09, 150, 7)], 128, 90),
+    # attention heads that fit the tiles beside states, ranks and gates that do not; no feed-forward anywhere
+    "uneven": O.random_config(
+        [O.parallel((3, 1, 32, 40, 0.2, 10, 700.0, YARN), (3, 21), (1.2, 0.9)),
+         O.windowed(5, 1, 40, 16, 0.2, 50, 2, dims=6, v_mix=False),
+         O.parallel((7, 7, 16, 8, 0.3, 16, 700.0, None), (1, 50), (0.9, 1.4))], 68, 59),
     # one kind of layer only; factors of one
     "windowed": O.random_config([O.windowed(4, 2, 32, 32, 0.2, 64, 2, mlp=O.dense(64)),
                                  O.windowed(8, 2, 64, 32, 0.1, 20, 129, dims=2)], 72, 64),
@@ -41,7 +46,7 @@ CONFIGS = {
 
 def make(tmp_path, name, dtype, device, seed=0, cfg=None, weights=None):
     cfg = cfg or CONFIGS[name]
-    w = weights or O.random_weights(cfg, seed, rank=5 if name == "odd" else 24 if name == "wide" else 8)
+    w = weights or O.random_weights(cfg, seed, rank=5 if name in ("odd", "uneven") else 24 if name == "wide" else 8)
     return cfg, w, load(write_checkpoint(tmp_path / name, cfg, w), dtype, device)
 
 
